@@ -10,7 +10,7 @@ the paged design instead:
   page, -1 where no page is held;
 * pages are taken before a step writes into them (:meth:`CacheManager.reserve`), and
   given back when the request ends (:meth:`release`) or, in a window group, once every
-  position of the page is older than the window (:meth:`commit`);
+  position of the page is older than the window (:meth:`commit`), except pages that hold a first token the group keeps;
 * free pages are handed out most-recently-freed first, so reuse happens quickly and
   tests can force it;
 * every request also holds one **state slot**, an index into per-call arrays of
@@ -74,8 +74,10 @@ class PagePool:
 
 @dataclass
 class GroupNeed:
-    """What a cache group needs to know to place tokens: the window, or None for all keys."""
+    """What a cache group needs to know to place tokens: the window, or None for all keys, and with a window how many of a
+    sequence's first keys stay besides."""
     window: Optional[int] = None
+    keep_first: int = 0
 
 
 @dataclass
@@ -182,7 +184,8 @@ class CacheManager:
         r.length += n_new
         for g, table in enumerate(r.tables):
             first = min(self._first_needed_page(g, r.length), len(table))   # the next query sits at r.length
-            for lp in range(first):
+            kept = (self.groups[g].keep_first + self.page_size - 1) // self.page_size     # pages that hold a kept first token
+            for lp in range(kept, first):
                 if table[lp] >= 0:
                     self.pools[g].give_back(table[lp])
                     table[lp] = -1

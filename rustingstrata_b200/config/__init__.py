@@ -3,6 +3,7 @@ from .lokinex_config import LokinexConfig
 from .tabedra_config import TabedraConfig
 from .kupelix_config import KupelixConfig
 from .kozasun_config import KozasunConfig
+from .sefelorn_config import SefelornConfig
 from .engine_config import EngineConfig
 from .registry import (Architecture, register_architecture, unregister_architecture, registered_architectures,
                        resolve_architecture, load_model_config)

@@ -49,16 +49,35 @@ __device__ __forceinline__ float gelu_tanh_mul_fast(float gate, float up) {
     const float y = 0.7978845608028654f * fmaf(0.044715f * gate * gate, gate, gate);
     return __fdividef(gate, 1.0f + __expf(-2.0f * y)) * up;
 }
-// Epilogue codes of the bfloat16 products that gate: 3 SiLU(gate) * up, 4 GELU(gate) * up (tanh form).
-#define RS_EPI_GATED(e) ((e) == 3 || (e) == 4)
+// The clamped gate: with g = min(gate, limit) and u = up held in [-limit, limit], g sigmoid(alpha g) (u + 1).
+struct GateParams { float alpha, limit; };
+__device__ __forceinline__ float clamped_mul_fast(float gate, float up, GateParams gp) {
+    const float g = fminf(gate, gp.limit), u = fminf(fmaxf(up, -gp.limit), gp.limit);
+    return __fdividef(g, 1.0f + __expf(-gp.alpha * g)) * (u + 1.0f);
+}
+// Epilogue codes of the bfloat16 products that gate: 3 SiLU(gate) * up, 4 GELU(gate) * up (tanh form), 5 the clamped gate
+// (its two constants are the launch's; the other codes ignore them).
+#define RS_EPI_GATED(e) ((e) == 3 || (e) == 4 || (e) == 5)
 template <int EPI>
-__device__ __forceinline__ float gated_mul_fast(float gate, float up) {
-    return EPI == 4 ? gelu_tanh_mul_fast(gate, up) : silu_mul_fast(gate, up);
+__device__ __forceinline__ float gated_mul_fast(float gate, float up, GateParams gp) {
+    return EPI == 5 ? clamped_mul_fast(gate, up, gp) : EPI == 4 ? gelu_tanh_mul_fast(gate, up) : silu_mul_fast(gate, up);
 }
 __device__ __forceinline__ float fast_exp2(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
+}
+
+// four weights (float32 or bfloat16, by code) from element 4 i on; four values rounded to bfloat16 in 8 bytes
+__device__ __forceinline__ float4 load_weights4(const void* w, int w_dt, int i) {
+    if (w_dt == RS_F32) return reinterpret_cast<const float4*>(w)[i];
+    const uint2 h = reinterpret_cast<const uint2*>(w)[i];
+    const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&h.x), b = *reinterpret_cast<const __nv_bfloat162*>(&h.y);
+    return make_float4(__low2float(a), __high2float(a), __low2float(b), __high2float(b));
+}
+__device__ __forceinline__ uint2 pack_bf16x4(float x, float y, float z, float w) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(x, y), hi = __floats2bfloat162_rn(z, w);
+    return make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

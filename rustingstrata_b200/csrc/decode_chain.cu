@@ -304,7 +304,7 @@ decode_chain_kernel(const __grid_constant__ ChainMaps maps, const __grid_constan
                 const int KB = (op.K + TILE_K - 1) / TILE_K;
                 const int U = ((op.N + TILE_N - 1) / TILE_N) * KB;
                 const int u0 = first_unit(blockIdx.x, U, G), u1 = first_unit(blockIdx.x + 1, U, G);
-                SkinnyParams sp;
+                SkinnyParams sp; sp.gate = {0.f, 0.f};
                 sp.C = op.C; sp.ldc = op.ldc; sp.M = op.M; sp.N = op.N; sp.K = op.K; sp.stages = stages;
                 sp.workspace = p.workspace; sp.status = p.status;
                 float acc[NT][4], acc2[NT][4];
@@ -349,7 +349,7 @@ decode_chain_kernel(const __grid_constant__ ChainMaps maps, const __grid_constan
                 if (ok && (int)blockIdx.x < G - 1) {
                     const SharedTile st = shared_tile_of_boundary(blockIdx.x + 1, op.N, op.K, G);
                     if (st.acts) {
-                        SkinnyParams sp;
+                        SkinnyParams sp; sp.gate = {0.f, 0.f};
                         sp.C = op.C; sp.ldc = op.ldc; sp.M = op.M; sp.N = op.N; sp.K = op.K; sp.stages = stages;
                         sp.workspace = p.workspace; sp.status = p.status;
                         if (op.epi == EPI_STORE_BF16) finish_shared_tile<NT, EPI_STORE_BF16>(sp, st, G, warp, g, t);

@@ -42,7 +42,7 @@ RS_EXPORT int rs_embed(const void* table, int table_dt, const int* ids, float* o
 template <typename TO>
 __global__ void rmsnorm_kernel(const float* __restrict__ x, long x_stride, const int* __restrict__ rows,
                                const void* __restrict__ w, int w_dt, float eps, TO* __restrict__ out, long out_stride,
-                               int n) {
+                               const void* __restrict__ w2, TO* __restrict__ out2, long out2_stride, int n) {
     __shared__ float scratch[33];
     pdl_launch_dependents();
     pdl_wait();
@@ -53,34 +53,32 @@ __global__ void rmsnorm_kernel(const float* __restrict__ x, long x_stride, const
     ss = block_sum(ss, scratch);
     const float s = 1.0f / sqrtf(ss / (float)n + eps);
     TO* o = out + (size_t)r * out_stride;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) o[i] = from_f32<TO>(ld_dep(xr + i) * s * load_any(w, w_dt, i));
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const float y = ld_dep(xr + i) * s;
+        o[i] = from_f32<TO>(y * load_any(w, w_dt, i));
+        if (w2) out2[(size_t)r * out2_stride + i] = from_f32<TO>(y * load_any(w2, w_dt, i));
+    }
 }
 
 // The same for a bfloat16 output when the row fits the block's registers (n <= 512 * 4 * VPT, n % 4 == 0, 16-byte
-// aligned rows): one read of x with float4 loads, the row kept in registers between the sum and the scaling.
-template <int VPT>
+// aligned rows): one read of x with float4 loads, the row kept in registers between the sum and the scaling.  PAIR: a
+// second output with weights of its own, from the same read and the same sum.
+template <int VPT, bool PAIR>
 __global__ void __launch_bounds__(512) rmsnorm_bf16_vec_kernel(const float* x, long x_stride, const int* __restrict__ rows,
                                                                const void* __restrict__ w, int w_dt, float eps,
-                                                               __nv_bfloat16* __restrict__ out, long out_stride, int n) {
+                                                               __nv_bfloat16* __restrict__ out, long out_stride,
+                                                               const void* __restrict__ w2, __nv_bfloat16* __restrict__ out2,
+                                                               long out2_stride, int n) {
     __shared__ float scratch[33];
     pdl_launch_dependents();
     const int n4 = n >> 2;
     // the weights are the model's, not the previous kernel's: they are fetched while that kernel is still at work
-    float wv[VPT][4];
+    float4 wv[VPT], wv2[PAIR ? VPT : 1];
 #pragma unroll
     for (int u = 0; u < VPT; ++u) {
         const int i = threadIdx.x + u * 512;
-        wv[u][0] = wv[u][1] = wv[u][2] = wv[u][3] = 0.f;
-        if (i < n4) {
-            if (w_dt == RS_F32) {
-                const float4 f = reinterpret_cast<const float4*>(w)[i];
-                wv[u][0] = f.x; wv[u][1] = f.y; wv[u][2] = f.z; wv[u][3] = f.w;
-            } else {
-                const uint2 h = reinterpret_cast<const uint2*>(w)[i];
-                const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&h.x), b = *reinterpret_cast<const __nv_bfloat162*>(&h.y);
-                wv[u][0] = __low2float(a); wv[u][1] = __high2float(a); wv[u][2] = __low2float(b); wv[u][3] = __high2float(b);
-            }
-        }
+        wv[u] = i < n4 ? load_weights4(w, w_dt, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        if (PAIR) wv2[u] = i < n4 ? load_weights4(w2, w_dt, i) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     pdl_wait();
     const int r = blockIdx.x;
@@ -100,30 +98,34 @@ __global__ void __launch_bounds__(512) rmsnorm_bf16_vec_kernel(const float* x, l
     for (int u = 0; u < VPT; ++u) {
         const int i = threadIdx.x + u * 512;
         if (i < n4) {
-            const __nv_bfloat162 lo = __floats2bfloat162_rn(v[u].x * s * wv[u][0], v[u].y * s * wv[u][1]);
-            const __nv_bfloat162 hi = __floats2bfloat162_rn(v[u].z * s * wv[u][2], v[u].w * s * wv[u][3]);
-            uint2 pk;
-            pk.x = *reinterpret_cast<const uint32_t*>(&lo); pk.y = *reinterpret_cast<const uint32_t*>(&hi);
-            reinterpret_cast<uint2*>(o)[i] = pk;
+            reinterpret_cast<uint2*>(o)[i] = pack_bf16x4(v[u].x * s * wv[u].x, v[u].y * s * wv[u].y, v[u].z * s * wv[u].z, v[u].w * s * wv[u].w);
+            if (PAIR)
+                reinterpret_cast<uint2*>(out2 + (size_t)r * out2_stride)[i] =
+                    pack_bf16x4(v[u].x * s * wv2[u].x, v[u].y * s * wv2[u].y, v[u].z * s * wv2[u].z, v[u].w * s * wv2[u].w);
         }
     }
 }
 
+// out[r] = RMSNorm(x[r]) * w; with w2 also out2[r] = RMSNorm(x[r]) * w2 (the row is read and its square summed once).
 RS_EXPORT int rs_rmsnorm(const float* x, long x_stride, const int* rows, const void* w, int w_dt, float eps,
-                         void* out, int out_dt, long out_stride, int n_rows, int n, void* stream) {
+                         void* out, int out_dt, long out_stride, const void* w2, void* out2, long out2_stride, int n_rows, int n,
+                         void* stream) {
     if (n_rows <= 0) return 0;
+    if ((w2 == nullptr) != (out2 == nullptr)) return (int)cudaErrorInvalidValue;
     if (out_dt == RS_BF16 && n % 4 == 0 && n <= 512 * 4 * 4 && x_stride % 4 == 0 && out_stride % 4 == 0 && ((long)x & 15) == 0 &&
-        ((long)out & 7) == 0 && ((long)w & 15) == 0) {
-        auto* o = (__nv_bfloat16*)out;
+        ((long)out & 7) == 0 && ((long)w & 15) == 0 && ((long)w2 & 15) == 0 && ((long)out2 & 7) == 0 && out2_stride % 4 == 0) {
+        auto *o = (__nv_bfloat16*)out, *o2 = (__nv_bfloat16*)out2;
         cudaStream_t s = (cudaStream_t)stream;
-        if (n <= 512 * 4) return rs_launch_pdl(rmsnorm_bf16_vec_kernel<1>, dim3(n_rows), dim3(512), 0, s, x, x_stride, rows, w, w_dt, eps, o, out_stride, n);
-        if (n <= 512 * 8) return rs_launch_pdl(rmsnorm_bf16_vec_kernel<2>, dim3(n_rows), dim3(512), 0, s, x, x_stride, rows, w, w_dt, eps, o, out_stride, n);
-        return rs_launch_pdl(rmsnorm_bf16_vec_kernel<4>, dim3(n_rows), dim3(512), 0, s, x, x_stride, rows, w, w_dt, eps, o, out_stride, n);
+#define RS_NORM(V, P) rs_launch_pdl(rmsnorm_bf16_vec_kernel<V, P>, dim3(n_rows), dim3(512), 0, s, x, x_stride, rows, w, w_dt, eps, o, out_stride, w2, o2, out2_stride, n)
+        if (n <= 512 * 4) return w2 ? RS_NORM(1, true) : RS_NORM(1, false);
+        if (n <= 512 * 8) return w2 ? RS_NORM(2, true) : RS_NORM(2, false);
+        return w2 ? RS_NORM(4, true) : RS_NORM(4, false);
+#undef RS_NORM
     }
     const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : 128);
     RS_DISPATCH_DTYPE(out_dt, TO,
         return rs_launch_pdl(rmsnorm_kernel<TO>, dim3(n_rows), dim3(threads), 0, (cudaStream_t)stream, x, x_stride, rows, w,
-                             w_dt, eps, (TO*)out, out_stride, n));
+                             w_dt, eps, (TO*)out, out_stride, w2, (TO*)out2, out2_stride, n));
     return 0;
 }
 
@@ -363,26 +365,33 @@ RS_EXPORT int rs_qk_norm_rope_kv(void* qkv, int dt, long row_stride, int n_q, in
 
 // --------------------------------------------------------------------------- act(gate) * up
 // in: [rows, 2*I] with gate in columns [0, I) and up in [I, 2I); out: [rows, I].  act: 0 SiLU, 1 the tanh form of GELU,
-// 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))); float32 arithmetic.
+// 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), 2 the clamped gate: with g = min(gate, limit) and u = up held in
+// [-limit, limit], g sigmoid(alpha g) (u + 1); float32 arithmetic.
 template <typename T>
 __global__ void silu_mul_kernel(const T* __restrict__ in, long in_stride, T* __restrict__ out, long out_stride,
-                                int rows, int I, int act) {
+                                int rows, int I, int act, GateParams gp) {
     const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= (long)rows * I) return;
     const int r = (int)(idx / I), c = (int)(idx % I);
-    const float g = to_f32<T>(in[(size_t)r * in_stride + c]);
-    const float u = to_f32<T>(in[(size_t)r * in_stride + I + c]);
+    float g = to_f32<T>(in[(size_t)r * in_stride + c]);
+    float u = to_f32<T>(in[(size_t)r * in_stride + I + c]);
+    if (act == 2) {
+        g = fminf(g, gp.limit);
+        u = fminf(fmaxf(u, -gp.limit), gp.limit);
+        out[(size_t)r * out_stride + c] = from_f32<T>(g / (1.0f + expf(-gp.alpha * g)) * (u + 1.0f));
+        return;
+    }
     const float a = act == 1 ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g / (1.0f + expf(-g));
     out[(size_t)r * out_stride + c] = from_f32<T>(a * u);
 }
 
 RS_EXPORT int rs_silu_mul(const void* in, long in_stride, void* out, long out_stride, int dt, int rows, int I, int act,
-                          void* stream) {
+                          float gate_alpha, float gate_limit, void* stream) {
     if (rows <= 0) return 0;
     const long n = (long)rows * I;
     RS_DISPATCH_DTYPE(dt, T,
         silu_mul_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>((const T*)in, in_stride,
-                                                                                       (T*)out, out_stride, rows, I, act));
+                                                                                       (T*)out, out_stride, rows, I, act, GateParams{gate_alpha, gate_limit}));
     return rs_launch_result();
 }
 
@@ -399,6 +408,28 @@ RS_EXPORT int rs_residual_add(float* x, const void* delta, int dt, long n, void*
     RS_DISPATCH_DTYPE(dt, T,
         residual_add_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(x, (const T*)delta, n));
     return rs_launch_result();
+}
+
+// x[t, :] += scale * table[ids[t], :] in float32
+__global__ void add_embed_kernel(float* x, long x_stride, const void* __restrict__ table, int table_dt, const int* __restrict__ ids,
+                                 int V, float scale, int n, int* status) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    int id = ld_dep(ids + t);
+    if (id < 0 || id >= V) {
+        if (threadIdx.x == 0) atomicOr(status, RS_STATUS_BAD_TOKEN);
+        id = 0;
+    }
+    float* xr = x + (size_t)t * x_stride;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) xr[i] = fmaf(scale, load_any(table, table_dt, (size_t)id * n + i), ld_dep(xr + i));
+}
+
+RS_EXPORT int rs_add_embed(float* x, long x_stride, const void* table, int table_dt, const int* ids, int V, float scale, int n_tokens,
+                           int n, int* status, void* stream) {
+    if (n_tokens <= 0) return 0;
+    return rs_launch_pdl(add_embed_kernel, dim3(n_tokens), dim3(n >= 512 ? 256 : 128), 0, (cudaStream_t)stream, x, x_stride, table, table_dt,
+                         ids, V, scale, n, status);
 }
 
 // dst[i] = src[idx[i]]: the ids a step chose, brought into the order of the next step's rows on the device

@@ -27,7 +27,7 @@ constexpr int UMMA_K = 16;
 constexpr int A_BYTES = BM * BK * 2;      // 16 KiB
 constexpr int THREADS = 192;
 
-enum Epilogue : int { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_GEGLU_BF16 = 4 };
+enum Epilogue : int { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_GEGLU_BF16 = 4, EPI_CLAMPED_BF16 = 5 };
 
 template <int BN> struct Cfg {
     static constexpr int B_BYTES = BN * BK * 2;
@@ -111,6 +111,7 @@ struct GemmParams {
     int vec_ok;            // C rows allow 16-byte vector access
     int bn;                // columns per tile: the template's BN, or less (a multiple of 16) in buffers sized for BN
     int out_by_tma;        // float32 results leave through shared memory and the TMA unit (map_c is valid)
+    GateParams gate;       // constants of the clamped gate
     int* status;
 };
 
@@ -128,7 +129,7 @@ __device__ __forceinline__ void epilogue_chunk(const GemmParams& p, const uint32
             for (int j = 0; j < 8; ++j) {
                 const float g0 = __uint_as_float(r[4 * j]), u0 = __uint_as_float(r[4 * j + 1]);
                 const float g1 = __uint_as_float(r[4 * j + 2]), u1 = __uint_as_float(r[4 * j + 3]);
-                __nv_bfloat162 v = __floats2bfloat162_rn(gated_mul_fast<EPI>(g0, u0), gated_mul_fast<EPI>(g1, u1));
+                __nv_bfloat162 v = __floats2bfloat162_rn(gated_mul_fast<EPI>(g0, u0, p.gate), gated_mul_fast<EPI>(g1, u1, p.gate));
                 packed[j] = *reinterpret_cast<uint32_t*>(&v);
             }
             reinterpret_cast<uint4*>(out)[0] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
@@ -138,7 +139,7 @@ __device__ __forceinline__ void epilogue_chunk(const GemmParams& p, const uint32
             for (int j = 0; j < 16; ++j) {
                 if (oc0 + j < half_n) {
                     const float g = __uint_as_float(r[2 * j]), u = __uint_as_float(r[2 * j + 1]);
-                    out[j] = __float2bfloat16_rn(gated_mul_fast<EPI>(g, u));
+                    out[j] = __float2bfloat16_rn(gated_mul_fast<EPI>(g, u, p.gate));
                 }
             }
         }
@@ -341,7 +342,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                             for (int j = 0; j < 4; ++j) {
                                 const float g0 = __uint_as_float(r[16 * q + 4 * j]), u0 = __uint_as_float(r[16 * q + 4 * j + 1]);
                                 const float g1 = __uint_as_float(r[16 * q + 4 * j + 2]), u1 = __uint_as_float(r[16 * q + 4 * j + 3]);
-                                __nv_bfloat162 v = __floats2bfloat162_rn(gated_mul_fast<EPI>(g0, u0), gated_mul_fast<EPI>(g1, u1));
+                                __nv_bfloat162 v = __floats2bfloat162_rn(gated_mul_fast<EPI>(g0, u0, p.gate), gated_mul_fast<EPI>(g1, u1, p.gate));
                                 w[j] = *reinterpret_cast<uint32_t*>(&v);
                             }
                             *reinterpret_cast<uint4*>(dst + lane * 128 + (((part * 2 + q) ^ (lane & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -437,6 +438,7 @@ int launch_epi(int epi, const CUtensorMap& ma, const CUtensorMap& mw, const CUte
         case EPI_ADD_F32: return launch<BN, EPI_ADD_F32>(ma, mw, mc, p, max_ctas, s);
         case EPI_SWIGLU_BF16: return launch<BN, EPI_SWIGLU_BF16>(ma, mw, mc, p, max_ctas, s);
         case EPI_GEGLU_BF16: return launch<BN, EPI_GEGLU_BF16>(ma, mw, mc, p, max_ctas, s);
+        case EPI_CLAMPED_BF16: return launch<BN, EPI_CLAMPED_BF16>(ma, mw, mc, p, max_ctas, s);
     }
     return (int)cudaErrorInvalidValue;
 }
@@ -453,10 +455,12 @@ RS_EXPORT int rs_gemm_tc_supported(long a_ptr, long lda, long w_ptr, long ldw, i
 
 // C[M, N] (=|+=) A[M, K] . W[N, K]^T with bf16 inputs.  a_rows is the row capacity of A's buffer (>= M): the
 // tensor map covers the whole buffer, rows beyond M are computed and dropped.  epi: 0 bf16 store, 1 f32 store,
-// 2 f32 accumulate, 3 SiLU(gate)*up over interleaved columns into a bf16 [M, N/2] output.  bn: columns per tile, 64, 128,
+// 2 f32 accumulate, 3 to 5 act(gate)*up over interleaved columns into a bf16 [M, N/2] output (common.cuh; gate_alpha and
+// gate_limit are code 5's constants).  bn: columns per tile, 64, 128,
 // a multiple of 16 from 144 to 256, or 0 to choose.  max_ctas > 0 caps the grid (tests use it to force several tiles per CTA).
 RS_EXPORT int rs_gemm_bf16_tc(const void* A, long lda, long a_rows, const void* W, long ldw, void* C, long ldc, int M,
-                              int N, int K, int epi, int bn, int max_ctas, int* status, void* stream) {
+                              int N, int K, int epi, int bn, int max_ctas, float gate_alpha, float gate_limit, int* status,
+                              void* stream) {
     if (M <= 0 || N <= 0) return 0;
     if (!rs_gemm_tc_supported((long)A, lda, (long)W, ldw, N, K, epi) || a_rows < M) return (int)cudaErrorInvalidValue;
     int tpl = bn;                                        // template instantiation (buffer sizes): 64, 128 or 256
@@ -485,7 +489,7 @@ RS_EXPORT int rs_gemm_bf16_tc(const void* A, long lda, long a_rows, const void* 
     rc = get_map(W, N, K, ldw, bn, &mw);
     if (rc) return rc;
     GemmParams p;
-    p.C = C; p.ldc = ldc; p.M = M; p.N = N; p.K = K; p.status = status; p.bn = bn;
+    p.C = C; p.ldc = ldc; p.M = M; p.N = N; p.K = K; p.status = status; p.bn = bn; p.gate = {gate_alpha, gate_limit};
     const int out_elem = (epi == EPI_STORE_BF16 || RS_EPI_GATED(epi)) ? 2 : 4;
     p.vec_ok = (((long)C & 15) == 0 && (ldc * out_elem) % 16 == 0) ? 1 : 0;
     // results go out through the TMA unit when a tile's columns fill whole 128-byte rows of the staging tiles

@@ -41,7 +41,7 @@ constexpr int W_BYTES = W_BOX_BYTES * BOXES;
 constexpr int THREADS = 192;
 constexpr int SMEM_BUDGET = 200 * 1024;
 
-enum Epilogue : int { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_GEGLU_BF16 = 4 };
+enum Epilogue : int { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_GEGLU_BF16 = 4, EPI_CLAMPED_BF16 = 5 };
 
 struct MidParams {
     void* C; long ldc;
@@ -49,6 +49,7 @@ struct MidParams {
     int stages;
     int vec_ok;                // rows of C allow 16-byte (f32) / 8-byte (bf16) access at every fourth column
     float* workspace;          // [grid][2][MP][128] float32 partials
+    GateParams gate;           // constants of the clamped gate
     int* status;
 };
 
@@ -97,7 +98,7 @@ __device__ __forceinline__ void store_value(const MidParams& p, float v, int m, 
         // rows of W alternate gate, up: the even lane of a pair writes
         const float up = __shfl_xor_sync(0xffffffffu, v, 1);
         if ((n & 1) == 0 && n + 1 < p.N)
-            ((__nv_bfloat16*)p.C)[(size_t)m * p.ldc + (n >> 1)] = __float2bfloat16_rn(gated_mul_fast<EPI>(v, up));
+            ((__nv_bfloat16*)p.C)[(size_t)m * p.ldc + (n >> 1)] = __float2bfloat16_rn(gated_mul_fast<EPI>(v, up, p.gate));
     } else if (n < p.N) {
         const size_t o = (size_t)m * p.ldc + n;
         if (EPI == EPI_STORE_BF16) ((__nv_bfloat16*)p.C)[o] = __float2bfloat16_rn(v);
@@ -112,7 +113,7 @@ template <int EPI>
 __device__ __forceinline__ void store_four(const MidParams& p, float4 v, float4 old, int m, int n0) {
     if (RS_EPI_GATED(EPI)) {
         __nv_bfloat16* out = (__nv_bfloat16*)p.C + (size_t)m * p.ldc + (n0 >> 1);
-        const float a = gated_mul_fast<EPI>(v.x, v.y), b = gated_mul_fast<EPI>(v.z, v.w);
+        const float a = gated_mul_fast<EPI>(v.x, v.y, p.gate), b = gated_mul_fast<EPI>(v.z, v.w, p.gate);
         if (p.vec_ok && n0 + 3 < p.N) {
             *reinterpret_cast<__nv_bfloat162*>(out) = __floats2bfloat162_rn(a, b);
         } else {
@@ -414,6 +415,7 @@ int launch_epi(int epi, const CUtensorMap& mw, const CUtensorMap& ma, const MidP
         case EPI_ADD_F32: return launch<MP, EPI_ADD_F32>(mw, ma, p, max_ctas, defer, s);
         case EPI_SWIGLU_BF16: return launch<MP, EPI_SWIGLU_BF16>(mw, ma, p, max_ctas, defer, s);
         case EPI_GEGLU_BF16: return launch<MP, EPI_GEGLU_BF16>(mw, ma, p, max_ctas, defer, s);
+        case EPI_CLAMPED_BF16: return launch<MP, EPI_CLAMPED_BF16>(mw, ma, p, max_ctas, defer, s);
     }
     return (int)cudaErrorInvalidValue;
 }
@@ -430,7 +432,8 @@ RS_EXPORT long rs_mid_gemm_workspace_floats() { return (long)rs_tma::sm_count() 
 // rs_mid_finish or rs_mid_finish_rmsnorm is launched with the same C, shape, workspace and max_ctas; no other product
 // of this kind may run in between.
 RS_EXPORT int rs_mid_gemm_bf16(const void* A, long lda, long a_rows, const void* W, long ldw, void* C, long ldc, int M, int N,
-                               int K, int epi, float* workspace, int max_ctas, int defer, int* status, void* stream) {
+                               int K, int epi, float* workspace, int max_ctas, int defer, float gate_alpha, float gate_limit,
+                               int* status, void* stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M > 128 || K <= 0 || K % 8 || lda % 8 || ldw % 8 || ((long)A & 15) || ((long)W & 15) || a_rows < M ||
         workspace == nullptr)
@@ -445,7 +448,7 @@ RS_EXPORT int rs_mid_gemm_bf16(const void* A, long lda, long a_rows, const void*
     if (rc) return rc;
     MidParams p;
     p.C = C; p.ldc = ldc; p.M = M; p.N = N; p.K = K; p.stages = 0; p.workspace = workspace;
-    p.status = status;
+    p.status = status; p.gate = {gate_alpha, gate_limit};
     const int out_elem = (epi == EPI_STORE_BF16 || RS_EPI_GATED(epi)) ? 2 : 4;
     p.vec_ok = (((long)C & 15) == 0 && (ldc * out_elem) % 16 == 0) ? 1 : 0;
     cudaStream_t s = (cudaStream_t)stream;
@@ -459,7 +462,7 @@ RS_EXPORT int rs_mid_gemm_bf16(const void* A, long lda, long a_rows, const void*
 RS_EXPORT int rs_mid_finish(void* C, long ldc, int M, int N, int K, float* workspace, int max_ctas, void* stream) {
     if (M <= 0 || M > 128 || N <= 0 || K <= 0 || workspace == nullptr) return (int)cudaErrorInvalidValue;
     MidParams p;
-    p.C = C; p.ldc = ldc; p.M = M; p.N = N; p.K = K; p.stages = 0; p.workspace = workspace; p.status = nullptr;
+    p.C = C; p.ldc = ldc; p.M = M; p.N = N; p.K = K; p.stages = 0; p.workspace = workspace; p.status = nullptr; p.gate = {0.f, 0.f};
     p.vec_ok = (((long)C & 15) == 0 && (ldc * 4) % 16 == 0) ? 1 : 0;
     const long grid = grid_of(N, K, max_ctas);
     if (grid < 2) return 0;
@@ -473,11 +476,13 @@ RS_EXPORT int rs_mid_finish(void* C, long ldc, int M, int N, int K, float* works
     }
 }
 
-// Finishes a deferred product and writes out[m] = RMSNorm(C[m]) * w as bfloat16, in one kernel (one CTA per row).
+// Finishes a deferred product and writes out[m] = RMSNorm(C[m]) * w as bfloat16 (with w2 also out2[m] = RMSNorm(C[m]) * w2),
+// in one kernel (one CTA per row).
 RS_EXPORT int rs_mid_finish_rmsnorm(void* C, long ldc, int M, int N, int K, float* workspace, int max_ctas, const void* w,
-                                    int w_dt, float eps, void* out, long out_stride, void* stream) {
+                                    int w_dt, float eps, void* out, long out_stride, const void* w2, void* out2, long out2_stride,
+                                    void* stream) {
     if (M <= 0 || M > 128) return (int)cudaErrorInvalidValue;
     const rs_streamk::Layout L = {TILE_N, TILE_K, padded_rows(M)};
     return rs_streamk::launch_finish_rmsnorm(C, ldc, M, N, K, workspace, (int)grid_of(N, K, max_ctas), L, w, w_dt, eps, out, out_stride,
-                                             (cudaStream_t)stream);
+                                             w2, out2, out2_stride, (cudaStream_t)stream);
 }

@@ -210,6 +210,7 @@ int launch_epi(int epi, const CUtensorMap& mw, const CUtensorMap& ma, const Skin
         case EPI_ADD_F32: return launch<NT, EPI_ADD_F32>(mw, ma, p, max_ctas, defer, s);
         case EPI_SWIGLU_BF16: return launch<NT, EPI_SWIGLU_BF16>(mw, ma, p, max_ctas, defer, s);
         case EPI_GEGLU_BF16: return launch<NT, EPI_GEGLU_BF16>(mw, ma, p, max_ctas, defer, s);
+        case EPI_CLAMPED_BF16: return launch<NT, EPI_CLAMPED_BF16>(mw, ma, p, max_ctas, defer, s);
     }
     return (int)cudaErrorInvalidValue;
 }
@@ -226,8 +227,8 @@ RS_EXPORT long rs_skinny_gemm_workspace_floats() { return (long)rs_tma::sm_count
 // rs_skinny_finish or rs_skinny_finish_rmsnorm is launched with the same C, shape, workspace and max_ctas; no other
 // product may use the workspace in between.
 RS_EXPORT int rs_skinny_gemm_bf16(const void* A, long lda, long a_rows, const void* W, long ldw, void* C, long ldc, int M,
-                                  int N, int K, int epi, float* workspace, int max_ctas, int defer, int* status,
-                                  void* stream) {
+                                  int N, int K, int epi, float* workspace, int max_ctas, int defer, float gate_alpha,
+                                  float gate_limit, int* status, void* stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M > 64 || K <= 0 || K % 8 || lda % 8 || ldw % 8 || ((long)A & 15) || ((long)W & 15) || a_rows < M ||
         workspace == nullptr)
@@ -242,7 +243,7 @@ RS_EXPORT int rs_skinny_gemm_bf16(const void* A, long lda, long a_rows, const vo
     if (rc) return rc;
     SkinnyParams p;
     p.C = C; p.ldc = ldc; p.M = M; p.N = N; p.K = K; p.stages = 0; p.workspace = workspace;
-    p.status = status;
+    p.status = status; p.gate = {gate_alpha, gate_limit};
     cudaStream_t s = (cudaStream_t)stream;
     switch (nt) {
         case 1: return launch_epi<1>(epi, mw, ma, p, max_ctas, defer != 0, s);
@@ -256,7 +257,7 @@ RS_EXPORT int rs_skinny_gemm_bf16(const void* A, long lda, long a_rows, const vo
 RS_EXPORT int rs_skinny_finish(void* C, long ldc, int M, int N, int K, float* workspace, int max_ctas, void* stream) {
     if (M <= 0 || M > 8 || N <= 0 || K <= 0 || workspace == nullptr) return (int)cudaErrorInvalidValue;
     SkinnyParams p;
-    p.C = C; p.ldc = ldc; p.M = M; p.N = N; p.K = K; p.stages = 0; p.workspace = workspace; p.status = nullptr;
+    p.C = C; p.ldc = ldc; p.M = M; p.N = N; p.K = K; p.stages = 0; p.workspace = workspace; p.status = nullptr; p.gate = {0.f, 0.f};
     const long grid = grid_of(N, K, max_ctas);
     if (grid < 2) return 0;
     return rs_launch_pdl(skinny_reduce_kernel<1, EPI_ADD_F32>, dim3((unsigned)(grid - 1)), dim3(CONSUMER_WARPS * 32), 0,
@@ -269,11 +270,14 @@ namespace rs_streamk {
 // the same arithmetic in the same order (partials in CTA order, then added to C; the sum of squares by thread-strided
 // float4 partials and a tree), so the bits are those of the two kernels.  It saves a kernel boundary and a round trip
 // to memory between two small dependent kernels.  Rows of up to 512 * 4 * VPT values.
-// C[M, N] float32 with row pitch ldc; workspace, N, K, G, L: the product's; w: the norm's weights (float32 or bfloat16).
-template <int VPT>
+// C[M, N] float32 with row pitch ldc; workspace, N, K, G, L: the product's; w: the norm's weights (float32 or bfloat16).  PAIR: a
+// second output out2 with weights w2 from the same rows and sums.
+template <int VPT, bool PAIR>
 __global__ void __launch_bounds__(512) finish_rmsnorm_kernel(float* C, long ldc, int N, int K, const float* workspace, int G,
                                                              const Layout L, const void* __restrict__ w, int w_dt, float eps,
-                                                             __nv_bfloat16* __restrict__ out, long out_stride) {
+                                                             __nv_bfloat16* __restrict__ out, long out_stride,
+                                                             const void* __restrict__ w2, __nv_bfloat16* __restrict__ out2,
+                                                             long out2_stride) {
     constexpr int MAX_TILES = 512 * 4 * VPT / 64;              // tiles are at least 64 wide
     __shared__ float scratch[33];
     __shared__ int2 sharers[MAX_TILES];                        // per row tile: first and last CTA of the product that worked on it
@@ -287,21 +291,12 @@ __global__ void __launch_bounds__(512) finish_rmsnorm_kernel(float* C, long ldc,
     const int per_cta = U / G, extra = U % G;                  // the first `extra` CTAs take one unit more
     for (int tile = threadIdx.x; tile < n_tiles; tile += 512) sharers[tile] = sharers_of_tile(tile, KB, U, G);
     const int n4 = N >> 2;
-    float wv[VPT][4];
+    float4 wv[VPT], wv2[PAIR ? VPT : 1];
 #pragma unroll
     for (int u = 0; u < VPT; ++u) {
         const int idx = threadIdx.x + u * 512;
-        wv[u][0] = wv[u][1] = wv[u][2] = wv[u][3] = 0.f;
-        if (idx < n4) {
-            if (w_dt == RS_F32) {
-                const float4 f = reinterpret_cast<const float4*>(w)[idx];
-                wv[u][0] = f.x; wv[u][1] = f.y; wv[u][2] = f.z; wv[u][3] = f.w;
-            } else {
-                const uint2 h = reinterpret_cast<const uint2*>(w)[idx];
-                const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&h.x), b = *reinterpret_cast<const __nv_bfloat162*>(&h.y);
-                wv[u][0] = __low2float(a); wv[u][1] = __high2float(a); wv[u][2] = __low2float(b); wv[u][3] = __high2float(b);
-            }
-        }
+        wv[u] = idx < n4 ? load_weights4(w, w_dt, idx) : make_float4(0.f, 0.f, 0.f, 0.f);
+        if (PAIR) wv2[u] = idx < n4 ? load_weights4(w2, w_dt, idx) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     __syncthreads();
     pdl_wait();
@@ -339,11 +334,11 @@ __global__ void __launch_bounds__(512) finish_rmsnorm_kernel(float* C, long ldc,
     for (int u = 0; u < VPT; ++u) {
         const int idx = threadIdx.x + u * 512;
         if (idx < n4) {
-            const __nv_bfloat162 lo = __floats2bfloat162_rn(v[u].x * sc * wv[u][0], v[u].y * sc * wv[u][1]);
-            const __nv_bfloat162 hi2 = __floats2bfloat162_rn(v[u].z * sc * wv[u][2], v[u].w * sc * wv[u][3]);
-            uint2 pk;
-            pk.x = *reinterpret_cast<const uint32_t*>(&lo); pk.y = *reinterpret_cast<const uint32_t*>(&hi2);
-            reinterpret_cast<uint2*>(o)[idx] = pk;
+            reinterpret_cast<uint2*>(o)[idx] =
+                pack_bf16x4(v[u].x * sc * wv[u].x, v[u].y * sc * wv[u].y, v[u].z * sc * wv[u].z, v[u].w * sc * wv[u].w);
+            if (PAIR)
+                reinterpret_cast<uint2*>(out2 + (size_t)m * out2_stride)[idx] =
+                    pack_bf16x4(v[u].x * sc * wv2[u].x, v[u].y * sc * wv2[u].y, v[u].z * sc * wv2[u].z, v[u].w * sc * wv2[u].w);
         }
     }
 }
@@ -354,15 +349,19 @@ bool finish_rmsnorm_supported(const void* C, long ldc, int N, const void* w, con
 }
 
 int launch_finish_rmsnorm(void* C, long ldc, int M, int N, int K, const float* workspace, int G, Layout L, const void* w,
-                                 int w_dt, float eps, void* out, long out_stride, cudaStream_t s) {
+                                 int w_dt, float eps, void* out, long out_stride, const void* w2, void* out2, long out2_stride,
+                                 cudaStream_t s) {
     if (M <= 0 || M > L.rows_padded || K <= 0 || workspace == nullptr || G < 1 || (w_dt != RS_F32 && w_dt != RS_BF16) ||
-        L.tile_n < 64 || L.tile_n % 4 || !finish_rmsnorm_supported(C, ldc, N, w, out, out_stride))
+        L.tile_n < 64 || L.tile_n % 4 || !finish_rmsnorm_supported(C, ldc, N, w, out, out_stride) || (w2 == nullptr) != (out2 == nullptr) ||
+        (w2 && !finish_rmsnorm_supported(C, ldc, N, w2, out2, out2_stride)))
         return (int)cudaErrorInvalidValue;
     float* c = (float*)C;
-    auto* o = (__nv_bfloat16*)out;
-    if (N <= 512 * 4) return rs_launch_pdl(finish_rmsnorm_kernel<1>, dim3(M), dim3(512), 0, s, c, ldc, N, K, workspace, G, L, w, w_dt, eps, o, out_stride);
-    if (N <= 512 * 8) return rs_launch_pdl(finish_rmsnorm_kernel<2>, dim3(M), dim3(512), 0, s, c, ldc, N, K, workspace, G, L, w, w_dt, eps, o, out_stride);
-    return rs_launch_pdl(finish_rmsnorm_kernel<4>, dim3(M), dim3(512), 0, s, c, ldc, N, K, workspace, G, L, w, w_dt, eps, o, out_stride);
+    auto *o = (__nv_bfloat16*)out, *o2 = (__nv_bfloat16*)out2;
+#define RS_FINISH(V, P) rs_launch_pdl(finish_rmsnorm_kernel<V, P>, dim3(M), dim3(512), 0, s, c, ldc, N, K, workspace, G, L, w, w_dt, eps, o, out_stride, w2, o2, out2_stride)
+    if (N <= 512 * 4) return w2 ? RS_FINISH(1, true) : RS_FINISH(1, false);
+    if (N <= 512 * 8) return w2 ? RS_FINISH(2, true) : RS_FINISH(2, false);
+    return w2 ? RS_FINISH(4, true) : RS_FINISH(4, false);
+#undef RS_FINISH
 }
 }  // namespace rs_streamk
 
@@ -371,13 +370,15 @@ RS_EXPORT int rs_skinny_finish_rmsnorm_supported(const void* C, long ldc, int N,
     return rs_streamk::finish_rmsnorm_supported(C, ldc, N, w, out, out_stride) ? 1 : 0;
 }
 
-// Finishes a deferred product and writes out[m] = RMSNorm(C[m]) * w as bfloat16, in one kernel.
+// Finishes a deferred product and writes out[m] = RMSNorm(C[m]) * w as bfloat16 (with w2 also out2[m] = RMSNorm(C[m]) * w2),
+// in one kernel.
 RS_EXPORT int rs_skinny_finish_rmsnorm(void* C, long ldc, int M, int N, int K, float* workspace, int max_ctas, const void* w,
-                                       int w_dt, float eps, void* out, long out_stride, void* stream) {
+                                       int w_dt, float eps, void* out, long out_stride, const void* w2, void* out2,
+                                       long out2_stride, void* stream) {
     if (M > 8) return (int)cudaErrorInvalidValue;
     const rs_streamk::Layout L = {TILE_N, TILE_K, 8};
     return rs_streamk::launch_finish_rmsnorm(C, ldc, M, N, K, workspace, (int)grid_of(N, K, max_ctas), L, w, w_dt, eps, out, out_stride,
-                                             (cudaStream_t)stream);
+                                             w2, out2, out2_stride, (cudaStream_t)stream);
 }
 
 // Turns programmatic dependent launch on or off for every kernel of this library (default on).

@@ -20,7 +20,7 @@ constexpr int CONSUMER_WARPS = 4;
 constexpr int THREADS = (CONSUMER_WARPS + 1) * 32;
 constexpr int SMEM_BUDGET = 200 * 1024;
 
-enum Epilogue : int { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_GEGLU_BF16 = 4 };
+enum Epilogue : int { EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU_BF16 = 3, EPI_GEGLU_BF16 = 4, EPI_CLAMPED_BF16 = 5 };
 
 struct SkinnyParams {
     void* C; long ldc;
@@ -28,6 +28,7 @@ struct SkinnyParams {
     int stages;
     float* workspace;          // [grid][2][8 NT activation rows][TILE_N] float32 partials
     int* status;
+    GateParams gate;           // constants of the clamped gate
 };
 
 __device__ __forceinline__ uint4 lds128(uint32_t addr) {
@@ -54,7 +55,7 @@ __device__ __forceinline__ void store_tile(const SkinnyParams& p, const float (&
                     const int m = m0 + (i & 1), n = (i >> 1) ? nb : na;
                     if (m < p.M && n + 1 < p.N) {
                         const float gate = acc[j][i], up = partner[i];
-                        out[(size_t)m * p.ldc + (n >> 1)] = __float2bfloat16_rn(gated_mul_fast<EPI>(gate, up));
+                        out[(size_t)m * p.ldc + (n >> 1)] = __float2bfloat16_rn(gated_mul_fast<EPI>(gate, up, p.gate));
                     }
                 }
             }

@@ -1,11 +1,16 @@
 // Mixers that keep a matrix of state per head instead of a cache of keys, for both engines:
-//   * state_recurrence: per (sequence, head) a [rows, columns] float32 state walked token by token, in two forms:
+//   * state_recurrence: per (sequence, head) a [rows, columns] float32 state walked token by token, in three forms:
 //       gated write   S = diag(g) S + w v^T,                                    o = S^T q      (HGRN2: g = f, w = 1 - f)
 //       delta rule    S = diag(g) S;  u = beta (v - S^T k);  S = S + k u^T;     o = S^T q      (decay per key channel)
+//       head decay    S = a S + beta k v^T,                  o = S^T q + skip v                (a, beta one number per head)
 //   * hgrn2_prep: q = silu(.), forget gate with a lower bound, both laid out in padded rows;
 //   * retention_prep: q and k rotated by position (halves of the rotated prefix paired), k scaled, in padded rows;
 //   * delta_prep: short convolution over time + silu on q, k, v; unit-length q and k; decay and write strength;
+//   * mamba2_prep: short convolution over time + bias + silu of [x | B | C]; step size and decay of every head;
+//   * low_rank_decay: alpha = sigmoid(W2 u + b)^(1 / tau) per key channel from the inner rows u of a low-rank map;
+//   * pad_heads: heads of any width into rows of a padded width;
 //   * conv_tail_update: a request's last taps - 1 projected rows after the step;
+//   * gated_group_norm: rows times silu(z), then divided part by part by the part's root mean square, times a weight;
 //   * head_norm_gate: every head's read-out divided by its root mean square, times a weight and a sigmoid or SiLU gate;
 //   * activation: elementwise xIELU / tanh-GELU;  scale_rows: float32 rows times one number.
 // Gates, decays, norms and the state are float32 whatever the engine's element type.
@@ -32,16 +37,20 @@ constexpr int ROW_LANES = 8;
 constexpr int COLS_PER_CTA = 32;
 
 struct RecurrenceParams {
-    const float* q; long q_stride;          // [T, q heads * rows_pad]
-    const float* k; long k_stride;          // delta rule: keys [T, q heads * rows_pad]; gated write: w [T, heads * rows_pad]
-    const float* g; long g_stride;          // [T, heads * rows_pad] decay of every row
-    const float* beta; long beta_stride;    // [T, heads] (delta rule)
+    const float* q; long q_stride;          // [T, q heads * rows]
+    const float* k; long k_stride;          // keys [T, q heads * rows] (gated write: what is written, w)
+    const float* g; long g_stride;          // [T, heads * rows] decay of every row; head decay: [T, heads]
+    const float* beta; long beta_stride;    // [T, heads] write strength (delta rule, head decay)
     const float* v; long v_stride;          // [T, heads * columns]
     float* out; long out_stride;            // [T, heads * columns]
     float* state; long state_stride;        // [slots, heads * columns * rows_pad]
     const int* q_start; const int* slots;
-    int heads, group, columns;              // group: state heads per q/k head (delta rule)
+    int heads, group, columns;              // group: state heads per q/k head
+    int rows;                               // rows of a head in q, k and g (a multiple of 4, at most the padded rows)
+    float q_scale;                          // multiplies the read-out S^T q
+    const float* skip;                      // [heads] or null: head decay only, o += skip v
 };
+enum RecurrenceForm : int { REC_GATED = 0, REC_DELTA = 1, REC_HEAD = 2 };
 
 template <int RL>
 __device__ __forceinline__ float sum_row_lanes(float v) {
@@ -80,8 +89,9 @@ __device__ __forceinline__ void cp_async_4(void* dst, const void* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-template <int RPT, bool DELTA, int RL>
+template <int RPT, int FORM, int RL>
 __global__ void __launch_bounds__(256) state_recurrence_kernel(RecurrenceParams p) {
+    constexpr bool DELTA = FORM == REC_DELTA, HEAD = FORM == REC_HEAD;
     using St = RecurrenceStage<RPT * RL>;
     constexpr int RP = St::RP, CHUNK = St::CHUNK, ROW = St::ROW;
     extern __shared__ __align__(16) float stage[];         // [2][CHUNK][ROW]
@@ -98,13 +108,13 @@ __global__ void __launch_bounds__(256) state_recurrence_kernel(RecurrenceParams 
     float* sp = p.state + (size_t)p.slots[s] * p.state_stride + ((size_t)h * p.columns + jc) * RP + rl * 4;
     float S[RPT];
     load_rows<RPT, RL>(sp, S);
-    const size_t q_off = (size_t)(DELTA ? h / p.group : h) * RP;
-    const size_t k_off = DELTA ? q_off : (size_t)h * RP;
-    const size_t g_off = (size_t)h * RP;
+    const size_t q_off = (size_t)(h / p.group) * p.rows;
+    const size_t g_off = (size_t)h * p.rows;
 
-    // what this thread copies of every token: pieces tid, tid + threads, .. of the 3 RP / 4 16-byte pieces of q | k | g,
-    // and one of the CTA's values or the write strength
-    constexpr int PIECES = 3 * RP / 4, MAX_OWN = (PIECES + 63) / 64;
+    // what this thread copies of every token: pieces tid, tid + threads, .. of the 16-byte pieces of q | k | g (RP / 4
+    // each, head decay: q | k only), and one of the CTA's values, the write strength or the head's decay.  Rows beyond
+    // p.rows are not copied: they are zero in both buffers from the start.
+    constexpr int PIECES = (HEAD ? 2 : 3) * RP / 4, MAX_OWN = (PIECES + 63) / 64;
     const float* own_src[MAX_OWN];
     long own_step[MAX_OWN];
     int own_dst[MAX_OWN];
@@ -112,15 +122,21 @@ __global__ void __launch_bounds__(256) state_recurrence_kernel(RecurrenceParams 
     for (int e = 0; e < MAX_OWN; ++e) {
         const int piece = tid + e * nthreads;
         const int which = piece / (RP / 4), off = (piece % (RP / 4)) * 4;
-        own_dst[e] = piece < PIECES ? which * RP + off : -1;
+        own_dst[e] = piece < PIECES && off < p.rows ? which * RP + off : -1;
         own_step[e] = which == 0 ? p.q_stride : which == 1 ? p.k_stride : p.g_stride;
-        own_src[e] = (which == 0 ? p.q + q_off : which == 1 ? p.k + k_off : p.g + g_off) + (size_t)t0 * own_step[e] + off;
+        own_src[e] = (which == 0 ? p.q + q_off : which == 1 ? p.k + q_off : p.g + g_off) + (size_t)t0 * own_step[e] + off;
     }
-    const bool own_v = tid < cols_cta, own_b = DELTA && tid == cols_cta;
+    if (p.rows < RP)
+        for (int i = tid; i < 2 * CHUNK * 3 * RP; i += nthreads) {
+            const int tt = i / (3 * RP), c = i % (3 * RP);
+            if (c % RP >= p.rows) stage[tt * ROW + c] = 0.f;
+        }
+    const bool own_v = tid < cols_cta, own_b = FORM != REC_GATED && tid == cols_cta, own_a = HEAD && tid == cols_cta + 1;
     const float* small_src = own_v ? p.v + (size_t)t0 * p.v_stride + (size_t)h * p.columns + min((int)blockIdx.y * cols_cta + tid, p.columns - 1)
-                                   : p.beta + (size_t)t0 * p.beta_stride + h;
-    const long small_step = own_v ? p.v_stride : p.beta_stride;
-    const int small_dst = 3 * RP + (own_v ? tid : COLS_PER_CTA);
+                           : own_a ? p.g + (size_t)t0 * p.g_stride + h : p.beta + (size_t)t0 * p.beta_stride + h;
+    const long small_step = own_v ? p.v_stride : own_a ? p.g_stride : p.beta_stride;
+    const int small_dst = 3 * RP + (own_v ? tid : own_a ? COLS_PER_CTA + 1 : COLS_PER_CTA);
+    const float skip = HEAD && p.skip ? p.skip[h] : 0.f;
 
     auto fetch = [&](int c) {                               // chunk c of the step's tokens into buffer c & 1
         float* dst = stage + (size_t)(c & 1) * CHUNK * ROW;
@@ -131,7 +147,7 @@ __global__ void __launch_bounds__(256) state_recurrence_kernel(RecurrenceParams 
             const float* src = own_src[e] + (size_t)first * own_step[e];
             for (int tt = 0; tt < count; ++tt) cp_async_16(dst + tt * ROW + own_dst[e], src + (size_t)tt * own_step[e]);
         }
-        if (own_v || own_b) {
+        if (own_v || own_b || own_a) {
             const float* src = small_src + (size_t)first * small_step;
             for (int tt = 0; tt < count; ++tt) cp_async_4(dst + tt * ROW + small_dst, src + (size_t)tt * small_step);
         }
@@ -167,7 +183,7 @@ __global__ void __launch_bounds__(256) state_recurrence_kernel(RecurrenceParams 
             float qc[RPT], kc[RPT], gc[RPT];
             load_rows<RPT, RL>(row + rl * 4, qc);
             load_rows<RPT, RL>(row + RP + rl * 4, kc);
-            load_rows<RPT, RL>(row + 2 * RP + rl * 4, gc);
+            if (!HEAD) load_rows<RPT, RL>(row + 2 * RP + rl * 4, gc);
             const float vc = row[3 * RP + jl];
             float acc;
             if (DELTA) {
@@ -186,12 +202,18 @@ __global__ void __launch_bounds__(256) state_recurrence_kernel(RecurrenceParams 
                 const float u = bc * (vc - r);
 #pragma unroll
                 for (int m = 0; m < RPT; ++m) S[m] = fmaf(kc[m], u, S[m]);
-                acc = fmaf(u, d, a);
+                acc = fmaf(u, d, a) * p.q_scale;
+            } else if (HEAD) {
+                const float a = row[3 * RP + COLS_PER_CTA + 1], wv = row[3 * RP + COLS_PER_CTA] * vc;
+                float a4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int m = 0; m < RPT; ++m) { S[m] = fmaf(a, S[m], kc[m] * wv); a4[m & 3] = fmaf(S[m], qc[m], a4[m & 3]); }
+                acc = fmaf(skip, vc, sum_row_lanes<RL>((a4[0] + a4[1]) + (a4[2] + a4[3])) * p.q_scale);
             } else {
                 float a4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int m = 0; m < RPT; ++m) { S[m] = fmaf(gc[m], S[m], kc[m] * vc); a4[m & 3] = fmaf(S[m], qc[m], a4[m & 3]); }
-                acc = sum_row_lanes<RL>((a4[0] + a4[1]) + (a4[2] + a4[3]));
+                acc = sum_row_lanes<RL>((a4[0] + a4[1]) + (a4[2] + a4[3])) * p.q_scale;
             }
             if (rl == 0 && live) p.out[(size_t)(t0 + c * CHUNK + tt) * p.out_stride + (size_t)h * p.columns + j] = acc;
         }
@@ -364,7 +386,146 @@ __global__ void conv_tail_update_kernel(const float* proj, long proj_stride, flo
     }
 }
 
+// ------------------------------------------------------------------------------------------------ Mamba-2: inputs
+struct Mamba2PrepParams {
+    const float* proj; long proj_stride;      // [T, ...]: convolved channels from conv_off on, step sizes from dt_off on
+    const float* conv; const float* bias;     // [taps, C] tap-major, [C] or null
+    const float* tail; long tail_stride;      // [slots, (taps - 1) * C]
+    const float* dt_bias; const float* a_log; // [heads]
+    float* out; long out_stride;              // [T, C]
+    float* dt; float* decay;                  // [T, heads]
+    const int* seq_of_token; const int* q_start; const int* slots;
+    int C, taps, heads, conv_off, dt_off, n_tokens;
+};
+
+// V neighbouring channels of one token per thread (V = 4: 16-byte accesses), then one thread per (token, head).
+template <int V>
+__global__ void __launch_bounds__(256) mamba2_prep_kernel(Mamba2PrepParams p) {
+    const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    const int groups = p.C / V;
+    const long n_conv = (long)p.n_tokens * groups;
+    if (idx >= n_conv) {
+        const long i = idx - n_conv;
+        if (i >= (long)p.n_tokens * p.heads) return;
+        const int t = (int)(i / p.heads), h = (int)(i % p.heads);
+        const float step = softplus_f(p.proj[(size_t)t * p.proj_stride + p.dt_off + h] + p.dt_bias[h]);
+        p.dt[i] = step;
+        p.decay[i] = expf(-expf(p.a_log[h]) * step);
+        return;
+    }
+    const int t = (int)(idx / groups), c = (int)(idx % groups) * V;
+    const int s = p.seq_of_token[t], t0 = p.q_start[s];
+    float acc[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) acc[e] = p.bias ? p.bias[c + e] : 0.f;
+    for (int jt = 0; jt < p.taps; ++jt) {
+        const int from = t - (p.taps - 1 - jt);                  // the token this tap reads
+        const float* src = from >= t0 ? p.proj + (size_t)from * p.proj_stride + p.conv_off + c
+                                      : p.tail + (size_t)p.slots[s] * p.tail_stride + (size_t)(p.taps - 1 - (t0 - from)) * p.C + c;
+        const float* w = p.conv + (size_t)jt * p.C + c;
+        if (V == 4) {
+            const float4 x4 = *reinterpret_cast<const float4*>(src), w4 = *reinterpret_cast<const float4*>(w);
+            acc[0] = fmaf(w4.x, x4.x, acc[0]); acc[1 % V] = fmaf(w4.y, x4.y, acc[1 % V]);
+            acc[2 % V] = fmaf(w4.z, x4.z, acc[2 % V]); acc[3 % V] = fmaf(w4.w, x4.w, acc[3 % V]);
+        } else {
+            acc[0] = fmaf(w[0], src[0], acc[0]);
+        }
+    }
+    float* dst = p.out + (size_t)t * p.out_stride + c;
+    if (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(silu_f(acc[0]), silu_f(acc[1 % V]), silu_f(acc[2 % V]), silu_f(acc[3 % V]));
+    else dst[0] = silu_f(acc[0]);
+}
+
+// ------------------------------------------------------------------------------------------------ decay of a low-rank map
+// g[t, h * rows + i] = sigmoid(z)^(1 / tau) = exp(log sigmoid(z) / tau), z = sum_r w[h * dim + i, r] u[t, r] + bias: a
+// thread per channel and DECAY_TOKENS tokens, whose u rows lie in shared memory.  Rows beyond dim are zero.
+constexpr int DECAY_TOKENS = 16;
+__global__ void __launch_bounds__(256) low_rank_decay_kernel(const float* u, long u_stride, const void* w, int w_dt, const float* bias,
+                                                             float inv_tau, float* g, long g_stride, int heads, int dim, int rows,
+                                                             int rank, int n_tokens) {
+    extern __shared__ __align__(16) float us[];                  // [DECAY_TOKENS][rank]
+    const int t0 = blockIdx.y * DECAY_TOKENS, nt = min(DECAY_TOKENS, n_tokens - t0);
+    for (int i = threadIdx.x; i < nt * rank; i += blockDim.x) us[i] = u[(size_t)(t0 + i / rank) * u_stride + i % rank];
+    __syncthreads();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= heads * rows) return;
+    const int h = c / rows, i = c % rows;
+    float acc[DECAY_TOKENS];
+    const bool live = i < dim;
+    const float b = live && bias ? bias[h * dim + i] : 0.f;
+#pragma unroll
+    for (int e = 0; e < DECAY_TOKENS; ++e) acc[e] = b;
+    if (live) {
+        const size_t row = (size_t)(h * dim + i) * rank;
+        for (int r = 0; r < rank; ++r) {
+            const float wv = load_any(w, w_dt, row + r);
+#pragma unroll
+            for (int e = 0; e < DECAY_TOKENS; ++e)
+                if (e < nt) acc[e] = fmaf(wv, us[e * rank + r], acc[e]);
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < DECAY_TOKENS; ++e)
+        if (e < nt) {
+            const float z = acc[e];
+            const float log_sig = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+            g[(size_t)(t0 + e) * g_stride + c] = live ? expf(log_sig * inv_tau) : 0.f;
+        }
+}
+
+// dst[t, h * rows + i] = src[t, h * dim + i] for i < dim, zero up to rows
+__global__ void pad_heads_kernel(const float* src, long src_stride, float* dst, int heads, int dim, int rows, long n) {
+    const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= n) return;
+    const int i = (int)(idx % rows), h = (int)((idx / rows) % heads);
+    const long t = idx / ((long)rows * heads);
+    dst[idx] = i < dim ? src[t * src_stride + (long)h * dim + i] : 0.f;
+}
+
 // ------------------------------------------------------------------------------------------------ read-out
+// A CTA per (token, part of the row): u = y silu(z), then u / sqrt(mean(u^2) + eps) * weight over the part's ``width``
+// columns.  NV: 16-byte pieces of the part a thread keeps in registers (0: one value at a time, computed twice).
+template <int NV>
+__global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* y, long y_stride, const float* z, long z_stride,
+                                                               const float* weight, void* out, int out_dt, long out_stride, int width,
+                                                               int parts, float eps) {
+    __shared__ float scratch[33];
+    const int t = blockIdx.x / parts, part = blockIdx.x % parts, tid = threadIdx.x;
+    const float* yr = y + (size_t)t * y_stride + (size_t)part * width;
+    const float* zr = z + (size_t)t * z_stride + (size_t)part * width;
+    const float* w = weight + (size_t)part * width;
+    const size_t o = (size_t)t * out_stride + (size_t)part * width;
+    float ss = 0.f;
+    if (NV > 0) {
+        float4 u[NV > 0 ? NV : 1];
+#pragma unroll
+        for (int e = 0; e < NV; ++e) {
+            const int i = tid + e * blockDim.x;
+            u[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (4 * i < width) {
+                const float4 a = reinterpret_cast<const float4*>(yr)[i], b = reinterpret_cast<const float4*>(zr)[i];
+                u[e] = make_float4(a.x * silu_f(b.x), a.y * silu_f(b.y), a.z * silu_f(b.z), a.w * silu_f(b.w));
+            }
+            ss = fmaf(u[e].x, u[e].x, ss); ss = fmaf(u[e].y, u[e].y, ss); ss = fmaf(u[e].z, u[e].z, ss); ss = fmaf(u[e].w, u[e].w, ss);
+        }
+        const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+#pragma unroll
+        for (int e = 0; e < NV; ++e) {
+            const int i = tid + e * blockDim.x;
+            if (4 * i < width) {
+                const float4 g = reinterpret_cast<const float4*>(w)[i];
+                const float4 v = make_float4(u[e].x * r * g.x, u[e].y * r * g.y, u[e].z * r * g.z, u[e].w * r * g.w);
+                if (out_dt == RS_F32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + o + 4 * i) = v;
+                else *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out) + o + 4 * i) = pack_bf16x4(v.x, v.y, v.z, v.w);
+            }
+        }
+    } else {
+        for (int i = tid; i < width; i += blockDim.x) { const float u = yr[i] * silu_f(zr[i]); ss = fmaf(u, u, ss); }
+        const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+        for (int i = tid; i < width; i += blockDim.x) store_any(out, out_dt, o + i, yr[i] * silu_f(zr[i]) * r * w[i]);
+    }
+}
+
 // A warp per (token, head): o / sqrt(mean(o^2) + eps) * weight * sigmoid(gate) (weight and gate optional).
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, long o_stride, const void* weight, int w_dt, const float* gate,
                                                             long gate_stride, void* out, int out_dt, long out_stride, int heads, int vdim,
@@ -386,6 +547,49 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, lon
             y *= gate_silu ? silu_f(z) : sigmoid_f(z);
         }
         store_any(out, out_dt, (size_t)t * out_stride + (size_t)h * vdim + d, y);
+    }
+}
+
+// The same, 16 bytes a lane: heads of up to 128 NV columns (a multiple of 4) in aligned rows.
+template <int NV>
+__global__ void __launch_bounds__(256) head_norm_gate_vec_kernel(const float* o, long o_stride, const float* weight, const float* gate,
+                                                                 long gate_stride, void* out, int out_dt, long out_stride, int heads,
+                                                                 int vdim, float eps, int n_tokens, int gate_silu) {
+    const int lane = threadIdx.x & 31;
+    const long wid = (long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (wid >= (long)n_tokens * heads) return;
+    const int t = (int)(wid / heads), h = (int)(wid % heads);
+    const float4* row = reinterpret_cast<const float4*>(o + (size_t)t * o_stride + (size_t)h * vdim);
+    const float4* gr = reinterpret_cast<const float4*>(gate ? gate + (size_t)t * gate_stride + (size_t)h * vdim : nullptr);
+    const int n4 = vdim >> 2;
+    float4 x[NV], z[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < NV; ++e) {
+        const int i = lane + 32 * e;
+        x[e] = i < n4 ? row[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        z[e] = gate && i < n4 ? gr[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss = fmaf(x[e].x, x[e].x, ss); ss = fmaf(x[e].y, x[e].y, ss); ss = fmaf(x[e].z, x[e].z, ss); ss = fmaf(x[e].w, x[e].w, ss);
+    }
+    ss = warp_sum(ss);
+    const float r = 1.0f / sqrtf(ss / (float)vdim + eps);
+    const size_t base = (size_t)t * out_stride + (size_t)h * vdim;
+#pragma unroll
+    for (int e = 0; e < NV; ++e) {
+        const int i = lane + 32 * e;
+        if (i >= n4) continue;
+        float v[4] = {x[e].x * r, x[e].y * r, x[e].z * r, x[e].w * r};
+        if (weight) {
+            const float4 w = reinterpret_cast<const float4*>(weight)[i];
+            v[0] *= w.x; v[1] *= w.y; v[2] *= w.z; v[3] *= w.w;
+        }
+        if (gate) {
+            const float zz[4] = {z[e].x, z[e].y, z[e].z, z[e].w};
+#pragma unroll
+            for (int q = 0; q < 4; ++q) v[q] *= gate_silu ? silu_f(zz[q]) : sigmoid_f(zz[q]);
+        }
+        if (out_dt == RS_F32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + base + 4 * i) = make_float4(v[0], v[1], v[2], v[3]);
+        else *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out) + base + 4 * i) = pack_bf16x4(v[0], v[1], v[2], v[3]);
     }
 }
 
@@ -444,10 +648,12 @@ RS_EXPORT int rs_state_recurrence_rows_pad(int rows) {
 RS_EXPORT int rs_state_recurrence(const float* q, long q_stride, const float* k, long k_stride, const float* g, long g_stride,
                                   const float* beta, long beta_stride, const float* v, long v_stride, float* out, long out_stride,
                                   float* state, long state_stride, const int* q_start, const int* slots, int n_seqs, int heads,
-                                  int group, int rows_pad, int columns, int delta, cudaStream_t stream) {
+                                  int group, int rows, int rows_pad, int columns, int form, float q_scale, const float* skip,
+                                  cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
+    if (rows < 4 || rows % 4 || rows > rows_pad || form < REC_GATED || form > REC_HEAD) return (int)cudaErrorInvalidValue;
     RecurrenceParams p{q, q_stride, k, k_stride, g, g_stride, beta, beta_stride, v, v_stride, out, out_stride, state, state_stride,
-                       q_start, slots, heads, group < 1 ? 1 : group, columns};
+                       q_start, slots, heads, group < 1 ? 1 : group, columns, rows, q_scale, skip};
     // Narrower CTAs while the step has fewer than two per multiprocessor: the walk is a chain of dependent steps, so its
     // time is that of one CTA, and more of them only cost reads of q, k and g that the second-level cache serves.  A
     // small step (no more than a warp per scheduler even so) puts a column over 16 lanes instead of 8: half the
@@ -461,9 +667,11 @@ RS_EXPORT int rs_state_recurrence(const float* q, long q_stride, const float* k,
     const int threads = cols_cta * rl;
     static bool sized = false;          // once: the attribute is a property of the function, not of a launch
 #define RS_REC_SIZE(RPT, RL)                                                                                                    \
-    cudaFuncSetAttribute(state_recurrence_kernel<RPT, true, RL>, cudaFuncAttributeMaxDynamicSharedMemorySize,                  \
+    cudaFuncSetAttribute(state_recurrence_kernel<RPT, REC_GATED, RL>, cudaFuncAttributeMaxDynamicSharedMemorySize,             \
                          (int)RecurrenceStage<RPT * RL>::BYTES);                                                                \
-    cudaFuncSetAttribute(state_recurrence_kernel<RPT, false, RL>, cudaFuncAttributeMaxDynamicSharedMemorySize,                 \
+    cudaFuncSetAttribute(state_recurrence_kernel<RPT, REC_DELTA, RL>, cudaFuncAttributeMaxDynamicSharedMemorySize,             \
+                         (int)RecurrenceStage<RPT * RL>::BYTES);                                                                \
+    cudaFuncSetAttribute(state_recurrence_kernel<RPT, REC_HEAD, RL>, cudaFuncAttributeMaxDynamicSharedMemorySize,              \
                          (int)RecurrenceStage<RPT * RL>::BYTES);
     if (!sized) {
         RS_REC_SIZE(4, 8) RS_REC_SIZE(8, 8) RS_REC_SIZE(16, 8) RS_REC_SIZE(32, 8)
@@ -473,8 +681,10 @@ RS_EXPORT int rs_state_recurrence(const float* q, long q_stride, const float* k,
 #undef RS_REC_SIZE
 #define RS_REC(RPT, RL)                                                                                                         \
     if (rows_pad == RPT * RL && rl == RL) {                                                                                     \
-        if (delta) state_recurrence_kernel<RPT, true, RL><<<grid, threads, RecurrenceStage<RPT * RL>::BYTES, stream>>>(p);      \
-        else state_recurrence_kernel<RPT, false, RL><<<grid, threads, RecurrenceStage<RPT * RL>::BYTES, stream>>>(p);           \
+        constexpr size_t bytes = RecurrenceStage<RPT * RL>::BYTES;                                                              \
+        if (form == REC_DELTA) state_recurrence_kernel<RPT, REC_DELTA, RL><<<grid, threads, bytes, stream>>>(p);                \
+        else if (form == REC_HEAD) state_recurrence_kernel<RPT, REC_HEAD, RL><<<grid, threads, bytes, stream>>>(p);             \
+        else state_recurrence_kernel<RPT, REC_GATED, RL><<<grid, threads, bytes, stream>>>(p);                                  \
         return rs_launch_result();                                                                                              \
     }
     RS_REC(4, 8) RS_REC(8, 8) RS_REC(16, 8) RS_REC(32, 8) RS_REC(4, 16) RS_REC(8, 16) RS_REC(16, 16)
@@ -511,11 +721,84 @@ RS_EXPORT int rs_delta_prep(const float* proj, long proj_stride, const void* con
     return rs_launch_result();
 }
 
+RS_EXPORT int rs_mamba2_prep(const float* proj, long proj_stride, int conv_off, int dt_off, const float* conv, const float* bias,
+                             float* tail, long tail_stride, const float* dt_bias, const float* a_log, float* out, long out_stride,
+                             float* dt, float* decay, const int* seq_of_token, const int* q_start, const int* slots, int channels,
+                             int taps, int heads, int n_tokens, int n_seqs, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (taps < 1 || channels < 1 || heads < 1 || (taps > 1 && !tail)) return (int)cudaErrorInvalidValue;
+    Mamba2PrepParams p{proj, proj_stride, conv, bias, tail, tail_stride, dt_bias, a_log, out, out_stride, dt, decay, seq_of_token,
+                       q_start, slots, channels, taps, heads, conv_off, dt_off, n_tokens};
+    const bool vec = channels % 4 == 0 && conv_off % 4 == 0 && proj_stride % 4 == 0 && out_stride % 4 == 0 &&
+                     (((uintptr_t)proj | (uintptr_t)conv | (uintptr_t)out) & 15) == 0 &&
+                     (!tail || (tail_stride % 4 == 0 && ((uintptr_t)tail & 15) == 0));
+    const long n = (long)n_tokens * (vec ? channels / 4 : channels) + (long)n_tokens * heads;
+    const unsigned blocks = (unsigned)((n + 255) / 256);
+    if (vec) mamba2_prep_kernel<4><<<blocks, 256, 0, stream>>>(p);
+    else mamba2_prep_kernel<1><<<blocks, 256, 0, stream>>>(p);
+    int rc = rs_launch_result();
+    if (rc || taps == 1) return rc;
+    const long m = (long)n_seqs * channels;
+    conv_tail_update_kernel<<<(unsigned)((m + 255) / 256), 256, 0, stream>>>(proj + conv_off, proj_stride, tail, tail_stride, q_start,
+                                                                            slots, channels, taps, n_seqs);
+    return rs_launch_result();
+}
+
+RS_EXPORT int rs_low_rank_decay(const float* u, long u_stride, const void* w, int w_dt, const float* bias, float inv_tau, float* g,
+                                long g_stride, int heads, int dim, int rows, int rank, int n_tokens, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (rank < 1 || rank > 512 || rows < dim) return (int)cudaErrorInvalidValue;
+    const dim3 grid((unsigned)((heads * rows + 255) / 256), (unsigned)((n_tokens + DECAY_TOKENS - 1) / DECAY_TOKENS));
+    low_rank_decay_kernel<<<grid, 256, DECAY_TOKENS * rank * sizeof(float), stream>>>(u, u_stride, w, w_dt, bias, inv_tau, g, g_stride,
+                                                                                      heads, dim, rows, rank, n_tokens);
+    return rs_launch_result();
+}
+
+RS_EXPORT int rs_pad_heads(const float* src, long src_stride, float* dst, int heads, int dim, int rows, int n_tokens,
+                           cudaStream_t stream) {
+    const long n = (long)n_tokens * heads * rows;
+    if (n <= 0) return 0;
+    pad_heads_kernel<<<(unsigned)((n + 255) / 256), 256, 0, stream>>>(src, src_stride, dst, heads, dim, rows, n);
+    return rs_launch_result();
+}
+
+RS_EXPORT int rs_gated_group_norm(const float* y, long y_stride, const float* z, long z_stride, const float* weight, void* out,
+                                  int out_dt, long out_stride, int width, int parts, float eps, int n_tokens, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (parts < 1 || width < 1) return (int)cudaErrorInvalidValue;
+    const int out_align = out_dt == RS_F32 ? 15 : 7;
+    const bool vec = width % 4 == 0 && y_stride % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0 && width <= 8 * 4 * 256 &&
+                     (((uintptr_t)y | (uintptr_t)z | (uintptr_t)weight) & 15) == 0 && ((uintptr_t)out & out_align) == 0;
+    const unsigned blocks = (unsigned)n_tokens * parts;
+#define RS_GGN(NV, TH) gated_group_norm_kernel<NV><<<blocks, TH, 0, stream>>>(y, y_stride, z, z_stride, weight, out, out_dt, out_stride, width, parts, eps)
+    if (!vec) RS_GGN(0, 128);
+    else if (width <= 4 * 32) RS_GGN(1, 32);
+    else if (width <= 4 * 64) RS_GGN(1, 64);
+    else if (width <= 4 * 128) RS_GGN(1, 128);
+    else if (width <= 4 * 256) RS_GGN(1, 256);
+    else if (width <= 2 * 4 * 256) RS_GGN(2, 256);
+    else if (width <= 4 * 4 * 256) RS_GGN(4, 256);
+    else RS_GGN(8, 256);
+#undef RS_GGN
+    return rs_launch_result();
+}
+
 RS_EXPORT int rs_head_norm_gate(const float* o, long o_stride, const void* weight, int w_dt, const float* gate, long gate_stride,
                                 void* out, int out_dt, long out_stride, int heads, int vdim, float eps, int n_tokens,
                                 int gate_silu, cudaStream_t stream) {
     const long warps = (long)n_tokens * heads;
     if (warps <= 0) return 0;
+    const bool vec = vdim % 4 == 0 && vdim <= 512 && o_stride % 4 == 0 && out_stride % 4 == 0 && (!gate || gate_stride % 4 == 0) &&
+                     (!weight || w_dt == RS_F32) && (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)weight) & 15) == 0 &&
+                     ((uintptr_t)out & (out_dt == RS_F32 ? 15 : 7)) == 0;
+    if (vec) {
+        const unsigned blocks = (unsigned)((warps + 7) / 8);
+        const float* w = reinterpret_cast<const float*>(weight);
+        if (vdim <= 128) head_norm_gate_vec_kernel<1><<<blocks, 256, 0, stream>>>(o, o_stride, w, gate, gate_stride, out, out_dt, out_stride, heads, vdim, eps, n_tokens, gate_silu);
+        else if (vdim <= 256) head_norm_gate_vec_kernel<2><<<blocks, 256, 0, stream>>>(o, o_stride, w, gate, gate_stride, out, out_dt, out_stride, heads, vdim, eps, n_tokens, gate_silu);
+        else head_norm_gate_vec_kernel<4><<<blocks, 256, 0, stream>>>(o, o_stride, w, gate, gate_stride, out, out_dt, out_stride, heads, vdim, eps, n_tokens, gate_silu);
+        return rs_launch_result();
+    }
     head_norm_gate_kernel<<<(unsigned)((warps + 7) / 8), 256, 0, stream>>>(o, o_stride, weight, w_dt, gate, gate_stride, out, out_dt,
                                                                           out_stride, heads, vdim, eps, n_tokens, gate_silu);
     return rs_launch_result();

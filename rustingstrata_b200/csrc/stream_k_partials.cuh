@@ -71,7 +71,7 @@ bool finish_rmsnorm_supported(const void* C, long ldc, int N, const void* w, con
 
 // RMSNorm of the M rows of C straight after a product with the f32 += epilogue whose shared tiles were left unfinished
 // (workspace, N, K, G, L: the product's), one CTA per row: out[m] = RMSNorm(C[m] + partials) * w as bfloat16, and C[m]
-// made whole.  Defined once, in skinny_gemm_tma.cu, for both products.
+// made whole; with w2 also out2[m] = the same row times w2 (both null: one output).  Defined once, in skinny_gemm_tma.cu, for both products.
 int launch_finish_rmsnorm(void* C, long ldc, int M, int N, int K, const float* workspace, int G, Layout L, const void* w, int w_dt,
-                          float eps, void* out, long out_stride, cudaStream_t s);
+                          float eps, void* out, long out_stride, const void* w2, void* out2, long out2_stride, cudaStream_t s);
 }  // namespace rs_streamk

@@ -7,7 +7,8 @@
 //     mixed[h] = sum_g talk[h, g] raw[g], online softmax per (head, query) whose running maximum and sum start at
 //     (sink, 1) instead of (-inf, 0), weighted sum of values, and at the end o / l * gate.
 // A query sees the keys up to its own position, within ``window`` keys if there is a window, and within its own block
-// of ``chunk`` positions (counted from the sequence's first) if the attention is chunked.
+// of ``chunk`` positions (counted from the sequence's first) if the attention is chunked; the sequence's first ``keep``
+// keys stay visible however far behind they are.  The heads' results are multiplied by ``out_scale``.
 // Scores, weights, the mix and the sums are float32; keys and values have the cache's element type.  Key tiles start
 // at multiples of KEY_TILE counted from the sequence's first key, so the order in which a query's keys enter its sums
 // does not depend on how the sequence was cut into steps or on what else is in the batch.
@@ -184,7 +185,7 @@ struct AttnParams {
     const int* q_start; const int* kv_len; const int* work;     // work: (sequence, first query of the tile) pairs
     const float* talk; const float* sink;     // [H, H], [H]; either may be null
     void* out; int out_dt; long out_stride;   // [T, H * dv]
-    int H, G, dk, dv, window, chunk, QT; float scale;
+    int H, G, dk, dv, window, chunk, keep, QT; float scale, out_scale;
     int* status;
 };
 
@@ -220,12 +221,16 @@ __global__ void __launch_bounds__(THREADS) talking_attention_kernel(AttnParams p
     for (int i = tid; i < H * QT * dv; i += THREADS) O[i] = 0.f;
     if (p.talk) for (int i = tid; i < H * H; i += THREADS) Tm[i] = p.talk[i];
 
-    for (int k0 = (k_begin / KEY_TILE) * KEY_TILE; k0 < k_end; k0 += KEY_TILE) {
+    // the tiles that hold kept first keys, as far as they lie before the window's, then the window's
+    const int kt0 = k_begin / KEY_TILE, n_keep = min((p.keep + KEY_TILE - 1) / KEY_TILE, kt0);
+    const int n_tiles = n_keep + (k_end + KEY_TILE - 1) / KEY_TILE - kt0;
+    for (int u = 0; u < n_tiles; ++u) {
+        const int k0 = (u < n_keep ? u : kt0 + u - n_keep) * KEY_TILE;
         __syncthreads();                                 // the tile before this one is done with key_at, Ks and the scores
         if (tid < KEY_TILE) {
             const int kpos = k0 + tid;
             long long at = -1;
-            if (kpos >= k_begin && kpos < k_end) {
+            if ((kpos >= k_begin || kpos < p.keep) && kpos < k_end) {
                 const int page = p.block_table[(size_t)s * p.table_stride + kpos / p.page_size];
                 if (page < 0 || page >= p.num_pages) atomicOr(p.status, RS_STATUS_BAD_PAGE);
                 else at = (long long)page * p.page_stride + (long long)(kpos % p.page_size) * p.hdp;
@@ -272,8 +277,8 @@ __global__ void __launch_bounds__(THREADS) talking_attention_kernel(AttnParams p
             const int kk = i % KEY_TILE, qi = (i / KEY_TILE) % nq, h = i / (KEY_TILE * nq);
             const int kpos = k0 + kk, qpos = pos0 + qi;
             float v = -INFINITY;
-            if (kpos <= qpos && kpos >= k_begin && (p.window <= 0 || kpos > qpos - p.window)
-                && (p.chunk <= 0 || kpos >= qpos / p.chunk * p.chunk) && key_at[kk] >= 0) {
+            if (kpos <= qpos && key_at[kk] >= 0 && (kpos < p.keep || ((p.window <= 0 || kpos > qpos - p.window)
+                && (p.chunk <= 0 || kpos >= qpos / p.chunk * p.chunk)))) {
                 if (p.talk) {
                     v = 0.f;
                     for (int g = 0; g < H; ++g) v = fmaf(Tm[h * H + g], Sraw[(g * QT + qi) * KEY_TILE + kk], v);
@@ -316,7 +321,7 @@ __global__ void __launch_bounds__(THREADS) talking_attention_kernel(AttnParams p
         const int d = i % dv, h = (i / dv) % H, qi = i / (dv * H);
         const int ri = h * QT + qi;
         const float l = L[ri];
-        float y = l > 0.f ? O[ri * dv + d] / l : 0.f;
+        float y = l > 0.f ? O[ri * dv + d] / l * p.out_scale : 0.f;
         if (p.gate) y *= p.gate[(size_t)(t_first + qi) * H + h];
         store_any(p.out, p.out_dt, (size_t)(t_first + qi) * p.out_stride + (size_t)h * dv + d, y);
     }
@@ -357,12 +362,14 @@ RS_EXPORT int rs_talking_attention(const float* q, long q_stride, const float* g
                                    int num_pages, int page_size, int hdp, const int* block_table, int table_stride,
                                    const int* q_start, const int* kv_len, const int* work, int n_work, const float* talk,
                                    const float* sink, void* out, int out_dt, long out_stride, int H, int G, int dk, int dv,
-                                   int window, int chunk, int QT, float scale, int* status, cudaStream_t stream) {
+                                   int window, int chunk, int keep, int QT, float scale, float out_scale, int* status,
+                                   cudaStream_t stream) {
     if (n_work <= 0) return 0;
     const size_t smem = attn_smem_bytes(H, QT, dk, dv);
     if (QT < 1 || smem > SMEM_LIMIT || H % G) return (int)cudaErrorInvalidValue;
     AttnParams p{q, q_stride, gate, cache, page_stride, (long)G * page_size * hdp, num_pages, page_size, hdp, block_table, table_stride,
-                 q_start, kv_len, work, talk, sink, out, out_dt, out_stride, H, G, dk, dv, window, chunk, QT, scale, status};
+                 q_start, kv_len, work, talk, sink, out, out_dt, out_stride, H, G, dk, dv, window, chunk, keep, QT, scale, out_scale,
+                 status};
     static bool sized = false;          // once: the attribute is a property of the function, not of a launch
     if (!sized) {
         cudaFuncSetAttribute(talking_attention_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_LIMIT);

@@ -8,8 +8,8 @@
 //      bfloat16 terms (x = hi + lo, |lo| <= 2^-9 |x|) and both are multiplied, so the score carries the float32
 //      query and not its 8-bit rounding; accumulation is float32.  Scaled scores go to shared memory.
 //   2. mixed[h] = sum_g talk[h, g] raw[g] on the CUDA cores in float32: a thread owns four neighbouring keys of one
-//      query and eight output heads, so one 16-byte read of raw[g] feeds 32 multiply-adds; the causal and window
-//      masks are applied here.
+//      query and eight output heads, so one 16-byte read of raw[g] feeds 32 multiply-adds; the masks are applied here.
+//      Without a mix this step falls away and step 1 applies the masks.
 //   3. online softmax per (head, query) in float32, the running maximum and sum starting at (sink, 1); the weights,
 //      split in two bfloat16 terms like the queries, times V on the tensor cores; a warp per head (two, each with half
 //      of the value columns, when there are 8 heads or fewer).
@@ -36,7 +36,7 @@ struct MmaParams {
     const float* talk; const float* sink;     // [H, H], [H]; either may be null
     void* out; int out_dt; long out_stride;   // [T, H * dv]
     float* partial; long partial_rows;        // [rows, H, dv + 2]: sums, maximum, denominator
-    int H, G, dk, dv, window, chunk, QT; float scale;
+    int H, G, dk, dv, window, chunk, keep, QT; float scale, out_scale;
     int* status;
 };
 
@@ -77,12 +77,18 @@ __device__ __forceinline__ void split_bf16(float x, __nv_bfloat16& hi, __nv_bflo
 __device__ __forceinline__ void locate_keys(const MmaParams& p, long long* key_at, int s, int k0, int k_begin, int k_end, int lane) {
     const int kpos = k0 + lane;
     long long at = -1;
-    if (kpos >= k_begin && kpos < k_end) {
+    if ((kpos >= k_begin || kpos < p.keep) && kpos < k_end) {
         const int page = p.block_table[(size_t)s * p.table_stride + kpos / p.page_size];
         if (page < 0 || page >= p.num_pages) atomicOr(p.status, RS_STATUS_BAD_PAGE);
         else at = (long long)page * p.page_stride + (long long)(kpos % p.page_size) * p.hdp;
     }
     key_at[lane] = at;
+}
+
+// whether the query at qpos sees the key at kpos, whose row starts at ``at`` (negative: no key there)
+__device__ __forceinline__ bool sees(const MmaParams& p, int qpos, int kpos, long long at) {
+    return kpos <= qpos && at >= 0 && (kpos < p.keep || ((p.window <= 0 || kpos > qpos - p.window)
+           && (p.chunk <= 0 || kpos >= qpos / p.chunk * p.chunk)));
 }
 
 // rows [KEY_TILE][G * width] of one plane of the cache into shared memory, 16 bytes per copy; rows without a key are zero.
@@ -132,13 +138,18 @@ __global__ void __launch_bounds__(THREADS, 1) talking_mma_kernel(MmaParams p) {
     int k_begin = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
     if (p.chunk > 0) k_begin = max(k_begin, pos0 / p.chunk * p.chunk);      // chunked: nothing before the first query's block
     const int kt0 = k_begin / KEY_TILE, kt1 = (k_end + KEY_TILE - 1) / KEY_TILE;
-    const int per = (kt1 - kt0 + parts - 1) / parts;
-    const int t_begin = kt0 + part * per, t_end = min(kt1, t_begin + per);
+    // the tiles that hold kept first keys, as far as they lie before the window's, then the window's: a tile's place in
+    // this walk is what the parts share out and the loop counts
+    const int n_keep = min((p.keep + KEY_TILE - 1) / KEY_TILE, kt0), n_walk = n_keep + kt1 - kt0;
+    const auto tile_at = [&](int t) { return t < n_keep ? t : kt0 + t - n_keep; };
+    const int per = (n_walk + parts - 1) / parts;
+    const int t_begin = part * per, t_end = min(n_walk, t_begin + per);
     const size_t plane = (size_t)p.plane_stride;
     const int qt_shift = QT == 16 ? 4 : QT == 8 ? 3 : 2;
     const uint32_t q_hi_addr = smem_addr(Qhi), q_lo_addr = smem_addr(Qlo), ks_addr = smem_addr(Ks), vs_addr = smem_addr(Vs);
     // step 3: a warp per head; with 8 heads or fewer two warps per head, each holding half of the value columns
     const bool pair = HPW == 1 && 2 * H <= WARPS;
+    const float* Sm = p.talk ? Smix : Sraw;      // what the softmax reads
     const int col_half = pair ? (warp & 1) : 0;
 
     for (int i = tid; i < QT * H * dk; i += THREADS) {
@@ -168,7 +179,7 @@ __global__ void __launch_bounds__(THREADS, 1) talking_mma_kernel(MmaParams p) {
                 for (int c = 0; c < 4; ++c) O[i][a][b][c] = 0.f;
     }
     if (t_begin < t_end) {
-        if (tid < KEY_TILE) locate_keys(p, key_at + (t_begin & 1) * KEY_TILE, s, t_begin * KEY_TILE, k_begin, k_end, lane);
+        if (tid < KEY_TILE) locate_keys(p, key_at + (t_begin & 1) * KEY_TILE, s, tile_at(t_begin) * KEY_TILE, k_begin, k_end, lane);
         __syncthreads();
         fetch_plane(p, key_at + (t_begin & 1) * KEY_TILE, Ks, L.k_pitch, dk, 0, tid);
         cp_async_commit();
@@ -176,13 +187,13 @@ __global__ void __launch_bounds__(THREADS, 1) talking_mma_kernel(MmaParams p) {
         cp_async_commit();
     }
     for (int t = t_begin; t < t_end; ++t) {
-        const int k0 = t * KEY_TILE;
+        const int k0 = tile_at(t) * KEY_TILE;
         const long long* at_now = key_at + (t & 1) * KEY_TILE;
         long long* at_next = key_at + ((t + 1) & 1) * KEY_TILE;
         cp_async_wait<1>();                                  // this tile's K has landed (its V may still be on the way)
         __syncthreads();
         // ---- 1: raw scores, a warp per head
-        if (t + 1 < t_end && tid >= THREADS - KEY_TILE) locate_keys(p, at_next, s, k0 + KEY_TILE, k_begin, k_end, lane);
+        if (t + 1 < t_end && tid >= THREADS - KEY_TILE) locate_keys(p, at_next, s, tile_at(t + 1) * KEY_TILE, k_begin, k_end, lane);
         for (int task = warp; task < 2 * H; task += WARPS) {
             const int g = task >> 1, half = task & 1, c = g / r;
             float acc[2][4];
@@ -209,6 +220,11 @@ __global__ void __launch_bounds__(THREADS, 1) talking_mma_kernel(MmaParams p) {
 #pragma unroll
             for (int nb = 0; nb < 2; ++nb) {
                 const int col = (2 * half + nb) * 8 + 2 * tig;
+                if (!p.talk) {                               // no mix: what the query does not see is masked here
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        if (!sees(p, pos0 + gid + 8 * (e >> 1), k0 + col + (e & 1), at_now[col + (e & 1)])) acc[nb][e] = -INFINITY;
+                }
                 if (gid < QT)
                     *reinterpret_cast<float2*>(Sraw + ((size_t)g * QT + gid) * SROW + col) =
                         make_float2(acc[nb][0] * p.scale, acc[nb][1] * p.scale);
@@ -217,11 +233,12 @@ __global__ void __launch_bounds__(THREADS, 1) talking_mma_kernel(MmaParams p) {
                         make_float2(acc[nb][2] * p.scale, acc[nb][3] * p.scale);
             }
         }
+        if (!p.talk) cp_async_wait<0>();                     // this tile's V has landed: the barrier below serves steps 1 and 2
         __syncthreads();
         if (t + 1 < t_end) fetch_plane(p, at_next, Ks, L.k_pitch, dk, 0, tid);
         cp_async_commit();
         // ---- 2: the mix across heads and the masks
-        const int items = (L.h8 / 8) * QT * 8;
+        const int items = p.talk ? (L.h8 / 8) * QT * 8 : 0;
         for (int i = tid; i < items; i += THREADS) {
             const int kq = i & 7, qi = (i >> 3) & (QT - 1), hc = i >> (3 + qt_shift);
             if (qi >= nq) continue;
@@ -246,8 +263,7 @@ __global__ void __launch_bounds__(THREADS, 1) talking_mma_kernel(MmaParams p) {
 #pragma unroll
             for (int b = 0; b < 4; ++b) {
                 const int kpos = k0 + kq * 4 + b;
-                seen[b] = kpos <= qpos && (p.window <= 0 || kpos > qpos - p.window)
-                          && (p.chunk <= 0 || kpos >= qpos / p.chunk * p.chunk) && at_now[kq * 4 + b] >= 0;
+                seen[b] = sees(p, qpos, kpos, at_now[kq * 4 + b]);
             }
 #pragma unroll
             for (int a = 0; a < 8; ++a) {
@@ -258,8 +274,10 @@ __global__ void __launch_bounds__(THREADS, 1) talking_mma_kernel(MmaParams p) {
                                     seen[2] ? acc[a][2] : -INFINITY, seen[3] ? acc[a][3] : -INFINITY);
             }
         }
-        cp_async_wait<1>();                                  // this tile's V has landed (the next K may still be on the way)
-        __syncthreads();
+        if (p.talk) {
+            cp_async_wait<1>();                              // this tile's V has landed (the next K may still be on the way)
+            __syncthreads();
+        }
         // ---- 3: online softmax and weighted values, a warp per head
 #pragma unroll
         for (int i = 0; i < HPW; ++i) {
@@ -269,8 +287,8 @@ __global__ void __launch_bounds__(THREADS, 1) talking_mma_kernel(MmaParams p) {
 #pragma unroll
             for (int nb = 0; nb < 4; ++nb) {
                 float2 lo2 = make_float2(-INFINITY, -INFINITY), hi2 = lo2;
-                if (gid < nq) lo2 = *reinterpret_cast<const float2*>(Smix + ((size_t)h * QT + gid) * SROW + nb * 8 + 2 * tig);
-                if (gid + 8 < nq) hi2 = *reinterpret_cast<const float2*>(Smix + ((size_t)h * QT + gid + 8) * SROW + nb * 8 + 2 * tig);
+                if (gid < nq) lo2 = *reinterpret_cast<const float2*>(Sm + ((size_t)h * QT + gid) * SROW + nb * 8 + 2 * tig);
+                if (gid + 8 < nq) hi2 = *reinterpret_cast<const float2*>(Sm + ((size_t)h * QT + gid + 8) * SROW + nb * 8 + 2 * tig);
                 sc[nb][0] = lo2.x; sc[nb][1] = lo2.y; sc[nb][2] = hi2.x; sc[nb][3] = hi2.y;
             }
             float mx[2] = {-INFINITY, -INFINITY};
@@ -352,7 +370,7 @@ __global__ void __launch_bounds__(THREADS, 1) talking_mma_kernel(MmaParams p) {
             const int qi = gid + 8 * e;
             if (qi >= nq) continue;
             if (parts == 1) {
-                float f = l_run[i][e] > 0.f ? 1.0f / l_run[i][e] : 0.f;
+                float f = l_run[i][e] > 0.f ? p.out_scale / l_run[i][e] : 0.f;
                 if (p.gate) f *= p.gate[(size_t)(t_first + qi) * H + h];
                 const size_t o = (size_t)(t_first + qi) * p.out_stride + (size_t)h * dv;
 #pragma unroll
@@ -408,7 +426,7 @@ __global__ void __launch_bounds__(1024) talking_combine_kernel(MmaParams p) {
         float den = wi * li;
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
-        float f = den > 0.f ? 1.0f / den : 0.f;
+        float f = den > 0.f ? p.out_scale / den : 0.f;
         if (p.gate) f *= p.gate[(size_t)(t_first + qi) * H + h];
         const size_t o0 = (size_t)(t_first + qi) * p.out_stride + (size_t)h * dv;
         for (int d0 = 0; d0 < dv; d0 += 64) {                                   // every lane walks every round: the shuffles need them
@@ -462,7 +480,7 @@ RS_EXPORT int rs_talking_attention_mma(const float* q, long q_stride, const floa
                                        const int* q_start, const int* kv_len, const int* work, int n_work, int any_parts,
                                        const float* talk, const float* sink, void* out, int out_dt, long out_stride,
                                        float* partial, long partial_rows, int H, int G, int dk, int dv, int window, int chunk,
-                                       int QT, float scale, int* status, cudaStream_t stream) {
+                                       int keep, int QT, float scale, float out_scale, int* status, cudaStream_t stream) {
     if (n_work <= 0) return 0;
     if (!shape_ok(H, G, dk, dv) || (QT != 4 && QT != 8 && QT != 16) || hdp % 8 || (any_parts && !partial))
         return (int)cudaErrorInvalidValue;
@@ -470,7 +488,7 @@ RS_EXPORT int rs_talking_attention_mma(const float* q, long q_stride, const floa
     if (smem > SMEM_LIMIT) return (int)cudaErrorInvalidValue;
     MmaParams p{q, q_stride, gate, reinterpret_cast<const __nv_bfloat16*>(cache), page_stride, (long)G * page_size * hdp, num_pages,
                 page_size, hdp, block_table, table_stride, q_start, kv_len, work, talk, sink, out, out_dt, out_stride, partial,
-                partial_rows, H, G, dk, dv, window, chunk, QT, scale, status};
+                partial_rows, H, G, dk, dv, window, chunk, keep, QT, scale, out_scale, status};
     int rc;
     if (H > WARPS) rc = launch<2, 4>(p, n_work, smem, stream);
     else if (dv <= 64) rc = launch<1, 4>(p, n_work, smem, stream);

@@ -73,7 +73,7 @@ class ModelRunner:
         self.max_positions = self.spec.max_positions
         # ---- cache and state
         m = self.model
-        self.cache = CacheManager([GroupNeed(n.window) for n in m.cache_groups], self.page_size, self.num_pages,
+        self.cache = CacheManager([GroupNeed(n.window, n.keep_first) for n in m.cache_groups], self.page_size, self.num_pages,
                                   engine.max_seqs)
         self.caches = allocate_caches(m.cache_groups, m.group_calls, self.num_pages, self.page_size, self.dtype,
                                       self.device)

@@ -103,11 +103,11 @@ class Scheduler:
             raise RequestRejected(f"request {req.rid!r}: context full ({total} tokens; the model has "
                                   f"{self.max_positions} positions)")
         for g, (pool, need) in enumerate(zip(self.cache.pools, self.cache.groups)):
-            # a group that keeps every key must hold the whole request; a window group the window and the page
-            # that is being written
+            # a group that keeps every key must hold the whole request; a window group the window, the page that is
+            # being written and the first tokens it keeps
             most = self._pages_for(total)
             if need.window is not None:
-                most = min(most, self._pages_for(need.window) + 1)
+                most = min(most, self._pages_for(need.window) + 1 + self._pages_for(need.keep_first))
             if most > pool.num_pages:
                 raise RequestRejected(f"request {req.rid!r}: context full ({total} tokens; cache group {g} holds "
                                       f"{pool.num_pages * self.cache.page_size})")

@@ -89,12 +89,13 @@ def core():
         lib.rs_embed.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p]
         lib.rs_gather_i32.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_void_p]
         lib.rs_rmsnorm.argtypes = [c_void_p, c_long, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_long,
-                                   c_int, c_int, c_void_p]
+                                   c_void_p, c_void_p, c_long, c_int, c_int, c_void_p]
         lib.rs_qk_norm_rope_kv.argtypes = [c_void_p, c_int, c_long, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                                            c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
                                            c_int, c_int, c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_void_p]
-        lib.rs_silu_mul.argtypes = [c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_void_p]
+        lib.rs_silu_mul.argtypes = [c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p]
         lib.rs_head_sigmoid_gate.argtypes = [c_void_p, c_int, c_long, c_void_p, c_long, c_int, c_int, c_int, c_void_p]
+        lib.rs_add_embed.argtypes = [c_void_p, c_long, c_void_p, c_int, c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p]
         lib.rs_residual_add.argtypes = [c_void_p, c_void_p, c_int, c_long, c_void_p]
         lib.rs_linear_simt.argtypes = [c_void_p, c_int, c_long, c_void_p, c_int, c_long, c_void_p, c_int, c_long,
                                        c_int, c_int, c_int, c_int, c_void_p]
@@ -160,13 +161,20 @@ def gather_i32(dst: torch.Tensor, src: torch.Tensor, idx: torch.Tensor, n: int) 
 
 
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
-            rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None, pending=None) -> None:
+            rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None, pending=None,
+            weight2: Optional[torch.Tensor] = None, out2: Optional[torch.Tensor] = None) -> None:
     """out[r] = x[rows[r] or r] * rsqrt(mean(x^2) + eps) * weight.  x float32 [*, n].
+
+    ``weight2`` and ``out2``: a second norm of the same rows with weights of its own, from the same read of ``x``.
 
     ``pending``: a :class:`PendingSum` still owed to ``x``.  If it covers exactly the rows that are normed, one kernel
     adds the partial sums and norms the rows (the same bits as the two kernels in turn); else it is finished first."""
-    _cuda(x, weight, out, rows)
-    if _ACTIVE_CHAIN is not None and _ACTIVE_CHAIN.ops and pending is None and rows is None:
+    _cuda(x, weight, out, rows, weight2, out2)
+    if (weight2 is None) != (out2 is None) or (weight2 is not None and (
+            weight2.dtype != weight.dtype or weight2.numel() != weight.numel() or not weight2.is_contiguous()
+            or out2.dtype != out.dtype or out2.shape[1] != out.shape[1] or out2.shape[0] < out.shape[0] or out2.stride(1) != 1)):
+        raise KernelError("rmsnorm: the second norm has the first one's width and element types")
+    if _ACTIVE_CHAIN is not None and _ACTIVE_CHAIN.ops and pending is None and rows is None and weight2 is None:
         nr = n_rows if n_rows is not None else x.shape[0]
         lib = bf16lib()
         if (nr <= lib.rs_decode_chain_max_rows() and x.dtype == torch.float32 and out.dtype == torch.bfloat16
@@ -184,8 +192,10 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
                 and pending.n_rows == nr and pending.N == x.shape[1] == weight.numel() == out.shape[1]
                 and x.dtype == torch.float32 and out.dtype == torch.bfloat16 and weight.is_contiguous()
                 and weight.dtype in (torch.float32, torch.bfloat16) and nr <= out.shape[0] and x.stride(1) == 1 and out.stride(1) == 1
-                and lib.rs_skinny_finish_rmsnorm_supported(_ptr(x), x.stride(0), pending.N, _ptr(weight), _ptr(out), out.stride(0))):
-            pending.finish_with_rmsnorm(weight, eps, out)
+                and lib.rs_skinny_finish_rmsnorm_supported(_ptr(x), x.stride(0), pending.N, _ptr(weight), _ptr(out), out.stride(0))
+                and (weight2 is None or lib.rs_skinny_finish_rmsnorm_supported(_ptr(x), x.stride(0), pending.N, _ptr(weight2),
+                                                                               _ptr(out2), out2.stride(0)))):
+            pending.finish_with_rmsnorm(weight, eps, out, weight2, out2)
             return
         pending.finish()
     _rows_contiguous(x, "rmsnorm x")
@@ -202,7 +212,8 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
     if rows is not None and (rows.dtype != torch.int32 or rows.numel() < n_rows):
         raise KernelError("rmsnorm: rows must be int32 with n_rows entries")
     _check(core().rs_rmsnorm(_ptr(x), x.stride(0), _ptr(rows), _ptr(weight), dtype_code(weight), float(eps),
-                             _ptr(out), dtype_code(out), out.stride(0), n_rows, n, _stream()), "rmsnorm")
+                             _ptr(out), dtype_code(out), out.stride(0), _ptr(weight2), _ptr(out2),
+                             0 if out2 is None else out2.stride(0), n_rows, n, _stream()), "rmsnorm")
 
 
 def qk_norm_rope_kv(qkv: torch.Tensor, n_tokens: int, n_q: int, n_kv: int, head_dim: int,
@@ -253,12 +264,15 @@ def qk_norm_rope_kv(qkv: torch.Tensor, n_tokens: int, n_q: int, n_kv: int, head_
         n_tokens, _ptr(status), _stream()), "qk_norm_rope_kv")
 
 
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped": 2}
+NO_GATE_CONSTANTS = (0.0, 0.0)      # (alpha, limit) of the clamped gate; the other activations have no constants
 
 
-def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, n_rows: int, activation: str = "silu") -> None:
+def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, n_rows: int, activation: str = "silu",
+             gate=NO_GATE_CONSTANTS) -> None:
     """out[r, c] = act(gate_up[r, c]) * gate_up[r, I + c], I = out.shape[1]; act is SiLU or ("gelu_tanh") the tanh
-    form of GELU."""
+    form of GELU; "clamped" with ``gate`` = (alpha, limit): g sigmoid(alpha g) (u + 1), g = min(gate, limit) and u = up
+    held in [-limit, limit]."""
     if activation not in GATE_ACTIVATIONS:
         raise KernelError(f"silu_mul: unknown activation '{activation}' (known: {', '.join(sorted(GATE_ACTIVATIONS))})")
     _cuda(gate_up, out)
@@ -268,7 +282,7 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, n_rows: int, activation: 
     if gate_up.shape[1] != 2 * I or gate_up.dtype != out.dtype or n_rows > min(gate_up.shape[0], out.shape[0]):
         raise KernelError(f"silu_mul: gate_up {tuple(gate_up.shape)} does not fit out {tuple(out.shape)}")
     _check(core().rs_silu_mul(_ptr(gate_up), gate_up.stride(0), _ptr(out), out.stride(0), dtype_code(out), n_rows, I,
-                              GATE_ACTIVATIONS[activation], _stream()), "silu_mul")
+                              GATE_ACTIVATIONS[activation], float(gate[0]), float(gate[1]), _stream()), "silu_mul")
 
 
 def head_sigmoid_gate(a: torch.Tensor, gate: torch.Tensor, n_heads: int, dv: int, n_tokens: int) -> None:
@@ -280,6 +294,18 @@ def head_sigmoid_gate(a: torch.Tensor, gate: torch.Tensor, n_heads: int, dv: int
         raise KernelError("head_sigmoid_gate: a [T, heads * dv], gate float32 [T, heads]")
     _check(core().rs_head_sigmoid_gate(_ptr(a), dtype_code(a), a.stride(0), _ptr(gate), gate.stride(0), n_heads, dv, n_tokens,
                                        _stream()), "head_sigmoid_gate")
+
+
+def add_embed(x: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float, n_tokens: int, status: torch.Tensor) -> None:
+    """x[t] += scale * table[ids[t]] in float32."""
+    _cuda(x, table, ids, status)
+    _rows_contiguous(x, "add_embed x")
+    n = x.shape[1]
+    if x.dtype != torch.float32 or ids.dtype != torch.int32 or table.shape[1] != n or not table.is_contiguous() \
+            or n_tokens > min(x.shape[0], ids.numel()):
+        raise KernelError("add_embed: x float32 [T, n], table [V, n], ids int32 [T]")
+    _check(core().rs_add_embed(_ptr(x), x.stride(0), _ptr(table), dtype_code(table), _ptr(ids), table.shape[0], float(scale), n_tokens,
+                               n, _ptr(status), _stream()), "add_embed")
 
 
 def residual_add(x: torch.Tensor, delta: torch.Tensor, n_rows: int) -> None:
@@ -333,17 +359,17 @@ def bf16lib():
     if _bf16 is None:
         lib = load_library("bf16")
         lib.rs_gemm_bf16_tc.argtypes = [c_void_p, c_long, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int,
-                                        c_int, c_int, c_int, c_void_p, c_void_p]
+                                        c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p]
         lib.rs_skinny_gemm_bf16.argtypes = [c_void_p, c_long, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int,
-                                            c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]
+                                            c_int, c_void_p, c_int, c_int, c_float, c_float, c_void_p, c_void_p]
         lib.rs_skinny_gemm_workspace_floats.restype = c_long
         lib.rs_skinny_finish.argtypes = [c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_int, c_void_p]
         lib.rs_skinny_finish_rmsnorm_supported.argtypes = [c_void_p, c_long, c_int, c_void_p, c_void_p, c_long]
         lib.rs_skinny_finish_rmsnorm.argtypes = [c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int,
-                                                 c_float, c_void_p, c_long, c_void_p]
+                                                 c_float, c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p]
         lib.rs_decode_chain.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         lib.rs_mid_gemm_bf16.argtypes = [c_void_p, c_long, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int,
-                                         c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]
+                                         c_int, c_void_p, c_int, c_int, c_float, c_float, c_void_p, c_void_p]
         lib.rs_mid_finish.argtypes = lib.rs_skinny_finish.argtypes
         lib.rs_mid_finish_rmsnorm.argtypes = lib.rs_skinny_finish_rmsnorm.argtypes
         lib.rs_mid_gemm_workspace_floats.restype = c_long
@@ -377,7 +403,8 @@ def bf16lib():
     return _bf16
 
 
-EPI_STORE_BF16, EPI_STORE_F32, EPI_ADD_F32, EPI_SWIGLU_BF16, EPI_GEGLU_BF16 = 0, 1, 2, 3, 4
+EPI_STORE_BF16, EPI_STORE_F32, EPI_ADD_F32, EPI_SWIGLU_BF16, EPI_GEGLU_BF16, EPI_CLAMPED_BF16 = 0, 1, 2, 3, 4, 5
+GATED_EPILOGUES = {"silu": EPI_SWIGLU_BF16, "gelu_tanh": EPI_GEGLU_BF16, "clamped": EPI_CLAMPED_BF16}
 
 
 def tensor_core_shape_ok(a: torch.Tensor, weight: torch.Tensor) -> bool:
@@ -391,11 +418,12 @@ def tensor_core_shape_ok(a: torch.Tensor, weight: torch.Tensor) -> bool:
 
 
 def _epilogue_code(out: torch.Tensor, accumulate: bool, swiglu) -> int:
-    """``swiglu``: False, or which gated epilogue: True or "silu" for SiLU(gate) * up, "gelu_tanh" for the tanh form of GELU."""
+    """``swiglu``: False, or which gated epilogue: True or "silu" for SiLU(gate) * up, "gelu_tanh" for the tanh form of GELU,
+    "clamped" for the clamped gate."""
     if swiglu:
         if out.dtype != torch.bfloat16 or accumulate:
             raise KernelError("the fused act(gate)*up epilogue writes bfloat16 and does not accumulate")
-        return EPI_GEGLU_BF16 if swiglu == "gelu_tanh" else EPI_SWIGLU_BF16
+        return GATED_EPILOGUES["silu" if swiglu is True else swiglu]
     if out.dtype == torch.bfloat16:
         if accumulate:
             raise KernelError("accumulating products go into the float32 residual stream")
@@ -419,7 +447,8 @@ def _check_product(a, weight, out, n_rows, swiglu):
 
 
 def gemm_bf16_tc(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_rows: int, accumulate: bool = False,
-                 swiglu: bool = False, status: Optional[torch.Tensor] = None, bn: int = 0, max_ctas: int = 0) -> None:
+                 swiglu: bool = False, status: Optional[torch.Tensor] = None, bn: int = 0, max_ctas: int = 0,
+                 gate=NO_GATE_CONSTANTS) -> None:
     """out[:n_rows] (=|+=) a[:n_rows] @ weight.T on the tcgen05 tensor cores (csrc/gemm_tcgen05.cu).
     ``swiglu``: weight rows alternate gate, up and out[:, j] = silu(gate_j) * up_j."""
     N, K = _check_product(a, weight, out, n_rows, swiglu)
@@ -430,7 +459,7 @@ def gemm_bf16_tc(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_row
         status = _default_status(a.device)
     _check(bf16lib().rs_gemm_bf16_tc(_ptr(a), a.stride(0), a.shape[0], _ptr(weight), weight.stride(0), _ptr(out),
                                      out.stride(0), n_rows, N, K, _epilogue_code(out, accumulate, swiglu), bn, max_ctas,
-                                     _ptr(status), _stream()), "gemm_bf16_tc")
+                                     float(gate[0]), float(gate[1]), _ptr(status), _stream()), "gemm_bf16_tc")
 
 
 SKINNY_MAX_ROWS = 64     # what the kernel takes
@@ -469,13 +498,14 @@ class PendingSum:
             _check(fn(_ptr(self.out), self.out.stride(0), self.n_rows, self.N, self.K, _ptr(self.workspace), self.max_ctas,
                       _stream()), self.kind + "_finish")
 
-    def finish_with_rmsnorm(self, weight: torch.Tensor, eps: float, out: torch.Tensor) -> None:
-        """The same and out[r] = RMSNorm(self.out[r]) * weight, in one kernel."""
+    def finish_with_rmsnorm(self, weight: torch.Tensor, eps: float, out: torch.Tensor, weight2: Optional[torch.Tensor] = None,
+                            out2: Optional[torch.Tensor] = None) -> None:
+        """The same and out[r] = RMSNorm(self.out[r]) * weight (with ``weight2`` also out2[r]), in one kernel."""
         self.done = True
         fn = bf16lib().rs_skinny_finish_rmsnorm if self.kind == "skinny" else bf16lib().rs_mid_finish_rmsnorm
         _check(fn(_ptr(self.out), self.out.stride(0), self.n_rows, self.N, self.K, _ptr(self.workspace), self.max_ctas,
-                  _ptr(weight), dtype_code(weight), float(eps), _ptr(out), out.stride(0), _stream()),
-               self.kind + "_finish_rmsnorm")
+                  _ptr(weight), dtype_code(weight), float(eps), _ptr(out), out.stride(0), _ptr(weight2), _ptr(out2),
+                  0 if out2 is None else out2.stride(0), _stream()), self.kind + "_finish_rmsnorm")
 
 
 SKINNY_DEFER_ROWS = 8    # the deferred form exists for the thread layout of up to 8 rows
@@ -484,7 +514,7 @@ DEFER_SUMS = True        # whether linear() lets a product leave its last sum to
 
 def skinny_gemm_bf16(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_rows: int, accumulate: bool = False,
                      swiglu: bool = False, status: Optional[torch.Tensor] = None, max_ctas: int = 0,
-                     defer: bool = False) -> Optional[PendingSum]:
+                     defer: bool = False, gate=NO_GATE_CONSTANTS) -> Optional[PendingSum]:
     """out[:n_rows] (=|+=) a[:n_rows] @ weight.T for n_rows <= 64: persistent CTAs stream the weight through a
     TMA-fed ring of shared-memory stages (csrc/skinny_gemm_tma.cu).  With ``defer`` (float32 +=, up to 8 rows) the
     kernel that adds up the shared tiles is not launched and a :class:`PendingSum` is returned instead."""
@@ -499,7 +529,7 @@ def skinny_gemm_bf16(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n
     ws = _skinny_scratch(a.device)
     _check(bf16lib().rs_skinny_gemm_bf16(_ptr(a), a.stride(0), a.shape[0], _ptr(weight), weight.stride(0), _ptr(out),
                                          out.stride(0), n_rows, N, K, _epilogue_code(out, accumulate, swiglu), _ptr(ws),
-                                         max_ctas, 1 if defer else 0, _ptr(status), _stream()), "skinny_gemm_bf16", 1 if defer else 2)
+                                         max_ctas, 1 if defer else 0, float(gate[0]), float(gate[1]), _ptr(status), _stream()), "skinny_gemm_bf16", 1 if defer else 2)
     return PendingSum("skinny", out, n_rows, N, K, ws, max_ctas) if defer else None
 
 
@@ -518,7 +548,7 @@ def _mid_scratch(device):
 
 def mid_gemm_bf16(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_rows: int, accumulate: bool = False,
                   swiglu: bool = False, status: Optional[torch.Tensor] = None, max_ctas: int = 0,
-                  defer: bool = False) -> Optional[PendingSum]:
+                  defer: bool = False, gate=NO_GATE_CONSTANTS) -> Optional[PendingSum]:
     """out[:n_rows] (=|+=) a[:n_rows] @ weight.T for n_rows <= 128 on the tensor cores with the operands swapped
     (rows of the weight fill the 128-row side of the MMA) and the work dealt to the SMs in equal shares of k
     (csrc/mid_gemm_tcgen05.cu).  With ``defer`` (float32 += only) the kernel that adds up the shared tiles is not
@@ -534,7 +564,7 @@ def mid_gemm_bf16(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_ro
     ws = _mid_scratch(a.device)
     _check(bf16lib().rs_mid_gemm_bf16(_ptr(a), a.stride(0), a.shape[0], _ptr(weight), weight.stride(0), _ptr(out),
                                       out.stride(0), n_rows, N, K, _epilogue_code(out, accumulate, swiglu), _ptr(ws),
-                                      max_ctas, 1 if defer else 0, _ptr(status), _stream()), "mid_gemm_bf16",
+                                      max_ctas, 1 if defer else 0, float(gate[0]), float(gate[1]), _ptr(status), _stream()), "mid_gemm_bf16",
            1 if defer else 2)
     return PendingSum("mid", out, n_rows, N, K, ws, max_ctas) if defer else None
 
@@ -685,7 +715,7 @@ def reset_chain_barrier() -> None:
 def _chain_takes_product(a, weight, out, n_rows, swiglu: bool) -> bool:
     if _ACTIVE_CHAIN is None:            # asked first: the 32-bit engine must not load (or compile) the bfloat16 library
         return False
-    if swiglu == "gelu_tanh":            # the chained kernel has the SiLU gate only
+    if swiglu in ("gelu_tanh", "clamped"):   # the chained kernel has the SiLU gate only
         return False
     lib = bf16lib()
     return (n_rows <= lib.rs_decode_chain_max_rows() and tensor_core_shape_ok(a, weight)
@@ -718,9 +748,9 @@ def linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_rows: int
 
 
 def linear_swiglu(a: torch.Tensor, weight_interleaved: torch.Tensor, out: torch.Tensor, n_rows: int,
-                  status: Optional[torch.Tensor] = None, activation: str = "silu") -> None:
-    """out[:, j] = act(a @ w[2j]) * (a @ w[2j+1]) in one kernel, act SiLU or ("gelu_tanh") the tanh form of GELU; only for
-    shapes ``tensor_core_shape_ok`` takes."""
+                  status: Optional[torch.Tensor] = None, activation: str = "silu", gate=NO_GATE_CONSTANTS) -> None:
+    """out[:, j] = act(a @ w[2j]) * (a @ w[2j+1]) in one kernel, act SiLU or ("gelu_tanh") the tanh form of GELU, or the
+    clamped gate of :func:`silu_mul` with its constants ``gate``; only for shapes ``tensor_core_shape_ok`` takes."""
     if activation not in GATE_ACTIVATIONS:
         raise KernelError(f"linear_swiglu: unknown activation '{activation}' (known: {', '.join(sorted(GATE_ACTIVATIONS))})")
     if _chain_takes_product(a, weight_interleaved, out, n_rows, activation):
@@ -728,11 +758,11 @@ def linear_swiglu(a: torch.Tensor, weight_interleaved: torch.Tensor, out: torch.
         _ACTIVE_CHAIN.add_product(a, weight_interleaved, out, n_rows, _epilogue_code(out, False, True))
         return
     if n_rows <= SKINNY_ROWS:
-        skinny_gemm_bf16(a, weight_interleaved, out, n_rows, swiglu=activation, status=status)
+        skinny_gemm_bf16(a, weight_interleaved, out, n_rows, swiglu=activation, status=status, gate=gate)
     elif n_rows <= MID_MAX_ROWS:
-        mid_gemm_bf16(a, weight_interleaved, out, n_rows, swiglu=activation, status=status)
+        mid_gemm_bf16(a, weight_interleaved, out, n_rows, swiglu=activation, status=status, gate=gate)
     else:
-        gemm_bf16_tc(a, weight_interleaved, out, n_rows, swiglu=activation, status=status)
+        gemm_bf16_tc(a, weight_interleaved, out, n_rows, swiglu=activation, status=status, gate=gate)
 
 
 # ----------------------------------------------------------------------------- attention
@@ -1570,7 +1600,15 @@ def mixerslib():
         lib = load_library("mixers")
         lib.rs_state_recurrence_rows_pad.argtypes = [c_int]
         lib.rs_state_recurrence.argtypes = [c_void_p, c_long] * 7 + [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                                                     c_void_p]
+                                                                     c_int, c_float, c_void_p, c_void_p]
+        lib.rs_mamba2_prep.argtypes = [c_void_p, c_long, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p,
+                                       c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                       c_void_p]
+        lib.rs_low_rank_decay.argtypes = [c_void_p, c_long, c_void_p, c_int, c_void_p, c_float, c_void_p, c_long, c_int, c_int, c_int,
+                                          c_int, c_int, c_void_p]
+        lib.rs_pad_heads.argtypes = [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
+        lib.rs_gated_group_norm.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_int, c_long, c_int, c_int,
+                                            c_float, c_int, c_void_p]
         lib.rs_hgrn2_prep.argtypes = [c_void_p, c_long, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                       c_int, c_int, c_void_p]
         lib.rs_delta_prep.argtypes = [c_void_p, c_long, c_void_p, c_int, c_void_p, c_long, c_void_p, c_long, c_void_p, c_int, c_void_p,
@@ -1589,12 +1627,12 @@ def mixerslib():
                                                   c_void_p, c_void_p]
         lib.rs_talking_attention.argtypes = [c_void_p, c_long, c_void_p, c_void_p, c_int, c_long, c_int, c_int, c_int, c_void_p, c_int,
                                              c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_long, c_int,
-                                             c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p]
+                                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p]
         lib.rs_talking_attention_mma_q_per_cta.argtypes = [c_int, c_int, c_int, c_int]
         lib.rs_talking_attention_mma.argtypes = [c_void_p, c_long, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_int,
                                                  c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                                                 c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                                 c_void_p, c_void_p]
+                                                 c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                                 c_float, c_float, c_void_p, c_void_p]
         _mixerslib = lib
     return _mixerslib
 
@@ -1621,29 +1659,97 @@ def state_rows_pad(rows: int) -> int:
 
 def state_recurrence(q: torch.Tensor, k: torch.Tensor, g: torch.Tensor, beta: Optional[torch.Tensor], v: torch.Tensor,
                      out: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, n_seqs: int, heads: int,
-                     group: int, rows_pad: int, columns: int, delta: bool) -> None:
+                     group: int, rows_pad: int, columns: int, delta: bool = False, head_decay: bool = False,
+                     rows: Optional[int] = None, q_scale: float = 1.0, skip: Optional[torch.Tensor] = None) -> None:
     """Per (sequence, head) a float32 state S [rows, columns] walked over the step's tokens (csrc/state_mixers.cu).
 
-    ``delta`` False: S = diag(g) S + k v^T, out = S^T q, with q, k, g [T, heads * rows_pad].
-    ``delta`` True:  S = diag(g) S; u = beta (v - S^T k); S += k u^T; out = S^T q, with q and k [T, (heads / group) *
-    rows_pad] (state head h reads q/k head h // group), g [T, heads * rows_pad], beta [T, heads].
+    Gated write (default): S = diag(g) S + k v^T, out = S^T q, with g [T, heads * rows].
+    ``delta``:             S = diag(g) S; u = beta (v - S^T k); S += k u^T; out = S^T q, beta [T, heads].
+    ``head_decay``:        S = g S + beta k v^T, out = S^T q + skip v, with g and beta [T, heads], skip [heads] or None.
+    q and k [T, (heads / group) * rows] (state head h reads q/k head h // group); ``rows`` per head, a multiple of 4, at
+    most ``rows_pad`` (the default); every read-out S^T q times ``q_scale``.
     v, out [T, heads * columns]; state [slots, >= heads * columns * rows_pad], each head stored column by column."""
-    _cuda(q, k, g, beta, v, out, state, q_start, slots)
+    _cuda(q, k, g, beta, v, out, state, q_start, slots, skip)
     _f32_rows("state_recurrence", q=q, k=k, g=g, beta=beta, v=v, out=out, state=state)
+    rows = rows_pad if rows is None else int(rows)
     _i32("state_recurrence", q_start, slots)
-    if delta and beta is None:
-        raise KernelError("state_recurrence: the delta rule needs a write strength per head")
-    qk_heads = heads // group if delta else heads
-    if q.shape[1] < qk_heads * rows_pad or k.shape[1] < qk_heads * rows_pad or g.shape[1] < heads * rows_pad \
-            or v.shape[1] < heads * columns or out.shape[1] < heads * columns or state.shape[1] < heads * columns * rows_pad:
+    if (delta or head_decay) and (beta is None or delta and head_decay):
+        raise KernelError("state_recurrence: the delta rule and the decay per head (one of them) need a write strength per head")
+    if skip is not None and (not head_decay or skip.dtype != torch.float32 or skip.numel() != heads):
+        raise KernelError("state_recurrence: skip belongs to the decay per head, float32 [heads]")
+    qk_heads = heads // group
+    if heads % group or rows % 4 or not 4 <= rows <= rows_pad or q.shape[1] < qk_heads * rows or k.shape[1] < qk_heads * rows \
+            or g.shape[1] < heads * (1 if head_decay else rows) or v.shape[1] < heads * columns or out.shape[1] < heads * columns or state.shape[1] < heads * columns * rows_pad:
         raise KernelError("state_recurrence: an operand is narrower than heads x rows / columns ask for")
-    for name, t in (("q", q), ("k", k), ("g", g), ("state", state)):
+    for name, t in (("q", q), ("k", k), ("state", state)) + (() if head_decay else (("g", g),)):
         if t.stride(0) % 4 or t.data_ptr() % 16:
             raise KernelError(f"state_recurrence: {name} must start on 16 bytes with a row pitch that is a multiple of 4")
     _check(mixerslib().rs_state_recurrence(
         _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(g), g.stride(0), _ptr(beta), 0 if beta is None else beta.stride(0),
         _ptr(v), v.stride(0), _ptr(out), out.stride(0), _ptr(state), state.stride(0), _ptr(q_start), _ptr(slots), n_seqs, heads,
-        group, rows_pad, columns, 1 if delta else 0, _stream()), "state_recurrence")
+        group, rows, rows_pad, columns, 2 if head_decay else 1 if delta else 0, float(q_scale), _ptr(skip), _stream()),
+        "state_recurrence")
+
+
+def mamba2_prep(proj: torch.Tensor, conv_off: int, dt_off: int, conv: torch.Tensor, bias: Optional[torch.Tensor],
+                tail: Optional[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor, out: torch.Tensor, dt: torch.Tensor,
+                decay: torch.Tensor, seq_of_token: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, heads: int,
+                n_tokens: int, n_seqs: int) -> None:
+    """From proj (float32): the channels from ``conv_off`` on pass a causal convolution over time (``conv`` [taps, C]
+    tap-major, ``bias`` [C]; ``tail`` [slots, >= (taps - 1) * C] holds every request's last inputs and is updated) and silu
+    into ``out`` [T, C]; dt = softplus(. + dt_bias) of the columns from ``dt_off`` on and decay = exp(-exp(a_log) dt), both
+    [T, heads] contiguous."""
+    _cuda(proj, conv, bias, tail, dt_bias, a_log, out, dt, decay, seq_of_token, q_start, slots)
+    _f32_rows("mamba2_prep", proj=proj, conv=conv, tail=tail, out=out, dt=dt, decay=decay)
+    _i32("mamba2_prep", seq_of_token, q_start, slots)
+    taps, C = conv.shape
+    for name, t, n in (("bias", bias, C), ("dt_bias", dt_bias, heads), ("a_log", a_log, heads)):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous()):
+            raise KernelError(f"mamba2_prep: {name} must be contiguous float32 with {n} values")
+    if proj.shape[1] < max(conv_off + C, dt_off + heads) or out.shape[1] < C or not conv.is_contiguous() \
+            or any(t.shape[1] != heads or not t.is_contiguous() for t in (dt, decay)) \
+            or (taps > 1 and (tail is None or tail.shape[1] < (taps - 1) * C)):
+        raise KernelError("mamba2_prep: shapes do not fit the channels, taps and heads")
+    _check(mixerslib().rs_mamba2_prep(
+        _ptr(proj), proj.stride(0), conv_off, dt_off, _ptr(conv), _ptr(bias), _ptr(tail), 0 if tail is None else tail.stride(0),
+        _ptr(dt_bias), _ptr(a_log), _ptr(out), out.stride(0), _ptr(dt), _ptr(decay), _ptr(seq_of_token), _ptr(q_start), _ptr(slots),
+        C, taps, heads, n_tokens, n_seqs, _stream()), "mamba2_prep", 2 if taps > 1 else 1)
+
+
+def low_rank_decay(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], tau: float, g: torch.Tensor, heads: int,
+                   dim: int, rows: int, n_tokens: int) -> None:
+    """g[t, h * rows + i] = sigmoid(z)^(1 / tau), z = (weight u_t + bias)[h * dim + i], zero for dim <= i < rows; u float32
+    [T, rank], weight [heads * dim, rank], float32 arithmetic."""
+    _cuda(u, weight, bias, g)
+    _f32_rows("low_rank_decay", u=u, g=g)
+    if weight.shape[0] != heads * dim or not weight.is_contiguous() or u.shape[1] < weight.shape[1] or g.shape[1] < heads * rows \
+            or rows < dim or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != heads * dim)):
+        raise KernelError("low_rank_decay: shapes do not fit heads x dim")
+    _check(mixerslib().rs_low_rank_decay(_ptr(u), u.stride(0), _ptr(weight), dtype_code(weight), _ptr(bias), 1.0 / float(tau), _ptr(g),
+                                         g.stride(0), heads, dim, rows, weight.shape[1], n_tokens, _stream()), "low_rank_decay")
+
+
+def pad_heads(src: torch.Tensor, dst: torch.Tensor, heads: int, dim: int, rows: int, n_tokens: int) -> None:
+    """dst[t, h * rows + i] = src[t, h * dim + i] for i < dim, zero up to rows; float32, dst contiguous [T, heads * rows]."""
+    _cuda(src, dst)
+    _f32_rows("pad_heads", src=src, dst=dst)
+    if src.shape[1] < heads * dim or dst.shape[1] != heads * rows or not dst.is_contiguous() or rows < dim:
+        raise KernelError("pad_heads: shapes do not fit heads x rows")
+    _check(mixerslib().rs_pad_heads(_ptr(src), src.stride(0), _ptr(dst), heads, dim, rows, n_tokens, _stream()), "pad_heads")
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, parts: int, eps: float,
+                     n_tokens: int) -> None:
+    """u = y silu(z); each of the row's ``parts`` equal parts of u over its own root mean square (eps inside the root), times
+    weight; y, z, weight float32."""
+    _cuda(y, z, weight, out)
+    _f32_rows("gated_group_norm", y=y, z=z)
+    _rows_contiguous(out, "gated_group_norm out")
+    n = weight.numel()
+    if n % parts or y.shape[1] < n or z.shape[1] < n or out.shape[1] < n or weight.dtype != torch.float32 or not weight.is_contiguous():
+        raise KernelError(f"gated_group_norm: {n} weights in {parts} parts do not fit the rows")
+    _check(mixerslib().rs_gated_group_norm(_ptr(y), y.stride(0), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), dtype_code(out),
+                                           out.stride(0), n // parts, parts, float(eps), n_tokens, _stream()), "gated_group_norm")
 
 
 def hgrn2_prep(proj: torch.Tensor, f_bias: Optional[torch.Tensor], lower: torch.Tensor, q: torch.Tensor, g: torch.Tensor,
@@ -1794,11 +1900,13 @@ def talking_attention_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_n
 def talking_attention(q: torch.Tensor, gate: Optional[torch.Tensor], cache: torch.Tensor, block_table: torch.Tensor,
                       page_size: int, q_start: torch.Tensor, kv_len: torch.Tensor, work: torch.Tensor, n_work: int,
                       talk: Optional[torch.Tensor], sink: Optional[torch.Tensor], out: torch.Tensor, n_heads: int, n_kv: int,
-                      dk: int, dv: int, window: int, q_per_cta: int, scale: float, status: torch.Tensor, chunk: int = 0) -> None:
+                      dk: int, dv: int, window: int, q_per_cta: int, scale: float, status: torch.Tensor, chunk: int = 0,
+                      keep: int = 0, out_scale: float = 1.0) -> None:
     """Causal attention of the step's queries over the paged cache (within ``window`` keys if positive, within the query's
-    own block of ``chunk`` positions if positive) with scores mixed across heads (``talk`` float32
+    own block of ``chunk`` positions if positive, a sequence's first ``keep`` keys besides) with scores mixed across heads (``talk`` float32
     [heads, heads]: mixed[h] = sum_g talk[h, g] raw[g]) before a softmax whose denominator also holds exp(sink[h]);
-    every head's output times ``gate`` [T, heads].  ``work``: (sequence, first query) per tile of ``q_per_cta`` queries."""
+    every head's output times ``gate`` [T, heads] and ``out_scale``.  ``work``: (sequence, first query) per tile of
+    ``q_per_cta`` queries."""
     _cuda(q, gate, cache, block_table, q_start, kv_len, work, talk, sink, out, status)
     _f32_rows("talking_attention", q=q, gate=gate)
     _rows_contiguous(out, "talking_attention out")
@@ -1812,8 +1920,8 @@ def talking_attention(q: torch.Tensor, gate: Optional[torch.Tensor], cache: torc
     _check(mixerslib().rs_talking_attention(
         _ptr(q), q.stride(0), _ptr(gate), _ptr(cache), dtype_code(cache), cache.stride(0), cache.shape[0], page_size,
         cache.shape[-1], _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len), _ptr(work), n_work, _ptr(talk),
-        _ptr(sink), _ptr(out), dtype_code(out), out.stride(0), n_heads, n_kv, dk, dv, window, int(chunk), q_per_cta,
-        float(scale), _ptr(status), _stream()), "talking_attention")
+        _ptr(sink), _ptr(out), dtype_code(out), out.stride(0), n_heads, n_kv, dk, dv, window, int(chunk), int(keep),
+        q_per_cta, float(scale), float(out_scale), _ptr(status), _stream()), "talking_attention")
 
 
 def talking_attention_mma_q_per_cta(n_heads: int, n_kv: int, dk: int, dv: int) -> int:
@@ -1829,7 +1937,7 @@ def talking_attention_mma(q: torch.Tensor, gate: Optional[torch.Tensor], cache: 
                           page_size: int, q_start: torch.Tensor, kv_len: torch.Tensor, work: torch.Tensor, n_work: int,
                           any_parts: bool, talk: Optional[torch.Tensor], sink: Optional[torch.Tensor], out: torch.Tensor,
                           partial: Optional[torch.Tensor], n_heads: int, n_kv: int, dk: int, dv: int, window: int, q_per_cta: int,
-                          scale: float, status: torch.Tensor, chunk: int = 0) -> None:
+                          scale: float, status: torch.Tensor, chunk: int = 0, keep: int = 0, out_scale: float = 1.0) -> None:
     """``talking_attention`` for a bfloat16 cache on the tensor cores (csrc/talking_attention_mma.cu).  ``work`` rows are
     (sequence, first query, part, parts, first partial row): a tile's key tiles are dealt out over ``parts`` CTAs, whose
     sums meet in ``partial`` float32 [rows, >= heads * (dv + 2)] (part p of a tile of n queries uses rows first + p * n ..)."""
@@ -1855,4 +1963,4 @@ def talking_attention_mma(q: torch.Tensor, gate: Optional[torch.Tensor], cache: 
         _ptr(q), q.stride(0), _ptr(gate), _ptr(cache), cache.stride(0), cache.shape[0], page_size, cache.shape[-1],
         _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len), _ptr(work), n_work, 1 if any_parts else 0,
         _ptr(talk), _ptr(sink), _ptr(out), dtype_code(out), out.stride(0), _ptr(partial), rows, n_heads, n_kv, dk, dv, window,
-        int(chunk), q_per_cta, float(scale), _ptr(status), _stream()), "talking_attention_mma")
+        int(chunk), int(keep), q_per_cta, float(scale), float(out_scale), _ptr(status), _stream()), "talking_attention_mma")

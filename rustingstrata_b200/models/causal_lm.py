@@ -151,6 +151,8 @@ class CausalLM:
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         for p in self.parts():
             p.load(tensors)
+        for b in self.blocks:
+            b.finish_load()
 
     # ---------------------------------------------------------------- storage binding
     def bind_storage(self, caches: List[torch.Tensor], states: Dict[Tuple[int, str], torch.Tensor]) -> None:

@@ -198,8 +198,26 @@ class Mixer(Part):
         raise NotImplementedError
 
 
+    # ---- a mixer whose first and last steps are plain products may offer them to the block, which can then run several
+    # parts' products as one (see ParallelBlock): ``joinable`` True, ``in_cols`` and ``row_cols`` (columns of the float32
+    # projection it reads and of the rows its output matrix takes), ``w_in`` [in_cols, hidden] and ``w_o`` [hidden, row_cols]
+    # after load (the block may replace them by views of a joint matrix), and :meth:`forward_rows`.
+    joinable = False
+
+    def forward_rows(self, proj: torch.Tensor, rows: torch.Tensor, ctx: StepContext, call: CallInfo) -> None:
+        """From the projected rows ``proj`` [T, in_cols] (float32) to what the output matrix multiplies, ``rows``
+        [T, row_cols] in the engine's element type."""
+        raise NotImplementedError
+
+
 class FeedForward(Part):
     """Per-token feed-forward: reads ``h`` [T, hidden], adds its output into ``residual`` in place."""
+
+    # like a mixer's: ``row_cols``, ``w_down`` [hidden, row_cols] and ``forward_rows(h, rows, ctx)``
+    joinable = False
+
+    def forward_rows(self, h: torch.Tensor, rows: torch.Tensor, ctx: StepContext) -> None:
+        raise NotImplementedError
 
     def forward(self, h: torch.Tensor, residual: torch.Tensor, ctx: StepContext) -> None:
         raise NotImplementedError
@@ -214,6 +232,13 @@ class Norm(Part):
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, n_rows: int, rows: Optional[torch.Tensor] = None) -> None:
         raise NotImplementedError
+
+    def forward_pair(self, x: torch.Tensor, out: torch.Tensor, other: "Norm", out2: torch.Tensor, n_rows: int, owed=None) -> None:
+        """out = self(x), out2 = other(x); a norm that can takes both from one read of ``x``."""
+        if owed is not None:
+            owed.finish()
+        self.forward(x, out, n_rows)
+        other.forward(x, out2, n_rows)
 
     def forward_add(self, delta: torch.Tensor, x: torch.Tensor, n_rows: int, then: Optional["Norm"] = None,
                     out: Optional[torch.Tensor] = None) -> None:
@@ -271,6 +296,9 @@ class Block(Part):
 
     def mixers(self) -> Dict[str, Mixer]:
         return {r: p for r, p in self.parts.items() if self.roles.get(r) == "mixer"}
+
+    def finish_load(self) -> None:
+        """Called once after every part has taken its tensors: the place to join matrices of several parts."""
 
     @property
     def first_reader_takes_owed(self) -> bool:

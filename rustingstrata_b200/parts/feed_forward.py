@@ -17,8 +17,11 @@ from .spec import TensorNeed
 
 @register_part("feed_forward", "gated_mlp")
 class GatedMLP(FeedForward):
-    """params: hidden, intermediate, activation ("silu", the default, or "gelu_tanh").  tensors: gate_proj, up_proj, down_proj."""
+    """params: hidden, intermediate, activation ("silu", the default, "gelu_tanh", or "clamped": with g = min(gate, limit) and
+    u = up held in [-limit, limit], g sigmoid(alpha g) (u + 1)), and for "clamped" alpha and limit.
+    tensors: gate_proj, up_proj, down_proj."""
     chain_safe = True
+    joinable = True
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -28,6 +31,12 @@ class GatedMLP(FeedForward):
         if act not in ops.GATE_ACTIVATIONS:
             raise ValueError(f"gated_mlp: activation '{act}' has no kernel (known: {', '.join(sorted(ops.GATE_ACTIVATIONS))})")
         self.activation = act
+        self.gate_constants = ops.NO_GATE_CONSTANTS
+        if act == "clamped":
+            self.gate_constants = (float(spec.params["alpha"]), float(spec.params["limit"]))
+            if not self.gate_constants[1] > 0:
+                raise ValueError(f"gated_mlp: the clamped gate's limit must be positive, got {self.gate_constants[1]}")
+        self.row_cols = self.inter
         runtime.scratch("gate_up", runtime.max_batch_tokens, 2 * self.inter)
         runtime.scratch("ff_act", runtime.max_batch_tokens, self.inter)
         self.w_gate_up = self.w_down = None
@@ -53,16 +62,19 @@ class GatedMLP(FeedForward):
             self.w_gate_up = torch.cat([g, u], dim=0).contiguous()
         self.w_down = tensors[t["down_proj"]].contiguous()
 
-    def forward(self, h, residual, ctx):
-        rt = self.runtime
+    def forward_rows(self, h, rows, ctx):
         T = ctx.n_tokens
-        gate_up = rt.get_scratch("gate_up")[:, : 2 * self.inter]
-        act = rt.get_scratch("ff_act")[:, : self.inter]
         if self.fused:
-            ops.linear_swiglu(h, self.w_gate_up, act, T, status=ctx.status, activation=self.activation)
+            ops.linear_swiglu(h, self.w_gate_up, rows, T, status=ctx.status, activation=self.activation, gate=self.gate_constants)
         else:
+            gate_up = self.runtime.get_scratch("gate_up")[:, : 2 * self.inter]
             ops.linear(h, self.w_gate_up, gate_up, T)
-            ops.silu_mul(gate_up, act, T, self.activation)
+            ops.silu_mul(gate_up, rows, T, self.activation, self.gate_constants)
+
+    def forward(self, h, residual, ctx):
+        T = ctx.n_tokens
+        act = self.runtime.get_scratch("ff_act")[:, : self.inter]
+        self.forward_rows(h, act, ctx)
         ctx.owed = ops.linear(act, self.w_down, residual, T, accumulate=not ctx.store_output, status=ctx.status,
                               may_defer=ctx.may_owe and not ctx.store_output)
 

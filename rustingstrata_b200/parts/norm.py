@@ -34,6 +34,12 @@ class RMSNorm(Norm):
     def forward(self, x, out, n_rows, rows=None, owed=None):
         ops.rmsnorm(x, self.weight, self.eps, out, rows=rows, n_rows=n_rows, pending=owed)
 
+    def forward_pair(self, x, out, other, out2, n_rows, owed=None):
+        if isinstance(other, RMSNorm) and other.width == self.width and other.eps == self.eps and other.weight.dtype == self.weight.dtype:
+            ops.rmsnorm(x, self.weight, self.eps, out, n_rows=n_rows, pending=owed, weight2=other.weight, out2=out2)
+            return
+        super().forward_pair(x, out, other, out2, n_rows, owed)
+
     def forward_add(self, delta, x, n_rows, then=None, out=None):
         if then is not None and isinstance(then, RMSNorm) and then.width == self.width:
             ops.rmsnorm_add(x, delta, self.gain, self.eps, n_rows, then.gain, then.eps, out)

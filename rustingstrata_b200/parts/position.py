@@ -17,7 +17,8 @@ from .registry import register_part
 @register_part("position", "rope_neox")
 class RotaryNeox(PositionEncoding):
     """params: n_rot (rotated dims of a head), base, base_bits (32, the default: the base is held as float32 and widened,
-    as the reference holds it; 64: the base as config.json gives it).  Coordinate i < n_rot / 2 turns together with
+    as the reference holds it; 64: the base as config.json gives it), min_rows (0: the table holds at least so many positions,
+    for requests longer than the cache pool, which a window allows).  Coordinate i < n_rot / 2 turns together with
     i + n_rot / 2 (``pairing`` "half")."""
     chain_safe = True
     pairing = "half"
@@ -32,7 +33,7 @@ class RotaryNeox(PositionEncoding):
         if self.base_bits not in (32, 64):
             raise ValueError(f"rope_neox: base_bits {self.base_bits} (32 or 64)")
         # as many positions as a request can reach: the model's limit, or what the cache pool holds if that is less
-        self.rows = max(1, min(runtime.max_positions, runtime.pool_tokens))
+        self.rows = max(1, min(runtime.max_positions, max(runtime.pool_tokens, int(spec.params.get("min_rows", 0)))))
         self._key = ("rope_neox", self.n_rot, self.base, self.base_bits, self.rows)
 
     @property

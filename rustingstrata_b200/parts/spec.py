@@ -100,6 +100,7 @@ class CacheNeed:
 
     ``window`` None keeps every key; an integer keeps the most recent ``window`` keys
     (the current one included), so pages wholly older than that are given back.
+    ``keep_first``: with a window, the first so many keys of a sequence stay besides.
     ``planes``: 2 keeps a key row and a value row per token and head; 1 keeps one row that
     serves as both (a latent from which keys and values are expanded).
     Calls with equal needs share a page pool ("cache group").
@@ -108,6 +109,7 @@ class CacheNeed:
     head_dim: int
     window: Optional[int] = None
     planes: int = 2
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

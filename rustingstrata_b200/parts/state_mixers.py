@@ -1,5 +1,6 @@
 """Mixers that keep a matrix of state per head in place of a cache of keys: HGRN2, the gated delta rule with a decay
-per key channel, and retention with one fixed decay per head.  All walk a float32 state S [dim, vdim] per (request, head)
+per key channel, retention with one fixed decay per head, gated linear attention with a decay per key channel, and
+Mamba-2 with a decay per head that the input sets.  All walk a float32 state S [dim, vdim] per (request, head)
 token by token and read it out with a query.
 
 ``hgrn2`` (gated linear recurrence whose forget gate also decides what is written).  From the mixer's input h:
@@ -29,7 +30,24 @@ k times dim^-1/2 after the rotation;
 each head's o_t is divided by its root mean square over vdim (no weight), the heads are joined, multiplied by
 silu(W_g h) coordinate by coordinate, and W_o maps them back.
 
-Per request the state slot holds S for every head (zero at admission) and, for the convolution, the last taps - 1
+``gated_linear_attention``.  q = W_q h * q_scale (dim^-1/2), k = W_k h (heads x dim), v = W_v h (heads x vdim),
+alpha = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau) per head and key channel;
+
+    S_t = diag(alpha_t) S_(t-1) + k_t v_t^T,        o_t = S_t^T q_t;
+
+each head's o_t is divided by its root mean square over vdim and multiplied by a weight [vdim] shared by the heads, the
+heads are joined, multiplied by silu(W_g h), and W_o maps them back.
+
+``mamba2`` (state-space duality; N = state rows, G = groups, inner = heads x vdim).  W_in h = [z | x | B | C | dt] with
+widths inner, inner, G N, G N, heads; x, B and C pass a short causal convolution over time with a bias, and silu;
+dt <- softplus(dt + dt_bias); head h reads B and C of group h // (heads / G):
+
+    S_t = exp(-exp(A_h) dt) S_(t-1) + dt B_t x_t^T,        y_t = S_t^T C_t + D_h x_t;
+
+the joined y is multiplied by silu(z), each of ``norm_groups`` equal parts divided by its own root mean square, times a
+weight [inner]; then W_o.
+
+Per request the state slot holds S for every head (zero at admission) and, for a convolution, the last taps - 1
 projected rows.  The projections follow the engine's element type with float32 results; gates, decays, norms, the
 state and the recurrence are float32 in both engines.
 """
@@ -288,3 +306,186 @@ class Retention(Mixer):
         gate = proj[:, v_off + self.v_cols:] if self.has_gate else None
         ops.head_norm_gate(read, None, gate, out, H, self.dv, self.eps, T, gate_silu=True)
         ops.linear(out, self.w_o, residual, T, accumulate=not ctx.store_output, status=ctx.status)
+
+
+def _on_16_bytes(dim: int, *ts) -> bool:
+    """Whether every head of ``dim`` values in these float32 rows starts on 16 bytes (the recurrence can read them in place)."""
+    return dim % 4 == 0 and all(t.stride(0) % 4 == 0 and t.data_ptr() % 16 == 0 for t in ts)
+
+
+@register_part("mixer", "gated_linear_attention")
+class GatedLinearAttention(Mixer):
+    """params: hidden, n_heads, dim, vdim, tau, decay_rank (inner width of the decay's low-rank map), eps (of the read-out
+    norm), q_scale (default dim^-1/2), out_scale (default 1: multiplies the mixer's output).
+    tensors: q_proj, k_proj, v_proj, g_proj [heads * vdim, hidden], a1_proj [decay_rank, hidden], a2_proj [heads * dim,
+    decay_rank], a2_bias [heads * dim], norm [vdim], o_proj."""
+    joinable = True
+
+    def __init__(self, spec, runtime, position=None):
+        super().__init__(spec, runtime)
+        p = spec.params
+        self.hidden, self.n_heads = int(p["hidden"]), int(p["n_heads"])
+        self.dk, self.dv = int(p["dim"]), int(p["vdim"])
+        self.tau, self.rank = float(p["tau"]), int(p["decay_rank"])
+        self.eps = float(p.get("eps", 0.0))
+        self.q_scale = float(p["q_scale"]) if p.get("q_scale") is not None else float(self.dk) ** -0.5
+        self.out_scale = float(p.get("out_scale", 1.0))
+        if not self.tau > 0 or self.rank < 1:
+            raise ValueError(f"gated_linear_attention: tau {self.tau} and decay_rank {self.rank} must be positive")
+        self.rows_pad = ops.state_rows_pad(self.dk)
+        self.qk_cols, self.v_cols = self.n_heads * self.dk, self.n_heads * self.dv
+        self.v_off = 2 * self.qk_cols
+        self.g_off = self.v_off + self.v_cols
+        self.a1_off = self.g_off + self.v_cols
+        self.in_cols = self.a1_off + self.rank
+        self.row_cols = self.v_cols
+        rt = runtime
+        rt.scratch("state_proj", rt.max_batch_tokens, self.in_cols, torch.float32)
+        # decays, and where heads do not start on 16 bytes the padded queries and keys
+        rt.scratch("state_rows", 1, 3 * rt.max_batch_tokens * self.n_heads * self.rows_pad, torch.float32)
+        rt.scratch("state_read", rt.max_batch_tokens, self.v_cols, torch.float32)
+        rt.scratch("state_out", rt.max_batch_tokens, self.v_cols)
+
+    def tensor_needs(self):
+        t, D = self.spec.tensors, self.hidden
+        return {t["q_proj"]: TensorNeed((self.qk_cols, D)), t["k_proj"]: TensorNeed((self.qk_cols, D)),
+                t["v_proj"]: TensorNeed((self.v_cols, D)), t["g_proj"]: TensorNeed((self.v_cols, D)),
+                t["a1_proj"]: TensorNeed((self.rank, D)), t["a2_proj"]: TensorNeed((self.qk_cols, self.rank)),
+                t["a2_bias"]: TensorNeed((self.qk_cols,)), t["norm"]: TensorNeed((self.dv,), "norm"),
+                t["o_proj"]: TensorNeed((D, self.v_cols))}
+
+    def load(self, tensors):
+        t = self.spec.tensors
+        mats = [tensors[t[n]] for n in ("q_proj", "k_proj", "v_proj", "g_proj", "a1_proj")]
+        if len({m.dtype for m in mats}) != 1:
+            raise ValueError("gated_linear_attention: the input projections must share an element type")
+        self.w_in = torch.cat(mats, dim=0).contiguous()              # [q | k | v | gate | a1]: h is read by one product
+        self.w_a2 = tensors[t["a2_proj"]].contiguous()
+        self.a2_bias = tensors[t["a2_bias"]].to(torch.float32).contiguous()
+        # the output's factor rides on the read-out norm's weight, in float32
+        self.norm_w = (tensors[t["norm"]].to(torch.float32) * self.out_scale).contiguous()
+        self.w_o = tensors[t["o_proj"]].contiguous()
+
+    def state_need(self):
+        return StateNeed(self.n_heads * self.dv * self.rows_pad, "float32")
+
+    def flops_per_token(self) -> float:
+        return 2.0 * (self.hidden * (self.in_cols + self.v_cols) + self.qk_cols * self.rank) + 6.0 * self.n_heads * self.dk * self.dv
+
+    def forward(self, h, residual, ctx: StepContext, call: CallInfo):
+        rt, T = self.runtime, ctx.n_tokens
+        proj = rt.get_scratch("state_proj", torch.float32)[:, : self.in_cols]
+        out = rt.get_scratch("state_out")[:, : self.v_cols]
+        ops.linear(h, self.w_in, proj, T, status=ctx.status)
+        self.forward_rows(proj, out, ctx, call)
+        ops.linear(out, self.w_o, residual, T, accumulate=not ctx.store_output, status=ctx.status)
+
+    def forward_rows(self, proj, out, ctx: StepContext, call: CallInfo):
+        rt, T, H, RP = self.runtime, ctx.n_tokens, self.n_heads, self.rows_pad
+        mbt = rt.max_batch_tokens
+        n = mbt * H * RP
+        flat = rt.get_scratch("state_rows", torch.float32)[0]
+        q_buf, k_buf = flat[:n].view(mbt, H * RP), flat[n: 2 * n].view(mbt, H * RP)
+        read = rt.get_scratch("state_read", torch.float32)[:, : self.v_cols]
+        q, k, rows = proj[:, : self.qk_cols], proj[:, self.qk_cols: self.v_off], self.dk
+        if not _on_16_bytes(self.dk, q, k):
+            ops.pad_heads(q, q_buf, H, self.dk, RP, T)
+            ops.pad_heads(k, k_buf, H, self.dk, RP, T)
+            q, k, rows = q_buf, k_buf, RP
+        g = flat[2 * n: 2 * n + mbt * H * rows].view(mbt, H * rows)
+        ops.low_rank_decay(proj[:, self.a1_off: self.a1_off + self.rank], self.w_a2, self.a2_bias, self.tau, g, H, self.dk, rows, T)
+        ops.state_recurrence(q, k, g, None, proj[:, self.v_off: self.g_off], read, call.state, ctx.q_start, ctx.state_slots,
+                             ctx.n_seqs, H, 1, RP, self.dv, rows=rows, q_scale=self.q_scale)
+        ops.head_norm_gate(read, self.norm_w, proj[:, self.g_off: self.a1_off], out, H, self.dv, self.eps, T, gate_silu=True)
+
+
+@register_part("mixer", "mamba2")
+class Mamba2(Mixer):
+    """params: hidden, n_heads, vdim, state (rows of a head's state), groups (of B and C), taps, norm_groups, eps (of the
+    read-out norm), out_scale (default 1: multiplies the mixer's output).
+    tensors: in_proj [2 * inner + 2 * groups * state + heads, hidden], conv [inner + 2 * groups * state, taps], conv_bias,
+    dt_bias [heads], a_log [heads], d_skip [heads], norm [inner], o_proj [hidden, inner], inner = heads * vdim."""
+    joinable = True
+
+    def __init__(self, spec, runtime, position=None):
+        super().__init__(spec, runtime)
+        p = spec.params
+        self.hidden, self.n_heads, self.dv = int(p["hidden"]), int(p["n_heads"]), int(p["vdim"])
+        self.rows, self.groups, self.taps = int(p["state"]), int(p["groups"]), int(p["taps"])
+        self.norm_groups, self.eps = int(p["norm_groups"]), float(p.get("eps", 0.0))
+        self.out_scale = float(p.get("out_scale", 1.0))
+        if self.n_heads % self.groups:
+            raise ValueError(f"mamba2: {self.n_heads} heads are not a multiple of {self.groups} groups")
+        self.inner = self.row_cols = self.n_heads * self.dv
+        if self.inner % self.norm_groups:
+            raise ValueError(f"mamba2: {self.inner} inner channels do not divide into {self.norm_groups} norm groups")
+        if not 1 <= self.taps <= 64:
+            raise ValueError(f"mamba2: {self.taps} taps (1 to 64 are supported)")
+        self.rows_pad = ops.state_rows_pad(self.rows)
+        self.bc_cols = self.groups * self.rows
+        self.channels = self.inner + 2 * self.bc_cols
+        self.dt_off = self.inner + self.channels
+        self.in_cols = self.dt_off + self.n_heads
+        self.tail = (self.taps - 1) * self.channels
+        self.state_cols = self.n_heads * self.dv * self.rows_pad
+        rt, mbt = runtime, runtime.max_batch_tokens
+        rt.scratch("state_proj", mbt, self.in_cols, torch.float32)
+        self.conv_pitch = (self.channels + 3) // 4 * 4
+        rt.scratch("mamba_conv", mbt, self.conv_pitch, torch.float32)
+        rt.scratch("mamba_step", 1, 2 * mbt * self.n_heads, torch.float32)
+        if self.rows % 4 or self.inner % 4:
+            rt.scratch("state_rows", 1, 2 * mbt * self.groups * self.rows_pad, torch.float32)
+        rt.scratch("state_read", mbt, self.inner, torch.float32)
+        rt.scratch("state_out", mbt, self.inner)
+
+    def tensor_needs(self):
+        t, D, H = self.spec.tensors, self.hidden, self.n_heads
+        return {t["in_proj"]: TensorNeed((self.in_cols, D)), t["conv"]: TensorNeed((self.channels, self.taps)),
+                t["conv_bias"]: TensorNeed((self.channels,)), t["dt_bias"]: TensorNeed((H,)), t["a_log"]: TensorNeed((H,)),
+                t["d_skip"]: TensorNeed((H,)), t["norm"]: TensorNeed((self.inner,), "norm"),
+                t["o_proj"]: TensorNeed((D, self.inner))}
+
+    def load(self, tensors):
+        t = self.spec.tensors
+        f32 = lambda name: tensors[t[name]].to(torch.float32).contiguous()                        # noqa: E731
+        self.w_in, self.w_o = tensors[t["in_proj"]].contiguous(), tensors[t["o_proj"]].contiguous()
+        self.w_conv = f32("conv").t().contiguous()                   # tap-major, as the kernel reads it
+        self.conv_bias, self.dt_bias, self.a_log, self.d_skip = f32("conv_bias"), f32("dt_bias"), f32("a_log"), f32("d_skip")
+        self.norm_w = (f32("norm") * self.out_scale).contiguous()
+
+    def state_need(self):
+        # the slot's pitch stays a multiple of 16 bytes: the recurrence moves a state's rows in runs of four values
+        return StateNeed(self.state_cols + (self.tail + 3) // 4 * 4, "float32")
+
+    def flops_per_token(self) -> float:
+        return 2.0 * self.hidden * (self.in_cols + self.inner) + 6.0 * self.n_heads * self.rows * self.dv
+
+    def forward(self, h, residual, ctx: StepContext, call: CallInfo):
+        rt, T = self.runtime, ctx.n_tokens
+        proj = rt.get_scratch("state_proj", torch.float32)[:, : self.in_cols]
+        out = rt.get_scratch("state_out")[:, : self.inner]
+        ops.linear(h, self.w_in, proj, T, status=ctx.status)
+        self.forward_rows(proj, out, ctx, call)
+        ops.linear(out, self.w_o, residual, T, accumulate=not ctx.store_output, status=ctx.status)
+
+    def forward_rows(self, proj, out, ctx: StepContext, call: CallInfo):
+        rt, T, H, G, RP = self.runtime, ctx.n_tokens, self.n_heads, self.groups, self.rows_pad
+        mbt = rt.max_batch_tokens
+        conv = rt.get_scratch("mamba_conv", torch.float32)[:, : self.channels]
+        flat = rt.get_scratch("mamba_step", torch.float32)[0]
+        dt, decay = flat[: mbt * H].view(mbt, H), flat[mbt * H: 2 * mbt * H].view(mbt, H)
+        read = rt.get_scratch("state_read", torch.float32)[:, : self.inner]
+        state = call.state
+        ops.mamba2_prep(proj, self.inner, self.dt_off, self.w_conv, self.conv_bias, state[:, self.state_cols:] if self.tail else None,
+                        self.dt_bias, self.a_log, conv, dt, decay, ctx.seq_of_token, ctx.q_start, ctx.state_slots, H, T, ctx.n_seqs)
+        k, q, rows = conv[:, self.inner: self.inner + self.bc_cols], conv[:, self.inner + self.bc_cols:], self.rows
+        if not _on_16_bytes(self.rows, k, q):
+            n = mbt * G * RP
+            pads = rt.get_scratch("state_rows", torch.float32)[0]
+            k_buf, q_buf = pads[:n].view(mbt, G * RP), pads[n: 2 * n].view(mbt, G * RP)
+            ops.pad_heads(k, k_buf, G, self.rows, RP, T)
+            ops.pad_heads(q, q_buf, G, self.rows, RP, T)
+            k, q, rows = k_buf, q_buf, RP
+        ops.state_recurrence(q, k, decay, dt, conv[:, : self.inner], read, state, ctx.q_start, ctx.state_slots, ctx.n_seqs, H, H // G,
+                             RP, self.dv, head_decay=True, rows=rows, skip=self.d_skip)
+        ops.gated_group_norm(read, proj[:, : self.inner], self.norm_w, out, self.norm_groups, self.eps, T)

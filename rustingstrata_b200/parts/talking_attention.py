@@ -10,13 +10,14 @@ pairs halves, coordinate i with i + n_rot / 2.  With raw[g, i, j] = (q_gi . k_gj
 
     mixed[h, i, j] = sum_g talk[h, g] raw[g, i, j]                      (talk [heads, heads]; None: the raw score)
 
-and the weights of query i over the keys j <= i (within ``window`` if there is one; with ``chunk`` only keys of the
+and the weights of query i over the keys j <= i (within ``window`` if there is one; the sequence's first
+``keep_first`` keys stay visible however far behind they are, in their true positions; with ``chunk`` only keys of the
 query's own block of that many positions, floor(i / chunk) = floor(j / chunk), blocks counted from position 0) are
 
     exp(mixed[h, i, j]) / (exp(sink[h]) + sum_j' exp(mixed[h, i, j']))  (sink [heads]; None: no such term).
 
 The sink has no key and no value, is neither scaled nor mixed, and counts once.  Head h's weighted sum of values is
-multiplied by sigmoid(w_g[h] . h), and W_o maps the joined heads back to the stream.  Norms, angles, scores, the mix,
+multiplied by sigmoid(w_g[h] . h) and by ``out_scale``, and W_o maps the joined heads back to the stream.  Norms, angles, scores, the mix,
 weights and gates are float32 in both engines; keys and values are cached in the engine's element type, in rows
 padded to a common size.  Each of bias, norm, talk, sink and gate is a parameter of the part and may be left out.
 """
@@ -41,10 +42,12 @@ PARTIAL_ROWS = 4096        # (query, part) rows of partial sums the workspace ho
 
 @register_part("mixer", "talking_attention")
 class TalkingAttention(Mixer):
-    """params: hidden, n_heads, n_kv_heads, dim, vdim, scale, eps, window (None: every key), chunk (None: no blocks),
-    bias, qk_norm, talk, sink, gate (bools, default True), norm ("head", the default, or "row").  tensors: q_proj, k_proj,
+    """params: hidden, n_heads, n_kv_heads, dim, vdim, scale, eps, window (None: every key), keep_first (0), chunk (None: no
+    blocks), out_scale (1), bias, qk_norm, talk, sink, gate (bools, default True), norm ("head", the default, or "row").  tensors: q_proj, k_proj,
     v_proj, o_proj, and as the params ask q_bias, k_bias, v_bias, q_norm, k_norm ([dim] each; "row": [heads * dim] and
     [kv heads * dim]), talk [heads, heads], sink [heads], g_proj [heads, hidden]."""
+
+    joinable = True
 
     def __init__(self, spec, runtime, position=None):
         super().__init__(spec, runtime)
@@ -56,6 +59,12 @@ class TalkingAttention(Mixer):
         self.eps = float(p.get("eps", 0.0))
         self.window = int(p["window"]) if p.get("window") else 0
         self.chunk = int(p["chunk"]) if p.get("chunk") else 0
+        self.keep = int(p.get("keep_first") or 0)
+        if self.keep < 0 or (self.keep and self.chunk):
+            raise ValueError("talking_attention: keep_first counts a window's kept first keys (not negative, not with blocks)")
+        if not self.window:
+            self.keep = 0                    # every key is kept already
+        self.out_scale = float(p.get("out_scale", 1.0))
         self.row_norm = p.get("norm", "head") == "row"
         if p.get("norm", "head") not in ("head", "row"):
             raise ValueError(f"talking_attention: norm {p.get('norm')!r} (known: 'head', 'row')")
@@ -74,7 +83,7 @@ class TalkingAttention(Mixer):
         self.q_cols, self.k_cols, self.v_cols = self.n_heads * self.dk, self.n_kv * self.dk, self.n_kv * self.dv
         self.g_cols = self.n_heads if self.has_gate else 0
         self.in_cols = self.q_cols + self.k_cols + self.v_cols + self.g_cols
-        self.o_in = self.n_heads * self.dv
+        self.o_in = self.row_cols = self.n_heads * self.dv
         self.q_per_cta = None
         self.mma_q = 0
         rt = runtime
@@ -122,7 +131,7 @@ class TalkingAttention(Mixer):
     def cache_need(self):
         # a block of ``chunk`` positions never reaches further back than chunk keys, the query's own included
         reach = [w for w in (self.window, self.chunk) if w]
-        return CacheNeed(self.n_kv, self.head_pad, min(reach) if reach else None)
+        return CacheNeed(self.n_kv, self.head_pad, min(reach) if reach else None, keep_first=self.keep)
 
     def flops_per_token(self) -> float:
         return 2.0 * self.hidden * (self.in_cols + self.o_in)
@@ -132,6 +141,8 @@ class TalkingAttention(Mixer):
         for q, kv in zip(np.asarray(q_lens, dtype=np.int64), np.asarray(kv_lens, dtype=np.int64)):
             pos = np.arange(kv - q, kv, dtype=np.float64)
             seen = pos + 1 if not self.window else np.minimum(pos + 1, self.window)
+            if self.keep:              # kept first keys that the window has passed
+                seen = seen + np.clip(pos + 1 - self.window, 0, self.keep)
             if self.chunk:
                 seen = np.minimum(seen, pos % self.chunk + 1)
             pairs += float(seen.sum())
@@ -147,7 +158,7 @@ class TalkingAttention(Mixer):
 
     def plan_key(self):
         self._setup()
-        return ("talking_attention", self.q_per_cta, self.mma_q, self.window, self.chunk)
+        return ("talking_attention", self.q_per_cta, self.mma_q, self.window, self.chunk, self.keep)
 
     def build_plan(self, batch: HostBatch):
         """Tiles of neighbouring queries of one sequence, the ones with the most keys to walk first.  For the tensor-core
@@ -180,7 +191,8 @@ class TalkingAttention(Mixer):
                 begin = np.maximum(0, first - self.window + 1) if self.window else np.zeros(n, dtype=np.int64)
                 if self.chunk:
                     begin = np.maximum(begin, first // self.chunk * self.chunk)
-                key_tiles = -(-(first + nq) // KEY_TILE) - begin // KEY_TILE
+                kept = np.minimum(-(-self.keep // KEY_TILE), begin // KEY_TILE)
+                key_tiles = -(-(first + nq) // KEY_TILE) - begin // KEY_TILE + kept
                 parts = np.clip(key_tiles // MIN_PART_TILES, 1, share)
             while int((parts * nq)[parts > 1].sum()) > PARTIAL_ROWS:
                 parts = np.maximum(1, parts // 2)
@@ -194,14 +206,19 @@ class TalkingAttention(Mixer):
     # ---------------------------------------------------------------- the step
     def forward(self, h, residual, ctx: StepContext, call: CallInfo):
         rt, T = self.runtime, ctx.n_tokens
+        proj = rt.get_scratch("talk_proj", torch.float32)[:, : self.in_cols]
+        out = rt.get_scratch("talk_out")[:, : self.o_in]
+        ops.linear(h, self.w_in, proj, T, status=ctx.status)
+        self.forward_rows(proj, out, ctx, call)
+        ops.linear(out, self.w_o, residual, T, accumulate=not ctx.store_output, status=ctx.status)
+
+    def forward_rows(self, proj, out, ctx: StepContext, call: CallInfo):
+        rt, T = self.runtime, ctx.n_tokens
         if not call.writes_cache:
             raise RuntimeError("talking_attention: every call owns its cache")
-        proj = rt.get_scratch("talk_proj", torch.float32)[:, : self.in_cols]
         q = rt.get_scratch("talk_q", torch.float32)[:, : self.q_cols]
         gate = rt.get_scratch("talk_gate", torch.float32)[0, : rt.max_batch_tokens * self.n_heads] \
             .view(rt.max_batch_tokens, self.n_heads) if self.has_gate else None
-        out = rt.get_scratch("talk_out")[:, : self.o_in]
-        ops.linear(h, self.w_in, proj, T, status=ctx.status)
         table = ctx.block_tables[call.cache_group]
         pos = self.position
         rot = getattr(pos, "cos_sin", None) if pos is not None else None
@@ -214,10 +231,11 @@ class TalkingAttention(Mixer):
             partial = rt.get_scratch("talk_partial", torch.float32) if plan["any_parts"] else None
             ops.talking_attention_mma(q, gate, call.cache, table, rt.page_size, ctx.q_start, ctx.kv_len, plan["work"],
                                       plan["n_work"], bool(plan["any_parts"]), self.talk, self.sink, out, partial, self.n_heads,
-                                      self.n_kv, self.dk, self.dv, self.window, plan["qt"], self.scale, ctx.status, chunk=self.chunk)
+                                      self.n_kv, self.dk, self.dv, self.window, plan["qt"], self.scale, ctx.status, chunk=self.chunk,
+                                      keep=self.keep, out_scale=self.out_scale)
         else:
             # a step of single tokens: a CTA's shared memory is sized for its one query
             ops.talking_attention(q, gate, call.cache, table, rt.page_size, ctx.q_start, ctx.kv_len, plan["work"],
                                   plan["n_work"], self.talk, self.sink, out, self.n_heads, self.n_kv, self.dk, self.dv,
-                                  self.window, plan["qt"], self.scale, ctx.status, chunk=self.chunk)
-        ops.linear(out, self.w_o, residual, T, accumulate=not ctx.store_output, status=ctx.status)
+                                  self.window, plan["qt"], self.scale, ctx.status, chunk=self.chunk, keep=self.keep,
+                                  out_scale=self.out_scale)
