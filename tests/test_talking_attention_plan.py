@@ -6,9 +6,9 @@ from rustingstrata_b200.parts import talking_attention as TA
 from rustingstrata_b200.parts.base import HostBatch
 
 
-def make_part(mma_q=16, window=0, chunk=0):
+def make_part(mma_q=16, window=0, chunk=0, keep=0):
     att = TA.TalkingAttention.__new__(TA.TalkingAttention)
-    att.q_per_cta, att.mma_q, att.window, att.chunk = 8, mma_q, window, chunk
+    att.q_per_cta, att.mma_q, att.window, att.chunk, att.keep = 8, mma_q, window, chunk, keep
     att.n_heads, att.n_kv, att.dk, att.dv = 16, 4, 64, 64
     return att
 
@@ -90,3 +90,12 @@ def test_blocks_of_positions_bound_the_keys_that_are_shared_out():
     by_seq = {s: w[w[:, 0] == s] for s in range(2)}
     assert len(by_seq[0]) == by_seq[0][0, 3] == 29 // TA.MIN_PART_TILES
     assert len(by_seq[1]) == 1 and by_seq[1][0, 3] == 1
+
+
+def test_kept_first_keys_count_in_the_walk():
+    """A window that keeps first keys: their tiles join the share-out as far as they lie before the window's."""
+    plain = rows_of(make_part(window=512).build_plan(batch([1], [4000])))
+    kept = rows_of(make_part(window=512, keep=300).build_plan(batch([1], [4000])))
+    assert plain[0, 3] == 17 // TA.MIN_PART_TILES and kept[0, 3] == (17 + 10) // TA.MIN_PART_TILES
+    near = rows_of(make_part(window=512, keep=300).build_plan(batch([1], [520])))
+    assert near[0, 3] == rows_of(make_part().build_plan(batch([1], [520])))[0, 3]       # the window still reaches the first keys
