@@ -95,8 +95,8 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=0, help="run this many of the configuration's layers (0 = all)")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--no-points", action="store_true", help="skip decode at batch 1 and 64")
-    ap.add_argument("--workload", default="headline", choices=["headline", "14b-mixed", "32b-long", "lokinex", "tabedra", "kupelix", "kozasun"])
-    ap.add_argument("--sizes", default="1024,2048", help="with --workload lokinex, tabedra, kupelix or kozasun: widths to run")
+    ap.add_argument("--workload", default="headline", choices=["headline", "14b-mixed", "32b-long", "lokinex", "tabedra", "kupelix", "kozasun", "sefelorn"])
+    ap.add_argument("--sizes", default="1024,2048", help="with --workload lokinex, tabedra, kupelix, kozasun or sefelorn: widths to run")
     ap.add_argument("--marginal", action="store_true", help="marginal cost of each kernel family inside the decode step")
     ap.add_argument("--prompt-len", type=int, default=PROMPT, help="with --marginal: tokens each request holds")
     ap.add_argument("--marginal-prefill", action="store_true",
@@ -121,7 +121,7 @@ def main() -> int:
         return long_context_workload(args)
     if args.workload == "lokinex":
         return lokinex_workload(args)
-    if args.workload in ("tabedra", "kupelix", "kozasun"):
+    if args.workload in ("tabedra", "kupelix", "kozasun", "sefelorn"):
         return lokinex_workload(args, design=args.workload)
 
     import numpy as np
@@ -444,6 +444,27 @@ def kozasun_config(width: int) -> dict:
                        dict(att, mlp=dense, weights_of=0), dict(ret, mlp=moe), dict(lat, mlp=dense), dict(lat, mlp=moe)]}
 
 
+SEFELORN_WINDOW = 1024
+
+
+def sefelorn_config(width: int) -> dict:
+    """A Sefelorn model whose layers resemble real ones at this width: attention heads of 128 query/key and 128 value
+    coordinates with one key/value head per four query heads, half of each head rotated, a window of 1,024 keys that keeps
+    the first 16 tokens, beside gated linear attention with as many heads of 128 + 128 and a low-rank map of 16; Mamba-2
+    with twice the width inside, heads of 64, states of 128 rows, one group, 4 taps; a gated feed-forward of 8/3 width (as
+    many weights as two matrices of 4 x width); four layers (parallel, Mamba-2, parallel, Mamba-2) run twice by the loop."""
+    heads = width // 128
+    par = {"type": "parallel", "mixer": {
+        "left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                 "rot": {"base": 1000000.0, "dims": 64}, "mask": {"size": SEFELORN_WINDOW, "keep_first": 16}},
+        "right": {"heads": heads, "dim": 128, "vdim": 128, "tau": 16.0, "decay_rank": 16}, "left_scale": 0.5, "right_scale": 0.5}}
+    mamba = {"type": "mamba2", "mixer": {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}}
+    dense = {"kind": "dense", "ff": width * 8 // 3 // 64 * 64, "limit": 7.0}
+    return {"architecture": "Sefelorn", "vocab": 32768, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "logit_scale": 1.0, "layers": [dict(par, mlp=dense), dict(mamba, mlp=dense), dict(par, mlp=dense), dict(mamba, mlp=dense)],
+            "loop": {"start": 0, "stop": 4, "times": 2}}
+
+
 def qwen3_windowed(width: int) -> dict:
     """The closest existing model for the Tabedra design: the Qwen3 decoder of :func:`qwen3_like` with the same sliding
     window on every layer and as many key/value heads."""
@@ -469,7 +490,7 @@ class OpTimer:
              "attention_decode_items", "silu_mul", "residual_add", "sample", "latent_expand", "embed_sum", "stream_layernorm",
              "stream_update", "router_topk", "conv_norm_kv_write", "sigmoid_gate", "talking_attention_prep", "talking_attention", "talking_attention_mma",
              "state_recurrence", "hgrn2_prep", "delta_prep", "head_norm_gate", "activation", "scale_rows", "retention_prep",
-             "head_sigmoid_gate")
+             "head_sigmoid_gate", "mamba2_prep", "low_rank_decay", "pad_heads", "gated_group_norm", "add_embed")
 
     def __init__(self):
         self.events, self.real = [], {}
@@ -523,12 +544,13 @@ def lokinex_workload(args, design: str = "lokinex") -> int:
     clocks = ClockSampler()
     clocks.start()
     pair = {"lokinex": (lokinex_config, qwen3_like), "tabedra": (tabedra_config, qwen3_windowed),
-            "kupelix": (kupelix_config, qwen3_like), "kozasun": (kozasun_config, kupelix_config)}[design]
+            "kupelix": (kupelix_config, qwen3_like), "kozasun": (kozasun_config, kupelix_config),
+            "sefelorn": (sefelorn_config, kupelix_config)}[design]
     out = {"workload": design, "prompt_len": PROMPT, "batch": args.batch, "steps": args.steps, "dtype": "bf16",
            "data": "synthetic", "weights": "random N(0,0.02) bf16", "peaks": pk["source"], "sizes": {}}
     for width in [int(x) for x in args.sizes.split(",")]:
         rec = {}
-        other = "kupelix" if design == "kozasun" else "qwen3"        # the closest existing model of the design
+        other = "kupelix" if design in ("kozasun", "sefelorn") else "qwen3"        # the closest existing model of the design
         for name, cfg in ((design, pair[0](width)), (other, pair[1](width))):
             V = cfg.get("vocab", cfg.get("vocab_size"))
             eng = Engine(cfg, dtype="bfloat16", random_seed=0, page_size=16, max_tokens=args.batch * CONTEXT,

@@ -215,38 +215,43 @@ def test_mixed_batches_with_pages_and_slots_used_again(tmp_path_factory, name, d
 
 
 # ----------------------------------------------------------------------------- edges of windows and kept first tokens
+EDGE_TOL = {"float32": 1.5e-4, "bfloat16": 2e-2}   # root mean square over the vocabulary, over that of the reference
+
+
+def row_rms(d):
+    d = d - d.mean(axis=1, keepdims=True)
+    return np.sqrt((d * d).mean(axis=1))
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name", ["P", "R", "S"])
 def test_edges_of_windows_and_kept_tokens(tmp_path_factory, name, dtype):
     """Peaked attention, so that a key more or a key less shows.  The premise first, on the plain implementation: with
-    every window one key larger or smaller, or one first token more or less kept, the logits of many positions move by
-    more than three times the tolerance.  Then the engine: the prompt whole, a short prompt followed by single tokens that
-    pass every window's edge and the kept tokens' edge, and portions that start and end on and beside them."""
+    every window one key larger or smaller, or one first token more or less kept, the logits of several positions move by
+    more than twice the tolerance.  Then the engine: the prompt whole, a short prompt followed by single tokens that pass
+    every window's edge and the kept tokens' edge, and portions that start and end on and beside them."""
     path, cfg, w = model(tmp_path_factory, name + "_sharp", name, seed=21, sharp=SHARP[dtype])
-    tol = TOL_SHARP[dtype]
+    tol = EDGE_TOL[dtype]
     n = {"P": 150, "R": 330, "S": 120}[name]
     toks = tokens_for(cfg, n, 31)
     ref = plain_logits(cfg, w, toks)
-    scale = np.max(np.abs(ref))
+    scale = row_rms(ref).mean()
     for size, keep in ((1, 0), (-1, 0), (0, 1), (0, -1)):
         if size < 0 and any(L["mixer"]["left"]["mask"]["size"] == 1 for L in cfg["layers"] if L["type"] == "parallel"):
             continue
-        moved = np.max(np.abs(plain_logits(M.with_masks(cfg, size, keep), w, toks) - ref), axis=1) / scale
-        assert (moved > 3 * tol).sum() >= 5, f"premise: windows {size:+d}, kept {keep:+d}"
+        moved = row_rms(plain_logits(M.with_masks(cfg, size, keep), w, toks) - ref) / scale
+        assert (moved > 2 * tol).sum() >= 5, f"premise: windows {size:+d}, kept {keep:+d}"
     r = runner_for(path, dtype, page_size=16, pool_tokens=512, max_batch_tokens=512)
-    err = np.max(np.abs(step_all(r, "w", toks) - ref), axis=1) / scale
-    assert_rows_within(err, tol, "whole")
+    assert_rows_within(row_rms(step_all(r, "w", toks) - ref) / scale, tol, "whole")
     r.release("w")
     got = [step_all(r, "d", toks[:3])] + [step_all(r, "d", [t]) for t in toks[3:]]
-    err = np.max(np.abs(np.concatenate(got) - ref), axis=1) / scale
-    assert_rows_within(err, tol, "decoding")
+    assert_rows_within(row_rms(np.concatenate(got) - ref) / scale, tol, "decoding")
     r.release("d")
     edges = {p + d for L in cfg["layers"] if L["type"] == "parallel" for e in L["mixer"]["left"]["mask"].values()
              for p in range(e, n, max(e, 16)) for d in (-1, 0, 1)}
     marks = sorted({0, n} | {p for p in edges if 0 < p < n})
     got = [step_all(r, "p", toks[a:b]) for a, b in zip(marks[:-1], marks[1:])]
-    err = np.max(np.abs(np.concatenate(got) - ref), axis=1) / scale
-    assert_rows_within(err, tol, "portions cut at the edges")
+    assert_rows_within(row_rms(np.concatenate(got) - ref) / scale, tol, "portions cut at the edges")
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
