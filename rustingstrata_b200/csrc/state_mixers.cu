@@ -396,6 +396,7 @@ struct Mamba2PrepParams {
     float* dt; float* decay;                  // [T, heads]
     const int* seq_of_token; const int* q_start; const int* slots;
     int C, taps, heads, conv_off, dt_off, n_tokens;
+    int log_decay;                            // decay holds -exp(a_log) dt instead of its exponential
 };
 
 // V neighbouring channels of one token per thread (V = 4: 16-byte accesses), then one thread per (token, head).
@@ -410,7 +411,8 @@ __global__ void __launch_bounds__(256) mamba2_prep_kernel(Mamba2PrepParams p) {
         const int t = (int)(i / p.heads), h = (int)(i % p.heads);
         const float step = softplus_f(p.proj[(size_t)t * p.proj_stride + p.dt_off + h] + p.dt_bias[h]);
         p.dt[i] = step;
-        p.decay[i] = expf(-expf(p.a_log[h]) * step);
+        const float log_d = -expf(p.a_log[h]) * step;
+        p.decay[i] = p.log_decay ? log_d : expf(log_d);
         return;
     }
     const int t = (int)(idx / groups), c = (int)(idx % groups) * V;
@@ -438,11 +440,12 @@ __global__ void __launch_bounds__(256) mamba2_prep_kernel(Mamba2PrepParams p) {
 
 // ------------------------------------------------------------------------------------------------ decay of a low-rank map
 // g[t, h * rows + i] = sigmoid(z)^(1 / tau) = exp(log sigmoid(z) / tau), z = sum_r w[h * dim + i, r] u[t, r] + bias: a
-// thread per channel and DECAY_TOKENS tokens, whose u rows lie in shared memory.  Rows beyond dim are zero.
+// thread per channel and DECAY_TOKENS tokens, whose u rows lie in shared memory.  Rows beyond dim are zero.  log_decay:
+// g holds the exponent itself.
 constexpr int DECAY_TOKENS = 16;
 __global__ void __launch_bounds__(256) low_rank_decay_kernel(const float* u, long u_stride, const void* w, int w_dt, const float* bias,
                                                              float inv_tau, float* g, long g_stride, int heads, int dim, int rows,
-                                                             int rank, int n_tokens) {
+                                                             int rank, int n_tokens, int log_decay) {
     extern __shared__ __align__(16) float us[];                  // [DECAY_TOKENS][rank]
     const int t0 = blockIdx.y * DECAY_TOKENS, nt = min(DECAY_TOKENS, n_tokens - t0);
     for (int i = threadIdx.x; i < nt * rank; i += blockDim.x) us[i] = u[(size_t)(t0 + i / rank) * u_stride + i % rank];
@@ -469,7 +472,7 @@ __global__ void __launch_bounds__(256) low_rank_decay_kernel(const float* u, lon
         if (e < nt) {
             const float z = acc[e];
             const float log_sig = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
-            g[(size_t)(t0 + e) * g_stride + c] = live ? expf(log_sig * inv_tau) : 0.f;
+            g[(size_t)(t0 + e) * g_stride + c] = !live ? 0.f : log_decay ? log_sig * inv_tau : expf(log_sig * inv_tau);
         }
 }
 
@@ -724,11 +727,11 @@ RS_EXPORT int rs_delta_prep(const float* proj, long proj_stride, const void* con
 RS_EXPORT int rs_mamba2_prep(const float* proj, long proj_stride, int conv_off, int dt_off, const float* conv, const float* bias,
                              float* tail, long tail_stride, const float* dt_bias, const float* a_log, float* out, long out_stride,
                              float* dt, float* decay, const int* seq_of_token, const int* q_start, const int* slots, int channels,
-                             int taps, int heads, int n_tokens, int n_seqs, cudaStream_t stream) {
+                             int taps, int heads, int log_decay, int n_tokens, int n_seqs, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (taps < 1 || channels < 1 || heads < 1 || (taps > 1 && !tail)) return (int)cudaErrorInvalidValue;
     Mamba2PrepParams p{proj, proj_stride, conv, bias, tail, tail_stride, dt_bias, a_log, out, out_stride, dt, decay, seq_of_token,
-                       q_start, slots, channels, taps, heads, conv_off, dt_off, n_tokens};
+                       q_start, slots, channels, taps, heads, conv_off, dt_off, n_tokens, log_decay};
     const bool vec = channels % 4 == 0 && conv_off % 4 == 0 && proj_stride % 4 == 0 && out_stride % 4 == 0 &&
                      (((uintptr_t)proj | (uintptr_t)conv | (uintptr_t)out) & 15) == 0 &&
                      (!tail || (tail_stride % 4 == 0 && ((uintptr_t)tail & 15) == 0));
@@ -745,12 +748,13 @@ RS_EXPORT int rs_mamba2_prep(const float* proj, long proj_stride, int conv_off, 
 }
 
 RS_EXPORT int rs_low_rank_decay(const float* u, long u_stride, const void* w, int w_dt, const float* bias, float inv_tau, float* g,
-                                long g_stride, int heads, int dim, int rows, int rank, int n_tokens, cudaStream_t stream) {
+                                long g_stride, int heads, int dim, int rows, int rank, int log_decay, int n_tokens,
+                                cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (rank < 1 || rank > 512 || rows < dim) return (int)cudaErrorInvalidValue;
     const dim3 grid((unsigned)((heads * rows + 255) / 256), (unsigned)((n_tokens + DECAY_TOKENS - 1) / DECAY_TOKENS));
     low_rank_decay_kernel<<<grid, 256, DECAY_TOKENS * rank * sizeof(float), stream>>>(u, u_stride, w, w_dt, bias, inv_tau, g, g_stride,
-                                                                                      heads, dim, rows, rank, n_tokens);
+                                                                                      heads, dim, rows, rank, n_tokens, log_decay);
     return rs_launch_result();
 }
 

@@ -1602,10 +1602,12 @@ def mixerslib():
         lib.rs_state_recurrence.argtypes = [c_void_p, c_long] * 7 + [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                                      c_int, c_float, c_void_p, c_void_p]
         lib.rs_mamba2_prep.argtypes = [c_void_p, c_long, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p,
-                                       c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                       c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                        c_void_p]
+        lib.rs_state_chunks_supported.argtypes = [c_int, c_int, c_int]
+        lib.rs_state_recurrence_chunked.argtypes = [c_void_p, c_long] * 7 + [c_void_p] * 7 + [c_int] * 8 + [c_float, c_void_p, c_void_p]
         lib.rs_low_rank_decay.argtypes = [c_void_p, c_long, c_void_p, c_int, c_void_p, c_float, c_void_p, c_long, c_int, c_int, c_int,
-                                          c_int, c_int, c_void_p]
+                                          c_int, c_int, c_int, c_void_p]
         lib.rs_pad_heads.argtypes = [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.rs_gated_group_norm.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_int, c_long, c_int, c_int,
                                             c_float, c_int, c_void_p]
@@ -1691,14 +1693,59 @@ def state_recurrence(q: torch.Tensor, k: torch.Tensor, g: torch.Tensor, beta: Op
         "state_recurrence")
 
 
+STATE_CHUNK = 64               # tokens per chunk of the chunked recurrence
+
+
+def state_chunks_supported(rows_pad: int, columns: int, head_decay: bool) -> bool:
+    """Whether :func:`state_recurrence_chunked` takes heads of these sizes."""
+    return bool(mixerslib().rs_state_chunks_supported(2 if head_decay else 0, rows_pad, columns))
+
+
+def state_recurrence_chunked(q: torch.Tensor, k: torch.Tensor, g: torch.Tensor, beta: Optional[torch.Tensor], v: torch.Tensor,
+                             out: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, n_seqs: int, heads: int,
+                             group: int, rows_pad: int, columns: int, chunk_seq: torch.Tensor, chunk_start: torch.Tensor,
+                             seq_first_chunk: torch.Tensor, n_chunks: int, work: torch.Tensor, head_decay: bool = False,
+                             rows: Optional[int] = None, q_scale: float = 1.0, skip: Optional[torch.Tensor] = None) -> None:
+    """:func:`state_recurrence` (gated write or ``head_decay``) in chunks of STATE_CHUNK tokens on the tensor cores
+    (csrc/state_chunks.cu), with ``g`` the LOGARITHM of the decays.  chunk_seq, chunk_start [n_chunks]: sequence and first
+    token within its portion; seq_first_chunk [n_seqs + 1]; ``work``: float32 workspace of n_chunks * heads * (columns + 1) *
+    rows_pad values."""
+    _cuda(q, k, g, beta, v, out, state, q_start, slots, skip, chunk_seq, chunk_start, seq_first_chunk, work)
+    _f32_rows("state_recurrence_chunked", q=q, k=k, g=g, beta=beta, v=v, out=out, state=state)
+    _i32("state_recurrence_chunked", q_start, slots, chunk_seq, chunk_start, seq_first_chunk)
+    rows = rows_pad if rows is None else int(rows)
+    if head_decay and beta is None:
+        raise KernelError("state_recurrence_chunked: the decay per head needs a write strength per head")
+    if skip is not None and (not head_decay or skip.dtype != torch.float32 or skip.numel() != heads):
+        raise KernelError("state_recurrence_chunked: skip belongs to the decay per head, float32 [heads]")
+    qk_heads = heads // group
+    if heads % group or rows % 4 or not 4 <= rows <= rows_pad or q.shape[1] < qk_heads * rows or k.shape[1] < qk_heads * rows \
+            or g.shape[1] < heads * (1 if head_decay else rows) or v.shape[1] < heads * columns or out.shape[1] < heads * columns \
+            or state.shape[1] < heads * columns * rows_pad:
+        raise KernelError("state_recurrence_chunked: an operand is narrower than heads x rows / columns ask for")
+    for name, t in (("q", q), ("k", k), ("state", state)) + (() if head_decay else (("g", g),)):
+        if t.stride(0) % 4 or t.data_ptr() % 16:
+            raise KernelError(f"state_recurrence_chunked: {name} must start on 16 bytes with a row pitch that is a multiple of 4")
+    n_sums = n_chunks * heads * columns * rows_pad
+    if work.dtype != torch.float32 or not work.is_contiguous() or work.numel() < n_sums + n_chunks * heads * rows_pad \
+            or chunk_seq.numel() < n_chunks or chunk_start.numel() < n_chunks or seq_first_chunk.numel() < n_seqs + 1:
+        raise KernelError("state_recurrence_chunked: workspace or chunk lists are too small")
+    flat = work.view(-1)
+    _check(mixerslib().rs_state_recurrence_chunked(
+        _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(g), g.stride(0), _ptr(beta), 0 if beta is None else beta.stride(0),
+        _ptr(v), v.stride(0), _ptr(out), out.stride(0), _ptr(state), state.stride(0), _ptr(q_start), _ptr(slots), _ptr(chunk_seq),
+        _ptr(chunk_start), _ptr(seq_first_chunk), _ptr(flat), _ptr(flat[n_sums:]), n_chunks, n_seqs, heads, group, rows, rows_pad,
+        columns, 2 if head_decay else 0, float(q_scale), _ptr(skip), _stream()), "state_recurrence_chunked", 3)
+
+
 def mamba2_prep(proj: torch.Tensor, conv_off: int, dt_off: int, conv: torch.Tensor, bias: Optional[torch.Tensor],
                 tail: Optional[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor, out: torch.Tensor, dt: torch.Tensor,
                 decay: torch.Tensor, seq_of_token: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, heads: int,
-                n_tokens: int, n_seqs: int) -> None:
+                n_tokens: int, n_seqs: int, log_decay: bool = False) -> None:
     """From proj (float32): the channels from ``conv_off`` on pass a causal convolution over time (``conv`` [taps, C]
     tap-major, ``bias`` [C]; ``tail`` [slots, >= (taps - 1) * C] holds every request's last inputs and is updated) and silu
-    into ``out`` [T, C]; dt = softplus(. + dt_bias) of the columns from ``dt_off`` on and decay = exp(-exp(a_log) dt), both
-    [T, heads] contiguous."""
+    into ``out`` [T, C]; dt = softplus(. + dt_bias) of the columns from ``dt_off`` on and decay = exp(-exp(a_log) dt)
+    (``log_decay``: that exponent), both [T, heads] contiguous."""
     _cuda(proj, conv, bias, tail, dt_bias, a_log, out, dt, decay, seq_of_token, q_start, slots)
     _f32_rows("mamba2_prep", proj=proj, conv=conv, tail=tail, out=out, dt=dt, decay=decay)
     _i32("mamba2_prep", seq_of_token, q_start, slots)
@@ -1713,12 +1760,13 @@ def mamba2_prep(proj: torch.Tensor, conv_off: int, dt_off: int, conv: torch.Tens
     _check(mixerslib().rs_mamba2_prep(
         _ptr(proj), proj.stride(0), conv_off, dt_off, _ptr(conv), _ptr(bias), _ptr(tail), 0 if tail is None else tail.stride(0),
         _ptr(dt_bias), _ptr(a_log), _ptr(out), out.stride(0), _ptr(dt), _ptr(decay), _ptr(seq_of_token), _ptr(q_start), _ptr(slots),
-        C, taps, heads, n_tokens, n_seqs, _stream()), "mamba2_prep", 2 if taps > 1 else 1)
+        C, taps, heads, 1 if log_decay else 0, n_tokens, n_seqs, _stream()), "mamba2_prep", 2 if taps > 1 else 1)
 
 
 def low_rank_decay(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], tau: float, g: torch.Tensor, heads: int,
-                   dim: int, rows: int, n_tokens: int) -> None:
-    """g[t, h * rows + i] = sigmoid(z)^(1 / tau), z = (weight u_t + bias)[h * dim + i], zero for dim <= i < rows; u float32
+                   dim: int, rows: int, n_tokens: int, log_decay: bool = False) -> None:
+    """g[t, h * rows + i] = sigmoid(z)^(1 / tau), z = (weight u_t + bias)[h * dim + i] (``log_decay``: its logarithm), zero
+    for dim <= i < rows; u float32
     [T, rank], weight [heads * dim, rank], float32 arithmetic."""
     _cuda(u, weight, bias, g)
     _f32_rows("low_rank_decay", u=u, g=g)
@@ -1726,7 +1774,8 @@ def low_rank_decay(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.T
             or rows < dim or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != heads * dim)):
         raise KernelError("low_rank_decay: shapes do not fit heads x dim")
     _check(mixerslib().rs_low_rank_decay(_ptr(u), u.stride(0), _ptr(weight), dtype_code(weight), _ptr(bias), 1.0 / float(tau), _ptr(g),
-                                         g.stride(0), heads, dim, rows, weight.shape[1], n_tokens, _stream()), "low_rank_decay")
+                                         g.stride(0), heads, dim, rows, weight.shape[1], 1 if log_decay else 0, n_tokens, _stream()),
+           "low_rank_decay")
 
 
 def pad_heads(src: torch.Tensor, dst: torch.Tensor, heads: int, dim: int, rows: int, n_tokens: int) -> None:

@@ -53,10 +53,11 @@ state and the recurrence are float32 in both engines.
 """
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from ..kernels import ops
-from .base import CallInfo, Mixer, StepContext
+from .base import CallInfo, HostBatch, Mixer, StepContext
 from .registry import register_part
 from .spec import StateNeed, TensorNeed
 
@@ -308,13 +309,51 @@ class Retention(Mixer):
         ops.linear(out, self.w_o, residual, T, accumulate=not ctx.store_output, status=ctx.status)
 
 
+CHUNKED_FROM = 32      # the longest portion of a step from which on the bfloat16 engine walks it in chunks
+
+
+class ChunkedRecurrence(Mixer):
+    """What mixers share whose recurrence the chunked kernels take (csrc/state_chunks.cu): the step's list of chunks and the
+    workspace.  The 32-bit engine, captured steps and steps of short portions walk token by token."""
+
+    def _chunk_setup(self, n_heads: int, rows_pad: int, columns: int, head_decay: bool) -> None:
+        rt = self.runtime
+        self.chunks_ok = not rt.precise
+        self._chunk_shape = (rows_pad, columns, head_decay)
+        if self.chunks_ok:
+            most = rt.max_batch_tokens // ops.STATE_CHUNK + rt.max_seqs
+            rt.scratch("state_chunks", 1, most * n_heads * (columns + 1) * rows_pad, torch.float32)
+
+    def plan_key(self):
+        return ("state_chunks", ops.STATE_CHUNK) if self.chunks_ok else None
+
+    def build_plan(self, batch: HostBatch):
+        if batch.bucketed or int(batch.q_lens.max()) < CHUNKED_FROM:
+            return {"n_chunks": 0}
+        per_seq = -(-batch.q_lens // ops.STATE_CHUNK)
+        first = np.zeros(batch.n_seqs + 1, np.int32)
+        np.cumsum(per_seq, out=first[1:])
+        seq = np.repeat(np.arange(batch.n_seqs, dtype=np.int32), per_seq)
+        start = (np.arange(int(first[-1]), dtype=np.int32) - np.repeat(first[:-1], per_seq)) * ops.STATE_CHUNK
+        return {"chunk_seq": seq, "chunk_start": start.astype(np.int32), "seq_first_chunk": first, "n_chunks": int(first[-1])}
+
+    def _chunks(self, ctx: StepContext):
+        """The step's chunk lists as keywords of ``ops.state_recurrence_chunked``, or None: token by token."""
+        if not self.chunks_ok:
+            return None
+        plan = ctx.plans[self.plan_key()]
+        if not plan["n_chunks"] or not ops.state_chunks_supported(*self._chunk_shape):
+            return None
+        return dict(plan, work=self.runtime.get_scratch("state_chunks", torch.float32))
+
+
 def _on_16_bytes(dim: int, *ts) -> bool:
     """Whether every head of ``dim`` values in these float32 rows starts on 16 bytes (the recurrence can read them in place)."""
     return dim % 4 == 0 and all(t.stride(0) % 4 == 0 and t.data_ptr() % 16 == 0 for t in ts)
 
 
 @register_part("mixer", "gated_linear_attention")
-class GatedLinearAttention(Mixer):
+class GatedLinearAttention(ChunkedRecurrence):
     """params: hidden, n_heads, dim, vdim, tau, decay_rank (inner width of the decay's low-rank map), eps (of the read-out
     norm), q_scale (default dim^-1/2), out_scale (default 1: multiplies the mixer's output).
     tensors: q_proj, k_proj, v_proj, g_proj [heads * vdim, hidden], a1_proj [decay_rank, hidden], a2_proj [heads * dim,
@@ -345,6 +384,7 @@ class GatedLinearAttention(Mixer):
         rt.scratch("state_rows", 1, 3 * rt.max_batch_tokens * self.n_heads * self.rows_pad, torch.float32)
         rt.scratch("state_read", rt.max_batch_tokens, self.v_cols, torch.float32)
         rt.scratch("state_out", rt.max_batch_tokens, self.v_cols)
+        self._chunk_setup(self.n_heads, self.rows_pad, self.dv, False)
 
     def tensor_needs(self):
         t, D = self.spec.tensors, self.hidden
@@ -393,14 +433,17 @@ class GatedLinearAttention(Mixer):
             ops.pad_heads(k, k_buf, H, self.dk, RP, T)
             q, k, rows = q_buf, k_buf, RP
         g = flat[2 * n: 2 * n + mbt * H * rows].view(mbt, H * rows)
-        ops.low_rank_decay(proj[:, self.a1_off: self.a1_off + self.rank], self.w_a2, self.a2_bias, self.tau, g, H, self.dk, rows, T)
-        ops.state_recurrence(q, k, g, None, proj[:, self.v_off: self.g_off], read, call.state, ctx.q_start, ctx.state_slots,
-                             ctx.n_seqs, H, 1, RP, self.dv, rows=rows, q_scale=self.q_scale)
+        chunks = self._chunks(ctx)
+        ops.low_rank_decay(proj[:, self.a1_off: self.a1_off + self.rank], self.w_a2, self.a2_bias, self.tau, g, H, self.dk, rows, T,
+                           log_decay=chunks is not None)
+        walk = ops.state_recurrence if chunks is None else ops.state_recurrence_chunked
+        walk(q, k, g, None, proj[:, self.v_off: self.g_off], read, call.state, ctx.q_start, ctx.state_slots, ctx.n_seqs, H, 1, RP,
+             self.dv, rows=rows, q_scale=self.q_scale, **(chunks or {}))
         ops.head_norm_gate(read, self.norm_w, proj[:, self.g_off: self.a1_off], out, H, self.dv, self.eps, T, gate_silu=True)
 
 
 @register_part("mixer", "mamba2")
-class Mamba2(Mixer):
+class Mamba2(ChunkedRecurrence):
     """params: hidden, n_heads, vdim, state (rows of a head's state), groups (of B and C), taps, norm_groups, eps (of the
     read-out norm), out_scale (default 1: multiplies the mixer's output).
     tensors: in_proj [2 * inner + 2 * groups * state + heads, hidden], conv [inner + 2 * groups * state, taps], conv_bias,
@@ -437,6 +480,7 @@ class Mamba2(Mixer):
             rt.scratch("state_rows", 1, 2 * mbt * self.groups * self.rows_pad, torch.float32)
         rt.scratch("state_read", mbt, self.inner, torch.float32)
         rt.scratch("state_out", mbt, self.inner)
+        self._chunk_setup(self.n_heads, self.rows_pad, self.dv, True)
 
     def tensor_needs(self):
         t, D, H = self.spec.tensors, self.hidden, self.n_heads
@@ -475,9 +519,10 @@ class Mamba2(Mixer):
         flat = rt.get_scratch("mamba_step", torch.float32)[0]
         dt, decay = flat[: mbt * H].view(mbt, H), flat[mbt * H: 2 * mbt * H].view(mbt, H)
         read = rt.get_scratch("state_read", torch.float32)[:, : self.inner]
-        state = call.state
+        state, chunks = call.state, self._chunks(ctx)
         ops.mamba2_prep(proj, self.inner, self.dt_off, self.w_conv, self.conv_bias, state[:, self.state_cols:] if self.tail else None,
-                        self.dt_bias, self.a_log, conv, dt, decay, ctx.seq_of_token, ctx.q_start, ctx.state_slots, H, T, ctx.n_seqs)
+                        self.dt_bias, self.a_log, conv, dt, decay, ctx.seq_of_token, ctx.q_start, ctx.state_slots, H, T, ctx.n_seqs,
+                        log_decay=chunks is not None)
         k, q, rows = conv[:, self.inner: self.inner + self.bc_cols], conv[:, self.inner + self.bc_cols:], self.rows
         if not _on_16_bytes(self.rows, k, q):
             n = mbt * G * RP
@@ -486,6 +531,7 @@ class Mamba2(Mixer):
             ops.pad_heads(k, k_buf, G, self.rows, RP, T)
             ops.pad_heads(q, q_buf, G, self.rows, RP, T)
             k, q, rows = k_buf, q_buf, RP
-        ops.state_recurrence(q, k, decay, dt, conv[:, : self.inner], read, state, ctx.q_start, ctx.state_slots, ctx.n_seqs, H, H // G,
-                             RP, self.dv, head_decay=True, rows=rows, skip=self.d_skip)
+        walk = ops.state_recurrence if chunks is None else ops.state_recurrence_chunked
+        walk(q, k, decay, dt, conv[:, : self.inner], read, state, ctx.q_start, ctx.state_slots, ctx.n_seqs, H, H // G, RP, self.dv,
+             head_decay=True, rows=rows, skip=self.d_skip, **(chunks or {}))
         ops.gated_group_norm(read, proj[:, : self.inner], self.norm_w, out, self.norm_groups, self.eps, T)

@@ -80,3 +80,76 @@ def test_recurrence(case, delta):
     got = state.cpu().double().view(n + 3, heads, cols, rp)
     assert (got - ref_state).abs().max().item() <= 2e-5 * ref_state.abs().max().item()
     assert (got[..., rows:] == 0).all()
+
+
+# ----------------------------------------------------------------------------- the chunked form
+def reference_walk(q, k, log_g, beta, v, S, skip, head_decay, q_scale):
+    """float64: q, k [T, H, rows], log_g [T, H, rows] or [T, H], beta [T, H] or None, v [T, H, cols], S [H, rows, cols]."""
+    out = torch.zeros_like(v)
+    for t in range(q.shape[0]):
+        d = torch.exp(log_g[t])
+        d = d[:, None, None] if head_decay else d[:, :, None]
+        kv = k[t][:, :, None] * v[t][:, None, :]
+        S = d * S + (kv if beta is None else beta[t][:, None, None] * kv)
+        out[t] = q_scale * torch.einsum("hij,hi->hj", S, q[t])
+        if skip is not None:
+            out[t] += skip[:, None] * v[t]
+    return out, S
+
+
+@pytest.mark.parametrize("strength", [0.02, 1.0, 30.0])
+@pytest.mark.parametrize("form", ["rows", "head"])
+@pytest.mark.parametrize("shape", [(4, 2, 24, 16), (2, 1, 64, 40), (6, 3, 100, 64), (2, 2, 128, 128), (1, 1, 48, 264), (8, 8, 32, 8)])
+def test_chunked_recurrence_against_float64(shape, form, strength):
+    """Chunks of 64 tokens on the tensor cores against the walk in float64: sequences of 1 to 200 tokens in one step, states
+    that are not zero at the start, slots in another order, decays from next to none (the state lasts for the whole
+    sequence) to strong ones (factors that underflow), head sizes that need padding, several heads per key."""
+    from rustingstrata_b200.kernels import ops
+    H, group, rows, cols = shape
+    head_decay = form == "head"
+    if not head_decay:
+        group = 1
+    gen = torch.Generator().manual_seed(rows * cols)
+    lens = [130, 1, 64, 200, 17, 65]
+    T, S = sum(lens), len(lens)
+    RP = ops.state_rows_pad(rows)
+    G = H // group
+    rnd = lambda *s: torch.randn(*s, generator=gen)                           # noqa: E731
+    q, k, v = rnd(T, G, rows), rnd(T, G, rows), rnd(T, H, cols)
+    log_g = -strength * torch.rand(*((T, H) if head_decay else (T, H, rows)), generator=gen) ** 3
+    beta = torch.rand(T, H, generator=gen) + 0.2 if head_decay else None
+    skip = rnd(H) if head_decay else None
+    state = torch.zeros(S + 2, H, cols, RP)
+    state[:, :, :, :rows] = rnd(S + 2, H, cols, rows)
+    slots = torch.tensor([5, 0, 3, 7, 2, 1], dtype=torch.int32)
+    starts = np.concatenate([[0], np.cumsum(lens)]).astype(np.int32)
+    per = [-(-n // ops.STATE_CHUNK) for n in lens]
+    first = np.concatenate([[0], np.cumsum(per)]).astype(np.int32)
+    seq = np.repeat(np.arange(S), per).astype(np.int32)
+    start = np.concatenate([np.arange(n) * ops.STATE_CHUNK for n in per]).astype(np.int32)
+    cu = lambda a: torch.from_numpy(a).cuda() if isinstance(a, np.ndarray) else a.cuda()        # noqa: E731
+    dev_state = state.reshape(S + 2, -1).clone().cuda()
+    out = torch.full((T, H * cols), 9.0, device="cuda")
+    n_chunks = int(first[-1])
+    work = torch.full((n_chunks * H * (cols + 1) * RP,), float("nan"), device="cuda")
+    q2, k2 = q.reshape(T, -1).contiguous(), k.reshape(T, -1).contiguous()
+    if not ops.state_chunks_supported(RP, cols, head_decay):
+        pytest.skip("not a shape of the chunked form")
+    ops.state_recurrence_chunked(cu(q2), cu(k2), cu(log_g.reshape(T, -1).contiguous()), None if beta is None else cu(beta),
+                                 cu(v.reshape(T, -1).contiguous()), out, dev_state, cu(starts), cu(slots), S, H, group, RP, cols,
+                                 cu(seq), cu(start), cu(first), n_chunks, work, head_decay=head_decay, rows=rows, q_scale=0.25,
+                                 skip=None if skip is None else cu(skip))
+    f64 = lambda x: None if x is None else x.double()                         # noqa: E731
+    qh, kh = q.repeat_interleave(group, dim=1).double(), k.repeat_interleave(group, dim=1).double()
+    got, new = out.cpu().double().view(T, H, cols), dev_state.cpu().double().view(S + 2, H, cols, RP)
+    for s in range(S):
+        a, b = int(starts[s]), int(starts[s + 1])
+        S0 = state[int(slots[s])].double()[:, :, :rows].transpose(1, 2)
+        want, S1 = reference_walk(qh[a:b], kh[a:b], log_g[a:b].double(), f64(beta)[a:b] if head_decay else None, v[a:b].double(),
+                                  S0, f64(skip), head_decay, 0.25)
+        scale = want.abs().max()
+        assert (got[a:b] - want).abs().max() <= 1e-5 * scale, f"sequence {s}"
+        assert (new[int(slots[s])][:, :, :rows].transpose(1, 2) - S1).abs().max() <= 1e-5 * max(1.0, float(S1.abs().max())), f"state {s}"
+        assert (new[int(slots[s])][:, :, rows:] == 0).all()
+    for s in set(range(S + 2)) - set(slots.tolist()):
+        assert torch.equal(dev_state.cpu().view(S + 2, -1)[s], state.reshape(S + 2, -1)[s])
