@@ -16,12 +16,12 @@
 
 namespace {
 constexpr int CHUNK = 64;
-constexpr int COLS = 128;                 // columns a CTA takes: of one head, or of HP whole heads that share q and k
+constexpr int COLS = 128;                 // columns a CTA takes: of one head, or of two whole heads that share q and k
 constexpr int BLOCK = 16;
 constexpr int VP = COLS + 8;              // pitch of the staged values: fragment reads without bank conflicts
 constexpr int AP = CHUNK + 4;             // pitch of the chunk's token x token matrix
 constexpr float LOG2E = 1.4426950408889634f;
-constexpr int MAX_HP = COLS / 8;
+constexpr int MAX_HP = 2;
 
 enum Form : int { GATED = 0, HEAD = 2 };  // the codes of rs_state_recurrence
 
@@ -44,8 +44,8 @@ struct ChunkParams {
 __device__ __forceinline__ float exp_of(float x) { return fast_exp2(x * LOG2E); }
 
 __device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(lo) : "f"(x - __uint_as_float(hi)));
+    hi = __float_as_uint(x) & 0xffffe000u;                   // the leading 10 bits of the mantissa, then the next ones
+    lo = __float_as_uint(x - __uint_as_float(hi)) & 0xffffe000u;
 }
 __device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -85,41 +85,42 @@ __device__ __forceinline__ Place place_of(const ChunkParams& p) {
     c.ncols = p.hp > 1 ? p.hp * p.columns : min(COLS, p.columns - c.col0);
     return c;
 }
-// head (within the CTA's) and column of a staged column
-__device__ __forceinline__ int head_of(const ChunkParams& p, int cc) { return p.hp > 1 ? cc / p.columns : 0; }
-__device__ __forceinline__ int column_of(const ChunkParams& p, const Place& c, int cc) { return p.hp > 1 ? cc % p.columns : c.col0 + cc; }
+// Staged column cc is column (first_column + cc) of the row that all heads' columns make; which of the CTA's heads it is of:
+__device__ __forceinline__ size_t first_column(const ChunkParams& p, const Place& c) { return (size_t)c.h0 * p.columns + c.col0; }
+__device__ __forceinline__ int head_of(const ChunkParams& p, int cc) { return p.hp > 1 && cc >= p.columns ? 1 : 0; }
 
-// values of the CTA's columns, zero beyond the chunk's tokens and the columns, times scale[head][token] if given
+// values of the CTA's columns, zero beyond the chunk's tokens and the columns (asynchronous copies where rows are aligned)
 template <int THREADS>
-__device__ __forceinline__ void stage_values(const ChunkParams& p, const Place& c, float* Vs, const float (*scale)[CHUNK]) {
+__device__ __forceinline__ void stage_values(const ChunkParams& p, const Place& c, float* Vs) {
     const float* v = p.v + (size_t)c.t0 * p.v_stride + (size_t)c.h0 * p.columns + c.col0;
+    const bool aligned = ((uintptr_t)v & 15) == 0 && p.v_stride % 4 == 0;
+#pragma unroll 4
     for (int i = threadIdx.x; i < CHUNK * (COLS / 4); i += THREADS) {
         const int j = i / (COLS / 4), cc = (i % (COLS / 4)) * 4;
-        float x[4];
         const float* src = v + (size_t)j * p.v_stride + cc;
-        if (j < c.nt && cc + 3 < c.ncols && ((uintptr_t)src & 15) == 0) {
-            const float4 f = *reinterpret_cast<const float4*>(src);
-            x[0] = f.x; x[1] = f.y; x[2] = f.z; x[3] = f.w;
+        float* dst = Vs + j * VP + cc;
+        if (aligned && j < c.nt && cc + 3 < c.ncols) {
+            cp_async16(smem_addr(dst), src);
         } else {
 #pragma unroll
-            for (int e = 0; e < 4; ++e) x[e] = j < c.nt && cc + e < c.ncols ? src[e] : 0.f;
+            for (int e = 0; e < 4; ++e) dst[e] = j < c.nt && cc + e < c.ncols ? src[e] : 0.f;
         }
-        if (scale) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) x[e] *= cc + e < c.ncols ? scale[head_of(p, cc + e)][j] : 0.f;
-        }
-        *reinterpret_cast<float4*>(Vs + j * VP + cc) = make_float4(x[0], x[1], x[2], x[3]);
     }
 }
 
-// rows of q, k or g of one head: [CHUNK][pitch], zero beyond the chunk's tokens and the head's rows
-template <int RP, int PITCH, int THREADS>
+// Rows of RP values with 16-byte fragment reads: row r's halves of 32 values trade places when bit 0 of r ^ (r >> 1) is
+// set, so that neither rows r, r + 1 nor rows r, r + 2 side by side meet in a bank.
+__device__ __forceinline__ int turned(int r) { return ((r ^ (r >> 1)) & 1) << 4; }
+
+// rows of q, k or g of one head: [CHUNK][RP] turned, zero beyond the chunk's tokens and the head's rows
+template <int RP, int THREADS>
 __device__ __forceinline__ void stage_rows(const float* src, long stride, float* dst, int nt, int rows) {
+#pragma unroll 4
     for (int i = threadIdx.x; i < CHUNK * (RP / 4); i += THREADS) {
         const int j = i / (RP / 4), d = (i % (RP / 4)) * 4;
-        float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (j < nt && d < rows) f = *reinterpret_cast<const float4*>(src + (size_t)j * stride + d);
-        *reinterpret_cast<float4*>(dst + j * PITCH + d) = f;
+        float* to = dst + j * RP + (d ^ turned(j));
+        if (j < nt && d < rows) cp_async16(smem_addr(to), src + (size_t)j * stride + d);
+        else *reinterpret_cast<float4*>(to) = make_float4(0.f, 0.f, 0.f, 0.f);
     }
 }
 
@@ -132,29 +133,43 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ChunkParams p) {
     float* Vs = Ks + CHUNK * KP;                             // [CHUNK][VP]
     float (*scale)[CHUNK] = reinterpret_cast<float (*)[CHUNK]>(Vs + CHUNK * VP);      // head decay: [HP][CHUNK]
     float* part = Vs + CHUNK * VP;                           // gated: [SEGS][RP]
+    (void)scale; (void)part;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
     const Place c = place_of(p);
+    stage_values<256>(p, c, Vs);
     if (FORM == GATED) {
         const int d = tid % RP, seg = tid / RP;
         const bool live = d < p.rows;
         const float* g = p.g + (size_t)c.t0 * p.g_stride + (size_t)c.h0 * p.rows + d;
         const float* k = p.k + (size_t)c.t0 * p.k_stride + (size_t)c.qk * p.rows + d;
-        float sum = 0.f;
-#pragma unroll 8
-        for (int j = seg * SEG; j < (seg + 1) * SEG; ++j) if (live && j < c.nt) sum += g[(size_t)j * p.g_stride];
+        float gv[SEG], kv[SEG], sum = 0.f;
+#pragma unroll
+        for (int e = 0; e < SEG; ++e) {
+            const int j = seg * SEG + e;
+            const bool on = live && j < c.nt;
+            gv[e] = on ? g[(size_t)j * p.g_stride] : 0.f;
+            kv[e] = on ? k[(size_t)j * p.k_stride] : 0.f;
+        }
+#pragma unroll
+        for (int e = 0; e < SEG; ++e) sum += gv[e];
         part[seg * RP + d] = sum;
         __syncthreads();
         float suffix = 0.f;                                  // log decay from token j to the chunk's end
         for (int e = SEGS - 1; e > seg; --e) suffix += part[e * RP + d];
-#pragma unroll 8
-        for (int j = (seg + 1) * SEG - 1; j >= seg * SEG; --j) {
-            const bool on = live && j < c.nt;
-            Ks[j * KP + d] = on ? k[(size_t)j * p.k_stride] * exp_of(suffix) : 0.f;
-            if (on) suffix += g[(size_t)j * p.g_stride];
+#pragma unroll
+        for (int e = SEG - 1; e >= 0; --e) {
+            Ks[(seg * SEG + e) * KP + d] = kv[e] * exp_of(suffix);
+            suffix += gv[e];
         }
         if (seg == 0 && c.col0 == 0) p.decays[((size_t)blockIdx.x * p.heads + c.h0) * RP + d] = live ? exp_of(suffix) : 0.f;
-        stage_values<256>(p, c, Vs, nullptr);
     } else {
+        const float* k = p.k + (size_t)c.t0 * p.k_stride + (size_t)c.qk * p.rows;
+#pragma unroll 4
+        for (int i = tid; i < CHUNK * (RP / 4); i += 256) {
+            const int j = i / (RP / 4), d = (i % (RP / 4)) * 4;
+            if (j < c.nt && d < p.rows) cp_async16(smem_addr(Ks + j * KP + d), k + (size_t)j * p.k_stride + d);
+            else *reinterpret_cast<float4*>(Ks + j * KP + d) = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
         // per head: beta_j times the decay from j to the end, by a scan from the end (two tokens a lane)
         for (int hh = warp; hh < p.hp; hh += 8) {
             const int h = c.h0 + hh, j0 = 2 * lane, j1 = j0 + 1;
@@ -173,10 +188,8 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ChunkParams p) {
             scale[hh][j0] = j0 < c.nt ? b[(size_t)j0 * p.beta_stride] * exp_of(after + g1) : 0.f;
             if (lane == 0 && c.col0 == 0) p.decays[(size_t)blockIdx.x * p.heads + h] = exp_of(incl);
         }
-        stage_rows<RP, KP, 256>(p.k + (size_t)c.t0 * p.k_stride + (size_t)c.qk * p.rows, p.k_stride, Ks, c.nt, p.rows);
-        __syncthreads();
-        stage_values<256>(p, c, Vs, scale);
     }
+    cp_async_wait_all();
     __syncthreads();
     // U = K^T V: a warp takes 32 rows of the state and COLS / CP columns
     constexpr int PAIRS = RP / 32, CP = PAIRS >= 4 ? 2 : 8 / PAIRS, NBW = COLS / 8 / CP;
@@ -201,7 +214,12 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ChunkParams p) {
                 const int n = n_base + nb * 8;
                 if (n >= c.ncols) continue;
                 const float* vb = Vs + (ks * 8 + tig) * VP + n + gid;
-                const BFrag b = make_b(vb[0], vb[4 * VP]);
+                float v0 = vb[0], v1 = vb[4 * VP];
+                if (FORM == HEAD) {
+                    const float* sc = scale[head_of(p, n)];
+                    v0 *= sc[ks * 8 + tig]; v1 *= sc[ks * 8 + tig + 4];
+                }
+                const BFrag b = make_b(v0, v1);
                 mma_split(acc[0][nb], a[0], b);
                 mma_split(acc[1][nb], a[1], b);
             }
@@ -212,7 +230,7 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ChunkParams p) {
             for (int e = 0; e < 2; ++e) {
                 const int cc = n_base + nb * 8 + 2 * tig + e;
                 if (cc >= c.ncols) continue;
-                float* u = p.sums + (((size_t)blockIdx.x * p.heads + c.h0 + head_of(p, cc)) * p.columns + column_of(p, c, cc)) * RP + pair * 32 + gid;
+                float* u = p.sums + ((size_t)blockIdx.x * p.heads * p.columns + first_column(p, c) + cc) * RP + pair * 32 + gid;
 #pragma unroll
                 for (int m = 0; m < 2; ++m) { u[16 * m] = acc[m][nb][e]; u[16 * m + 8] = acc[m][nb][e + 2]; }
             }
@@ -255,30 +273,34 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(ChunkParams p, int rp) 
 // ------------------------------------------------------------------------------------------------ 3: the outputs
 template <int FORM, int RP>
 struct OutputLayout {
-    static constexpr int P = RP + 16;                        // pitch of q, k, g: 16-byte fragment reads without bank conflicts
-    static constexpr size_t q = 0, k = q + CHUNK * P, v = k + CHUNK * P, a = v + CHUNK * VP, x = a + CHUNK * AP;
+    static constexpr int P = RP;                             // pitch of q, k, g and the state's columns (turned rows)
+    static constexpr int A_HEADS = FORM == GATED ? 1 : MAX_HP;
+    static constexpr size_t q = 0, k = q + CHUNK * P, s = k + CHUNK * P, v = s + COLS * P, a = v + CHUNK * VP,
+                            x = a + A_HEADS * CHUNK * AP;
     // gated: g [CHUNK][P], block decays [4][RP], decays up to a block [4][RP]; head decay: cumulative log decay in two
     // terms, and strength
     static constexpr size_t total = FORM == GATED ? x + CHUNK * P + 8 * RP : x + 3 * MAX_HP * CHUNK;
 };
 
-// a 16 x 8 block of q k^T (rows of q from ri, rows of k from rj), q times factor[d] if given
-template <int RP, int P>
+// a 16 x 8 block of q k^T (rows of q from ri, rows of k from rj), q times f0[d] f1[d] if given
+template <int RP>
 __device__ __forceinline__ void token_block(const float* Q, const float* K, int ri, int rj, const float* f0, const float* f1, int gid,
                                             int tig, float (&acc)[4]) {
     acc[0] = acc[1] = acc[2] = acc[3] = 0.f;
-    const float *qa = Q + (ri + gid) * P + 4 * tig, *qb = qa + 8 * P, *kb = K + (rj + gid) * P + 4 * tig;
+    const float *qa = Q + (ri + gid) * RP, *qb = qa + 8 * RP, *kb = K + (rj + gid) * RP;
+    const int qt = turned(ri + gid), kt = turned(rj + gid);          // rows eight apart are turned alike
 #pragma unroll 4
-    for (int d = 0; d < RP; d += 16) {
-        float4 x = *reinterpret_cast<const float4*>(qa + d), y = *reinterpret_cast<const float4*>(qb + d);
-        const float4 z = *reinterpret_cast<const float4*>(kb + d);
+    for (int d0 = 0; d0 < RP; d0 += 16) {
+        const int d = d0 + 4 * tig;
+        float4 x = *reinterpret_cast<const float4*>(qa + (d ^ qt)), y = *reinterpret_cast<const float4*>(qb + (d ^ qt));
+        const float4 z = *reinterpret_cast<const float4*>(kb + (d ^ kt));
         if (f0) {
-            const float4 f = *reinterpret_cast<const float4*>(f0 + d + 4 * tig);
+            const float4 f = *reinterpret_cast<const float4*>(f0 + d);
             x.x *= f.x; x.y *= f.y; x.z *= f.z; x.w *= f.w;
             y.x *= f.x; y.y *= f.y; y.z *= f.z; y.w *= f.w;
         }
         if (f1) {
-            const float4 f = *reinterpret_cast<const float4*>(f1 + d + 4 * tig);
+            const float4 f = *reinterpret_cast<const float4*>(f1 + d);
             x.x *= f.x; x.y *= f.y; x.z *= f.z; x.w *= f.w;
             y.x *= f.x; y.y *= f.y; y.z *= f.z; y.w *= f.w;
         }
@@ -294,18 +316,29 @@ template <int FORM, int RP>
 __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
     using L = OutputLayout<FORM, RP>;
     constexpr int P = L::P;
+    static_assert(P == RP, "turned rows have no pad");
     extern __shared__ __align__(16) float smem[];
-    float *Q = smem + L::q, *K = smem + L::k, *Vs = smem + L::v, *A = smem + L::a;
+    float *Q = smem + L::q, *K = smem + L::k, *Ss = smem + L::s, *Vs = smem + L::v, *A = smem + L::a;
     float* G = smem + L::x;                                  // gated
     float *Pb = G + CHUNK * P, *E = Pb + 4 * RP;
     float (*bc)[CHUNK] = reinterpret_cast<float (*)[CHUNK]>(smem + L::x);                       // head decay
     float (*bl)[CHUNK] = bc + MAX_HP, (*wt)[CHUNK] = bl + MAX_HP;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
     const Place c = place_of(p);
-    stage_rows<RP, P, 512>(p.q + (size_t)c.t0 * p.q_stride + (size_t)c.qk * p.rows, p.q_stride, Q, c.nt, p.rows);
-    stage_rows<RP, P, 512>(p.k + (size_t)c.t0 * p.k_stride + (size_t)c.qk * p.rows, p.k_stride, K, c.nt, p.rows);
-    if (FORM == GATED) stage_rows<RP, P, 512>(p.g + (size_t)c.t0 * p.g_stride + (size_t)c.h0 * p.rows, p.g_stride, G, c.nt, p.rows);
-    stage_values<512>(p, c, Vs, nullptr);
+    stage_rows<RP, 512>(p.q + (size_t)c.t0 * p.q_stride + (size_t)c.qk * p.rows, p.q_stride, Q, c.nt, p.rows);
+    stage_rows<RP, 512>(p.k + (size_t)c.t0 * p.k_stride + (size_t)c.qk * p.rows, p.k_stride, K, c.nt, p.rows);
+    if (FORM == GATED) stage_rows<RP, 512>(p.g + (size_t)c.t0 * p.g_stride + (size_t)c.h0 * p.rows, p.g_stride, G, c.nt, p.rows);
+    cp_async_commit();
+    // the values and the state before the chunk are asked for now and needed last
+    stage_values<512>(p, c, Vs);
+#pragma unroll 4
+    for (int i = tid; i < COLS * (RP / 4); i += 512) {
+        const int cc = i / (RP / 4), d = (i % (RP / 4)) * 4;
+        if (cc < c.ncols)
+            cp_async16(smem_addr(Ss + cc * P + (d ^ turned(cc))),
+                       p.sums + ((size_t)blockIdx.x * p.heads * p.columns + first_column(p, c) + cc) * RP + d);
+    }
+    cp_async_commit();
     if (FORM == HEAD) {
         for (int hh = warp; hh < p.hp; hh += 16) {
             const int h = c.h0 + hh, j0 = 2 * lane, j1 = j0 + 1;
@@ -326,6 +359,7 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
             wt[hh][j1] = j1 < c.nt ? b[(size_t)j1 * p.beta_stride] : 0.f;
         }
     }
+    cp_async_wait<1>();
     __syncthreads();
     if (FORM == GATED) {
         // running log decay inside every block of 16 tokens, and the block's decay
@@ -333,7 +367,11 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
             const int d = i % RP, blk = i / RP;
             float b = 0.f;
 #pragma unroll
-            for (int j = 0; j < BLOCK; ++j) { b += G[(blk * BLOCK + j) * P + d]; G[(blk * BLOCK + j) * P + d] = b; }
+            for (int j = 0; j < BLOCK; ++j) {
+                float* gj = G + (blk * BLOCK + j) * P + (d ^ turned(j));      // a block's first row is turned like row 0
+                b += *gj;
+                *gj = b;
+            }
             Pb[blk * RP + d] = exp_of(b);
         }
         __syncthreads();
@@ -351,11 +389,12 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
             const float *q0 = Q + r0 * P, *q1 = q0 + P, *k0 = K + s0 * P, *k1 = k0 + P;
             const float *bq0 = G + r0 * P, *bq1 = bq0 + P, *bk0 = G + s0 * P, *bk1 = bk0 + P;
             float s00 = 0.f, s01 = 0.f, s10 = 0.f, s11 = 0.f;
+            const int u0 = turned(r0), u1 = turned(r0 + 1), w0 = turned(s0), w1 = turned(s0 + 1);
             for (int d = 4 * part; d < RP; d += 16) {
-                const float4 x0 = *reinterpret_cast<const float4*>(q0 + d), x1 = *reinterpret_cast<const float4*>(q1 + d);
-                const float4 y0 = *reinterpret_cast<const float4*>(k0 + d), y1 = *reinterpret_cast<const float4*>(k1 + d);
-                const float4 a0 = *reinterpret_cast<const float4*>(bq0 + d), a1 = *reinterpret_cast<const float4*>(bq1 + d);
-                const float4 c0 = *reinterpret_cast<const float4*>(bk0 + d), c1 = *reinterpret_cast<const float4*>(bk1 + d);
+                const float4 x0 = *reinterpret_cast<const float4*>(q0 + (d ^ u0)), x1 = *reinterpret_cast<const float4*>(q1 + (d ^ u1));
+                const float4 y0 = *reinterpret_cast<const float4*>(k0 + (d ^ w0)), y1 = *reinterpret_cast<const float4*>(k1 + (d ^ w1));
+                const float4 a0 = *reinterpret_cast<const float4*>(bq0 + (d ^ u0)), a1 = *reinterpret_cast<const float4*>(bq1 + (d ^ u1));
+                const float4 c0 = *reinterpret_cast<const float4*>(bk0 + (d ^ w0)), c1 = *reinterpret_cast<const float4*>(bk1 + (d ^ w1));
 #define RS_PAIRS(e)                                                                                                             \
                 s00 = fmaf(x0.e * y0.e, exp_of(a0.e - c0.e), s00); s10 = fmaf(x1.e * y0.e, exp_of(a1.e - c0.e), s10);           \
                 s01 = fmaf(x0.e * y1.e, exp_of(fminf(a0.e - c1.e, 0.f)), s01); s11 = fmaf(x1.e * y1.e, exp_of(a1.e - c1.e), s11);
@@ -380,9 +419,10 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
         // q by its decay since its block's start, k by its decay to its block's end
         for (int i = tid; i < CHUNK * RP; i += 512) {
             const int j = i / RP, d = i % RP;
-            const float b = G[j * P + d], end = G[(j / BLOCK * BLOCK + BLOCK - 1) * P + d];
-            Q[j * P + d] *= exp_of(b);
-            K[j * P + d] *= exp_of(end - b);
+            const int last = j | (BLOCK - 1), at = j * P + (d ^ turned(j));
+            const float b = G[at], end = G[last * P + (d ^ turned(last))];
+            Q[at] *= exp_of(b);
+            K[at] *= exp_of(end - b);
         }
         __syncthreads();
         // blocks of earlier tokens: q (block bi) . k (block bj) with the decays of the blocks between
@@ -392,7 +432,7 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
             float acc[4];
             const float* f0 = bi - bj >= 2 ? Pb + (bj + 1) * RP : nullptr;
             const float* f1 = bi - bj >= 3 ? Pb + (bj + 2) * RP : nullptr;
-            token_block<RP, P>(Q, K, bi * BLOCK, bj * BLOCK + half * 8, f0, f1, gid, tig, acc);
+            token_block<RP>(Q, K, bi * BLOCK, bj * BLOCK + half * 8, f0, f1, gid, tig, acc);
             float* a = A + (bi * BLOCK + gid) * AP + bj * BLOCK + half * 8 + 2 * tig;
             a[0] = acc[0]; a[1] = acc[1]; a[8 * AP] = acc[2]; a[8 * AP + 1] = acc[3];
         }
@@ -401,11 +441,18 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
             const int pair = task >> 1, half = task & 1;
             const int bi = pair < 1 ? 0 : pair < 3 ? 1 : pair < 6 ? 2 : 3, bj = pair - bi * (bi + 1) / 2;
             float acc[4];
-            token_block<RP, P>(Q, K, bi * BLOCK, bj * BLOCK + half * 8, nullptr, nullptr, gid, tig, acc);
-            float* a = A + (bi * BLOCK + gid) * AP + bj * BLOCK + half * 8 + 2 * tig;
-            a[0] = acc[0]; a[1] = acc[1]; a[8 * AP] = acc[2]; a[8 * AP + 1] = acc[3];
+            token_block<RP>(Q, K, bi * BLOCK, bj * BLOCK + half * 8, nullptr, nullptr, gid, tig, acc);
+            // times the decay from j to i and j's strength, head by head; nothing above the diagonal
+            for (int hh = 0; hh < p.hp; ++hh)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int i = bi * BLOCK + gid + 8 * (e >> 1), j = bj * BLOCK + half * 8 + 2 * tig + (e & 1);
+                    A[(hh * CHUNK + i) * AP + j] =
+                        j <= i ? acc[e] * wt[hh][j] * exp_of((bc[hh][i] - bc[hh][j]) + (bl[hh][i] - bl[hh][j])) : 0.f;
+                }
         }
     }
+    cp_async_wait_all();
     __syncthreads();
     // outputs: a warp takes 32 tokens and 16 columns
     const int rp2 = warp & 1, row0 = rp2 * 32, n_base = (warp >> 1) * 16;
@@ -419,21 +466,25 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
             for (int e = 0; e < 4; ++e) acc[m][nb][e] = 0.f;
     int hh[2];
     const float* sp[2];                                      // the state's column for this lane's fragment of each block of columns
+    int st[2];
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb) {
         const int cc = min(n_base + nb * 8 + gid, c.ncols - 1);
         hh[nb] = head_of(p, min(n_base + nb * 8, c.ncols - 1));
-        sp[nb] = p.sums + (((size_t)blockIdx.x * p.heads + c.h0 + head_of(p, cc)) * p.columns + column_of(p, c, cc)) * RP + 4 * tig;
+        sp[nb] = Ss + cc * P;
+        st[nb] = turned(cc);
     }
+    const int qt = turned(row0 + gid);                       // rows eight apart are turned alike
 #pragma unroll 2
-    for (int d = 0; d < RP; d += 16) {
+    for (int d0 = 0; d0 < RP; d0 += 16) {
+        const int d = d0 + 4 * tig;
         AFrag a0[2], a1[2];
 #pragma unroll
         for (int m = 0; m < 2; ++m) {
-            const float* qa = Q + (row0 + 16 * m + gid) * P + d + 4 * tig;
+            const float* qa = Q + (row0 + 16 * m + gid) * P + (d ^ qt);
             float4 x = *reinterpret_cast<const float4*>(qa), y = *reinterpret_cast<const float4*>(qa + 8 * P);
             if (FORM == GATED) {
-                const float4 f = *reinterpret_cast<const float4*>(E + (2 * rp2 + m) * RP + d + 4 * tig);
+                const float4 f = *reinterpret_cast<const float4*>(E + (2 * rp2 + m) * RP + d);
                 x.x *= f.x; x.y *= f.y; x.z *= f.z; x.w *= f.w;
                 y.x *= f.x; y.y *= f.y; y.z *= f.z; y.w *= f.w;
             }
@@ -442,7 +493,7 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
         }
 #pragma unroll
         for (int nb = 0; nb < 2; ++nb) {
-            const float4 z = __ldcg(reinterpret_cast<const float4*>(sp[nb] + d));
+            const float4 z = *reinterpret_cast<const float4*>(sp[nb] + (d ^ st[nb]));
             const BFrag b0 = make_b(z.x, z.y), b1 = make_b(z.z, z.w);
 #pragma unroll
             for (int m = 0; m < 2; ++m) { mma_split(acc[m][nb], a0[m], b0); mma_split(acc[m][nb], a1[m], b1); }
@@ -462,38 +513,32 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
         const int i0 = row0 + 16 * m + gid, i1 = i0 + 8, steps = 2 * (2 * rp2 + m + 1);
         for (int ks = 0; ks < steps; ++ks) {
             const int j0 = ks * 8 + tig, j1 = j0 + 4;
-            float x[4] = {A[i0 * AP + j0], A[i1 * AP + j0], A[i0 * AP + j1], A[i1 * AP + j1]};
             AFrag a;
-            if (FORM == GATED) make_a(a, x[0], x[1], x[2], x[3]);
 #pragma unroll
             for (int nb = 0; nb < 2; ++nb) {
-                if (FORM == HEAD && (nb == 0 || hh[1] != hh[0])) {
-                    const float *b = bc[hh[nb]], *l = bl[hh[nb]];
-                    const float w0 = wt[hh[nb]][j0], w1 = wt[hh[nb]][j1];
-                    const auto decay = [&](int i, int j) { return exp_of((b[i] - b[j]) + (l[i] - l[j])); };
-                    make_a(a, j0 <= i0 ? x[0] * w0 * decay(i0, j0) : 0.f, j0 <= i1 ? x[1] * w0 * decay(i1, j0) : 0.f,
-                           j1 <= i0 ? x[2] * w1 * decay(i0, j1) : 0.f, j1 <= i1 ? x[3] * w1 * decay(i1, j1) : 0.f);
+                if (nb == 0 || (FORM == HEAD && hh[1] != hh[0])) {
+                    const float* Ah = A + (FORM == HEAD ? hh[nb] * CHUNK * AP : 0);
+                    make_a(a, Ah[i0 * AP + j0], Ah[i1 * AP + j0], Ah[i0 * AP + j1], Ah[i1 * AP + j1]);
                 }
                 const float* vb = Vs + j0 * VP + n_base + nb * 8 + gid;
                 mma_split(acc[m][nb], a, make_b(vb[0], vb[4 * VP]));
             }
         }
     }
+    float* out = p.out + (size_t)c.t0 * p.out_stride + first_column(p, c);
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             const int cc = n_base + nb * 8 + 2 * tig + e;
             if (cc >= c.ncols) continue;
-            const int h = c.h0 + head_of(p, cc);
-            const float skip = FORM == HEAD && p.skip ? p.skip[h] : 0.f;
-            float* o = p.out + (size_t)c.t0 * p.out_stride + (size_t)h * p.columns + column_of(p, c, cc);
+            const float skip = FORM == HEAD && p.skip ? p.skip[c.h0 + hh[nb]] : 0.f;
 #pragma unroll
             for (int m = 0; m < 2; ++m)
 #pragma unroll
                 for (int r = 0; r < 2; ++r) {
                     const int i = row0 + 16 * m + gid + 8 * r;
-                    if (i < c.nt) o[(size_t)i * p.out_stride] = fmaf(skip, Vs[i * VP + cc], acc[m][nb][e + 2 * r] * p.q_scale);
+                    if (i < c.nt) out[(size_t)i * p.out_stride + cc] = fmaf(skip, Vs[i * VP + cc], acc[m][nb][e + 2 * r] * p.q_scale);
                 }
         }
 }
@@ -541,9 +586,7 @@ RS_EXPORT int rs_state_recurrence_chunked(const float* q, long q_stride, const f
     if (!rs_state_chunks_supported(form, rows_pad, columns) || rows < 4 || rows % 4 || rows > rows_pad || group < 1 || heads % group ||
         (form == HEAD && !beta))
         return (int)cudaErrorInvalidValue;
-    int hp = 1;                          // whole heads that share q and k side by side in a CTA
-    if (form == HEAD)
-        for (int n = 2; n <= group && n * columns <= COLS; ++n) if (group % n == 0) hp = n;
+    const int hp = form == HEAD && group % 2 == 0 && 2 * columns <= COLS ? 2 : 1;       // two heads that share q and k in a CTA
     ChunkParams p{q, q_stride, k, k_stride, g, g_stride, beta, beta_stride, v, v_stride, out, out_stride, state, state_stride, q_start,
                   slots, chunk_seq, chunk_start, seq_first_chunk, sums, decays, heads, group, columns, rows, hp,
                   hp > 1 ? 1 : (columns + COLS - 1) / COLS, q_scale, skip};
