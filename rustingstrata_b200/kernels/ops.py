@@ -1635,6 +1635,11 @@ def mixerslib():
                                                  c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                  c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                                  c_float, c_float, c_void_p, c_void_p]
+        lib.rs_grouped_attention_q_per_cta.argtypes = [c_int, c_int, c_int, c_int]
+        lib.rs_grouped_attention_single_ok.argtypes = [c_int, c_int, c_int, c_int]
+        lib.rs_grouped_attention_mma.argtypes = [c_void_p, c_long, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_int,
+                                                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_long,
+                                                 c_void_p, c_long] + [c_int] * 8 + [c_float, c_float, c_void_p, c_void_p]
         _mixerslib = lib
     return _mixerslib
 
@@ -2013,3 +2018,46 @@ def talking_attention_mma(q: torch.Tensor, gate: Optional[torch.Tensor], cache: 
         _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len), _ptr(work), n_work, 1 if any_parts else 0,
         _ptr(talk), _ptr(sink), _ptr(out), dtype_code(out), out.stride(0), _ptr(partial), rows, n_heads, n_kv, dk, dv, window,
         int(chunk), int(keep), q_per_cta, float(scale), float(out_scale), _ptr(status), _stream()), "talking_attention_mma")
+
+
+def grouped_attention_q_per_cta(n_heads: int, n_kv: int, dk: int, dv: int) -> int:
+    """Queries per tile of the grouped tensor-core attention for these sizes; 0: not one of its shapes (head sizes that are
+    no multiple of 16 or above 128, more than 64 query heads per key/value head)."""
+    return int(mixerslib().rs_grouped_attention_q_per_cta(n_heads, n_kv, dk, dv))
+
+
+def grouped_attention_single_ok(n_heads: int, n_kv: int, dk: int, dv: int) -> bool:
+    return bool(mixerslib().rs_grouped_attention_single_ok(n_heads, n_kv, dk, dv))
+
+
+def grouped_attention_mma(q: torch.Tensor, gate: Optional[torch.Tensor], cache: torch.Tensor, block_table: torch.Tensor,
+                          page_size: int, q_start: torch.Tensor, kv_len: torch.Tensor, work: torch.Tensor, n_work: int,
+                          any_parts: bool, single: bool, sink: Optional[torch.Tensor], out: torch.Tensor,
+                          partial: Optional[torch.Tensor], n_heads: int, n_kv: int, dk: int, dv: int, window: int, q_per_cta: int,
+                          scale: float, status: torch.Tensor, chunk: int = 0, keep: int = 0, out_scale: float = 1.0) -> None:
+    """``talking_attention_mma`` for heads that do not mix (csrc/grouped_attention_mma.cu): a CTA per tile and key/value head.
+    ``single``: tiles of one query, whose keys the CTA's warps share out."""
+    _cuda(q, gate, cache, block_table, q_start, kv_len, work, sink, out, partial, status)
+    _f32_rows("grouped_attention_mma", q=q, gate=gate, partial=partial)
+    _rows_contiguous(out, "grouped_attention_mma out")
+    _i32("grouped_attention_mma", block_table, q_start, kv_len, work)
+    if cache.dtype != torch.bfloat16:
+        raise KernelError("grouped_attention_mma: the cache must be bfloat16")
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != n_heads or not sink.is_contiguous()):
+        raise KernelError(f"grouped_attention_mma: sink must be contiguous float32 with {n_heads} values")
+    if q.shape[1] < n_heads * dk or out.shape[1] < n_heads * dv or work.numel() < TALKING_WORK_COLS * n_work \
+            or not cache.is_contiguous() or cache.shape[-1] < max(dk, dv) \
+            or (gate is not None and (gate.shape[1] != n_heads or not gate.is_contiguous())) \
+            or out.stride(0) % 2 or out.data_ptr() % 8:
+        raise KernelError("grouped_attention_mma: shapes do not fit the head counts and sizes")
+    rows = 0
+    if partial is not None:
+        if not partial.is_contiguous() or partial.shape[1] < n_heads * (dv + 2):
+            raise KernelError("grouped_attention_mma: the partial sums need contiguous rows of heads * (dv + 2) values")
+        rows = partial.numel() // (n_heads * (dv + 2))
+    _check(mixerslib().rs_grouped_attention_mma(
+        _ptr(q), q.stride(0), _ptr(gate), _ptr(cache), cache.stride(0), cache.shape[0], page_size, cache.shape[-1],
+        _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len), _ptr(work), n_work, 1 if any_parts else 0,
+        1 if single else 0, _ptr(sink), _ptr(out), dtype_code(out), out.stride(0), _ptr(partial), rows, n_heads, n_kv, dk, dv,
+        window, int(chunk), int(keep), q_per_cta, float(scale), float(out_scale), _ptr(status), _stream()),
+        "grouped_attention_mma", 2 if any_parts else 1)

@@ -37,6 +37,8 @@ MMA_SINGLE_Q = 4           # its query tile in a step of single tokens (the smal
 FILL_CTAS = 148            # one CTA per multiprocessor
 MAX_PARTS = 32
 MIN_PART_TILES = 4         # a part walks at least this many key tiles
+GROUPED_KEY_TILE = 64      # keys per tile of the grouped form, and the least tiles a part of it walks
+GROUPED_MIN_TILES = 2
 PARTIAL_ROWS = 4096        # (query, part) rows of partial sums the workspace holds
 
 
@@ -85,7 +87,7 @@ class TalkingAttention(Mixer):
         self.in_cols = self.q_cols + self.k_cols + self.v_cols + self.g_cols
         self.o_in = self.row_cols = self.n_heads * self.dv
         self.q_per_cta = None
-        self.mma_q = 0
+        self.mma_q = self.grouped_q = self.single_q = 0
         rt = runtime
         if not rt.precise:
             rt.scratch("talk_partial", PARTIAL_ROWS, self.n_heads * (self.dv + 2), torch.float32)
@@ -155,19 +157,22 @@ class TalkingAttention(Mixer):
             self.q_per_cta = ops.talking_attention_q_per_cta(self.n_heads, self.dk, self.dv)
             # the tensor-core form reads a bfloat16 cache; the 32-bit engine and shapes it does not take use the other
             self.mma_q = 0 if self.runtime.precise else ops.talking_attention_mma_q_per_cta(self.n_heads, self.n_kv, self.dk, self.dv)
+            # heads that do not mix need not share a CTA
+            if not self.runtime.precise and not self.has_talk:
+                self.grouped_q = ops.grouped_attention_q_per_cta(self.n_heads, self.n_kv, self.dk, self.dv)
+                self.single_q = int(ops.grouped_attention_single_ok(self.n_heads, self.n_kv, self.dk, self.dv))
 
     def plan_key(self):
         self._setup()
-        return ("talking_attention", self.q_per_cta, self.mma_q, self.window, self.chunk, self.keep)
+        return ("talking_attention", self.q_per_cta, self.mma_q, self.grouped_q, self.single_q, self.n_kv if self.grouped_q else 0,
+                self.window, self.chunk, self.keep)
 
-    def build_plan(self, batch: HostBatch):
-        """Tiles of neighbouring queries of one sequence, the ones with the most keys to walk first.  For the tensor-core
-        form a tile's key tiles are dealt out over several CTAs when the step has too few tiles to fill the device."""
-        self._setup()
-        single = int(batch.q_lens.max()) == 1
-        qt = (MMA_SINGLE_Q if single else self.mma_q) if self.mma_q else (1 if single else self.q_per_cta)
+    def _deal(self, batch: HostBatch, seqs, qt: int, key_tile: int, ctas_per_tile: int, fill: int, min_tiles: int):
+        """Rows (sequence, first query, part, parts, first partial row) for tiles of ``qt`` neighbouring queries of ``seqs``,
+        the ones with the most keys to walk first.  A tile's key tiles are dealt out over several CTAs when the tiles are
+        too few to fill ``fill`` CTAs."""
         tiles = []
-        for s in range(batch.n_seqs):
+        for s in seqs:
             offs = np.arange(0, batch.q_lens[s], qt, dtype=np.int32)
             tiles.append(np.stack([np.full_like(offs, s), offs], axis=1))
         work = np.concatenate(tiles, axis=0).astype(np.int32)
@@ -175,25 +180,25 @@ class TalkingAttention(Mixer):
         if len(work) > 1 and not batch.bucketed:
             order = np.argsort(-first, kind="stable")
             work, first = work[order], first[order]
-        if not self.mma_q:
-            return {"work": work.reshape(-1), "n_work": int(work.shape[0]), "any_parts": 0, "qt": qt}
         n = work.shape[0]
         nq = np.minimum(qt, batch.q_lens[work[:, 0]] - work[:, 1])
         parts = np.ones(n, dtype=np.int64)
-        # single tokens: one wave of CTAs (each is mostly fixed cost); portions: up to two, which also evens out the
-        # unequal walks of a causal portion's tiles
-        fill = FILL_CTAS if single else 2 * FILL_CTAS
-        if n <= fill // 2:
-            share = min(MAX_PARTS, fill // n)
+        if n * ctas_per_tile <= fill // 2:
+            share = min(MAX_PARTS, fill // (n * ctas_per_tile))
             if batch.bucketed:
-                parts[:] = share              # a captured step: the launch shape must not follow the lengths
+                # a captured step: the launch shape must not follow the lengths (a window bounds them)
+                reach = [w for w in (self.window, self.chunk) if w]
+                if reach and ctas_per_tile > 1:
+                    most = -(-min(reach) // key_tile) + 1 + -(-self.keep // key_tile)
+                    share = max(1, min(share, most // min_tiles))
+                parts[:] = share
             else:
                 begin = np.maximum(0, first - self.window + 1) if self.window else np.zeros(n, dtype=np.int64)
                 if self.chunk:
                     begin = np.maximum(begin, first // self.chunk * self.chunk)
-                kept = np.minimum(-(-self.keep // KEY_TILE), begin // KEY_TILE)
-                key_tiles = -(-(first + nq) // KEY_TILE) - begin // KEY_TILE + kept
-                parts = np.clip(key_tiles // MIN_PART_TILES, 1, share)
+                kept = np.minimum(-(-self.keep // key_tile), begin // key_tile)
+                key_tiles = -(-(first + nq) // key_tile) - begin // key_tile + kept
+                parts = np.clip(key_tiles // min_tiles, 1, share)
             while int((parts * nq)[parts > 1].sum()) > PARTIAL_ROWS:
                 parts = np.maximum(1, parts // 2)
         rows = np.where(parts > 1, parts * nq, 0)
@@ -201,7 +206,33 @@ class TalkingAttention(Mixer):
         rep = np.repeat(np.arange(n), parts)
         part = np.arange(len(rep)) - np.repeat(np.cumsum(parts) - parts, parts)
         full = np.stack([work[rep, 0], work[rep, 1], part, parts[rep], base[rep]], axis=1).astype(np.int32)
-        return {"work": full.reshape(-1), "n_work": int(full.shape[0]), "any_parts": int(bool((parts > 1).any())), "qt": qt}
+        return full, bool((parts > 1).any())
+
+    def build_plan(self, batch: HostBatch):
+        """Work lists of the form that runs (see :meth:`_deal`): the CUDA-core form (tiles without parts), the tensor-core
+        form with all heads in a CTA, or the grouped one, which takes single tokens apart from portions."""
+        self._setup()
+        single = int(batch.q_lens.max()) == 1
+        everyone = range(batch.n_seqs)
+        if self.grouped_q:
+            alone = [s for s in everyone if batch.q_lens[s] == 1] if self.single_q else []
+            rest = [s for s in everyone if batch.q_lens[s] > 1 or not self.single_q]
+            plan = {"n_work": 0, "any_parts": 0, "qt": self.grouped_q, "n_single": 0, "single_parts": 0}
+            if rest:
+                full, parts = self._deal(batch, rest, self.grouped_q, GROUPED_KEY_TILE, self.n_kv, 2 * FILL_CTAS, GROUPED_MIN_TILES)
+                plan.update(work=full.reshape(-1), n_work=int(full.shape[0]), any_parts=int(parts))
+            if alone:
+                full, parts = self._deal(batch, alone, 1, GROUPED_KEY_TILE, self.n_kv, 2 * FILL_CTAS, GROUPED_MIN_TILES)
+                plan.update(single_work=full.reshape(-1), n_single=int(full.shape[0]), single_parts=int(parts))
+            return plan
+        qt = (MMA_SINGLE_Q if single else self.mma_q) if self.mma_q else (1 if single else self.q_per_cta)
+        # single tokens: one wave of CTAs (each is mostly fixed cost); portions: up to two, which also evens out the
+        # unequal walks of a causal portion's tiles
+        fill = (FILL_CTAS if single else 2 * FILL_CTAS) if self.mma_q else 0
+        full, parts = self._deal(batch, everyone, qt, KEY_TILE, 1, fill, MIN_PART_TILES)
+        if not self.mma_q:
+            full = full[:, :2]
+        return {"work": full.reshape(-1), "n_work": int(full.shape[0]), "any_parts": int(parts), "qt": qt}
 
     # ---------------------------------------------------------------- the step
     def forward(self, h, residual, ctx: StepContext, call: CallInfo):
@@ -227,7 +258,15 @@ class TalkingAttention(Mixer):
                                    ctx.positions, ctx.seq_of_token, self.n_heads, self.n_kv, self.dk, self.dv, T, True, ctx.status,
                                    row_norm=self.row_norm, half_pairs=self.half_pairs)
         plan = ctx.plans[self.plan_key()]
-        if self.mma_q:
+        if self.grouped_q:
+            for work, n, parts, alone in ((plan.get("work"), plan["n_work"], plan["any_parts"], False),
+                                          (plan.get("single_work"), plan["n_single"], plan["single_parts"], True)):
+                if n:
+                    ops.grouped_attention_mma(q, gate, call.cache, table, rt.page_size, ctx.q_start, ctx.kv_len, work, n, bool(parts),
+                                              alone, self.sink, out, rt.get_scratch("talk_partial", torch.float32) if parts else None,
+                                              self.n_heads, self.n_kv, self.dk, self.dv, self.window, 1 if alone else plan["qt"],
+                                              self.scale, ctx.status, chunk=self.chunk, keep=self.keep, out_scale=self.out_scale)
+        elif self.mma_q:
             partial = rt.get_scratch("talk_partial", torch.float32) if plan["any_parts"] else None
             ops.talking_attention_mma(q, gate, call.cache, table, rt.page_size, ctx.q_start, ctx.kv_len, plan["work"],
                                       plan["n_work"], bool(plan["any_parts"]), self.talk, self.sink, out, partial, self.n_heads,

@@ -6,9 +6,10 @@ from rustingstrata_b200.parts import talking_attention as TA
 from rustingstrata_b200.parts.base import HostBatch
 
 
-def make_part(mma_q=16, window=0, chunk=0, keep=0):
+def make_part(mma_q=16, window=0, chunk=0, keep=0, grouped=0):
     att = TA.TalkingAttention.__new__(TA.TalkingAttention)
     att.q_per_cta, att.mma_q, att.window, att.chunk, att.keep = 8, mma_q, window, chunk, keep
+    att.grouped_q, att.single_q = grouped, int(grouped > 0)
     att.n_heads, att.n_kv, att.dk, att.dv = 16, 4, 64, 64
     return att
 
