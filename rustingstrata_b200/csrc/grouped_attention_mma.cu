@@ -131,7 +131,7 @@ __global__ void __launch_bounds__(THREADS) grouped_attention_kernel(MmaParams p)
         fetch(p, key_at, Vs, dv, (size_t)p.plane_stride, c, tid);
         cp_async_commit();
     }
-    constexpr int NB = SINGLE ? 2 : 8;                       // blocks of 8 keys a warp scores
+    constexpr int NB = SINGLE ? 2 : 8, STEP = SINGLE ? 1 : 2;         // blocks of 8 keys a warp scores; fragments of 16 keys at once
     const int key0 = SINGLE ? 16 * warp : 0;
     for (int t = t_begin; t < t_end; ++t) {
         const int i = t - t_begin, buf = i & 1, k0 = tile_at(t);
@@ -157,13 +157,15 @@ __global__ void __launch_bounds__(THREADS) grouped_attention_kernel(MmaParams p)
         for (int ks = 0; ks < DK; ++ks) {
             if (ks * 16 >= dk) break;
 #pragma unroll
-            for (int j = 0; j < NB / 2; ++j) {
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4(k_addr + (uint32_t)(j * 16 * kp + ks * 16) * 2u, b0, b1, b2, b3);
-                mma16816(S[2 * j], qh[ks], b0, b1);
-                mma16816(S[2 * j], ql[ks], b0, b1);
-                mma16816(S[2 * j + 1], qh[ks], b2, b3);
-                mma16816(S[2 * j + 1], ql[ks], b2, b3);
+            for (int j = 0; j < NB / 2; j += STEP) {
+                uint32_t b[STEP][4];                         // two products of one sum never follow each other directly
+#pragma unroll
+                for (int u = 0; u < STEP; ++u)
+                    ldmatrix_x4(k_addr + (uint32_t)((j + u) * 16 * kp + ks * 16) * 2u, b[u][0], b[u][1], b[u][2], b[u][3]);
+#pragma unroll
+                for (int u = 0; u < 2 * STEP; ++u) mma16816(S[2 * j + u], qh[ks], b[u >> 1][2 * (u & 1)], b[u >> 1][2 * (u & 1) + 1]);
+#pragma unroll
+                for (int u = 0; u < 2 * STEP; ++u) mma16816(S[2 * j + u], ql[ks], b[u >> 1][2 * (u & 1)], b[u >> 1][2 * (u & 1) + 1]);
             }
         }
         // ---- what the queries do not see (a tile that every query sees whole needs no look)
@@ -218,14 +220,18 @@ __global__ void __launch_bounds__(THREADS) grouped_attention_kernel(MmaParams p)
             for (int e = 0; e < 4; ++e)                      // rows gid, gid + 8, then the same of the next 8 keys
                 split_pair(S[2 * j + (e >> 1)][(e & 1) * 2], S[2 * j + (e >> 1)][(e & 1) * 2 + 1], ah[e], al[e]);
 #pragma unroll
-            for (int a = 0; a < DV; ++a) {
+            for (int a = 0; a < DV; a += 2) {
                 if (a * 16 >= dv) break;
-                uint32_t b0, b1, b2, b3;
-                ldmatrix_x4_trans(v_addr + (uint32_t)(j * 16 * vp + a * 16) * 2u, b0, b1, b2, b3);
-                mma16816(O[a][0], ah, b0, b1);
-                mma16816(O[a][0], al, b0, b1);
-                mma16816(O[a][1], ah, b2, b3);
-                mma16816(O[a][1], al, b2, b3);
+                const bool both = (a + 1) * 16 < dv;
+                uint32_t b[2][4];
+                ldmatrix_x4_trans(v_addr + (uint32_t)(j * 16 * vp + a * 16) * 2u, b[0][0], b[0][1], b[0][2], b[0][3]);
+                if (both) ldmatrix_x4_trans(v_addr + (uint32_t)(j * 16 * vp + a * 16 + 16) * 2u, b[1][0], b[1][1], b[1][2], b[1][3]);
+                mma16816(O[a][0], ah, b[0][0], b[0][1]);
+                mma16816(O[a][1], ah, b[0][2], b[0][3]);
+                if (both) { mma16816(O[a + 1][0], ah, b[1][0], b[1][1]); mma16816(O[a + 1][1], ah, b[1][2], b[1][3]); }
+                mma16816(O[a][0], al, b[0][0], b[0][1]);
+                mma16816(O[a][1], al, b[0][2], b[0][3]);
+                if (both) { mma16816(O[a + 1][0], al, b[1][0], b[1][1]); mma16816(O[a + 1][1], al, b[1][2], b[1][3]); }
             }
         }
     }

@@ -48,7 +48,7 @@ __device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) 
     lo = __float_as_uint(x - __uint_as_float(hi)) & 0xffffe000u;
 }
 __device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+    asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
@@ -68,6 +68,12 @@ __device__ __forceinline__ void mma_split(float (&d)[4], const AFrag& a, const B
     mma_tf32(d, a.lo, b.h0, b.h1);
     mma_tf32(d, a.hi, b.l0, b.l1);
     mma_tf32(d, a.hi, b.h0, b.h1);
+}
+// the same for two blocks of rows: two products of one sum do not follow each other directly
+__device__ __forceinline__ void mma_split2(float (&d0)[4], float (&d1)[4], const AFrag& a0, const AFrag& a1, const BFrag& b) {
+    mma_tf32(d0, a0.lo, b.h0, b.h1); mma_tf32(d1, a1.lo, b.h0, b.h1);
+    mma_tf32(d0, a0.hi, b.l0, b.l1); mma_tf32(d1, a1.hi, b.l0, b.l1);
+    mma_tf32(d0, a0.hi, b.h0, b.h1); mma_tf32(d1, a1.hi, b.h0, b.h1);
 }
 
 struct Place { int s, t0, nt, h0, qk, col0, ncols; };       // of a CTA: sequence, first token row, tokens, heads, columns
@@ -220,8 +226,7 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(ChunkParams p) {
                     v0 *= sc[ks * 8 + tig]; v1 *= sc[ks * 8 + tig + 4];
                 }
                 const BFrag b = make_b(v0, v1);
-                mma_split(acc[0][nb], a[0], b);
-                mma_split(acc[1][nb], a[1], b);
+                mma_split2(acc[0][nb], acc[1][nb], a[0], a[1], b);
             }
         }
 #pragma unroll
@@ -495,8 +500,8 @@ __global__ void __launch_bounds__(512, 1) chunk_output_kernel(ChunkParams p) {
         for (int nb = 0; nb < 2; ++nb) {
             const float4 z = *reinterpret_cast<const float4*>(sp[nb] + (d ^ st[nb]));
             const BFrag b0 = make_b(z.x, z.y), b1 = make_b(z.z, z.w);
-#pragma unroll
-            for (int m = 0; m < 2; ++m) { mma_split(acc[m][nb], a0[m], b0); mma_split(acc[m][nb], a1[m], b1); }
+            mma_split2(acc[0][nb], acc[1][nb], a0[0], a0[1], b0);
+            mma_split2(acc[0][nb], acc[1][nb], a1[0], a1[1], b1);
         }
     }
     if (FORM == HEAD) {

@@ -390,13 +390,14 @@ __global__ void conv_tail_update_kernel(const float* proj, long proj_stride, flo
 struct Mamba2PrepParams {
     const float* proj; long proj_stride;      // [T, ...]: convolved channels from conv_off on, step sizes from dt_off on
     const float* conv; const float* bias;     // [taps, C] tap-major, [C] or null
-    const float* tail; long tail_stride;      // [slots, (taps - 1) * C]
+    float* tail; long tail_stride;            // [slots, (taps - 1) * C]
     const float* dt_bias; const float* a_log; // [heads]
     float* out; long out_stride;              // [T, C]
     float* dt; float* decay;                  // [T, heads]
     const int* seq_of_token; const int* q_start; const int* slots;
     int C, taps, heads, conv_off, dt_off, n_tokens;
     int log_decay;                            // decay holds -exp(a_log) dt instead of its exponential
+    int shift_tail;                           // a step of single tokens: the tail moves on here, channel by channel
 };
 
 // V neighbouring channels of one token per thread (V = 4: 16-byte accesses), then one thread per (token, head).
@@ -433,6 +434,16 @@ __global__ void __launch_bounds__(256) mamba2_prep_kernel(Mamba2PrepParams p) {
             acc[0] = fmaf(w[0], src[0], acc[0]);
         }
     }
+    if (p.shift_tail) {
+        // nobody else reads this channel of the request's tail: every row takes the next one's place, the newest is the token's
+        float* row = p.tail + (size_t)p.slots[s] * p.tail_stride + c;
+        const float* now = p.proj + (size_t)t * p.proj_stride + p.conv_off + c;
+        for (int e = 0; e < p.taps - 1; ++e) {
+            const float* from = e + 2 < p.taps ? row + (size_t)(e + 1) * p.C : now;
+            if (V == 4) *reinterpret_cast<float4*>(row + (size_t)e * p.C) = *reinterpret_cast<const float4*>(from);
+            else row[(size_t)e * p.C] = from[0];
+        }
+    }
     float* dst = p.out + (size_t)t * p.out_stride + c;
     if (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(silu_f(acc[0]), silu_f(acc[1 % V]), silu_f(acc[2 % V]), silu_f(acc[3 % V]));
     else dst[0] = silu_f(acc[0]);
@@ -448,7 +459,7 @@ __global__ void __launch_bounds__(256) low_rank_decay_kernel(const float* u, lon
                                                              int rank, int n_tokens, int log_decay) {
     extern __shared__ __align__(16) float us[];                  // [DECAY_TOKENS][rank]
     const int t0 = blockIdx.y * DECAY_TOKENS, nt = min(DECAY_TOKENS, n_tokens - t0);
-    for (int i = threadIdx.x; i < nt * rank; i += blockDim.x) us[i] = u[(size_t)(t0 + i / rank) * u_stride + i % rank];
+    for (int i = threadIdx.x; i < DECAY_TOKENS * rank; i += blockDim.x) us[i] = i < nt * rank ? u[(size_t)(t0 + i / rank) * u_stride + i % rank] : 0.f;
     __syncthreads();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= heads * rows) return;
@@ -460,11 +471,26 @@ __global__ void __launch_bounds__(256) low_rank_decay_kernel(const float* u, lon
     for (int e = 0; e < DECAY_TOKENS; ++e) acc[e] = b;
     if (live) {
         const size_t row = (size_t)(h * dim + i) * rank;
-        for (int r = 0; r < rank; ++r) {
-            const float wv = load_any(w, w_dt, row + r);
+        if (w_dt == RS_BF16 && rank % 8 == 0) {              // a row of the matrix in 16-byte pieces (it starts on 16 bytes)
+            for (int r = 0; r < rank; r += 8) {
+                const uint4 raw = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(w) + row + r);
+                const __nv_bfloat162* pair = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
-            for (int e = 0; e < DECAY_TOKENS; ++e)
-                if (e < nt) acc[e] = fmaf(wv, us[e * rank + r], acc[e]);
+                for (int h2 = 0; h2 < 4; ++h2) {
+                    const float w0 = __low2float(pair[h2]), w1 = __high2float(pair[h2]);
+#pragma unroll
+                    for (int e = 0; e < DECAY_TOKENS; ++e) {
+                        const float2 x = *reinterpret_cast<const float2*>(us + e * rank + r + 2 * h2);
+                        acc[e] = fmaf(w1, x.y, fmaf(w0, x.x, acc[e]));
+                    }
+                }
+            }
+        } else {
+            for (int r = 0; r < rank; ++r) {
+                const float wv = load_any(w, w_dt, row + r);
+#pragma unroll
+                for (int e = 0; e < DECAY_TOKENS; ++e) acc[e] = fmaf(wv, us[e * rank + r], acc[e]);
+            }
         }
     }
 #pragma unroll
@@ -731,7 +757,8 @@ RS_EXPORT int rs_mamba2_prep(const float* proj, long proj_stride, int conv_off, 
     if (n_tokens <= 0) return 0;
     if (taps < 1 || channels < 1 || heads < 1 || (taps > 1 && !tail)) return (int)cudaErrorInvalidValue;
     Mamba2PrepParams p{proj, proj_stride, conv, bias, tail, tail_stride, dt_bias, a_log, out, out_stride, dt, decay, seq_of_token,
-                       q_start, slots, channels, taps, heads, conv_off, dt_off, n_tokens, log_decay};
+                       q_start, slots, channels, taps, heads, conv_off, dt_off, n_tokens, log_decay,
+                       taps > 1 && n_tokens == n_seqs};
     const bool vec = channels % 4 == 0 && conv_off % 4 == 0 && proj_stride % 4 == 0 && out_stride % 4 == 0 &&
                      (((uintptr_t)proj | (uintptr_t)conv | (uintptr_t)out) & 15) == 0 &&
                      (!tail || (tail_stride % 4 == 0 && ((uintptr_t)tail & 15) == 0));
@@ -740,7 +767,7 @@ RS_EXPORT int rs_mamba2_prep(const float* proj, long proj_stride, int conv_off, 
     if (vec) mamba2_prep_kernel<4><<<blocks, 256, 0, stream>>>(p);
     else mamba2_prep_kernel<1><<<blocks, 256, 0, stream>>>(p);
     int rc = rs_launch_result();
-    if (rc || taps == 1) return rc;
+    if (rc || taps == 1 || p.shift_tail) return rc;
     const long m = (long)n_seqs * channels;
     conv_tail_update_kernel<<<(unsigned)((m + 255) / 256), 256, 0, stream>>>(proj + conv_off, proj_stride, tail, tail_stride, q_start,
                                                                             slots, channels, taps, n_seqs);

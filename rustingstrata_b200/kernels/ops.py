@@ -1765,7 +1765,7 @@ def mamba2_prep(proj: torch.Tensor, conv_off: int, dt_off: int, conv: torch.Tens
     _check(mixerslib().rs_mamba2_prep(
         _ptr(proj), proj.stride(0), conv_off, dt_off, _ptr(conv), _ptr(bias), _ptr(tail), 0 if tail is None else tail.stride(0),
         _ptr(dt_bias), _ptr(a_log), _ptr(out), out.stride(0), _ptr(dt), _ptr(decay), _ptr(seq_of_token), _ptr(q_start), _ptr(slots),
-        C, taps, heads, 1 if log_decay else 0, n_tokens, n_seqs, _stream()), "mamba2_prep", 2 if taps > 1 else 1)
+        C, taps, heads, 1 if log_decay else 0, n_tokens, n_seqs, _stream()), "mamba2_prep", 2 if taps > 1 and n_tokens > n_seqs else 1)
 
 
 def low_rank_decay(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], tau: float, g: torch.Tensor, heads: int,
