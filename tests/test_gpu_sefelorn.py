@@ -398,6 +398,21 @@ def test_greedy_generation_through_the_scheduler(tmp_path_factory, chunk):
     assert eng.generate(prompts[::-1], max_new_tokens=12) == want[::-1]
 
 
+def test_generation_without_any_cache(tmp_path_factory):
+    """A model of state mixers only keeps no pages at all: the scheduler admits and decodes by slots alone."""
+    from rustingstrata_b200 import Engine
+    path, cfg, w = model(tmp_path_factory, "one_mamba2_groups_and_parts", ONE_LAYER["mamba2_groups_and_parts"], seed=5)
+    prompts = [tokens_for(cfg, n, 60 + n) for n in (5, 40, 1)]
+    want = []
+    for p in prompts:
+        seq = list(p)
+        for _ in range(8):
+            seq.append(int(np.argmax(plain_logits(cfg, w, seq)[-1])))
+        want.append(seq[len(p):])
+    eng = Engine(path, dtype="float32", page_size=8, max_tokens=64, max_batch_tokens=32, max_seqs=2, prefill_chunk=16)
+    assert eng.generate(prompts, max_new_tokens=8) == want
+
+
 def test_bfloat16_generation_picks_top_tokens(tmp_path_factory):
     from rustingstrata_b200 import Engine
     path, cfg, w = model(tmp_path_factory, "R", "R", seed=11)

@@ -100,3 +100,19 @@ def test_kept_first_keys_count_in_the_walk():
     assert plain[0, 3] == 17 // TA.MIN_PART_TILES and kept[0, 3] == (17 + 10) // TA.MIN_PART_TILES
     near = rows_of(make_part(window=512, keep=300).build_plan(batch([1], [520])))
     assert near[0, 3] == rows_of(make_part().build_plan(batch([1], [520])))[0, 3]       # the window still reaches the first keys
+
+
+def test_grouped_form_takes_single_tokens_apart():
+    """Heads that do not mix: tiles of several queries for portions, a list of its own for single tokens, parts counted in
+    key tiles of 64 and CTAs per key/value head; a captured step's shape does not follow the lengths."""
+    att = make_part(window=1024, keep=16, grouped=16)
+    plan = att.build_plan(batch([100, 1, 1], [100, 3000, 40]))
+    w, one = rows_of(plan), plan["single_work"].reshape(-1, 5)
+    assert plan["qt"] == 16 and set(w[:, 0]) == {0} and len(set(w[:, 1])) == 7
+    assert set(one[:, 0]) == {1, 2} and (one[one[:, 0] == 2][:, 3] == 1).all()
+    seen = one[one[:, 0] == 1]
+    assert len(seen) == seen[0, 3] == (17 + 1) // TA.GROUPED_MIN_TILES               # the window's tiles and the kept first one
+    a, b = (att.build_plan(batch([1, 1], kv, bucketed=True)) for kv in ([40, 60], [5000, 900]))
+    assert a["n_single"] == b["n_single"] and a["single_parts"] == b["single_parts"] and a["n_work"] == b["n_work"] == 0
+    att.single_q = 0
+    assert att.build_plan(batch([1, 1], [40, 60]))["n_single"] == 0
