@@ -50,17 +50,22 @@ def _tensors(part):
 
 
 def weight_bytes(model) -> int:
-    """Bytes of every weight one step reads once: all tensors of all parts, each once; the token table only when it is
-    also the output head (a step gathers a few rows of it otherwise)."""
-    seen, total = set(), 0
+    """Bytes of every weight one step reads once: all tensors of all parts, each once (a part may hold a view of a matrix
+    that its block joined out of several parts' ones); the token table only when it is also the output head (a step gathers
+    a few rows of it otherwise)."""
+    spans = []
     head_ptrs = {t.data_ptr() for t in _tensors(model.head)}
     for part in model.parts():
         for t in _tensors(part):
             if part is model.embedding and t.data_ptr() not in head_ptrs:
                 continue
-            if t.data_ptr() not in seen:
-                seen.add(t.data_ptr())
-                total += t.numel() * t.element_size()
+            if t.numel():
+                last = sum((n - 1) * st for n, st in zip(t.shape, t.stride()))
+                spans.append((t.data_ptr(), t.data_ptr() + (last + 1) * t.element_size()))
+    total, end = 0, 0
+    for a, b in sorted(spans):
+        total += max(0, b - max(a, end))
+        end = max(end, b)
     return total
 
 

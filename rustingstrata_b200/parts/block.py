@@ -105,6 +105,9 @@ class ParallelBlock(Block):
         if ff is not None:
             ff.w_down = self.w_out[:, at: at + ff.row_cols]
 
+    def flops_per_token(self) -> float:
+        return 0.0                           # the joined matrices are the parts', which count them
+
     @property
     def first_reader_takes_owed(self):
         return getattr(self.norm, "takes_owed", False)

@@ -564,3 +564,17 @@ def test_gated_group_norm(shape):
         out = torch.empty(T, n, dtype=dt, device="cuda")
         ops.gated_group_norm(y, z, w, out, parts, 1e-5, T)
         assert (out.double() - ref).abs().max() / ref.abs().max() < tol
+
+
+def test_joined_matrices_count_once(tmp_path_factory):
+    """The roofline's bytes and flops of a model whose blocks join their parts' matrices: every matrix once."""
+    from rustingstrata_b200.engine import roofline
+    path, cfg, w = model(tmp_path_factory, "R", "R", seed=11)
+    r = runner_for(path, "bfloat16", pool_tokens=64, max_batch_tokens=64)
+    assert any(getattr(b, "join_out", False) for b in r.model.blocks)
+    shapes = M.tensor_shapes(cfg)
+    total = sum(int(np.prod(s)) for s in shapes.values()) * 2
+    assert total <= roofline.weight_bytes(r.model) <= total * 1.05                   # small vectors are kept in float32
+    mats = sum(2 * int(np.prod(s)) for n, s in shapes.items() if len(s) == 2 and n != "embed" and not n.endswith("conv"))
+    state = 6.0 * (4 * 32 * 48 + 8 * 64 * 32)
+    assert abs(roofline.flops_per_token(r.model) - mats - state) <= 0.02 * mats
