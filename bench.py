@@ -490,7 +490,7 @@ class OpTimer:
              "attention_decode_items", "silu_mul", "residual_add", "sample", "latent_expand", "embed_sum", "stream_layernorm",
              "stream_update", "router_topk", "conv_norm_kv_write", "sigmoid_gate", "talking_attention_prep", "talking_attention", "talking_attention_mma", "grouped_attention_mma",
              "state_recurrence", "state_recurrence_chunked", "hgrn2_prep", "delta_prep", "head_norm_gate", "activation", "scale_rows", "retention_prep",
-             "head_sigmoid_gate", "mamba2_prep", "low_rank_decay", "pad_heads", "gated_group_norm", "add_embed")
+             "mamba2_prep", "low_rank_decay", "pad_heads", "gated_group_norm", "add_embed")
 
     def __init__(self):
         self.events, self.real = [], {}

@@ -17,7 +17,8 @@
 // Key tiles start at multiples of 64 from key 0 and the split form's splits at multiples of the split size, so the order
 // in which a query's keys are reduced depends on its position alone.  The split form leaves un-normalised partial
 // results (sum, maximum, denominator) per (sequence, split, head) that a second kernel merges in ascending order,
-// the layout and order of the CUDA-core kernel (attention_simt.cu).
+// the layout and order of the CUDA-core kernel (attention_simt.cu).  With a sink (one learned number per head) the softmax's
+// denominator also holds exp(sink): it joins once, where a row's sums are complete.
 #include "mma_helpers.cuh"
 #include <math.h>
 #include <atomic>
@@ -40,6 +41,7 @@ struct LatParams {
     int* status;
     int n_buf;                                      // key buffers in shared memory: 2 (tile i + 1 loads under tile i) or 1
     int split_p;                                    // 1: the softmax weights enter P V in two bfloat16 terms
+    const float* sink;                              // [n_heads] or null: exp(sink[h]) joins the softmax's denominator
 };
 
 __device__ __forceinline__ void ldmatrix_x2(uint32_t addr, uint32_t& r0, uint32_t& r1) {
@@ -268,7 +270,11 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_kernel(const LatP
             }
             if (warp == 0 && (lane & 3) == 0) { dst[lat] = stat_m[r]; dst[lat + 1] = stat_l[r]; }
         } else {
-            const float inv = 1.0f / stat_l[r];
+            float inv = 1.0f / stat_l[r];
+            if (p.sink != nullptr) {
+                const float sk = p.sink[h], M = fmaxf(stat_m[r], sk), e = __expf(stat_m[r] - M);
+                inv = e / fmaf(stat_l[r], e, __expf(sk - M));
+            }
             __nv_bfloat16* dst = p.out + (size_t)(row0 + q_off + tl) * p.out_stride + (size_t)h * lat;
 #pragma unroll
             for (int n = 0; n < NT_MAX; ++n) {
@@ -302,8 +308,10 @@ __global__ void latent_merge_kernel(const LatParams p) {
     float M = -INFINITY;
 #pragma unroll 4
     for (int s = 0; s < n_splits; ++s) M = fmaxf(M, base[s * split_stride + lat]);
+    if (p.sink != nullptr) M = fmaxf(M, p.sink[h]);
     if (threadIdx.x < 32) {
-        float den = 0.f;                                      // lanes take splits in turn, added lane by lane: a fixed order
+        float den = p.sink != nullptr && threadIdx.x == 0 ? __expf(p.sink[h] - M) : 0.f;
+        // lanes take splits in turn, added lane by lane: a fixed order
         for (int s = threadIdx.x; s < n_splits; s += 32) {
             const float* ps = base + s * split_stride;
             const float e = __expf(ps[lat] - M);
@@ -358,7 +366,7 @@ RS_EXPORT int rs_attention_latent_bf16(const void* q, long q_stride, void* out, 
                                        int table_stride, const int* q_start, const int* kv_len, const int* work, int n_work,
                                        int n_heads, int lat, int window, float scale, int decode, int split_keys,
                                        int max_splits, const int* split_start, float* partial, int partial_slots,
-                                       int split_p, int* status, void* stream) {
+                                       int split_p, const float* sink, int* status, void* stream) {
     if (n_work <= 0) return 0;
     if (!rs_attention_latent_supported(n_heads, lat, page_size) || q_stride % 8 || out_stride % 2 || page_stride % 8 ||
         ((size_t)q & 15) || ((size_t)cache & 15) || ((size_t)out & 3))
@@ -373,7 +381,7 @@ RS_EXPORT int rs_attention_latent_bf16(const void* q, long q_stride, void* out, 
     p.n_heads = n_heads; p.lat = lat; p.hc = heads_per_cta(n_heads, decode); p.tok_per_cta = decode ? 1 : ROWS / p.hc;
     p.window = window; p.scale = scale; p.decode = decode; p.split_keys = split_keys; p.max_splits = max_splits;
     p.split_start = split_start; p.partial = partial; p.partial_slots = partial_slots; p.status = status;
-    p.split_p = split_p ? 1 : 0;
+    p.split_p = split_p ? 1 : 0; p.sink = sink;
     p.n_buf = latent_smem_bytes(lat, 2) <= HALF_SM_SMEM ? 2 : 1;
     const size_t smem = latent_smem_bytes(lat, p.n_buf);
     static std::atomic<size_t> smem_allowed[64];

@@ -41,6 +41,7 @@ struct AttnParams {
     float scale;
     const float* slopes;                   // [n_q] or null: slopes[h] * (key position - query position) is added to a score
     const float* dist_bias; int n_dist;    // [n_dist][n_q] or null: dist_bias[min(query - key position, n_dist - 1)][h] is added
+    const float* sink;                     // [n_q] or null: exp(sink[h]) joins the softmax's denominator
     int decode, split_keys, max_splits;
     const int* split_start;                // decode: [n_work] first partial slot of each sequence
     float* partial;                        // decode: [slot][n_q][hd + 2], slot = split_start[w] + split
@@ -175,7 +176,11 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kernel(const AttnP
             if (lane == 0) { dst[hd] = m[rr]; dst[hd + 1] = l[rr]; }
         } else {
             T* dst = (T*)p.out + (size_t)tok * p.out_stride + (size_t)h * hd;
-            const float inv = 1.0f / l[rr];
+            float inv = 1.0f / l[rr];
+            if (p.sink != nullptr) {
+                const float sk = p.sink[h], M = fmaxf(m[rr], sk), e = PRECISE ? expf(m[rr] - M) : __expf(m[rr] - M);
+                inv = e / fmaf(l[rr], e, PRECISE ? expf(sk - M) : __expf(sk - M));
+            }
 #pragma unroll
             for (int i = 0; i < HDL; ++i) { const int d = lane + 32 * i; if (d < hd) dst[d] = from_f32<T>(acc[rr][i] * inv); }
         }
@@ -199,9 +204,11 @@ __global__ void attention_merge_kernel(const AttnParams p) {
     const size_t split_stride = (size_t)p.n_q * (hd + 2);
     float M = -INFINITY;
     for (int s = 0; s < n_splits; ++s) M = fmaxf(M, base[s * split_stride + hd]);
+    if (p.sink != nullptr) M = fmaxf(M, p.sink[h]);
     T* dst = (T*)p.out + (size_t)p.q_start[seq] * p.out_stride + (size_t)h * hd;
     for (int d = threadIdx.x; d < hd; d += blockDim.x) {
         float num = 0.f, den = 0.f;
+        if (p.sink != nullptr) den = PRECISE ? expf(p.sink[h] - M) : __expf(p.sink[h] - M);
         for (int s = 0; s < n_splits; ++s) {
             const float* ps = base + s * split_stride;
             const float e = PRECISE ? expf(ps[hd] - M) : __expf(ps[hd] - M);
@@ -265,7 +272,7 @@ RS_EXPORT int rs_attention_simt(const void* q, long q_stride, void* out, long ou
                                 int table_stride, const int* q_start, const int* kv_len, const int* work, int n_work,
                                 int n_q, int n_kv, int hd, int window, float scale, int decode, int split_keys,
                                 int max_splits, const int* split_start, float* partial, int partial_slots,
-                                const float* slopes, const float* dist_bias, int n_dist, int one_plane, int* status,
+                                const float* slopes, const float* dist_bias, int n_dist, const float* sink, int one_plane, int* status,
                                 void* stream) {
     if (n_work <= 0) return 0;
     if (dist_bias != nullptr && n_dist <= 0) return (int)cudaErrorInvalidValue;
@@ -283,7 +290,7 @@ RS_EXPORT int rs_attention_simt(const void* q, long q_stride, void* out, long ou
     p.q_per_cta = decode ? 1 : ROWS / p.heads_per_cta;
     p.window = window; p.scale = scale; p.decode = decode; p.split_keys = split_keys; p.max_splits = max_splits;
     p.split_start = split_start; p.partial = partial; p.partial_slots = partial_slots; p.status = status;
-    p.slopes = slopes; p.dist_bias = dist_bias; p.n_dist = n_dist;
+    p.slopes = slopes; p.dist_bias = dist_bias; p.n_dist = n_dist; p.sink = sink;
     p.v_offset = one_plane ? 0 : (long)n_kv * page_size * hd;
     cudaStream_t s = (cudaStream_t)stream;
     if (dt == RS_F32) return dispatch_hd<float, true>(p, n_work, s);
@@ -372,6 +379,7 @@ RS_EXPORT int rs_attention_decode_noalloc(const void* q, long q_stride, void* ou
     p.q_per_cta = 1;
     p.window = window; p.scale = scale; p.decode = 1; p.split_keys = split_keys; p.max_splits = max_splits;
     p.split_start = split_start; p.partial = partial; p.status = status; p.slopes = nullptr; p.dist_bias = nullptr; p.n_dist = 0;
+    p.sink = nullptr;
     p.v_offset = (long)n_kv * page_size * hd;
     // what the array really holds for this shape, not what the caller said it would use: a split list that
     // disagrees with total_splits is flagged by the kernels (RS_STATUS_BAD_PLAN) instead of written past the array

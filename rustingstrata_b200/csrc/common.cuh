@@ -68,6 +68,16 @@ __device__ __forceinline__ float fast_exp2(float x) {
     return y;
 }
 
+// What a product's output row is multiplied by on its way out, in float32: scale * sigmoid(g), g one number per (row, block
+// of columns) or per (row, column); scale alone without a gate.
+struct OutputGate {
+    const float* g; long stride; int per_block; float scale;
+    __device__ __forceinline__ float factor(long row, int block, int col) const {
+        if (g == nullptr) return scale;
+        return scale / (1.0f + expf(-g[row * stride + (per_block ? block : col)]));
+    }
+};
+
 // four weights (float32 or bfloat16, by code) from element 4 i on; four values rounded to bfloat16 in 8 bytes
 __device__ __forceinline__ float4 load_weights4(const void* w, int w_dt, int i) {
     if (w_dt == RS_F32) return reinterpret_cast<const float4*>(w)[i];

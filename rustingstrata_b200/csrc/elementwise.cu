@@ -34,6 +34,35 @@ RS_EXPORT int rs_embed(const void* table, int table_dt, const int* ids, float* o
     return 0;
 }
 
+// The same followed by a norm: out[t, :] = e * rsqrt(mean(e^2) + eps) * w with e = table[ids[t], :].
+__global__ void embed_rmsnorm_kernel(const void* __restrict__ table, int table_dt, const int* __restrict__ ids,
+                                     const void* __restrict__ w, int w_dt, float eps, float* __restrict__ out, long out_stride, int H,
+                                     int V, int* status) {
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    int id = ld_dep(ids + t);
+    if (id < 0 || id >= V) {
+        if (threadIdx.x == 0) atomicOr(status, RS_STATUS_BAD_TOKEN);
+        id = 0;
+    }
+    const size_t row = (size_t)id * H;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) { const float v = load_any(table, table_dt, row + i); ss = fmaf(v, v, ss); }
+    ss = block_sum(ss, scratch);
+    const float s = 1.0f / sqrtf(ss / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += blockDim.x)
+        out[(size_t)t * out_stride + i] = load_any(table, table_dt, row + i) * s * load_any(w, w_dt, i);
+}
+
+RS_EXPORT int rs_embed_rmsnorm(const void* table, int table_dt, const int* ids, const void* w, int w_dt, float eps, float* out,
+                               long out_stride, int n_tokens, int H, int V, int* status, void* stream) {
+    if (n_tokens <= 0) return 0;
+    return rs_launch_pdl(embed_rmsnorm_kernel, dim3(n_tokens), dim3(H >= 2048 ? 512 : 256), 0, (cudaStream_t)stream, table, table_dt,
+                         ids, w, w_dt, eps, out, out_stride, H, V, status);
+}
+
 // --------------------------------------------------------------------------- RMSNorm
 // out[r, i] = x[src(r), i] * rsqrt(mean(x[src(r), :]^2) + eps) * w[i], src(r) = rows ? rows[r] : r.
 // x is the float32 residual stream; w is float32 or bfloat16; out is the activation type.
@@ -430,6 +459,76 @@ RS_EXPORT int rs_add_embed(float* x, long x_stride, const void* table, int table
     if (n_tokens <= 0) return 0;
     return rs_launch_pdl(add_embed_kernel, dim3(n_tokens), dim3(n >= 512 ? 256 : 128), 0, (cudaStream_t)stream, x, x_stride, table, table_dt,
                          ids, V, scale, n, status);
+}
+
+// out[t, c] = gelu(z[t, c]) * table[ids[t], col0 + c] with the tanh form of GELU in float32: a projection gated by a part of
+// the token's row in a table.
+template <typename TO>
+__global__ void gelu_table_gate_kernel(const float* z, long z_stride, const void* __restrict__ table, int table_dt, long table_stride,
+                                       int V, int col0, const int* __restrict__ ids, TO* out, long out_stride, int n, long total,
+                                       int* status) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= total) return;
+    const long t = idx / n;
+    const int c = (int)(idx - t * n);
+    int id = ld_dep(ids + t);
+    if (id < 0 || id >= V) { atomicOr(status, RS_STATUS_BAD_TOKEN); id = 0; }
+    const float v = ld_dep(z + t * z_stride + c);
+    const float g = 0.5f * v * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * v * v, v, v)));
+    out[t * out_stride + c] = from_f32<TO>(g * load_any(table, table_dt, (size_t)id * table_stride + col0 + c));
+}
+
+RS_EXPORT int rs_gelu_table_gate(const float* z, long z_stride, const void* table, int table_dt, long table_stride, int V, int col0,
+                                 const int* ids, void* out, int out_dt, long out_stride, int n_tokens, int n, int* status,
+                                 void* stream) {
+    const long total = (long)n_tokens * n;
+    if (total <= 0) return 0;
+    RS_DISPATCH_DTYPE(out_dt, TO,
+        return rs_launch_pdl(gelu_table_gate_kernel<TO>, dim3((unsigned)((total + 127) / 128)), dim3(128), 0, (cudaStream_t)stream, z,
+                             z_stride, table, table_dt, table_stride, V, col0, ids, (TO*)out, out_stride, n, total, status));
+    return 0;
+}
+
+// out[r, c] = x[r, c] in the activation type
+template <typename TO>
+__global__ void cast_rows_kernel(const float* x, long x_stride, TO* out, long out_stride, int n, long total) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= total) return;
+    const long r = idx / n;
+    const int c = (int)(idx - r * n);
+    out[r * out_stride + c] = from_f32<TO>(ld_dep(x + r * x_stride + c));
+}
+
+RS_EXPORT int rs_cast_rows(const float* x, long x_stride, void* out, int out_dt, long out_stride, int n_rows, int n, void* stream) {
+    const long total = (long)n_rows * n;
+    if (total <= 0) return 0;
+    RS_DISPATCH_DTYPE(out_dt, TO,
+        return rs_launch_pdl(cast_rows_kernel<TO>, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, x,
+                             x_stride, (TO*)out, out_stride, n, total));
+    return 0;
+}
+
+// x[r, c] = cap * tanh(x[r, c] * scale / cap) in place
+__global__ void softcap_rows_kernel(float* x, long stride, int n, long total, float scale, float cap) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= total) return;
+    const long r = idx / n;
+    float* p = x + r * stride + (idx - r * n);
+    *p = cap * tanhf(ld_dep(p) * scale / cap);
+}
+
+RS_EXPORT int rs_softcap_rows(float* x, long stride, int n_rows, int n, float scale, float cap, void* stream) {
+    const long total = (long)n_rows * n;
+    if (total <= 0) return 0;
+    if (!(cap > 0.f)) return (int)cudaErrorInvalidValue;
+    return rs_launch_pdl(softcap_rows_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, x, stride, n,
+                         total, scale, cap);
 }
 
 // dst[i] = src[idx[i]]: the ids a step chose, brought into the order of the next step's rows on the device

@@ -22,6 +22,7 @@ struct GroupedMmaParams {
     const int* order; const int* tiles; const int* n_tiles;        // tiles == null: every expert takes all dense_rows rows
     int dense_rows, tiles_per_expert;
     int K, gated;                                                  // gated: 0 plain; 1 SiLU(gate) * up of alternating rows; 2 plain, then max(., 0)^2
+    int use_gate; OutputGate gate;                                 // plain products of blocks: the result times gate.factor(row, expert, column)
 };
 
 // BM x BN: the CTA's tile; WM x WN warps, each owning (BM / WM) x (BN / WN) of it.  64 x 64 with 2 x 2 warps where an
@@ -138,6 +139,10 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
                     c0 = fmaxf(c0, 0.f); c0 *= c0;
                     c1 = fmaxf(c1, 0.f); c1 *= c1;
                 }
+                if (p.use_gate) {
+                    if (gn < p.w_rows) c0 *= p.gate.factor(pr, e, e * p.w_rows + gn);
+                    if (gn + 1 < p.w_rows) c1 *= p.gate.factor(pr, e, e * p.w_rows + gn + 1);
+                }
                 if (p.gated == 1) {
                     if (gn + 1 < p.w_rows) {
                         const float v = silu_mul_fast(c0, c1);
@@ -174,7 +179,7 @@ RS_EXPORT int rs_grouped_gemm_mma(const void* a, long a_stride, int a_div, const
     if (K <= 0 || K % 8 || a_stride % 8 || w_expert_stride % 8 || ((size_t)a & 15) || ((size_t)w & 15) || (gated == 1 && w_rows % 2) || gated < 0 || gated > 2)
         return (int)cudaErrorInvalidValue;
     GroupedMmaParams p{a, RS_BF16, a_stride, a_div, 0, (const __nv_bfloat16*)w, w_expert_stride, w_rows, nullptr, 0, out, out_dt,
-                       out_stride, 0, order, tiles, n_tiles, 0, 1, K, gated};
+                       out_stride, 0, order, tiles, n_tiles, 0, 1, K, gated, 0, OutputGate{nullptr, 0, 0, 1.0f}};
     if (large) grouped_gemm_mma_kernel<128, 128, 2, 4><<<dim3((w_rows + 127) / 128, max_tiles), 256, 0, (cudaStream_t)stream>>>(p);
     else grouped_gemm_mma_kernel<64, 64, 2, 2><<<dim3((w_rows + 63) / 64, max_tiles), 128, 0, (cudaStream_t)stream>>>(p);
     return rs_launch_result();
@@ -182,11 +187,12 @@ RS_EXPORT int rs_grouped_gemm_mma(const void* a, long a_stride, int a_div, const
 
 // The block-diagonal product of sequence_parts.cu (rs_block_linear) for more than a few rows, through the same kernel:
 // block b is an "expert" that takes every row, reads columns from b * in_bs and writes columns from b * out_bs.
-//   out[t, b * out_bs + o] = bias[b, o] + sum_i W[b, o, i] * x[t, b * in_bs + i]
+//   out[t, b * out_bs + o] = (bias[b, o] + sum_i W[b, o, i] * x[t, b * in_bs + i]) * out_scale * sigmoid(gate)
+// (gate as in rs_block_linear; null: none).
 // x: bfloat16, or float32 (rounded to bfloat16 as it enters the product); W: bfloat16 [B, O, I], I a multiple of 8.
 RS_EXPORT int rs_block_linear_mma(const void* x, int x_dt, long x_stride, long in_bs, const void* w, const void* bias,
                                   int bias_dt, void* out, int out_dt, long out_stride, long out_bs, int T, int B, int O,
-                                  int I, void* stream) {
+                                  int I, const float* gate, long gate_stride, int gate_per_block, float out_scale, void* stream) {
     if (T <= 0 || B <= 0 || O <= 0) return 0;
     const int align = x_dt == RS_F32 ? 4 : 8;                  // elements per 16 bytes
     if (I <= 0 || I % 8 || x_stride % align || in_bs % align || ((size_t)x & 15) || ((size_t)w & 15))
@@ -194,7 +200,8 @@ RS_EXPORT int rs_block_linear_mma(const void* x, int x_dt, long x_stride, long i
     const int bm = T > 256 ? 128 : 64;
     const int tiles_per = (T + bm - 1) / bm;
     GroupedMmaParams p{x, x_dt, x_stride, 1, in_bs, (const __nv_bfloat16*)w, (long)O * I, O, bias, bias_dt, out, out_dt, out_stride,
-                       out_bs, nullptr, nullptr, nullptr, T, tiles_per, I, 0};
+                       out_bs, nullptr, nullptr, nullptr, T, tiles_per, I, 0, gate != nullptr || out_scale != 1.0f,
+                       OutputGate{gate, gate_stride, gate_per_block, out_scale}};
     if (bm == 128) grouped_gemm_mma_kernel<128, 128, 2, 4><<<dim3((O + 127) / 128, tiles_per * B), 256, 0, (cudaStream_t)stream>>>(p);
     else grouped_gemm_mma_kernel<64, 64, 2, 2><<<dim3((O + 63) / 64, tiles_per * B), 128, 0, (cudaStream_t)stream>>>(p);
     return rs_launch_result();

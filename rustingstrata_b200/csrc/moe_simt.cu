@@ -7,8 +7,10 @@
 //     Epilogues: plain store, or SiLU(gate) * up with gate rows [0, N) and up rows [N, 2N) of the expert's matrix.
 //     A tile of at most 8 rows takes the row-streaming form (a warp per output column, the expert's matrix read
 //     once, coalesced); larger tiles the 64 x 64 register-tiled form;
-//   * moe_combine: out[t] = sum_k pair_out[t, k] * weight + sigmoid(h[t] . w_gate) * shared[t], the sum over k in
-//     ascending k, so a token's result does not depend on the batch.
+//   * moe_combine: out[t] = sum_k pair_out[t, k] * weight + gate[t] * shared[t], the sum over k in ascending k, so a token's
+//     result does not depend on the batch; a pair whose choice is an identity expert contributes h[t]; the whole may be
+//     scaled, added to the residual stream, and the stream's new row left in the activation type for its next reader.
+// Choices from E on (up to ``identity`` of them) are identity experts: they have no matrices and get no rows in the lists.
 // Every pair's row is computed with k ascending whatever else is in the batch.
 #include "common.cuh"
 #include <math.h>
@@ -23,7 +25,7 @@ constexpr int MAX_EXPERTS = 4096;
 
 // order[P]: pair ids (t * top + k) grouped by expert; tiles[i] = (expert, first row in order, rows); n_tiles[0].
 __global__ void __launch_bounds__(1024) moe_route_kernel(const int* __restrict__ ids, const int* __restrict__ table, int V,
-                                                         int top, int E, int n_tokens, int rows_per_tile,
+                                                         int top, int E, int identity, int n_tokens, int rows_per_tile,
                                                          int* __restrict__ order, int* __restrict__ tiles,
                                                          int* __restrict__ n_tiles, int max_tiles, int* status) {
     __shared__ int counts[MAX_EXPERTS];
@@ -35,6 +37,7 @@ __global__ void __launch_bounds__(1024) moe_route_kernel(const int* __restrict__
         int id = ids != nullptr ? ids[pr / top] : pr / top;        // without ids the table has one row per token of the step
         if (id < 0 || id >= V) { atomicOr(status, RS_STATUS_BAD_TOKEN); id = 0; }
         int e = table[(size_t)id * top + pr % top];
+        if (e >= E && e < E + identity) continue;
         if (e < 0 || e >= E) { atomicOr(status, RS_STATUS_BAD_PLAN); e = 0; }
         atomicAdd(&counts[e], 1);
     }
@@ -60,16 +63,17 @@ __global__ void __launch_bounds__(1024) moe_route_kernel(const int* __restrict__
         int id = ids != nullptr ? ids[pr / top] : pr / top;
         if (id < 0 || id >= V) id = 0;
         int e = table[(size_t)id * top + pr % top];
+        if (e >= E && e < E + identity) continue;
         if (e < 0 || e >= E) e = 0;
         order[atomicAdd(&cursor[e], 1)] = pr;
     }
 }
 
-RS_EXPORT int rs_moe_route(const int* ids, const int* table, int V, int top, int E, int n_tokens, int rows_per_tile,
+RS_EXPORT int rs_moe_route(const int* ids, const int* table, int V, int top, int E, int identity, int n_tokens, int rows_per_tile,
                            int* order, int* tiles, int* n_tiles, int max_tiles, int* status, void* stream) {
     if (n_tokens <= 0) return 0;
-    if (E <= 0 || E > MAX_EXPERTS || top <= 0 || rows_per_tile <= 0) return (int)cudaErrorInvalidValue;
-    moe_route_kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(ids, table, V, top, E, n_tokens, rows_per_tile, order, tiles,
+    if (E <= 0 || E > MAX_EXPERTS || identity < 0 || top <= 0 || rows_per_tile <= 0) return (int)cudaErrorInvalidValue;
+    moe_route_kernel<<<1, 1024, 0, (cudaStream_t)stream>>>(ids, table, V, top, E, identity, n_tokens, rows_per_tile, order, tiles,
                                                            n_tiles, max_tiles, status);
     return rs_launch_result();
 }
@@ -254,44 +258,103 @@ RS_EXPORT int rs_grouped_linear(const void* a, int a_dt, long a_stride, int a_di
     return rs_launch_result();
 }
 
-// out[t, :] = weight * sum_k (pair_w[t * top + k] or 1) * pair_out[t * top + k, :] + sigmoid(h[t, :] . gate_w) * shared[t, :]
-// (shared == null: no shared expert).  out is float32 [T, n].
-__global__ void moe_combine_kernel(const float* __restrict__ pair_out, long pair_stride, int top, float weight,
-                                   const float* __restrict__ pair_w,
-                                   const void* __restrict__ shared, int shared_dt, long shared_stride,
-                                   const void* __restrict__ h, int h_dt, long h_stride, const void* __restrict__ gate_w,
-                                   int gate_dt, float* __restrict__ out, long out_stride, int n) {
+// y[t, :] = scale * (weight * sum_k (pair_w[t * top + k] or 1) * v_k + g * shared[t, :]), where v_k is pair_out[t * top + k, :],
+// or h[t, :] for a pair whose choice is an identity expert (choice[t * top + k] >= n_experts), and g is 1,
+// sigmoid(gate_z[t]) or sigmoid(h[t, :] . gate_w) (shared == null: no shared expert).
+// out (float32 [T, n]) = y, or += y with ``accumulate``; copy (activation type), when given, takes out's new row as well.
+struct CombineParams {
+    const float* pair_out; long pair_stride; int top; float weight; const float* pair_w; const int* choice; int n_experts;
+    const void* shared; int shared_dt; long shared_stride;
+    const void* h; int h_dt; long h_stride;
+    const void* gate_w; int gate_dt; const float* gate_z; long gate_z_stride;
+    float* out; long out_stride; float scale; int accumulate;
+    void* copy; int copy_dt; long copy_stride;
+    int n;
+};
+
+__device__ __forceinline__ float4 load4_any(const void* p, int dt, size_t i) {       // i a multiple of 4
+    if (dt == RS_F32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);
+    return load_weights4(reinterpret_cast<const __nv_bfloat16*>(p) + i, RS_BF16, 0);
+}
+
+template <int V>      // columns a thread takes at a time: 4 (16-byte aligned rows) or 1
+__global__ void __launch_bounds__(256) moe_combine_kernel(const CombineParams p) {
     __shared__ float scratch[33];
     const int t = blockIdx.x;
-    float gate = 0.f;
-    if (shared != nullptr && gate_w != nullptr) {
+    float gate = p.shared != nullptr ? 1.0f : 0.f;
+    if (p.shared != nullptr && p.gate_z != nullptr) {
+        gate = 1.0f / (1.0f + expf(-p.gate_z[(size_t)t * p.gate_z_stride]));
+    } else if (p.shared != nullptr && p.gate_w != nullptr) {
         float d = 0.f;
-        for (int i = threadIdx.x; i < n; i += blockDim.x)
-            d = fmaf(load_any(h, h_dt, (size_t)t * h_stride + i), load_any(gate_w, gate_dt, i), d);
+        for (int i = threadIdx.x; i < p.n; i += blockDim.x)
+            d = fmaf(load_any(p.h, p.h_dt, (size_t)t * p.h_stride + i), load_any(p.gate_w, p.gate_dt, i), d);
         d = block_sum(d, scratch);
         gate = 1.0f / (1.0f + expf(-d));
-    } else if (shared != nullptr) {
-        gate = 1.0f;
     }
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-        float v = 0.f;
-        if (pair_w != nullptr) {             // every pair with a weight of its own, k ascending
-            for (int k = 0; k < top; ++k) v = fmaf(pair_w[(size_t)t * top + k], pair_out[(size_t)(t * top + k) * pair_stride + i], v);
-        } else {
-            for (int k = 0; k < top; ++k) v += pair_out[(size_t)(t * top + k) * pair_stride + i];
+    for (int i = threadIdx.x * V; i < p.n; i += blockDim.x * V) {
+        float v[V];
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] = 0.f;
+        for (int k = 0; k < p.top; ++k) {                    // k ascending
+            const size_t pr = (size_t)t * p.top + k;
+            const float w = p.pair_w != nullptr ? p.pair_w[pr] : 1.0f;
+            const bool identity = p.choice != nullptr && p.choice[pr] >= p.n_experts;
+            const void* src = identity ? p.h : (const void*)p.pair_out;
+            const int dt = identity ? p.h_dt : (int)RS_F32;
+            const size_t at = identity ? (size_t)t * p.h_stride + i : pr * p.pair_stride + i;
+            if (V == 4) {
+                const float4 u = load4_any(src, dt, at);
+                v[0] = fmaf(w, u.x, v[0]); v[1 % V] = fmaf(w, u.y, v[1 % V]); v[2 % V] = fmaf(w, u.z, v[2 % V]); v[3 % V] = fmaf(w, u.w, v[3 % V]);
+            } else {
+                v[0] = fmaf(w, load_any(src, dt, at), v[0]);
+            }
         }
-        v *= weight;
-        if (shared != nullptr) v = fmaf(gate, load_any(shared, shared_dt, (size_t)t * shared_stride + i), v);
-        out[(size_t)t * out_stride + i] = v;
+        float sh[V];
+#pragma unroll
+        for (int j = 0; j < V; ++j) sh[j] = 0.f;
+        if (p.shared != nullptr) {
+            if (V == 4) {
+                const float4 u = load4_any(p.shared, p.shared_dt, (size_t)t * p.shared_stride + i);
+                sh[0] = u.x; sh[1 % V] = u.y; sh[2 % V] = u.z; sh[3 % V] = u.w;
+            } else {
+                sh[0] = load_any(p.shared, p.shared_dt, (size_t)t * p.shared_stride + i);
+            }
+        }
+        float* o = p.out + (size_t)t * p.out_stride + i;
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] = p.scale * fmaf(gate, sh[j], v[j] * p.weight);
+        if (V == 4) {
+            float4* o4 = reinterpret_cast<float4*>(o);
+            if (p.accumulate) { const float4 x = *o4; v[0] += x.x; v[1 % V] += x.y; v[2 % V] += x.z; v[3 % V] += x.w; }
+            *o4 = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
+        } else {
+            if (p.accumulate) v[0] += o[0];
+            o[0] = v[0];
+        }
+        if (p.copy != nullptr) {
+            const size_t at = (size_t)t * p.copy_stride + i;
+            if (V == 4 && p.copy_dt == RS_BF16)
+                *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.copy) + at) = pack_bf16x4(v[0], v[1 % V], v[2 % V], v[3 % V]);
+            else
+#pragma unroll
+                for (int j = 0; j < V; ++j) store_any(p.copy, p.copy_dt, at + j, v[j]);
+        }
     }
 }
 
-RS_EXPORT int rs_moe_combine(const float* pair_out, long pair_stride, int top, float weight, const float* pair_w, const void* shared,
-                             int shared_dt, long shared_stride, const void* h, int h_dt, long h_stride, const void* gate_w,
-                             int gate_dt, float* out, long out_stride, int n_tokens, int n, void* stream) {
+RS_EXPORT int rs_moe_combine(const float* pair_out, long pair_stride, int top, float weight, const float* pair_w, const int* choice,
+                             int n_experts, const void* shared, int shared_dt, long shared_stride, const void* h, int h_dt,
+                             long h_stride, const void* gate_w, int gate_dt, const float* gate_z, long gate_z_stride, float* out,
+                             long out_stride, float scale, int accumulate, void* copy, int copy_dt, long copy_stride, int n_tokens,
+                             int n, void* stream) {
     if (n_tokens <= 0) return 0;
-    moe_combine_kernel<<<n_tokens, 256, 0, (cudaStream_t)stream>>>(pair_out, pair_stride, top, weight, pair_w, shared, shared_dt,
-                                                                  shared_stride, h, h_dt, h_stride, gate_w, gate_dt, out,
-                                                                  out_stride, n);
+    if ((choice != nullptr || gate_w != nullptr) && h == nullptr) return (int)cudaErrorInvalidValue;
+    CombineParams p{pair_out, pair_stride, top, weight, pair_w, choice, n_experts, shared, shared_dt, shared_stride, h, h_dt, h_stride,
+                    gate_w, gate_dt, gate_z, gate_z_stride, out, out_stride, scale, accumulate, copy, copy_dt, copy_stride, n};
+    auto ok = [](const void* q, int dt, long stride) { return q == nullptr || ((size_t)q % (dt == RS_F32 ? 16 : 8) == 0 && stride % 4 == 0); };
+    const bool vec = n % 4 == 0 && ok(pair_out, RS_F32, pair_stride) && ok(shared, shared_dt, shared_stride) && ok(h, h_dt, h_stride) &&
+                     ok(out, RS_F32, out_stride) && ok(copy, copy_dt, copy_stride);
+    if (vec) moe_combine_kernel<4><<<n_tokens, 256, 0, (cudaStream_t)stream>>>(p);
+    else moe_combine_kernel<1><<<n_tokens, 256, 0, (cudaStream_t)stream>>>(p);
     return rs_launch_result();
 }

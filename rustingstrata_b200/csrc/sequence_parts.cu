@@ -263,8 +263,9 @@ RS_EXPORT int rs_short_conv(const void* in, int in_dt, long in_stride, const voi
 }
 
 // --------------------------------------------------------------------------- block-diagonal matrix product
-// out[t, b * out_bs + o] = bias[b * O + o] + sum_i W[b, o, i] * in[t, b * in_bs + i],  o < O, i < I, b < B.
-// W: [B, O, I] contiguous.  Tiles of 64 x 64 outputs, k ascending per output element.
+// out[t, b * out_bs + o] = (bias[b * O + o] + sum_i W[b, o, i] * in[t, b * in_bs + i]) * f,  o < O, i < I, b < B,
+// f = out_scale * sigmoid(gate) in float32, gate one float32 number per token and block (gate_per_block) or per token and
+// output, or f = out_scale without a gate.  W: [B, O, I] contiguous.  Tiles of 64 x 64 outputs, k ascending per output element.
 namespace {
 constexpr int BL_BM = 64, BL_BN = 64, BL_BK = 16;
 
@@ -274,6 +275,7 @@ struct BlockLinearParams {
     const void* bias; int bias_dt;
     void* out; int out_dt; long out_stride; long out_bs;
     int T, O, I;
+    OutputGate gate;
 };
 
 __global__ void __launch_bounds__(256) block_linear_kernel(const BlockLinearParams p) {
@@ -322,6 +324,7 @@ __global__ void __launch_bounds__(256) block_linear_kernel(const BlockLinearPara
             if (gn >= p.O) continue;
             float v = acc[i][j];
             if (p.bias != nullptr) v += load_any(p.bias, p.bias_dt, (size_t)b * p.O + gn);
+            v *= p.gate.factor(gm, b, b * p.O + gn);
             store_any(p.out, p.out_dt, (size_t)gm * p.out_stride + (size_t)b * p.out_bs + gn, v);
         }
     }
@@ -383,6 +386,7 @@ __global__ void __launch_bounds__(256) block_linear_rows_kernel(const BlockLinea
             float v = warp_sum(acc[c][r]);
             if (lane == 0 && o < p.O && r < p.T) {
                 if (p.bias != nullptr) v += load_any(p.bias, p.bias_dt, (size_t)b * p.O + o);
+                v *= p.gate.factor(r, b, b * p.O + o);
                 store_any(p.out, p.out_dt, (size_t)r * p.out_stride + (size_t)b * p.out_bs + o, v);
             }
         }
@@ -392,9 +396,11 @@ __global__ void __launch_bounds__(256) block_linear_rows_kernel(const BlockLinea
 
 RS_EXPORT int rs_block_linear(const void* in, int in_dt, long in_stride, long in_bs, const void* w, int w_dt,
                               const void* bias, int bias_dt, void* out, int out_dt, long out_stride, long out_bs, int T,
-                              int B, int O, int I, void* stream) {
+                              int B, int O, int I, const float* gate, long gate_stride, int gate_per_block, float out_scale,
+                              void* stream) {
     if (T <= 0 || B <= 0 || O <= 0) return 0;
-    BlockLinearParams p{in, in_dt, in_stride, in_bs, w, w_dt, bias, bias_dt, out, out_dt, out_stride, out_bs, T, O, I};
+    BlockLinearParams p{in, in_dt, in_stride, in_bs, w, w_dt, bias, bias_dt, out, out_dt, out_stride, out_bs, T, O, I,
+                        OutputGate{gate, gate_stride, gate_per_block, out_scale}};
     if (T <= BR_ROWS) {
         block_linear_rows_kernel<<<dim3((O + BR_COLS - 1) / BR_COLS, B), 256, 0, (cudaStream_t)stream>>>(p);
         return rs_launch_result();
@@ -557,6 +563,8 @@ RS_EXPORT int rs_gated_linear_recurrence(const float* gates, long gates_stride, 
 // and for every head h: q_lat[t, h * lat + rank + j] = rotate(q[t, h * q_head + q_nope + j]) for j < rot, zeros up to lat.
 // The rotation turns the pairs (2i, 2i + 1), i < n_rot / 2, by the angle whose cosine and sine lie in
 // cos_sin[position][i] and cos_sin[position][n_rot / 2 + i]; coordinates from n_rot on pass unchanged.
+// A query that comes through a latent of its own: c_q[t] = cq[t] * rsqrt(mean(cq^2) + eps) * cq_w besides; the rotation of the
+// queries, which are made from c_q, is then a launch of its own (cache == null).
 struct LatentParams {
     const float* dkv; long dkv_stride;
     const void* norm_w; int norm_dt; float eps;
@@ -567,6 +575,7 @@ struct LatentParams {
     const int* seq_of_token; const int* block_table; int table_stride, page_size;
     void* cache; int cache_dt; long page_stride; int num_pages;
     int rank, rot, lat, heads, n_tokens;
+    const float* cq; long cq_stride; const void* cq_w; int cq_w_dt; void* cq_out; int cq_dt; long cq_out_stride; int q_rank;
     int* status;
 };
 
@@ -602,6 +611,15 @@ __global__ void latent_kv_write_kernel(const LatentParams p) {
         }
         store_any(p.q_lat, p.q_lat_dt, (size_t)t * p.q_lat_stride + (size_t)h * p.lat + p.rank + j, v);
     }
+    if (p.cq_out != nullptr) {
+        const float* row = p.cq + (size_t)t * p.cq_stride;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
+        ss = block_sum(ss, scratch);
+        const float s = 1.0f / sqrtf(ss / (float)p.q_rank + p.eps);
+        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x)
+            store_any(p.cq_out, p.cq_dt, (size_t)t * p.cq_out_stride + i, row[i] * s * load_any(p.cq_w, p.cq_w_dt, i));
+    }
     if (p.cache == nullptr) return;
     const int page = p.block_table[(size_t)p.seq_of_token[t] * p.table_stride + pos / p.page_size];
     if (page < 0 || page >= p.num_pages) {
@@ -630,63 +648,16 @@ RS_EXPORT int rs_latent_kv_write(const float* dkv, long dkv_stride, const void* 
                                  long q_lat_stride, const float* cos_sin, int n_rot, int table_rows, const int* positions,
                                  int pos_stride, const int* seq_of_token, const int* block_table, int table_stride,
                                  int page_size, void* cache, int cache_dt, long page_stride, int num_pages, int rank, int rot,
-                                 int lat, int heads, int n_tokens, int* status, void* stream) {
+                                 int lat, int heads, int n_tokens, const float* cq, long cq_stride, const void* cq_w, int cq_w_dt,
+                                 void* cq_out, int cq_dt, long cq_out_stride, int q_rank, int* status, void* stream) {
     if (n_tokens <= 0) return 0;
+    if (cq_out != nullptr && (cq == nullptr || cq_w == nullptr || q_rank <= 0)) return (int)cudaErrorInvalidValue;
     if (n_rot % 2 || n_rot > rot || rank + rot > lat) return (int)cudaErrorInvalidValue;
     LatentParams p{dkv, dkv_stride, norm_w, norm_dt, eps, q, q_dt, q_stride, q_head, q_nope, q_lat, q_lat_dt, q_lat_stride,
                    cos_sin, n_rot, table_rows, positions, pos_stride, seq_of_token, block_table, table_stride, page_size,
-                   cache, cache_dt, page_stride, num_pages, rank, rot, lat, heads, n_tokens, status};
+                   cache, cache_dt, page_stride, num_pages, rank, rot, lat, heads, n_tokens, cq, cq_stride, cq_w, cq_w_dt, cq_out,
+                   cq_dt, cq_out_stride, q_rank, status};
     latent_kv_write_kernel<<<n_tokens, 128, 0, (cudaStream_t)stream>>>(p);
-    return rs_launch_result();
-}
-
-// --------------------------------------------------------------------------- a gate per head
-// a[t, h * dv + d] *= sigmoid(g[t, h]) in place; g float32 (pre-activations), the sigmoid in float32
-__global__ void head_sigmoid_gate_kernel(void* __restrict__ a, int dt, long a_stride, const float* __restrict__ g, long g_stride,
-                                         int heads, int dv, long n) {
-    const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (idx >= n) return;
-    const int w = heads * dv;
-    const long t = idx / w;
-    const int c = (int)(idx % w);
-    const float z = g[t * g_stride + c / dv];
-    const size_t at = (size_t)t * a_stride + c;
-    store_any(a, dt, at, load_any(a, dt, at) * (1.0f / (1.0f + expf(-z))));
-}
-
-// the same with 16 bytes per thread: eight bfloat16 or four float32 values of one head (dv a multiple of that many,
-// rows and the pointer aligned to 16 bytes)
-template <typename T>
-__global__ void head_sigmoid_gate_vec_kernel(T* __restrict__ a, long a_stride, const float* __restrict__ g, long g_stride,
-                                             int heads, int dv, long n_pieces) {
-    constexpr int V = 16 / sizeof(T);
-    const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (idx >= n_pieces) return;
-    const int per_row = heads * dv / V;
-    const long t = idx / per_row;
-    const int c = (int)(idx % per_row) * V;
-    const float s = 1.0f / (1.0f + expf(-g[t * g_stride + c / dv]));
-    uint4* at = reinterpret_cast<uint4*>(a + (size_t)t * a_stride + c);
-    uint4 raw = *at;
-    T* v = reinterpret_cast<T*>(&raw);
-#pragma unroll
-    for (int i = 0; i < V; ++i) v[i] = from_f32<T>(to_f32<T>(v[i]) * s);
-    *at = raw;
-}
-
-RS_EXPORT int rs_head_sigmoid_gate(void* a, int dt, long a_stride, const float* g, long g_stride, int heads, int dv,
-                                   int n_tokens, void* stream) {
-    const long n = (long)n_tokens * heads * dv;
-    if (n <= 0) return 0;
-    const int v = dt == RS_F32 ? 4 : 8;
-    if ((dt == RS_F32 || dt == RS_BF16) && dv % v == 0 && a_stride % v == 0 && (uintptr_t)a % 16 == 0) {
-        const long pieces = n / v;
-        RS_DISPATCH_DTYPE(dt, T, (head_sigmoid_gate_vec_kernel<T><<<(unsigned)((pieces + 255) / 256), 256, 0, (cudaStream_t)stream>>>(
-            reinterpret_cast<T*>(a), a_stride, g, g_stride, heads, dv, pieces)));
-        return rs_launch_result();
-    }
-    head_sigmoid_gate_kernel<<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(a, dt, a_stride, g, g_stride, heads,
-                                                                                           dv, n);
     return rs_launch_result();
 }
 

@@ -167,11 +167,11 @@ __global__ void stream_update_kernel(const StreamUpdateParams p) {
 
 // one warp per token: scores = softmax(logits), or sigmoid(logits) each for itself (``sigmoid``); the `top` largest of
 // scores + correction are chosen (the lower index on a tie); with ``n_groups`` > 0 the experts form that many equal
-// groups of neighbours, a group is worth the sum of its two largest scores + correction, and only experts of the
+// groups of neighbours, a group is worth the sum of its two largest scores + correction (``worth_one``: its largest), and only experts of the
 // ``keep`` groups worth most can be chosen (the lower index on a tie); weights = the chosen experts' scores times
 // ``scale``, divided by (their sum + 1e-20) first when ``renorm`` is set
 __global__ void router_topk_kernel(const float* __restrict__ logits, long l_stride, const void* __restrict__ corr,
-                                   int corr_dt, int E, int top, int n_tokens, int sigmoid, int n_groups, int keep, float scale,
+                                   int corr_dt, int E, int top, int n_tokens, int sigmoid, int n_groups, int keep, int worth_one, float scale,
                                    int renorm, int* __restrict__ choice, float* __restrict__ weight, int* status) {
     extern __shared__ float sm[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, wpb = blockDim.x >> 5;
@@ -210,7 +210,7 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, long l_stri
                 const float v = pick[e];
                 if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
             }
-            worth[g] = per > 1 ? a + b : a;
+            worth[g] = per > 1 && !worth_one ? a + b : a;
             kept[g] = 0.f;
         }
         __syncwarp();
@@ -304,7 +304,7 @@ RS_EXPORT int rs_stream_update(float* x, long x_stride, const float* y, long y_s
 }
 
 RS_EXPORT int rs_router_topk(const float* logits, long l_stride, const void* corr, int corr_dt, int E, int top, int n_tokens,
-                             int sigmoid, int n_groups, int keep, float scale, int renorm, int* choice, float* weight, int* status,
+                             int sigmoid, int n_groups, int keep, int worth_one, float scale, int renorm, int* choice, float* weight, int* status,
                              void* stream) {
     if (n_tokens <= 0) return 0;
     if (E <= 0 || top <= 0 || top > E || E > 1024) return (int)cudaErrorInvalidValue;
@@ -313,6 +313,6 @@ RS_EXPORT int rs_router_topk(const float* logits, long l_stride, const void* cor
     const int wpb = 4;
     router_topk_kernel<<<(n_tokens + wpb - 1) / wpb, wpb * 32, (size_t)wpb * (2 * E + 2 * n_groups) * sizeof(float),
                          (cudaStream_t)stream>>>(
-        logits, l_stride, corr, corr_dt, E, top, n_tokens, sigmoid, n_groups, keep, scale, renorm, choice, weight, status);
+        logits, l_stride, corr, corr_dt, E, top, n_tokens, sigmoid, n_groups, keep, worth_one, scale, renorm, choice, weight, status);
     return rs_launch_result();
 }

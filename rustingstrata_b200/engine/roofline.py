@@ -44,8 +44,9 @@ def peaks(path: Optional[str] = None) -> Dict:
 
 
 def _tensors(part):
-    for v in vars(part).values():
-        if hasattr(v, "data_ptr") and hasattr(v, "element_size") and v.dim() >= 1:
+    gathered = getattr(part, "gathered", ())           # tables of which a step reads a few rows
+    for name, v in vars(part).items():
+        if name not in gathered and hasattr(v, "data_ptr") and hasattr(v, "element_size") and v.dim() >= 1:
             yield v
 
 

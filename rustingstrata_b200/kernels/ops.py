@@ -94,7 +94,6 @@ def core():
                                            c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
                                            c_int, c_int, c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_void_p]
         lib.rs_silu_mul.argtypes = [c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p]
-        lib.rs_head_sigmoid_gate.argtypes = [c_void_p, c_int, c_long, c_void_p, c_long, c_int, c_int, c_int, c_void_p]
         lib.rs_add_embed.argtypes = [c_void_p, c_long, c_void_p, c_int, c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p]
         lib.rs_residual_add.argtypes = [c_void_p, c_void_p, c_int, c_long, c_void_p]
         lib.rs_linear_simt.argtypes = [c_void_p, c_int, c_long, c_void_p, c_int, c_long, c_void_p, c_int, c_long,
@@ -102,7 +101,7 @@ def core():
         lib.rs_attention_simt.argtypes = [c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_int,
                                           c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                           c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                                          c_int, c_int, c_void_p, c_void_p]
+                                          c_int, c_void_p, c_int, c_void_p, c_void_p]
         lib.rs_attention_simt_q_per_cta.argtypes = [c_int, c_int]
         lib.rs_attention_simt_partial_floats.argtypes = [c_int, c_int, c_int]
         lib.rs_attention_simt_partial_floats.restype = c_long
@@ -117,7 +116,7 @@ def core():
                                       c_int, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                       c_int, c_int, c_void_p]
         lib.rs_block_linear.argtypes = [c_void_p, c_int, c_long, c_long, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int,
-                                        c_long, c_long, c_int, c_int, c_int, c_int, c_void_p]
+                                        c_long, c_long, c_int, c_int, c_int, c_int, c_void_p, c_long, c_int, c_float, c_void_p]
         lib.rs_gated_linear_recurrence.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_void_p, c_int,
                                                    c_void_p, c_int, c_void_p, c_int, c_long, c_void_p, c_long, c_void_p,
                                                    c_void_p, c_int, c_int, c_float, c_int, c_void_p]
@@ -126,15 +125,23 @@ def core():
         lib.rs_latent_kv_write.argtypes = [c_void_p, c_long, c_void_p, c_int, c_float, c_void_p, c_int, c_long, c_int, c_int,
                                            c_void_p, c_int, c_long, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p,
                                            c_void_p, c_int, c_int, c_void_p, c_int, c_long, c_int, c_int, c_int, c_int,
-                                           c_int, c_int, c_void_p, c_void_p]
+                                           c_int, c_int, c_void_p, c_long, c_void_p, c_int, c_void_p, c_int, c_long, c_int,
+                                           c_void_p, c_void_p]
         lib.rs_relu_squared.argtypes = [c_void_p, c_int, c_long, c_void_p, c_long, c_int, c_int, c_void_p]
-        lib.rs_moe_route.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
+        lib.rs_moe_route.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                      c_int, c_void_p, c_void_p]
         lib.rs_grouped_linear_rows_per_tile.argtypes = [c_int]
         lib.rs_grouped_linear.argtypes = [c_void_p, c_int, c_long, c_int, c_void_p, c_int, c_long, c_void_p, c_int, c_long,
                                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
-        lib.rs_moe_combine.argtypes = [c_void_p, c_long, c_int, c_float, c_void_p, c_void_p, c_int, c_long, c_void_p, c_int, c_long,
-                                       c_void_p, c_int, c_void_p, c_long, c_int, c_int, c_void_p]
+        lib.rs_moe_combine.argtypes = [c_void_p, c_long, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int, c_long, c_void_p,
+                                       c_int, c_long, c_void_p, c_int, c_void_p, c_long, c_void_p, c_long, c_float, c_int,
+                                       c_void_p, c_int, c_long, c_int, c_int, c_void_p]
+        lib.rs_embed_rmsnorm.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_long, c_int, c_int, c_int,
+                                         c_void_p, c_void_p]
+        lib.rs_gelu_table_gate.argtypes = [c_void_p, c_long, c_void_p, c_int, c_long, c_int, c_int, c_void_p, c_void_p, c_int,
+                                           c_long, c_int, c_int, c_void_p, c_void_p]
+        lib.rs_cast_rows.argtypes = [c_void_p, c_long, c_void_p, c_int, c_long, c_int, c_int, c_void_p]
+        lib.rs_softcap_rows.argtypes = [c_void_p, c_long, c_int, c_int, c_float, c_float, c_void_p]
         _core = lib
     return _core
 
@@ -150,6 +157,55 @@ def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, status: tor
         raise KernelError(f"embed: table {tuple(table.shape)} / ids {ids.numel()} do not fit out {tuple(out.shape)}")
     _check(core().rs_embed(_ptr(table), dtype_code(table), _ptr(ids), _ptr(out), T, H, table.shape[0], _ptr(status),
                            _stream()), "embed")
+
+
+def embed_rmsnorm(table: torch.Tensor, ids: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, n_tokens: int,
+                  status: torch.Tensor) -> None:
+    """out[t] = RMSNorm(table[ids[t]]) * weight in float32 (eps inside the root)."""
+    _cuda(table, ids, weight, out, status)
+    _rows_contiguous(out, "embed_rmsnorm out")
+    H = table.shape[1]
+    if ids.dtype != torch.int32 or out.dtype != torch.float32 or not table.is_contiguous() or not weight.is_contiguous() \
+            or out.shape[1] != H or weight.numel() != H or min(ids.numel(), out.shape[0]) < n_tokens:
+        raise KernelError("embed_rmsnorm: ids int32, out float32 [T, H], table [V, H] and weight [H] contiguous")
+    _check(core().rs_embed_rmsnorm(_ptr(table), dtype_code(table), _ptr(ids), _ptr(weight), dtype_code(weight), float(eps), _ptr(out),
+                                   out.stride(0), n_tokens, H, table.shape[0], _ptr(status), _stream()), "embed_rmsnorm")
+
+
+def gelu_table_gate(z: torch.Tensor, table: torch.Tensor, col0: int, ids: torch.Tensor, out: torch.Tensor, n_tokens: int,
+                    status: torch.Tensor) -> None:
+    """out[t, c] = gelu(z[t, c]) * table[ids[t], col0 + c], the tanh form of GELU in float32; z float32 [T, n]."""
+    _cuda(z, table, ids, out, status)
+    _rows_contiguous(z, "gelu_table_gate z")
+    _rows_contiguous(out, "gelu_table_gate out")
+    _rows_contiguous(table, "gelu_table_gate table")
+    n = z.shape[1]
+    if z.dtype != torch.float32 or ids.dtype != torch.int32 or out.shape[1] != n or col0 < 0 or col0 + n > table.shape[1] \
+            or min(ids.numel(), z.shape[0], out.shape[0]) < n_tokens:
+        raise KernelError("gelu_table_gate: z float32 [T, n], out [T, n], and n columns of the table from col0 on")
+    _check(core().rs_gelu_table_gate(_ptr(z), z.stride(0), _ptr(table), dtype_code(table), table.stride(0), table.shape[0], col0,
+                                     _ptr(ids), _ptr(out), dtype_code(out), out.stride(0), n_tokens, n, _ptr(status), _stream()),
+           "gelu_table_gate")
+
+
+def cast_rows(x: torch.Tensor, out: torch.Tensor, n_rows: int) -> None:
+    """out[r] = x[r] in out's element type; x float32."""
+    _cuda(x, out)
+    _rows_contiguous(x, "cast_rows x")
+    _rows_contiguous(out, "cast_rows out")
+    if x.dtype != torch.float32 or x.shape[1] != out.shape[1] or n_rows > min(x.shape[0], out.shape[0]):
+        raise KernelError("cast_rows: x float32 [T, n] and out [T, n]")
+    _check(core().rs_cast_rows(_ptr(x), x.stride(0), _ptr(out), dtype_code(out), out.stride(0), n_rows, x.shape[1], _stream()),
+           "cast_rows")
+
+
+def softcap_rows(x: torch.Tensor, n_rows: int, cap: float, scale: float = 1.0) -> None:
+    """x[r, c] = cap * tanh(x[r, c] * scale / cap) in place for float32 rows."""
+    _cuda(x)
+    _rows_contiguous(x, "softcap_rows x")
+    if x.dtype != torch.float32 or n_rows > x.shape[0] or not cap > 0:
+        raise KernelError("softcap_rows: float32 rows and a positive cap")
+    _check(core().rs_softcap_rows(_ptr(x), x.stride(0), n_rows, x.shape[1], float(scale), float(cap), _stream()), "softcap_rows")
 
 
 def gather_i32(dst: torch.Tensor, src: torch.Tensor, idx: torch.Tensor, n: int) -> None:
@@ -285,17 +341,6 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, n_rows: int, activation: 
                               GATE_ACTIVATIONS[activation], float(gate[0]), float(gate[1]), _stream()), "silu_mul")
 
 
-def head_sigmoid_gate(a: torch.Tensor, gate: torch.Tensor, n_heads: int, dv: int, n_tokens: int) -> None:
-    """a[t, h * dv + d] *= sigmoid(gate[t, h]) in place; gate float32 [T, >= heads] (pre-activations)."""
-    _cuda(a, gate)
-    _rows_contiguous(a, "head_sigmoid_gate a")
-    if gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[1] < n_heads \
-            or a.shape[1] < n_heads * dv or n_tokens > min(a.shape[0], gate.shape[0]):
-        raise KernelError("head_sigmoid_gate: a [T, heads * dv], gate float32 [T, heads]")
-    _check(core().rs_head_sigmoid_gate(_ptr(a), dtype_code(a), a.stride(0), _ptr(gate), gate.stride(0), n_heads, dv, n_tokens,
-                                       _stream()), "head_sigmoid_gate")
-
-
 def add_embed(x: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float, n_tokens: int, status: torch.Tensor) -> None:
     """x[t] += scale * table[ids[t]] in float32."""
     _cuda(x, table, ids, status)
@@ -391,12 +436,12 @@ def bf16lib():
                                             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.rs_grouped_gemm_mma_rows_per_tile.argtypes = [c_int]
         lib.rs_block_linear_mma.argtypes = [c_void_p, c_int, c_long, c_long, c_void_p, c_void_p, c_int, c_void_p, c_int, c_long,
-                                            c_long, c_int, c_int, c_int, c_int, c_void_p]
+                                            c_long, c_int, c_int, c_int, c_int, c_void_p, c_long, c_int, c_float, c_void_p]
         lib.rs_attention_latent_supported.argtypes = [c_int, c_int, c_int]
         lib.rs_attention_latent_q_per_cta.argtypes = [c_int]
         lib.rs_attention_latent_bf16.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_void_p,
                                                  c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                                                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p]
+                                                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p]
         lib.rs_attention_prefill_bf16_supported.argtypes = [c_int, c_int, c_int]
         lib.rs_attention_prefill_bf16_q_per_cta.argtypes = [c_int, c_int]
         _bf16 = lib
@@ -780,7 +825,7 @@ def attention_simt(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bloc
                    split_keys: int = 128, max_splits: int = 1, split_start: Optional[torch.Tensor] = None,
                    total_splits: int = 0, partial: Optional[torch.Tensor] = None,
                    slopes: Optional[torch.Tensor] = None, one_plane: bool = False,
-                   dist_bias: Optional[torch.Tensor] = None) -> None:
+                   dist_bias: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> None:
     """Paged causal attention (see csrc/attention_simt.cu).  q/out: [T, >= n_q*head_dim] views.
 
     ``one_plane``: the cache is [pages, 1, n_kv, page_size, head_dim] and a row is key and value at once (a latent
@@ -791,6 +836,8 @@ def attention_simt(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bloc
 
     ``dist_bias``: float32 [n_dist, n_q] or None: row min(query position - key position, n_dist - 1) is added to the
     scaled scores, one value per head (a bias tabulated by distance; the last row serves every longer distance).
+
+    ``sink``: float32 [n_q] or None: exp(sink[h]) joins the denominator of head h's softmax, once per query.
 
     Decode form: ``partial`` is the workspace of un-normalised partial results, one slot of n_q * (head_dim + 2)
     float32 values per (sequence, split); ``split_start[w]`` is the first slot of sequence w and ``total_splits`` the
@@ -817,6 +864,7 @@ def attention_simt(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bloc
     if dist_bias is not None and (dist_bias.dtype != torch.float32 or dist_bias.dim() != 2 or dist_bias.shape[1] != n_q
                                   or dist_bias.shape[0] < 1 or not dist_bias.is_contiguous() or not dist_bias.is_cuda):
         raise KernelError(f"attention: dist_bias must be contiguous float32 [distances, {n_q}] on the device")
+    _check_sink(sink, n_q)
     slots = 0
     if decode:
         if split_start is None or split_start.dtype != torch.int32:
@@ -827,7 +875,12 @@ def attention_simt(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bloc
         page_size, _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len), _ptr(work), n_work, n_q,
         n_kv, head_dim, int(window), float(scale), 1 if decode else 0, split_keys, max_splits, _ptr(split_start),
         _ptr(partial), slots, _ptr(slopes), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0],
-        1 if one_plane else 0, _ptr(status), _stream()), "attention_simt", 2 if decode else 1)
+        _ptr(sink), 1 if one_plane else 0, _ptr(status), _stream()), "attention_simt", 2 if decode else 1)
+
+
+def _check_sink(sink: Optional[torch.Tensor], n_heads: int) -> None:
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != n_heads or not sink.is_contiguous() or not sink.is_cuda):
+        raise KernelError(f"attention: sink must be contiguous float32 [{n_heads}] on the device")
 
 
 def _partial_slots(partial: Optional[torch.Tensor], total_splits: int, n_q: int, head_dim: int, who: str) -> int:
@@ -884,16 +937,17 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, b
                       q_start: torch.Tensor, kv_len: torch.Tensor, work: torch.Tensor, n_work: int, n_q: int, n_kv: int,
                       head_dim: int, page_size: int, window: int, scale: float, status: torch.Tensor,
                       force: str = "", slopes: Optional[torch.Tensor] = None, one_plane: bool = False,
-                      dist_bias: Optional[torch.Tensor] = None, dist_bias_by_head: Optional[torch.Tensor] = None) -> None:
+                      dist_bias: Optional[torch.Tensor] = None, dist_bias_by_head: Optional[torch.Tensor] = None,
+                      sink: Optional[torch.Tensor] = None) -> None:
     """Attention of prompt portions; ``work`` lists (sequence, first query) tiles of ``attention_prefill_q_per_cta``
     tokens.  tcgen05 kernel (csrc/attention_prefill_tc.cu), mma.sync kernel (csrc/attention_prefill_mma.cu) or
     CUDA cores, whichever takes the shape; ``force`` names one.  Score slopes are the CUDA-core kernel's; a bias
     tabulated by distance (``dist_bias`` [distances, heads], see :func:`attention_simt`) is added by all three, the
     tcgen05 kernel reading its transpose ``dist_bias_by_head`` [heads, distances] (and wanting a positive scale)."""
     kind = attention_prefill_kernel(q.dtype, n_q, n_kv, head_dim, page_size, force)
-    if (slopes is not None or one_plane) and kind != "simt":
-        raise KernelError("attention_prefill: only the CUDA-core kernel (force='simt') adds score slopes or reads a "
-                          "one-plane cache")
+    if (slopes is not None or one_plane or sink is not None) and kind != "simt":
+        raise KernelError("attention_prefill: only the CUDA-core kernel (force='simt') adds score slopes or a sink or reads "
+                          "a one-plane cache")
     if dist_bias is not None and kind == "tc":
         if dist_bias_by_head is None or dist_bias_by_head.dtype != torch.float32 or not dist_bias_by_head.is_contiguous() \
                 or tuple(dist_bias_by_head.shape) != (n_q, dist_bias.shape[0]) or not dist_bias_by_head.is_cuda or scale <= 0:
@@ -901,7 +955,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, b
                               f"and wants a positive scale")
     if kind == "simt":
         attention_simt(q, out, cache, block_table, q_start, kv_len, work, n_work, n_q, n_kv, head_dim, page_size, window,
-                       scale, False, status, slopes=slopes, one_plane=one_plane, dist_bias=dist_bias)
+                       scale, False, status, slopes=slopes, one_plane=one_plane, dist_bias=dist_bias, sink=sink)
         return
     _cuda(q, out, cache, block_table, q_start, kv_len, work, status)
     _rows_contiguous(q, "q")
@@ -947,16 +1001,17 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
                      max_splits: int, split_start: torch.Tensor, total_splits: int, partial: torch.Tensor,
                      force_simt: bool = False, slopes: Optional[torch.Tensor] = None,
                      items: Optional[torch.Tensor] = None, one_plane: bool = False,
-                     dist_bias: Optional[torch.Tensor] = None) -> None:
+                     dist_bias: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> None:
     """Attention of sequences with one query token each: the tensor-core kernel (csrc/attention_decode_mma.cu)
     where it takes the shape, else the CUDA-core kernel's split form (always, when score biases are given).  Same
     partial-workspace layout.  ``items``: the step's list of live (sequence, kv head, split) items from
     :func:`attention_decode_items`, which a caller with several layers builds once per step; built here if not given."""
-    if (force_simt or slopes is not None or one_plane
+    if (force_simt or slopes is not None or one_plane or sink is not None
             or not attention_decode_fast_ok(q.dtype, n_q, n_kv, head_dim, page_size)):
         attention_simt(q, out, cache, block_table, q_start, kv_len, work, n_work, n_q, n_kv, head_dim, page_size, window,
                        scale, True, status, split_keys=split_keys, max_splits=max_splits, split_start=split_start,
-                       total_splits=total_splits, partial=partial, slopes=slopes, one_plane=one_plane, dist_bias=dist_bias)
+                       total_splits=total_splits, partial=partial, slopes=slopes, one_plane=one_plane, dist_bias=dist_bias,
+                       sink=sink)
         return
     _cuda(q, out, cache, block_table, q_start, kv_len, work, status, partial, split_start)
     _rows_contiguous(q, "q")
@@ -996,13 +1051,16 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
                      q_start: torch.Tensor, kv_len: torch.Tensor, work: torch.Tensor, n_work: int, n_heads: int, lat: int,
                      page_size: int, window: int, scale: float, decode: bool, status: torch.Tensor, split_keys: int = 128,
                      max_splits: int = 1, split_start: Optional[torch.Tensor] = None, total_splits: int = 0,
-                     partial: Optional[torch.Tensor] = None, split_weights: bool = False) -> None:
+                     partial: Optional[torch.Tensor] = None, split_weights: bool = False,
+                     sink: Optional[torch.Tensor] = None) -> None:
     """Attention of ``n_heads`` query heads over a one-plane cache [pages, 1, 1, page_size, lat] whose rows are key and
     value at once, on the tensor cores (csrc/attention_latent_mma.cu).  ``work``: (sequence, first query) tiles of
     :func:`attention_latent_q_per_cta` tokens, or with ``decode`` one sequence per entry, the keys cut into splits whose
     partial results (layout of :func:`attention_simt`) are merged by a second kernel.  ``split_weights``: the softmax weights
-    enter the weighted sum in two bfloat16 terms (the float32 weight to 2^-17) instead of rounded to bfloat16."""
+    enter the weighted sum in two bfloat16 terms (the float32 weight to 2^-17) instead of rounded to bfloat16.  ``sink``:
+    float32 [n_heads] or None: exp(sink[h]) joins the denominator of head h's softmax."""
     _cuda(q, out, cache, block_table, q_start, kv_len, work, status, partial, split_start)
+    _check_sink(sink, n_heads)
     _rows_contiguous(q, "q")
     _rows_contiguous(out, "out")
     if q.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or not cache.is_contiguous():
@@ -1023,7 +1081,7 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
         _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), cache.shape[0], page_size,
         _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len), _ptr(work), n_work, n_heads, lat, int(window),
         float(scale), 1 if decode else 0, split_keys, max_splits, _ptr(split_start), _ptr(partial), slots,
-        1 if split_weights else 0, _ptr(status), _stream()), "attention_latent", 2 if decode else 1)
+        1 if split_weights else 0, _ptr(sink), _ptr(status), _stream()), "attention_latent", 2 if decode else 1)
 
 
 def attention_decode_items(split_start: torch.Tensor, n_work: int, n_kv: int, max_splits: int, items: torch.Tensor) -> None:
@@ -1149,10 +1207,14 @@ BLOCK_LINEAR_ROWS_FORM = 8     # up to this many rows the CUDA-core kernel's row
 
 
 def block_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_rows: int, in_block_stride: int,
-                 out_block_stride: int, bias: Optional[torch.Tensor] = None) -> None:
+                 out_block_stride: int, bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                 out_scale: float = 1.0) -> None:
     """out[t, b * out_block_stride + o] = bias[b, o] + sum_i weight[b, o, i] * x[t, b * in_block_stride + i]: one small
-    matrix per block of channels (a block-diagonal product), float32 accumulation.  weight [B, O, I] contiguous."""
-    _cuda(x, weight, out, bias)
+    matrix per block of channels (a block-diagonal product), float32 accumulation.  weight [B, O, I] contiguous.
+
+    ``gate`` float32 [T, B] or [T, B * O] (rows may be strided) and ``out_scale``: the result is multiplied, still in
+    float32, by out_scale * sigmoid(gate) of its block or of its own column."""
+    _cuda(x, weight, out, bias, gate)
     _rows_contiguous(x, "block_linear x")
     _rows_contiguous(out, "block_linear out")
     if weight.dim() != 3 or not weight.is_contiguous():
@@ -1164,6 +1226,10 @@ def block_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_row
                           f"{I} -> {O} at strides {in_block_stride}, {out_block_stride}")
     if bias is not None and (bias.numel() != B * O or not bias.is_contiguous()):
         raise KernelError("block_linear: bias must hold blocks * out values")
+    if gate is not None and (gate.dtype != torch.float32 or gate.shape[1] not in (B, B * O) or gate.shape[0] < n_rows
+                             or gate.stride(1) != 1):
+        raise KernelError("block_linear: the gate holds float32 rows of one value per block or per output")
+    gate_args = (_ptr(gate), 0 if gate is None else gate.stride(0), 1 if gate is not None and gate.shape[1] == B else 0, float(out_scale))
     per16 = 4 if x.dtype == torch.float32 else 8
     if (n_rows > BLOCK_LINEAR_ROWS_FORM and weight.dtype == torch.bfloat16 and x.dtype in (torch.bfloat16, torch.float32)
             and out.dtype in (torch.bfloat16, torch.float32) and I % 8 == 0 and in_block_stride % per16 == 0
@@ -1172,11 +1238,11 @@ def block_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_row
         # that takes every row (float32 inputs are rounded to bfloat16 as they enter the product)
         _check(bf16lib().rs_block_linear_mma(_ptr(x), dtype_code(x), x.stride(0), in_block_stride, _ptr(weight), _ptr(bias),
                                              _any_code(bias), _ptr(out), dtype_code(out), out.stride(0), out_block_stride,
-                                             n_rows, B, O, I, _stream()), "block_linear_mma")
+                                             n_rows, B, O, I, *gate_args, _stream()), "block_linear_mma")
         return
     _check(core().rs_block_linear(_ptr(x), dtype_code(x), x.stride(0), in_block_stride, _ptr(weight), dtype_code(weight),
                                   _ptr(bias), _any_code(bias), _ptr(out), dtype_code(out), out.stride(0), out_block_stride,
-                                  n_rows, B, O, I, _stream()), "block_linear")
+                                  n_rows, B, O, I, *gate_args, _stream()), "block_linear")
 
 
 def gated_linear_recurrence(gates: torch.Tensor, u: torch.Tensor, y: torch.Tensor, y_bias: Optional[torch.Tensor],
@@ -1225,20 +1291,34 @@ def gated_linear_recurrence(gates: torch.Tensor, u: torch.Tensor, y: torch.Tenso
     _check(core().rs_gated_linear_recurrence(*args, _stream()), "gated_linear_recurrence")
 
 
-def latent_kv_write(dkv: torch.Tensor, norm_weight: torch.Tensor, eps: float, q: torch.Tensor, q_head: int, q_nope: int,
-                    q_lat: torch.Tensor, cos_sin: Optional[torch.Tensor], n_rot: int, positions: torch.Tensor,
-                    seq_of_token: torch.Tensor, block_table: torch.Tensor, page_size: int, cache: Optional[torch.Tensor],
-                    rank: int, rot: int, lat: int, heads: int, n_tokens: int, status: torch.Tensor) -> None:
+def latent_kv_write(dkv: Optional[torch.Tensor], norm_weight: Optional[torch.Tensor], eps: float, q: Optional[torch.Tensor],
+                    q_head: int, q_nope: int, q_lat: Optional[torch.Tensor], cos_sin: Optional[torch.Tensor], n_rot: int,
+                    positions: torch.Tensor, seq_of_token: torch.Tensor, block_table: torch.Tensor, page_size: int,
+                    cache: Optional[torch.Tensor], rank: int, rot: int, lat: int, heads: int, n_tokens: int, status: torch.Tensor,
+                    cq: Optional[torch.Tensor] = None, cq_weight: Optional[torch.Tensor] = None,
+                    cq_out: Optional[torch.Tensor] = None) -> None:
     """Latent norm + interleaved rotation + write of [latent | rotated key part | 0...] into a one-plane cache
-    [pages, 1, 1, page_size, lat], and the rotated parts of the queries into q_lat[t, h * lat + rank : ...]."""
-    _cuda(dkv, norm_weight, q, q_lat, cos_sin, positions, seq_of_token, block_table, cache, status)
-    _rows_contiguous(dkv, "latent_kv_write dkv")
-    _rows_contiguous(q, "latent_kv_write q")
-    _rows_contiguous(q_lat, "latent_kv_write q_lat")
-    if dkv.dtype != torch.float32 or dkv.shape[1] < rank + rot or norm_weight.numel() != rank or not norm_weight.is_contiguous():
-        raise KernelError("latent_kv_write: dkv must be float32 [T, >= rank + rot] and the norm weight [rank]")
-    if q.shape[1] < heads * q_head or q_lat.shape[1] < heads * lat or q_nope + rot > q_head or rank + rot > lat:
-        raise KernelError("latent_kv_write: query buffers do not hold the heads")
+    [pages, 1, 1, page_size, lat] (``dkv``, ``norm_weight`` and ``cache`` given), and the rotated parts of the queries into
+    q_lat[t, h * lat + rank : ...] (``q`` and ``q_lat`` given).  ``cq`` float32 [T, n]: besides, cq_out = RMSNorm(cq) *
+    cq_weight, the latent that queries are made from."""
+    _cuda(dkv, norm_weight, q, q_lat, cos_sin, positions, seq_of_token, block_table, cache, status, cq, cq_weight, cq_out)
+    if (q is None) != (q_lat is None) or (dkv is None) != (cache is None) or (dkv is None) != (norm_weight is None):
+        raise KernelError("latent_kv_write: q goes with q_lat, dkv with its norm weight and the cache")
+    if dkv is not None:
+        _rows_contiguous(dkv, "latent_kv_write dkv")
+        if dkv.dtype != torch.float32 or dkv.shape[1] < rank + rot or norm_weight.numel() != rank or not norm_weight.is_contiguous():
+            raise KernelError("latent_kv_write: dkv must be float32 [T, >= rank + rot] and the norm weight [rank]")
+    if q is not None:
+        _rows_contiguous(q, "latent_kv_write q")
+        _rows_contiguous(q_lat, "latent_kv_write q_lat")
+        if q.shape[1] < heads * q_head or q_lat.shape[1] < heads * lat or q_nope + rot > q_head:
+            raise KernelError("latent_kv_write: query buffers do not hold the heads")
+    if rank + rot > lat:
+        raise KernelError("latent_kv_write: a cache row does not hold the latent and the rotated part")
+    if (cq is None) != (cq_out is None) or (cq is not None and (
+            cq.dtype != torch.float32 or cq.stride(1) != 1 or cq_out.stride(1) != 1 or cq_weight.numel() != cq.shape[1]
+            or not cq_weight.is_contiguous() or cq_out.shape[1] != cq.shape[1] or min(cq.shape[0], cq_out.shape[0]) < n_tokens)):
+        raise KernelError("latent_kv_write: cq float32 [T, n] with a weight of n values and an output of n columns")
     if cache is not None and (tuple(cache.shape[1:]) != (1, 1, page_size, lat) or not cache.is_contiguous()):
         raise KernelError(f"latent_kv_write: cache shape {tuple(cache.shape)} is not [pages, 1, 1, {page_size}, {lat}]")
     if cos_sin is not None and (cos_sin.dtype != torch.float32 or cos_sin.shape[1] != n_rot or not cos_sin.is_contiguous()):
@@ -1247,12 +1327,15 @@ def latent_kv_write(dkv: torch.Tensor, norm_weight: torch.Tensor, eps: float, q:
         if t.dtype != torch.int32:
             raise KernelError(f"latent_kv_write: {name} must be int32")
     pos_stride = 1 if positions.dim() == 1 else positions.shape[1]
+    stride = lambda t: 0 if t is None else t.stride(0)                                                   # noqa: E731
     _check(core().rs_latent_kv_write(
-        _ptr(dkv), dkv.stride(0), _ptr(norm_weight), dtype_code(norm_weight), float(eps), _ptr(q), dtype_code(q), q.stride(0),
-        q_head, q_nope, _ptr(q_lat), dtype_code(q_lat), q_lat.stride(0), _ptr(cos_sin), n_rot if cos_sin is not None else 0,
+        _ptr(dkv), stride(dkv), _ptr(norm_weight), _any_code(norm_weight), float(eps), _ptr(q), _any_code(q), stride(q),
+        q_head, q_nope, _ptr(q_lat), _any_code(q_lat), stride(q_lat), _ptr(cos_sin), n_rot if cos_sin is not None else 0,
         0 if cos_sin is None else cos_sin.shape[0], _ptr(positions), pos_stride, _ptr(seq_of_token), _ptr(block_table),
-        block_table.stride(0), page_size, _ptr(cache), _any_code(cache), 0 if cache is None else cache.stride(0),
-        0 if cache is None else cache.shape[0], rank, rot, lat, heads, n_tokens, _ptr(status), _stream()), "latent_kv_write")
+        block_table.stride(0), page_size, _ptr(cache), _any_code(cache), stride(cache),
+        0 if cache is None else cache.shape[0], rank, rot, lat, heads if q is not None else 0, n_tokens, _ptr(cq), stride(cq),
+        _ptr(cq_weight), _any_code(cq_weight), _ptr(cq_out), _any_code(cq_out), stride(cq_out), 0 if cq is None else cq.shape[1],
+        _ptr(status), _stream()), "latent_kv_write")
 
 
 def relu_squared(x: torch.Tensor, out: torch.Tensor, n_rows: int) -> None:
@@ -1282,10 +1365,11 @@ def grouped_rows_per_tile(small: bool) -> int:
 
 
 def moe_route(ids: Optional[torch.Tensor], table: torch.Tensor, n_experts: int, n_tokens: int, rows_per_tile: int,
-              order: torch.Tensor, tiles: torch.Tensor, n_tiles: torch.Tensor, status: torch.Tensor) -> None:
+              order: torch.Tensor, tiles: torch.Tensor, n_tiles: torch.Tensor, status: torch.Tensor, identity: int = 0) -> None:
     """Sorts the step's (token, k) pairs by the expert that ``table[ids[t], k]`` names: ``order`` [T * top] pair ids
     grouped by expert, ``tiles`` [max_tiles, 3] (expert, first row in order, rows), ``n_tiles`` [1].  Without ``ids``
-    the table has one row per token of the step (the choice a router made): pair (t, k) goes to ``table[t, k]``."""
+    the table has one row per token of the step (the choice a router made): pair (t, k) goes to ``table[t, k]``.  Pairs whose
+    choice is one of the ``identity`` numbers behind the last expert (experts without matrices) are left out of the lists."""
     _cuda(ids, table, order, tiles, n_tiles, status)
     V, top = table.shape
     for name, t in (("ids", ids), ("table", table), ("order", order), ("tiles", tiles), ("n_tiles", n_tiles)):
@@ -1295,7 +1379,7 @@ def moe_route(ids: Optional[torch.Tensor], table: torch.Tensor, n_experts: int, 
         raise KernelError("moe_route: order must hold tokens * top entries")
     if rows_per_tile not in (grouped_rows_per_tile(True), grouped_rows_per_tile(False), GROUPED_ROWS_LARGE):
         raise KernelError("moe_route: rows_per_tile must be a tile size of the grouped product")
-    _check(core().rs_moe_route(_ptr(ids), _ptr(table), V, top, n_experts, n_tokens, rows_per_tile, _ptr(order), _ptr(tiles),
+    _check(core().rs_moe_route(_ptr(ids), _ptr(table), V, top, n_experts, int(identity), n_tokens, rows_per_tile, _ptr(order), _ptr(tiles),
                                _ptr(n_tiles), tiles.numel() // 3, _ptr(status), _stream()), "moe_route")
 
 
@@ -1362,33 +1446,51 @@ def grouped_gemm_mma(a: torch.Tensor, a_div: int, weight: torch.Tensor, out: tor
 
 def moe_combine(pair_out: torch.Tensor, top: int, weight: float, out: torch.Tensor, n_tokens: int,
                 shared: Optional[torch.Tensor] = None, h: Optional[torch.Tensor] = None,
-                gate_weight: Optional[torch.Tensor] = None, pair_weights: Optional[torch.Tensor] = None) -> None:
-    """out[t] = weight * sum_k pair_out[t * top + k] + sigmoid(h[t] . gate_weight) * shared[t]  (float32 out; the
-    second term only with ``shared``, its factor 1 without ``gate_weight``).  ``pair_weights`` float32 [T * top]:
-    every pair is multiplied by its own weight in the sum."""
-    _cuda(pair_out, out, shared, h, gate_weight, pair_weights)
+                gate_weight: Optional[torch.Tensor] = None, pair_weights: Optional[torch.Tensor] = None,
+                choice: Optional[torch.Tensor] = None, n_experts: int = 0, gate_logit: Optional[torch.Tensor] = None,
+                scale: float = 1.0, accumulate: bool = False, copy: Optional[torch.Tensor] = None) -> None:
+    """y[t] = scale * (weight * sum_k pair_out[t * top + k] + g * shared[t]), g = sigmoid(h[t] . gate_weight) or
+    sigmoid(gate_logit[t, 0]) or 1 (the second term only with ``shared``); out = y, or out += y with ``accumulate`` (float32).
+    ``pair_weights`` float32 [T * top]: every pair is multiplied by its own weight in the sum.  ``choice`` int32 [T * top]: a
+    pair whose choice is ``n_experts`` or more is an identity expert's, and h[t] stands in for its row of ``pair_out``.
+    ``copy``: takes out's new rows in its own element type besides."""
+    _cuda(pair_out, out, shared, h, gate_weight, pair_weights, choice, gate_logit, copy)
     if pair_weights is not None and (pair_weights.dtype != torch.float32 or not pair_weights.is_contiguous()
                                      or pair_weights.numel() < n_tokens * top):
         raise KernelError("moe_combine: pair_weights must be contiguous float32 [T * top]")
+    if choice is not None and (choice.dtype != torch.int32 or not choice.is_contiguous() or choice.numel() < n_tokens * top
+                               or h is None):
+        raise KernelError("moe_combine: choice must be contiguous int32 [T * top] and identity experts need h")
     _rows_contiguous(pair_out, "moe_combine pair_out")
     _rows_contiguous(out, "moe_combine out")
     n = out.shape[1]
     if pair_out.dtype != torch.float32 or out.dtype != torch.float32 or pair_out.shape[1] != n \
             or pair_out.shape[0] < n_tokens * top or out.shape[0] < n_tokens:
         raise KernelError("moe_combine: pair_out float32 [T * top, n], out float32 [T, n]")
+    reads_h = choice is not None or gate_weight is not None
+    if reads_h:
+        _rows_contiguous(h, "moe_combine h")
+        if h.shape[1] != n or h.shape[0] < n_tokens:
+            raise KernelError("moe_combine: h must be [T, n]")
     if shared is not None:
         _rows_contiguous(shared, "moe_combine shared")
         if shared.shape[1] != n or shared.shape[0] < n_tokens:
             raise KernelError("moe_combine: shared must be [T, n]")
-        if gate_weight is not None:
-            _rows_contiguous(h, "moe_combine h")
-            if gate_weight.numel() != n or not gate_weight.is_contiguous() or h.shape[1] != n:
-                raise KernelError("moe_combine: the gate reads h [T, n] with a weight of n values")
-    _check(core().rs_moe_combine(_ptr(pair_out), pair_out.stride(0), top, float(weight), _ptr(pair_weights), _ptr(shared),
-                                 _any_code(shared),
-                                 0 if shared is None else shared.stride(0), _ptr(h if gate_weight is not None else None),
-                                 _any_code(h), 0 if h is None else h.stride(0), _ptr(gate_weight), _any_code(gate_weight),
-                                 _ptr(out), out.stride(0), n_tokens, n, _stream()), "moe_combine")
+        if gate_weight is not None and (gate_weight.numel() != n or not gate_weight.is_contiguous()):
+            raise KernelError("moe_combine: the gate reads h [T, n] with a weight of n values")
+        if gate_logit is not None and (gate_logit.dtype != torch.float32 or gate_logit.shape[0] < n_tokens or gate_logit.shape[1] < 1):
+            raise KernelError("moe_combine: gate_logit must be float32 [T, >= 1]")
+    if copy is not None:
+        _rows_contiguous(copy, "moe_combine copy")
+        if copy.shape[1] != n or copy.shape[0] < n_tokens:
+            raise KernelError("moe_combine: copy must be [T, n]")
+    stride = lambda t: 0 if t is None else t.stride(0)                                                   # noqa: E731
+    hh = h if reads_h else None
+    _check(core().rs_moe_combine(_ptr(pair_out), pair_out.stride(0), top, float(weight), _ptr(pair_weights), _ptr(choice), int(n_experts),
+                                 _ptr(shared), _any_code(shared), stride(shared), _ptr(hh), _any_code(hh), stride(hh),
+                                 _ptr(gate_weight), _any_code(gate_weight), _ptr(gate_logit), stride(gate_logit), _ptr(out),
+                                 out.stride(0), float(scale), 1 if accumulate else 0, _ptr(copy), _any_code(copy), stride(copy),
+                                 n_tokens, n, _stream()), "moe_combine")
 
 
 # ----------------------------------------------------------------------------- several residual streams, summed embeddings
@@ -1407,7 +1509,7 @@ def streamlib():
         lib.rs_stream_update.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int,
                                          c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_long, c_int, c_int, c_int,
                                          c_void_p]
-        lib.rs_router_topk.argtypes = [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
+        lib.rs_router_topk.argtypes = [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
                                        c_void_p, c_void_p, c_void_p, c_void_p]
         lib.rs_conv_norm_kv_write.argtypes = [c_void_p, c_int, c_long, c_void_p, c_int, c_void_p, c_long, c_int, c_int, c_int,
                                               c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_long, c_void_p, c_long,
@@ -1512,11 +1614,11 @@ def stream_update(x: torch.Tensor, n_streams: int, y: torch.Tensor, mix: torch.T
 
 def router_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, n_tokens: int, choice: torch.Tensor,
                 weights: torch.Tensor, status: torch.Tensor, sigmoid: bool = False, groups: int = 0, keep: int = 0,
-                scale: float = 1.0, renormalize: bool = True) -> None:
+                scale: float = 1.0, renormalize: bool = True, group_worth: str = "top2") -> None:
     """scores = softmax(logits[t]) (float32 [T, E]; ``sigmoid``: the sigmoid of every logit); choice[t] = the ``top``
     experts with the largest score + correction (int32 [T, top], the lower index on a tie); with ``groups`` > 0 only
     experts of the ``keep`` best of that many equal groups of neighbours (a group is worth its two largest scores +
-    correction added); weights[t] = their scores times ``scale``, over (the sum of their scores + 1e-20) first if
+    correction added, or with ``group_worth`` "max" its largest); weights[t] = their scores times ``scale``, over (the sum of their scores + 1e-20) first if
     ``renormalize``."""
     _cuda(logits, correction, choice, weights, status)
     _rows_contiguous(logits, "router_topk logits")
@@ -1526,10 +1628,12 @@ def router_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: i
         raise KernelError("router_topk: logits float32 [T, E], choice int32 and weights float32 [T * top] contiguous")
     if not 1 <= top <= E <= 1024 or (correction is not None and correction.numel() != E):
         raise KernelError(f"router_topk: top {top} of {E} experts (up to 1024), one correction per expert")
+    if group_worth not in ("top2", "max"):
+        raise KernelError(f"router_topk: unknown group worth '{group_worth}'")
     if groups and (E % groups or not 1 <= keep <= groups or top > keep * (E // groups)):
         raise KernelError(f"router_topk: {groups} groups of {E} experts, {keep} kept, top {top}")
     _check(streamlib().rs_router_topk(_ptr(logits), logits.stride(0), _ptr(correction), _any_code(correction), E, top,
-                                      n_tokens, 1 if sigmoid else 0, int(groups), int(keep), float(scale),
+                                      n_tokens, 1 if sigmoid else 0, int(groups), int(keep), 1 if group_worth == "max" else 0, float(scale),
                                       1 if renormalize else 0, _ptr(choice), _ptr(weights), _ptr(status), _stream()),
            "router_topk")
 

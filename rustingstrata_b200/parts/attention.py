@@ -140,6 +140,11 @@ class PagedAttention(Mixer):
         row min(query position - key position, last row) is added to every scaled score."""
         return None
 
+    def _sink(self):
+        """A number per head whose exponential joins the softmax's denominator, if the mixer has one: float32 [n_heads] on
+        the device.  The CUDA-core attention kernels take it."""
+        return None
+
     def _cuda_cores_only(self) -> bool:
         """Whether only the CUDA-core attention kernels can run this mixer (score slopes they alone add, a one-plane cache)."""
         return self._score_slopes() is not None or self.one_plane
@@ -227,7 +232,7 @@ class PagedAttention(Mixer):
         plan = ctx.plans[self.plan_key()]
         common = dict(q=q, out=out, cache=call.cache, block_table=table, q_start=ctx.q_start, kv_len=ctx.kv_len,
                       n_q=self.n_heads, n_kv=self.n_kv, head_dim=self.hd, page_size=rt.page_size, window=self.window,
-                      scale=self.scale, status=ctx.status, one_plane=self.one_plane)
+                      scale=self.scale, status=ctx.status, one_plane=self.one_plane, sink=self._sink())
         slopes = self._score_slopes()
         dist_bias = self._distance_bias()
         simt = self._cuda_cores_only()

@@ -139,8 +139,13 @@ class StepContext:
     # A block that norms a sublayer's output before it joins the stream hands the mixer or feed-forward a buffer of
     # its own in place of the stream and sets ``store_output``: the part then stores its output there instead of adding.
     store_output: bool = False
+    # A block whose next step reads the stream itself in the activation type sets ``stream_copy`` (a [T, hidden] buffer) around
+    # its feed-forward's call: a feed-forward that adds its output in a kernel of its own may leave the stream's new rows there
+    # and set the field to None; if it does not, the block makes the copy.
+    stream_copy: Any = None
     # A block that rewrites the whole stream at its end can run the first norm of the next block in the same pass:
-    # ``next_reader`` (set by the model before each block) is what that block's ``stream_reader()`` returned, or None;
+    # ``next_reader`` (set by the model before each block) is what that block's ``stream_reader()`` returned (a norm part, or
+    # the tuple of a block of several streams), or None;
     # ``normed_ready`` is set by the block that did so and cleared by the block that finds its input normed already.
     next_reader: Any = None
     normed_ready: bool = False

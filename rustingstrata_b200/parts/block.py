@@ -15,32 +15,88 @@ from .spec import TensorNeed
 
 @register_part("block", "pre_norm")
 class PreNormBlock(Block):
-    """params: hidden.  Made of: mixer_norm, mixer, feed_forward_norm, feed_forward (and a position encoding for
-    the mixer, if the layer lists one)."""
+    """x += mixer(norm(x)); x += feed_forward(norm(x)); x += norm(side(x)).
+
+    params: hidden, ignored_norms (names of norm weights a checkpoint may carry for a sublayer that the layer lacks).
+    Made of: mixer_norm, mixer; optionally feed_forward_norm with feed_forward (both or neither), and side with
+    side_norm: a per-token sublayer that reads the stream as it is (in the activation type) and whose output is normed before
+    it joins; and a position encoding for the mixer, if the layer lists one.
+
+    The side's norm adds to the stream and, in the same kernel, applies the next layer's first norm where that layer is of
+    this kind."""
     chain_safe = True
-    roles = {"mixer_norm": "norm", "mixer": "mixer", "feed_forward_norm": "norm", "feed_forward": "feed_forward"}
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "feed_forward_norm": "norm", "feed_forward": "feed_forward",
+             "side": "feed_forward", "side_norm": "norm"}
+    optional = ("feed_forward_norm", "feed_forward", "side", "side_norm")
 
     def __init__(self, spec, runtime, parts):
         super().__init__(spec, runtime, parts)
         self.mixer_norm, self.mixer = parts["mixer_norm"], parts["mixer"]
-        self.ff_norm, self.feed_forward = parts["feed_forward_norm"], parts["feed_forward"]
+        self.ff_norm, self.feed_forward = parts.get("feed_forward_norm"), parts.get("feed_forward")
+        self.side, self.side_norm = parts.get("side"), parts.get("side_norm")
+        if (self.ff_norm is None) != (self.feed_forward is None):
+            raise ValueError("block 'pre_norm' has a feed-forward with its norm or neither")
+        if (self.side is None) != (self.side_norm is None):
+            raise ValueError("block 'pre_norm' has a side sublayer with its norm or neither")
+        if self.side_norm is not None and type(self.side_norm).forward_add is Norm.forward_add:
+            raise ValueError("block 'pre_norm': the side_norm part cannot norm a sublayer's output into the stream")
         self.hidden = int(spec.params["hidden"])
         runtime.scratch("normed", runtime.max_batch_tokens, self.hidden)
+        if self.side is not None:
+            runtime.scratch("stream_rows", runtime.max_batch_tokens, self.hidden)
+            runtime.scratch("sublayer_out", runtime.max_batch_tokens, self.hidden, torch.float32)
+
+    def tensor_needs(self):
+        return {name: TensorNeed((self.hidden,), "norm", optional=True) for name in self.spec.params.get("ignored_norms", ())}
 
     @property
     def first_reader_takes_owed(self):
         return getattr(self.mixer_norm, "takes_owed", False)
 
+    def stream_reader(self):
+        """The norm a block before this one may apply for it (see StepContext.next_reader)."""
+        return self.mixer_norm
+
     def forward(self, residual, ctx, call):
+        T = ctx.n_tokens
         h = self.runtime.get_scratch("normed")[:, : self.hidden]
-        self.norm_of_stream(self.mixer_norm, residual, h, ctx)
-        ctx.may_owe = getattr(self.ff_norm, "takes_owed", False)
+        if ctx.normed_ready:
+            ctx.normed_ready = False             # the block before this one left the normed stream in h
+        else:
+            self.norm_of_stream(self.mixer_norm, residual, h, ctx)
+        # a sublayer may leave its last sum to the norm that reads the stream next
+        last = ctx.next_block_takes_owed and self.side is None
+        ctx.may_owe = getattr(self.ff_norm, "takes_owed", False) if self.ff_norm is not None else last
         self.mixer.forward(h, residual, ctx, call.mixers["mixer"])
         ctx.may_owe = False
-        self.norm_of_stream(self.ff_norm, residual, h, ctx)
-        ctx.may_owe = ctx.next_block_takes_owed
-        self.feed_forward.forward(h, residual, ctx)
-        ctx.may_owe = False
+        copy = None
+        if self.side is not None:
+            # the product that reads the stream takes it in the activation type: the stream itself, or a rounded copy
+            copy = None if self.runtime.precise else self.runtime.get_scratch("stream_rows")[:, : self.hidden]
+        if self.feed_forward is not None:
+            self.norm_of_stream(self.ff_norm, residual, h, ctx)
+            ctx.may_owe, ctx.stream_copy = last, copy
+            self.feed_forward.forward(h, residual, ctx)
+            ctx.may_owe = False
+            copied, ctx.stream_copy = copy is not None and ctx.stream_copy is None, None
+        else:
+            copied = False
+        if self.side is None:
+            return
+        if ctx.owed is not None:
+            ctx.owed.finish()
+            ctx.owed = None
+        if copy is not None and not copied:
+            ops.cast_rows(residual[:, : self.hidden], copy, T)
+        delta = self.runtime.get_scratch("sublayer_out", torch.float32)[:, : self.hidden]
+        ctx.store_output = True
+        try:
+            self.side.forward(residual[:, : self.hidden] if copy is None else copy, delta, ctx)
+        finally:
+            ctx.store_output = False
+        nxt = ctx.next_reader if isinstance(ctx.next_reader, Norm) else None
+        self.side_norm.forward_add(delta, residual, T, then=nxt, out=h if nxt is not None else None)
+        ctx.normed_ready = nxt is not None
 
 
 @register_part("block", "parallel")

@@ -73,7 +73,6 @@ class TableMoE(FeedForward):
         rt.scratch("moe_pair_out", pairs, self.hidden, torch.float32)
         rt.scratch("moe_order", 1, pairs, torch.int32)
         rt.scratch("moe_tiles", 1, 3 * self._max_tiles(pairs, min(_ROWS_PER_TILE.values())) + 4, torch.int32)
-        rt.scratch("moe_delta", rt.max_batch_tokens, self.hidden, torch.float32)
         if self.shared_ff:
             rt.scratch("moe_shared_act", rt.max_batch_tokens, self.shared_ff)
             rt.scratch("moe_shared_gu", rt.max_batch_tokens, 2 * self.shared_ff)
@@ -157,16 +156,8 @@ class TableMoE(FeedForward):
                 ops.linear(h, self.w_shared_gu, gu, T)
                 ops.silu_mul(gu, sact, T)
             ops.linear(sact, self.w_shared_down, shared_out, T, status=ctx.status)
-        if ctx.store_output:
-            ops.moe_combine(pair_out, top, 1.0 / top, residual, T, shared=shared_out, h=h,
-                            gate_weight=self.w_shared_scale if self.shared_ff else None)
-        else:
-            delta = rt.get_scratch("moe_delta", torch.float32)[:, : self.hidden]
-            ops.moe_combine(pair_out, top, 1.0 / top, delta, T, shared=shared_out, h=h,
-                            gate_weight=self.w_shared_scale if self.shared_ff else None)
-            ops.residual_add(residual, delta, T)
-
-
+        ops.moe_combine(pair_out, top, 1.0 / top, residual, T, shared=shared_out, h=h,
+                        gate_weight=self.w_shared_scale if self.shared_ff else None, accumulate=not ctx.store_output)
 
 
 @register_part("feed_forward", "routed_moe")
@@ -176,16 +167,20 @@ class RoutedMoE(FeedForward):
     Router logits z = W_r h are float32 in both engines; the scores s are softmax(z) over all experts (``score``
     "softmax") or sigmoid(z), each expert for itself ("sigmoid").  The ``top`` experts with the largest s + correction are
     chosen (``correction``: one learned number per expert that steers the choice only).  With ``groups`` the experts form
-    that many equal groups of neighbours; a group is worth the sum of its two largest s + correction, and only experts
-    of the ``keep`` groups worth most can be chosen.  The weights are the chosen experts' scores s times ``route_scale``,
+    that many equal groups of neighbours; a group is worth the sum of its two largest s + correction (``group_worth``
+    "top2") or its largest ("max"), and only experts of the ``keep`` groups worth most can be chosen.  The weights are the chosen experts' scores s times ``route_scale``,
     divided by the sum of the chosen scores (+ 1e-20) first if ``renormalize``.  An expert (``expert``) is "relu2":
     down(relu(up h)^2), or "gated_silu": down(silu(gate h) * (up h)), without biases; a shared expert of the same form
-    runs for every token and is added unweighted.
+    runs for every token and is added unweighted, or with ``shared_scale`` multiplied by sigmoid(w_sg . h), one number per
+    token.  The last ``identity`` of the router's outputs are identity experts: they take part in scores, groups and choice
+    like the others, have no tensors, and give h itself.  ``out_scale`` multiplies the whole output.
 
-    params: hidden, experts, top, expert_ff, shared_ff (0 or None: no shared expert), correction (bool), score, groups
-    (0 or None: none), keep, route_scale (default 1), renormalize (default True), expert (default "relu2").
-    tensors: router [experts, hidden], correction [experts]; expert_up / expert_down (and expert_gate): name patterns
-    with ``{e}`` for the expert's number; shared_up, shared_down (and shared_gate).  The step's (token, k) pairs are sorted
+    params: hidden, experts (with tensors), identity (default 0), top, expert_ff, shared_ff (0 or None: no shared expert),
+    shared_scale (bool, default False), correction (bool), score, groups (0 or None: none), keep, group_worth (default "top2"),
+    route_scale (default 1), renormalize (default True), expert (default "relu2"), out_scale (default 1).
+    tensors: router [experts + identity, hidden], correction [experts + identity]; expert_up / expert_down (and expert_gate):
+    name patterns with ``{e}`` for the expert's number; shared_up, shared_down (and shared_gate); shared_scale [1, hidden],
+    whose product with h is one more row of the router's.  The step's (token, k) pairs are sorted
     by expert on the device and one grouped product per projection serves all experts, as in :class:`TableMoE`."""
     SMALL_PAIRS_PER_EXPERT = TableMoE.SMALL_PAIRS_PER_EXPERT
     LARGE_PAIRS_PER_EXPERT = TableMoE.LARGE_PAIRS_PER_EXPERT
@@ -195,8 +190,15 @@ class RoutedMoE(FeedForward):
         p = spec.params
         self.hidden = int(p["hidden"])
         self.n_experts, self.top = int(p["experts"]), int(p["top"])
+        self.identity = int(p.get("identity") or 0)
+        self.n_choices = self.n_experts + self.identity
         self.ff = int(p["expert_ff"])
         self.shared_ff = int(p.get("shared_ff") or 0)
+        self.has_shared_scale = bool(p.get("shared_scale", False)) and self.shared_ff > 0
+        self.out_scale = float(p.get("out_scale", 1.0))
+        self.group_worth = p.get("group_worth", "top2")
+        if self.group_worth not in ("top2", "max"):
+            raise ValueError(f"routed_moe: group_worth {self.group_worth!r} (known: 'top2', 'max')")
         self.has_correction = bool(p.get("correction", False))
         self.score = p.get("score", "softmax")
         self.groups, self.keep = int(p.get("groups") or 0), int(p.get("keep") or 0)
@@ -208,11 +210,11 @@ class RoutedMoE(FeedForward):
         if self.form not in ("relu2", "gated_silu"):
             raise ValueError(f"routed_moe: expert form {self.form!r} (known: 'relu2', 'gated_silu')")
         self.gated = self.form == "gated_silu"
-        if not 1 <= self.top <= self.n_experts <= 1024:
-            raise ValueError(f"routed_moe: top {self.top} of {self.n_experts} experts (up to 1024)")
-        if self.groups and (self.n_experts % self.groups or not 1 <= self.keep <= self.groups
-                            or self.top > self.keep * (self.n_experts // self.groups)):
-            raise ValueError(f"routed_moe: {self.groups} groups of {self.n_experts} experts with {self.keep} kept cannot "
+        if self.identity < 0 or self.n_experts < 1 or not 1 <= self.top <= self.n_choices <= 1024:
+            raise ValueError(f"routed_moe: top {self.top} of {self.n_choices} experts (up to 1024)")
+        if self.groups and (self.n_choices % self.groups or not 1 <= self.keep <= self.groups
+                            or self.top > self.keep * (self.n_choices // self.groups)):
+            raise ValueError(f"routed_moe: {self.groups} groups of {self.n_choices} experts with {self.keep} kept cannot "
                              f"give {self.top} experts")
         rt = runtime
         pairs = rt.max_batch_tokens * self.top
@@ -221,8 +223,7 @@ class RoutedMoE(FeedForward):
         rt.scratch("moe_pair_out", pairs, self.hidden, torch.float32)
         rt.scratch("moe_order", 1, pairs, torch.int32)
         rt.scratch("moe_tiles", 1, 3 * self._max_tiles(pairs, min(_ROWS_PER_TILE.values())) + 4, torch.int32)
-        rt.scratch("moe_delta", rt.max_batch_tokens, self.hidden, torch.float32)
-        rt.scratch("router_logits", rt.max_batch_tokens, self.n_experts, torch.float32)
+        rt.scratch("router_logits", rt.max_batch_tokens, self.n_choices + self.has_shared_scale, torch.float32)
         rt.scratch("router_choice", 1, pairs, torch.int32)
         rt.scratch("router_weights", 1, pairs, torch.float32)
         if self.shared_ff:
@@ -236,9 +237,11 @@ class RoutedMoE(FeedForward):
 
     def tensor_needs(self):
         t = self.spec.tensors
-        needs = {t["router"]: TensorNeed((self.n_experts, self.hidden))}
+        needs = {t["router"]: TensorNeed((self.n_choices, self.hidden))}
         if self.has_correction:
-            needs[t["correction"]] = TensorNeed((self.n_experts,))
+            needs[t["correction"]] = TensorNeed((self.n_choices,))
+        if self.has_shared_scale:
+            needs[t["shared_scale"]] = TensorNeed((1, self.hidden))
         for e in range(self.n_experts):
             if self.gated:
                 needs[t["expert_gate"].format(e=e)] = TensorNeed((self.ff, self.hidden))
@@ -254,6 +257,11 @@ class RoutedMoE(FeedForward):
     def load(self, tensors):
         t, E = self.spec.tensors, self.n_experts
         self.w_router = tensors[t["router"]].contiguous()
+        if self.has_shared_scale:
+            sg = tensors[t["shared_scale"]].reshape(1, self.hidden)
+            if sg.dtype != self.w_router.dtype:
+                raise ValueError("routed_moe: the router and the shared expert's factor must share an element type")
+            self.w_router = torch.cat([self.w_router, sg], dim=0).contiguous()
         self.correction = tensors[t["correction"]].to(torch.float32).contiguous() if self.has_correction else None
         u0 = tensors[t["expert_up"].format(e=0)]
         # bfloat16 engine with 16-byte aligned rows: the grouped products run on the tensor cores
@@ -282,7 +290,8 @@ class RoutedMoE(FeedForward):
 
     def flops_per_token(self) -> float:
         m = 3 if self.gated else 2
-        return 2.0 * (m * self.top * self.ff * self.hidden + m * self.shared_ff * self.hidden + self.n_experts * self.hidden)
+        return 2.0 * (m * self.top * self.ff * self.hidden + m * self.shared_ff * self.hidden
+                      + (self.n_choices + self.has_shared_scale) * self.hidden)
 
     def forward(self, h, residual, ctx: StepContext):
         rt, T, top = self.runtime, ctx.n_tokens, self.top
@@ -297,13 +306,14 @@ class RoutedMoE(FeedForward):
         n_tiles, tiles = tiles[:1], tiles[4:]
         act = rt.get_scratch(self.act_name)[:, : self.ff]
         pair_out = rt.get_scratch("moe_pair_out", torch.float32)[:, : self.hidden]
-        logits = rt.get_scratch("router_logits", torch.float32)[:, : self.n_experts]
+        logits = rt.get_scratch("router_logits", torch.float32)[:, : self.w_router.shape[0]]
         choice = rt.get_scratch("router_choice", torch.int32).view(-1)[:pairs]
         weights = rt.get_scratch("router_weights", torch.float32).view(-1)[:pairs]
         ops.linear(h, self.w_router, logits, T, status=ctx.status)
-        ops.router_topk(logits, self.correction, top, T, choice, weights, ctx.status, sigmoid=self.score == "sigmoid",
-                        groups=self.groups, keep=self.keep, scale=self.route_scale, renormalize=self.renormalize)
-        ops.moe_route(None, choice.view(T, top), self.n_experts, T, rows, order, tiles, n_tiles, ctx.status)
+        ops.router_topk(logits[:, : self.n_choices], self.correction, top, T, choice, weights, ctx.status,
+                        sigmoid=self.score == "sigmoid", groups=self.groups, keep=self.keep, scale=self.route_scale,
+                        renormalize=self.renormalize, group_worth=self.group_worth)
+        ops.moe_route(None, choice.view(T, top), self.n_experts, T, rows, order, tiles, n_tiles, ctx.status, identity=self.identity)
         if tensor_cores:
             ops.grouped_gemm_mma(h, top, self.w_up, act, order, tiles, n_tiles, max_tiles, gated=self.gated, large=large,
                                  relu2=not self.gated)
@@ -326,9 +336,8 @@ class RoutedMoE(FeedForward):
                 ops.linear(h, self.w_shared_up, gu, T)
                 ops.silu_mul(gu, sact, T)
             ops.linear(sact, self.w_shared_down, shared_out, T, status=ctx.status)
-        if ctx.store_output:
-            ops.moe_combine(pair_out, top, 1.0, residual, T, shared=shared_out, pair_weights=weights)
-        else:
-            delta = rt.get_scratch("moe_delta", torch.float32)[:, : self.hidden]
-            ops.moe_combine(pair_out, top, 1.0, delta, T, shared=shared_out, pair_weights=weights)
-            ops.residual_add(residual, delta, T)
+        copy, ctx.stream_copy = ctx.stream_copy, None
+        ops.moe_combine(pair_out, top, 1.0, residual, T, shared=shared_out, h=h if self.identity else None, pair_weights=weights,
+                        choice=choice if self.identity else None, n_experts=self.n_experts,
+                        gate_logit=logits[:, self.n_choices:] if self.has_shared_scale else None, scale=self.out_scale,
+                        accumulate=not ctx.store_output, copy=copy)

@@ -121,3 +121,47 @@ class ActivationMLP(FeedForward):
         ops.linear(h, self.w_up, act, T, status=ctx.status)
         ops.activation(act, act, T, self.activation, self.act_params)
         ops.linear(act, self.w_down, residual, T, accumulate=not ctx.store_output, status=ctx.status)
+
+
+@register_part("feed_forward", "token_gate")
+class TokenGate(FeedForward):
+    """What a layer takes from the token itself: W_out (gelu(W_gate h) * e), gelu in its tanh form and float32, e the columns
+    [column, column + dim) of the token's row in a table.
+
+    params: hidden, dim, vocab, column (first column of this layer's part of the table), table_width (columns of the table).
+    tensors: gate_proj [dim, hidden], out_proj [hidden, dim], table [vocab, table_width]."""
+    gathered = ("table",)         # a step reads rows of it, not the whole
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        p = spec.params
+        self.hidden, self.dim, self.vocab = int(p["hidden"]), int(p["dim"]), int(p["vocab"])
+        self.column, self.table_width = int(p["column"]), int(p["table_width"])
+        if not 0 <= self.column <= self.table_width - self.dim:
+            raise ValueError(f"token_gate: columns {self.column} to {self.column + self.dim} of a table of {self.table_width}")
+        pad = (self.dim + 7) // 8 * 8
+        self.pre_name, self.act_name = f"token_gate_pre_{pad}", f"token_gate_act_{pad}"
+        runtime.scratch(self.pre_name, runtime.max_batch_tokens, pad, torch.float32)
+        runtime.scratch(self.act_name, runtime.max_batch_tokens, pad)
+
+    def tensor_needs(self):
+        t = self.spec.tensors
+        return {t["gate_proj"]: TensorNeed((self.dim, self.hidden)), t["out_proj"]: TensorNeed((self.hidden, self.dim)),
+                t["table"]: TensorNeed((self.vocab, self.table_width), "embedding")}
+
+    def load(self, tensors):
+        t = self.spec.tensors
+        self.w_gate = tensors[t["gate_proj"]].contiguous()
+        self.w_out = tensors[t["out_proj"]].contiguous()
+        self.table = tensors[t["table"]]
+
+    def flops_per_token(self) -> float:
+        return 4.0 * self.hidden * self.dim
+
+    def forward(self, h, residual, ctx):
+        rt, T = self.runtime, ctx.n_tokens
+        pre = rt.get_scratch(self.pre_name, torch.float32)[:, : self.dim]
+        act = rt.get_scratch(self.act_name)[:, : self.dim]
+        ops.linear(h, self.w_gate, pre, T, status=ctx.status)
+        ops.gelu_table_gate(pre, self.table, self.column, ctx.token_ids, act, T, ctx.status)
+        ops.linear(act, self.w_out, residual, T, accumulate=not ctx.store_output, status=ctx.status)

@@ -15,7 +15,7 @@ from .spec import TensorNeed
 
 @register_part("norm", "rmsnorm")
 class RMSNorm(Norm):
-    """params: width, eps.  tensors: weight."""
+    """params: width, eps, gain_scale (default 1: a constant that multiplies the weight, in float32).  tensors: weight."""
     chain_safe = True
     takes_owed = True
 
@@ -23,6 +23,7 @@ class RMSNorm(Norm):
         super().__init__(spec, runtime)
         self.width = int(spec.params["width"])
         self.eps = float(spec.params["eps"])
+        self.gain_scale = float(spec.params.get("gain_scale", 1.0))
         self.weight = None
 
     def tensor_needs(self):
@@ -30,6 +31,8 @@ class RMSNorm(Norm):
 
     def load(self, tensors):
         self.weight = tensors[self.spec.tensors["weight"]].contiguous()
+        if self.gain_scale != 1.0:
+            self.weight = (self.weight.to(torch.float32) * self.gain_scale).contiguous()
 
     def forward(self, x, out, n_rows, rows=None, owed=None):
         ops.rmsnorm(x, self.weight, self.eps, out, rows=rows, n_rows=n_rows, pending=owed)
@@ -63,6 +66,8 @@ class ScalarRMSNorm(RMSNorm):
 
     def load(self, tensors):
         self._gain = tensors[self.spec.tensors["weight"]].reshape(1).contiguous()
+        if self.gain_scale != 1.0:
+            self._gain = self._gain.to(torch.float32) * self.gain_scale
         # the row kernels shared with the vector kind read one weight per coordinate
         self.weight = self._gain.expand(self.width).contiguous()
 

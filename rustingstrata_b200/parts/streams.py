@@ -184,7 +184,7 @@ class HyperConnectionBlock(Block):
         else:
             ops.stream_layernorm(residual, S, m_in, n1.weight, n1.bias, n1.eps, h, T)
         nxt = ctx.next_reader
-        fuse_next = nxt is not None and nxt[0] == S and nxt[1] == self.hidden
+        fuse_next = isinstance(nxt, tuple) and nxt[0] == S and nxt[1] == self.hidden
         tail = dict(next_coef=nxt[2], next_weight=nxt[3], next_bias=nxt[4], next_eps=nxt[5], next_out=h) if fuse_next else {}
         ctx.store_output = True
         try:
