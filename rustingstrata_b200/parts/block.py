@@ -28,6 +28,7 @@ class PreNormBlock(Block):
     roles = {"mixer_norm": "norm", "mixer": "mixer", "feed_forward_norm": "norm", "feed_forward": "feed_forward",
              "side": "feed_forward", "side_norm": "norm"}
     optional = ("feed_forward_norm", "feed_forward", "side", "side_norm")
+    side = side_norm = None
 
     def __init__(self, spec, runtime, parts):
         super().__init__(spec, runtime, parts)
@@ -60,7 +61,7 @@ class PreNormBlock(Block):
     def forward(self, residual, ctx, call):
         T = ctx.n_tokens
         h = self.runtime.get_scratch("normed")[:, : self.hidden]
-        if ctx.normed_ready:
+        if getattr(ctx, "normed_ready", False):
             ctx.normed_ready = False             # the block before this one left the normed stream in h
         else:
             self.norm_of_stream(self.mixer_norm, residual, h, ctx)

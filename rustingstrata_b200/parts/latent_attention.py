@@ -37,7 +37,7 @@ from .spec import CacheNeed, PartSpec, TensorNeed
 @register_part("mixer", "latent_attention")
 class LatentAttention(PagedAttention):
     """params: hidden, n_heads, dim (unrotated query/key size per head), rot_dim, vdim, kv_rank, scale, eps (of the
-    latents' norms), window (None: every key), q_rank (None: q = W_q h), sink (bool, default False), gate (None, "head" or
+    latents' norms), window (None: every key), q_rank (None: q = W_q h), sink (bool, default False), gate (None, "head" or True, or
     "element"), out_scale (default 1), weights_bits (16, the default: the tensor-core kernel rounds the softmax weights to
     bfloat16 for the weighted sum; 32: it multiplies them in two bfloat16 terms).  tensors: q_proj [heads * (dim + rot_dim),
     hidden], or with q_rank dq_proj [q_rank, hidden], q_latent_norm [q_rank] and q_proj [heads * (dim + rot_dim), q_rank];
@@ -63,7 +63,7 @@ class LatentAttention(PagedAttention):
         self.spec = spec
         self._tensor_cores = None
         self.latent_eps = float(p["eps"])
-        self.gate = p.get("gate") or None
+        self.gate = {True: "head"}.get(p.get("gate"), p.get("gate") or None)
         if self.gate not in (None, "head", "element"):
             raise ValueError(f"latent_attention: gate {self.gate!r} (known: None, 'head', 'element')")
         self.gate_cols = {None: 0, "head": self.n_heads, "element": self.n_heads * self.vdim}[self.gate]
