@@ -95,8 +95,8 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=0, help="run this many of the configuration's layers (0 = all)")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--no-points", action="store_true", help="skip decode at batch 1 and 64")
-    ap.add_argument("--workload", default="headline", choices=["headline", "14b-mixed", "32b-long", "lokinex", "tabedra", "kupelix", "kozasun", "sefelorn"])
-    ap.add_argument("--sizes", default="1024,2048", help="with --workload lokinex, tabedra, kupelix, kozasun or sefelorn: widths to run")
+    ap.add_argument("--workload", default="headline", choices=["headline", "14b-mixed", "32b-long", "lokinex", "tabedra", "kupelix", "kozasun", "sefelorn", "gemodra"])
+    ap.add_argument("--sizes", default="1024,2048", help="with --workload lokinex, tabedra, kupelix, kozasun, sefelorn or gemodra: widths to run")
     ap.add_argument("--marginal", action="store_true", help="marginal cost of each kernel family inside the decode step")
     ap.add_argument("--prompt-len", type=int, default=PROMPT, help="with --marginal: tokens each request holds")
     ap.add_argument("--marginal-prefill", action="store_true",
@@ -121,7 +121,7 @@ def main() -> int:
         return long_context_workload(args)
     if args.workload == "lokinex":
         return lokinex_workload(args)
-    if args.workload in ("tabedra", "kupelix", "kozasun", "sefelorn"):
+    if args.workload in ("tabedra", "kupelix", "kozasun", "sefelorn", "gemodra"):
         return lokinex_workload(args, design=args.workload)
 
     import numpy as np
@@ -465,6 +465,24 @@ def sefelorn_config(width: int) -> dict:
             "loop": {"start": 0, "stop": 4, "times": 2}}
 
 
+def gemodra_config(width: int) -> dict:
+    """A Gemodra model whose layers resemble real ones at this width: latent attention with heads of 128 query/key and 128
+    value coordinates over a latent of width / 4, with 64 rotated ones besides and queries through a latent of 3/4 width in
+    two layers of three, without positions and queries through half the width in the third; 32 experts of 3/4 width and 8
+    identity experts in 4 groups of which 2 are kept, 4 per token, and a shared expert of 3/2 width; a per-layer token input
+    of width / 8; eight layers."""
+    heads = width // 128
+    rot = {"type": "latent_attention", "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": width // 4,
+                                                 "q_rank": width * 3 // 4, "scale": 192 ** -0.5, "rot": {"base": 1000000.0, "dims": 64}}}
+    flat = {"type": "latent_attention_2", "mixer": {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": width // 4,
+                                                    "q_rank": width // 2, "scale": 128 ** -0.5}}
+    moe = {"kind": "moe", "router": {"experts": 32, "identity": 8, "top": 4, "scale": 2.5, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": width * 3 // 4}, "shared": {"ff": width * 3 // 2}}
+    return {"architecture": "Gemodra", "vocab": 32768, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "token_side": {"dim": width // 8}, "logit_softcap": 30.0, "max_positions": 8192,
+            "layers": [dict(flat if i % 3 == 2 else rot, mlp=moe) for i in range(8)]}
+
+
 def qwen3_windowed(width: int) -> dict:
     """The closest existing model for the Tabedra design: the Qwen3 decoder of :func:`qwen3_like` with the same sliding
     window on every layer and as many key/value heads."""
@@ -490,7 +508,8 @@ class OpTimer:
              "attention_decode_items", "silu_mul", "residual_add", "sample", "latent_expand", "embed_sum", "stream_layernorm",
              "stream_update", "router_topk", "conv_norm_kv_write", "sigmoid_gate", "talking_attention_prep", "talking_attention", "talking_attention_mma", "grouped_attention_mma",
              "state_recurrence", "state_recurrence_chunked", "hgrn2_prep", "delta_prep", "head_norm_gate", "activation", "scale_rows", "retention_prep",
-             "mamba2_prep", "low_rank_decay", "pad_heads", "gated_group_norm", "add_embed")
+             "mamba2_prep", "low_rank_decay", "pad_heads", "gated_group_norm", "add_embed", "embed_rmsnorm",
+             "gelu_table_gate", "cast_rows", "softcap_rows")
 
     def __init__(self):
         self.events, self.real = [], {}
@@ -545,12 +564,13 @@ def lokinex_workload(args, design: str = "lokinex") -> int:
     clocks.start()
     pair = {"lokinex": (lokinex_config, qwen3_like), "tabedra": (tabedra_config, qwen3_windowed),
             "kupelix": (kupelix_config, qwen3_like), "kozasun": (kozasun_config, kupelix_config),
-            "sefelorn": (sefelorn_config, kupelix_config)}[design]
+            "sefelorn": (sefelorn_config, kupelix_config), "gemodra": (gemodra_config, kozasun_config)}[design]
     out = {"workload": design, "prompt_len": PROMPT, "batch": args.batch, "steps": args.steps, "dtype": "bf16",
            "data": "synthetic", "weights": "random N(0,0.02) bf16", "peaks": pk["source"], "sizes": {}}
     for width in [int(x) for x in args.sizes.split(",")]:
         rec = {}
-        other = "kupelix" if design in ("kozasun", "sefelorn") else "qwen3"        # the closest existing model of the design
+        # the closest existing model of the design
+        other = {"kozasun": "kupelix", "sefelorn": "kupelix", "gemodra": "kozasun"}.get(design, "qwen3")
         for name, cfg in ((design, pair[0](width)), (other, pair[1](width))):
             V = cfg.get("vocab", cfg.get("vocab_size"))
             eng = Engine(cfg, dtype="bfloat16", random_seed=0, page_size=16, max_tokens=args.batch * CONTEXT,

@@ -22,13 +22,14 @@ struct GroupedMmaParams {
     const int* order; const int* tiles; const int* n_tiles;        // tiles == null: every expert takes all dense_rows rows
     int dense_rows, tiles_per_expert;
     int K, gated;                                                  // gated: 0 plain; 1 SiLU(gate) * up of alternating rows; 2 plain, then max(., 0)^2
-    int use_gate; OutputGate gate;                                 // plain products of blocks: the result times gate.factor(row, expert, column)
+    OutputGate gate;                                               // GATE: the result times gate.factor(row, expert, column)
 };
 
 // BM x BN: the CTA's tile; WM x WN warps, each owning (BM / WM) x (BN / WN) of it.  64 x 64 with 2 x 2 warps where an
 // expert has few rows (a decode step reads every expert's matrix for a handful of rows: the weights are the cost), 128 x
 // 128 with 2 x 4 warps for prompt portions, where the traffic from L2 per multiply-add halves with the tile's edge.
-template <int BM, int BN, int WM, int WN>
+// GATE (plain products): the epilogue of a product behind a gate, compiled apart because it costs registers.
+template <int BM, int BN, int WM, int WN, bool GATE>
 __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const GroupedMmaParams p) {
     constexpr int THREADS = WM * WN * 32, MT = BM / WM / 16, NT = BN / WN / 8;
     int e, row0, rows;
@@ -127,6 +128,8 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
         for (int half = 0; half < 2; ++half) {
             const int pr = pair_of_row[m_base + i * 16 + (lane >> 2) + 8 * half];
             if (pr < 0) continue;
+            const bool row_gate = GATE && (p.gate.g == nullptr || p.gate.per_block);
+            const float row_factor = row_gate ? p.gate.factor(pr, e, 0) : 1.0f;
 #pragma unroll
             for (int j = 0; j < NT; ++j) {
                 const int gn = n0 + n_base + j * 8 + (lane & 3) * 2;
@@ -139,9 +142,9 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
                     c0 = fmaxf(c0, 0.f); c0 *= c0;
                     c1 = fmaxf(c1, 0.f); c1 *= c1;
                 }
-                if (p.use_gate) {
-                    if (gn < p.w_rows) c0 *= p.gate.factor(pr, e, e * p.w_rows + gn);
-                    if (gn + 1 < p.w_rows) c1 *= p.gate.factor(pr, e, e * p.w_rows + gn + 1);
+                if (GATE) {
+                    c0 *= row_gate ? row_factor : gn < p.w_rows ? p.gate.factor(pr, e, e * p.w_rows + gn) : 0.f;
+                    c1 *= row_gate ? row_factor : gn + 1 < p.w_rows ? p.gate.factor(pr, e, e * p.w_rows + gn + 1) : 0.f;
                 }
                 if (p.gated == 1) {
                     if (gn + 1 < p.w_rows) {
@@ -179,9 +182,9 @@ RS_EXPORT int rs_grouped_gemm_mma(const void* a, long a_stride, int a_div, const
     if (K <= 0 || K % 8 || a_stride % 8 || w_expert_stride % 8 || ((size_t)a & 15) || ((size_t)w & 15) || (gated == 1 && w_rows % 2) || gated < 0 || gated > 2)
         return (int)cudaErrorInvalidValue;
     GroupedMmaParams p{a, RS_BF16, a_stride, a_div, 0, (const __nv_bfloat16*)w, w_expert_stride, w_rows, nullptr, 0, out, out_dt,
-                       out_stride, 0, order, tiles, n_tiles, 0, 1, K, gated, 0, OutputGate{nullptr, 0, 0, 1.0f}};
-    if (large) grouped_gemm_mma_kernel<128, 128, 2, 4><<<dim3((w_rows + 127) / 128, max_tiles), 256, 0, (cudaStream_t)stream>>>(p);
-    else grouped_gemm_mma_kernel<64, 64, 2, 2><<<dim3((w_rows + 63) / 64, max_tiles), 128, 0, (cudaStream_t)stream>>>(p);
+                       out_stride, 0, order, tiles, n_tiles, 0, 1, K, gated, OutputGate{nullptr, 0, 0, 1.0f}};
+    if (large) grouped_gemm_mma_kernel<128, 128, 2, 4, false><<<dim3((w_rows + 127) / 128, max_tiles), 256, 0, (cudaStream_t)stream>>>(p);
+    else grouped_gemm_mma_kernel<64, 64, 2, 2, false><<<dim3((w_rows + 63) / 64, max_tiles), 128, 0, (cudaStream_t)stream>>>(p);
     return rs_launch_result();
 }
 
@@ -200,9 +203,13 @@ RS_EXPORT int rs_block_linear_mma(const void* x, int x_dt, long x_stride, long i
     const int bm = T > 256 ? 128 : 64;
     const int tiles_per = (T + bm - 1) / bm;
     GroupedMmaParams p{x, x_dt, x_stride, 1, in_bs, (const __nv_bfloat16*)w, (long)O * I, O, bias, bias_dt, out, out_dt, out_stride,
-                       out_bs, nullptr, nullptr, nullptr, T, tiles_per, I, 0, gate != nullptr || out_scale != 1.0f,
-                       OutputGate{gate, gate_stride, gate_per_block, out_scale}};
-    if (bm == 128) grouped_gemm_mma_kernel<128, 128, 2, 4><<<dim3((O + 127) / 128, tiles_per * B), 256, 0, (cudaStream_t)stream>>>(p);
-    else grouped_gemm_mma_kernel<64, 64, 2, 2><<<dim3((O + 63) / 64, tiles_per * B), 128, 0, (cudaStream_t)stream>>>(p);
+                       out_bs, nullptr, nullptr, nullptr, T, tiles_per, I, 0, OutputGate{gate, gate_stride, gate_per_block, out_scale}};
+    const cudaStream_t s = (cudaStream_t)stream;
+    const dim3 wide((O + 127) / 128, tiles_per * B), narrow((O + 63) / 64, tiles_per * B);
+    if (gate != nullptr || out_scale != 1.0f) {
+        if (bm == 128) grouped_gemm_mma_kernel<128, 128, 2, 4, true><<<wide, 256, 0, s>>>(p);
+        else grouped_gemm_mma_kernel<64, 64, 2, 2, true><<<narrow, 128, 0, s>>>(p);
+    } else if (bm == 128) grouped_gemm_mma_kernel<128, 128, 2, 4, false><<<wide, 256, 0, s>>>(p);
+    else grouped_gemm_mma_kernel<64, 64, 2, 2, false><<<narrow, 128, 0, s>>>(p);
     return rs_launch_result();
 }
