@@ -438,10 +438,10 @@ def bf16lib():
         lib.rs_block_linear_mma.argtypes = [c_void_p, c_int, c_long, c_long, c_void_p, c_void_p, c_int, c_void_p, c_int, c_long,
                                             c_long, c_int, c_int, c_int, c_int, c_void_p, c_long, c_int, c_float, c_void_p]
         lib.rs_attention_latent_supported.argtypes = [c_int, c_int, c_int]
-        lib.rs_attention_latent_q_per_cta.argtypes = [c_int]
+        lib.rs_attention_latent_q_per_cta.argtypes = [c_int, c_int]
         lib.rs_attention_latent_bf16.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_void_p,
                                                  c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                                                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p]
+                                                 c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]
         lib.rs_attention_prefill_bf16_supported.argtypes = [c_int, c_int, c_int]
         lib.rs_attention_prefill_bf16_q_per_cta.argtypes = [c_int, c_int]
         _bf16 = lib
@@ -1042,9 +1042,12 @@ def attention_latent_ok(dtype: torch.dtype, n_heads: int, lat: int, page_size: i
     return dtype == torch.bfloat16 and bool(bf16lib().rs_attention_latent_supported(n_heads, lat, page_size))
 
 
-def attention_latent_q_per_cta(n_heads: int) -> int:
+LATENT_WIDE_ROWS = 64     # query rows (tokens x heads) of a CTA of the wide portion kernel
+
+
+def attention_latent_q_per_cta(n_heads: int, wide: bool = False) -> int:
     """Query tokens per work item of the portion form of :func:`attention_latent`."""
-    return int(bf16lib().rs_attention_latent_q_per_cta(n_heads))
+    return int(bf16lib().rs_attention_latent_q_per_cta(n_heads, 1 if wide else 0))
 
 
 def attention_latent(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
@@ -1052,13 +1055,15 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
                      page_size: int, window: int, scale: float, decode: bool, status: torch.Tensor, split_keys: int = 128,
                      max_splits: int = 1, split_start: Optional[torch.Tensor] = None, total_splits: int = 0,
                      partial: Optional[torch.Tensor] = None, split_weights: bool = False,
-                     sink: Optional[torch.Tensor] = None) -> None:
+                     sink: Optional[torch.Tensor] = None, wide: bool = False, v_cols: Optional[int] = None) -> None:
     """Attention of ``n_heads`` query heads over a one-plane cache [pages, 1, 1, page_size, lat] whose rows are key and
     value at once, on the tensor cores (csrc/attention_latent_mma.cu).  ``work``: (sequence, first query) tiles of
     :func:`attention_latent_q_per_cta` tokens, or with ``decode`` one sequence per entry, the keys cut into splits whose
     partial results (layout of :func:`attention_simt`) are merged by a second kernel.  ``split_weights``: the softmax weights
     enter the weighted sum in two bfloat16 terms (the float32 weight to 2^-17) instead of rounded to bfloat16.  ``sink``:
-    float32 [n_heads] or None: exp(sink[h]) joins the denominator of head h's softmax."""
+    float32 [n_heads] or None: exp(sink[h]) joins the denominator of head h's softmax.  ``wide`` (portions): tiles of 64 query rows,
+    of ``attention_latent_q_per_cta(n_heads, wide=True)`` tokens.  ``v_cols``: only the first so many columns of a row (a multiple
+    of 8; default all) are summed and written."""
     _cuda(q, out, cache, block_table, q_start, kv_len, work, status, partial, split_start)
     _check_sink(sink, n_heads)
     _rows_contiguous(q, "q")
@@ -1081,7 +1086,8 @@ def attention_latent(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
         _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(cache), cache.stride(0), cache.shape[0], page_size,
         _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len), _ptr(work), n_work, n_heads, lat, int(window),
         float(scale), 1 if decode else 0, split_keys, max_splits, _ptr(split_start), _ptr(partial), slots,
-        1 if split_weights else 0, _ptr(sink), _ptr(status), _stream()), "attention_latent", 2 if decode else 1)
+        1 if split_weights else 0, _ptr(sink), lat if v_cols is None else int(v_cols), 1 if wide else 0, _ptr(status), _stream()),
+        "attention_latent", 2 if decode else 1)
 
 
 def attention_decode_items(split_start: torch.Tensor, n_work: int, n_kv: int, max_splits: int, items: torch.Tensor) -> None:

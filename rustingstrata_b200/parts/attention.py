@@ -167,10 +167,14 @@ class PagedAttention(Mixer):
                                                               self.runtime.page_size, force)
         return ("paged_attention", self.q_per_cta, self.window)
 
+    def _tile_tokens(self, q_lens: np.ndarray) -> int:
+        """Query tokens per tile of this step's portions (``q_lens``: the portions' lengths)."""
+        return self.q_per_cta
+
     def build_plan(self, batch: HostBatch):
         """Work lists: sequences with one query take the split (decode) form, the rest are cut into query tiles."""
-        qpc = self.q_per_cta
         single = batch.q_lens == 1
+        qpc = self._tile_tokens(batch.q_lens[~single])
         dec = np.nonzero(single)[0].astype(np.int32)
         splits = decode_splits(batch.kv_lens[dec], self.window).astype(np.int32) if len(dec) else np.zeros(0, np.int32)
         split_start = np.zeros(len(dec) + 1, np.int32)
@@ -198,7 +202,7 @@ class PagedAttention(Mixer):
             max_splits = (max_splits + SPLIT_BUCKET - 1) // SPLIT_BUCKET * SPLIT_BUCKET
             total_splits = 0
         return {"decode_work": dec, "split_start": split_start, "prefill_work": pre.reshape(-1),
-                "n_decode": int(len(dec)), "n_prefill": int(pre.shape[0]),
+                "n_decode": int(len(dec)), "n_prefill": int(pre.shape[0]), "tile_tokens": int(qpc),
                 "max_splits": max_splits, "total_splits": total_splits}
 
     # ---------------------------------------------------------------- the step

@@ -34,6 +34,9 @@ from .registry import register_part
 from .spec import CacheNeed, PartSpec, TensorNeed
 
 
+WIDE_TILES = 64        # tiles of 64 query rows from which a step's portions take the wide kernel
+
+
 @register_part("mixer", "latent_attention")
 class LatentAttention(PagedAttention):
     """params: hidden, n_heads, dim (unrotated query/key size per head), rot_dim, vdim, kv_rank, scale, eps (of the
@@ -141,9 +144,20 @@ class LatentAttention(PagedAttention):
         return self._tensor_cores
 
     def plan_key(self):
-        if self.q_per_cta is None and self.tensor_cores:
+        if not self.tensor_cores:
+            return super().plan_key()
+        if self.q_per_cta is None:
             self.q_per_cta = ops.attention_latent_q_per_cta(self.n_heads)
-        return super().plan_key()
+            self.q_per_wide_cta = ops.attention_latent_q_per_cta(self.n_heads, wide=True)
+        return ("latent_attention", self.n_heads, self.window)
+
+    def _tile_tokens(self, q_lens):
+        """Wide tiles (64 query rows) where the step's portions give the device enough of them, else narrow ones (16)."""
+        if not self.tensor_cores:
+            return super()._tile_tokens(q_lens)
+        head_parts = -(-self.n_heads // ops.LATENT_WIDE_ROWS)
+        tiles = int(sum(-(-int(n) // self.q_per_wide_cta) for n in q_lens)) * head_parts
+        return self.q_per_wide_cta if tiles >= WIDE_TILES else self.q_per_cta
 
     def _attend(self, q, ctx: StepContext, call: CallInfo):
         if not self.tensor_cores:
@@ -153,9 +167,11 @@ class LatentAttention(PagedAttention):
         plan = ctx.plans[self.plan_key()]
         common = dict(q=q, out=out, cache=call.cache, block_table=ctx.block_tables[call.cache_group], q_start=ctx.q_start,
                       kv_len=ctx.kv_len, n_heads=self.n_heads, lat=self.lat, page_size=rt.page_size, window=self.window,
-                      scale=self.scale, status=ctx.status, split_weights=self.split_weights, sink=self.sink)
+                      scale=self.scale, status=ctx.status, split_weights=self.split_weights, sink=self.sink,
+                      v_cols=(self.rank + 7) // 8 * 8)
         if plan["n_prefill"]:
-            ops.attention_latent(work=plan["prefill_work"], n_work=plan["n_prefill"], decode=False, **common)
+            ops.attention_latent(work=plan["prefill_work"], n_work=plan["n_prefill"], decode=False,
+                                 wide=plan["tile_tokens"] != self.q_per_cta, **common)
         if plan["n_decode"]:
             ops.attention_latent(work=plan["decode_work"], n_work=plan["n_decode"], decode=True, split_keys=SPLIT_KEYS,
                                  max_splits=plan["max_splits"], split_start=plan["split_start"],

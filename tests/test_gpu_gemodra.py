@@ -420,14 +420,15 @@ def test_block_product_behind_a_gate(rows, dtype, per):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("H,lat", [(3, 48), (20, 128), (8, 576)])
-def test_attention_over_latents_with_a_sink(dtype, H, lat):
-    """Both kernels of latent attention (portions and the split form over several splits) with sinks from next to nothing to
+@pytest.mark.parametrize("window", [0, 37])
+@pytest.mark.parametrize("H,lat,v", [(3, 48, 40), (20, 128, 128), (8, 576, 512), (70, 80, 72), (16, 320, 256), (33, 304, 304)])
+def test_attention_over_latents_with_a_sink(dtype, H, lat, v, window):
+    """The kernels of latent attention (narrow and wide portions, the split form over several splits) with sinks from next to nothing to
     far above every score, over scattered pages, against float64."""
     from rustingstrata_b200.kernels import ops
-    from rustingstrata_b200.parts.attention import SPLIT_KEYS
+    from rustingstrata_b200.parts.attention import SPLIT_KEYS, decode_splits
     g = torch.Generator().manual_seed(4)
-    page, kv_lens, q_lens = 16, [300, 41, 1], [1, 20, 1]
+    page, kv_lens, q_lens = 16, [300, 241, 1], [1, 120, 1]
     pages = [(n + page - 1) // page for n in kv_lens]
     ids = torch.randperm(sum(pages) + 5, generator=g)[: sum(pages)].to(torch.int32)
     table = torch.full((3, max(pages)), -1, dtype=torch.int32)
@@ -443,36 +444,44 @@ def test_attention_over_latents_with_a_sink(dtype, H, lat):
     for s in range(3):
         keys = torch.stack([cache[table[s, p // page], 0, 0, p % page] for p in range(kv_lens[s])]).double()
         for j in range(q_lens[s]):
-            t, seen = q_start[-1] + j, kv_lens[s] - q_lens[s] + j + 1
-            sc = q[t].double().view(H, lat) @ keys[:seen].T * scale
+            t, end = q_start[-1] + j, kv_lens[s] - q_lens[s] + j + 1
+            seen = slice(max(0, end - window) if window else 0, end)
+            sc = q[t].double().view(H, lat) @ keys[seen].T * scale
             m = torch.maximum(sc.max(-1).values, sink.double())
             e = torch.exp(sc - m[:, None])
-            want[t] = e @ keys[:seen] / (e.sum(-1) + torch.exp(sink.double() - m))[:, None]
+            want[t] = e @ keys[seen] / (e.sum(-1) + torch.exp(sink.double() - m))[:, None]
         q_start.append(q_start[-1] + q_lens[s])
     dev = lambda x: torch.as_tensor(x, dtype=torch.int32).cuda()                                    # noqa: E731
     out, status = torch.zeros(T, H * lat, dtype=dtype, device="cuda"), _status()
     singles = [s for s in range(3) if q_lens[s] == 1]
-    splits = [(kv_lens[s] + SPLIT_KEYS - 1) // SPLIT_KEYS for s in singles]
+    splits = [int(n) for n in decode_splits(np.array([kv_lens[s] for s in singles]), window)]
     split_start = dev([0] + list(np.cumsum(splits)))
     partial = torch.zeros(1, (sum(splits) + 2) * H * (lat + 2), device="cuda")
     common = dict(q=q.cuda(), out=out, cache=cache.cuda(), block_table=table.cuda(), q_start=dev(q_start), kv_len=dev(kv_lens),
-                  page_size=page, window=0, scale=scale, status=status, sink=sink.cuda())
+                  page_size=page, window=window, scale=scale, status=status, sink=sink.cuda())
     split = dict(split_keys=SPLIT_KEYS, max_splits=max(splits), split_start=split_start, total_splits=sum(splits), partial=partial)
     if dtype == torch.bfloat16:
-        qpc = ops.attention_latent_q_per_cta(H)
-        work = [(1, o) for o in range(0, q_lens[1], qpc)]
-        ops.attention_latent(work=dev(work).view(-1), n_work=len(work), decode=False, n_heads=H, lat=lat, split_weights=True, **common)
-        ops.attention_latent(work=dev(singles), n_work=len(singles), decode=True, n_heads=H, lat=lat, split_weights=True, **common, **split)
+        shape = dict(n_heads=H, lat=lat, split_weights=True, v_cols=v)
+        outs = {}
+        for wide in (False, True):
+            qpc = ops.attention_latent_q_per_cta(H, wide)
+            work = [(1, o) for o in range(0, q_lens[1], qpc)]
+            outs[wide] = torch.zeros_like(out)
+            ops.attention_latent(work=dev(work).view(-1), n_work=len(work), decode=False, wide=wide, **shape, **dict(common, out=outs[wide]))
+            ops.attention_latent(work=dev(singles), n_work=len(singles), decode=True, **shape, **dict(common, out=outs[wide]), **split)
     else:
         qpc = ops.attention_q_per_cta(H, 1)
         work = [(1, o) for o in range(0, q_lens[1], qpc)]
         shape = dict(n_q=H, n_kv=1, head_dim=lat, one_plane=True)
         ops.attention_simt(work=dev(work).view(-1), n_work=len(work), decode=False, **shape, **common)
         ops.attention_simt(work=dev(singles), n_work=len(singles), decode=True, **shape, **common, **split)
+        outs, v = {False: out}, lat
     assert int(status.item()) == 0
-    got = out.float().cpu().double().view(T, H, lat)
-    for h in range(H):
-        assert rel_err(got[:, h], want[:, h]) <= (2e-5 if dtype == torch.float32 else 1.2e-2), (h, float(sink[h]))
+    for form, x in outs.items():
+        got = x.float().cpu().double().view(T, H, lat)
+        for h in range(H):
+            assert rel_err(got[:, h, :v], want[:, h, :v]) <= (2e-5 if dtype == torch.float32 else 1.2e-2), (form, h, float(sink[h]))
+        assert dtype == torch.float32 or not got[:, :, v:].any()
 
 
 def test_small_row_kernels():
