@@ -4,14 +4,15 @@
 //
 // A CTA takes one row tile of one expert and a tile of rows of the expert's matrix (64 x 64 with 4 warps, or 128 x 128
 // with 8); it gathers its input rows through the sorted list (pair p reads row p / a_div of A), streams A and W in steps
-// of 32 of k through two shared-memory buffers with cp.async, and writes every pair's result to the pair's own row of the
+// of 32 of k through four shared-memory stages with cp.async, and writes every pair's result to the pair's own row of the
 // output.  Epilogues: plain store (float32 or bfloat16), or SiLU(gate) * up for a matrix whose rows
 // alternate gate, up: the two lie in neighbouring accumulator columns of one thread, and the output has half the columns.
 // Every output element accumulates k in ascending order, whatever else is in the batch.
 #include "mma_helpers.cuh"
+#include <atomic>
 
 namespace {
-constexpr int BK = 32, PITCH = BK + 8;
+constexpr int BK = 32, PITCH = BK + 8, STAGES = 4;
 
 struct GroupedMmaParams {
     const void* a; int a_dt; long a_stride; int a_div;             // bfloat16, or float32 rounded to bfloat16 on the way in
@@ -41,46 +42,57 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
         row0 = (blockIdx.y % p.tiles_per_expert) * BM;
         rows = min(BM, p.dense_rows - row0);
     }
-    __shared__ __align__(16) __nv_bfloat16 As[2][BM][PITCH];
-    __shared__ __align__(16) __nv_bfloat16 Ws[2][BN][PITCH];
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __nv_bfloat16* As = reinterpret_cast<__nv_bfloat16*>(smem_raw);                  // [STAGES][BM][PITCH]
+    __nv_bfloat16* Ws = As + STAGES * BM * PITCH;                                    // [STAGES][BN][PITCH]
     __shared__ int pair_of_row[BM];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int n0 = blockIdx.x * BN;
     if (tid < BM) pair_of_row[tid] = tid < rows ? (p.order != nullptr ? p.order[row0 + tid] : row0 + tid) : -1;
     __syncthreads();
-    const __nv_bfloat16* wbase = p.w + (size_t)e * p.w_expert_stride;
-    const size_t a_col0 = (size_t)e * p.a_expert_cols;
 
-    auto load = [&](int buf, int k0) {
+    // a thread fetches the same 16-byte column of the same rows at every step: their addresses are found once
+    constexpr int QA = BM * 4 / THREADS, QW = BN * 4 / THREADS;
+    const int ch8 = (tid & 3) * 8;
+    size_t a_at[QA];
+    const __nv_bfloat16* w_at[QW];
+    bool a_ok[QA], w_ok[QW];
 #pragma unroll
-        for (int q = 0; q < BM * 4 / THREADS; ++q) {
-            const int i = tid + q * THREADS;               // BM * 4 chunks of 16 bytes
-            const int r = i >> 2, ch = i & 3;
-            const int k = k0 + ch * 8;
-            const int pr = pair_of_row[r];
-            if (pr >= 0 && k < p.K) {
-                const size_t ai = (size_t)(pr / p.a_div) * p.a_stride + a_col0 + k;
+    for (int q = 0; q < QA; ++q) {
+        const int pr = pair_of_row[(tid + q * THREADS) >> 2];
+        a_ok[q] = pr >= 0;
+        a_at[q] = a_ok[q] ? (size_t)(pr / p.a_div) * p.a_stride + (size_t)e * p.a_expert_cols + ch8 : 0;
+    }
+#pragma unroll
+    for (int q = 0; q < QW; ++q) {
+        const int gn = n0 + ((tid + q * THREADS) >> 2);
+        w_ok[q] = gn < p.w_rows;
+        w_at[q] = p.w + (size_t)e * p.w_expert_stride + (w_ok[q] ? (size_t)gn * p.K + ch8 : 0);
+    }
+    auto load = [&](int stage, int k0) {
+        const bool k_ok = k0 + ch8 < p.K;
+#pragma unroll
+        for (int q = 0; q < QA; ++q) {
+            __nv_bfloat16* dst = As + (stage * BM + ((tid + q * THREADS) >> 2)) * PITCH + ch8;
+            if (a_ok[q] && k_ok) {
                 if (p.a_dt == RS_BF16) {
-                    cp_async16(smem_addr(&As[buf][r][ch * 8]), reinterpret_cast<const __nv_bfloat16*>(p.a) + ai);
+                    cp_async16(smem_addr(dst), reinterpret_cast<const __nv_bfloat16*>(p.a) + a_at[q] + k0);
                 } else {
-                    const float4 lo = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.a) + ai);
-                    const float4 hi = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.a) + ai + 4);
+                    const float* src = reinterpret_cast<const float*>(p.a) + a_at[q] + k0;
+                    const float4 lo = *reinterpret_cast<const float4*>(src), hi = *reinterpret_cast<const float4*>(src + 4);
                     uint4 u;
                     u.x = pack_bf16(lo.x, lo.y); u.y = pack_bf16(lo.z, lo.w); u.z = pack_bf16(hi.x, hi.y); u.w = pack_bf16(hi.z, hi.w);
-                    *reinterpret_cast<uint4*>(&As[buf][r][ch * 8]) = u;
+                    *reinterpret_cast<uint4*>(dst) = u;
                 }
             } else {
-                *reinterpret_cast<uint4*>(&As[buf][r][ch * 8]) = make_uint4(0, 0, 0, 0);
+                *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
             }
         }
 #pragma unroll
-        for (int q = 0; q < BN * 4 / THREADS; ++q) {
-            const int i = tid + q * THREADS;
-            const int r = i >> 2, ch = i & 3;
-            const int k = k0 + ch * 8;
-            const int gn = n0 + r;
-            if (gn < p.w_rows && k < p.K) cp_async16(smem_addr(&Ws[buf][r][ch * 8]), wbase + (size_t)gn * p.K + k);
-            else *reinterpret_cast<uint4*>(&Ws[buf][r][ch * 8]) = make_uint4(0, 0, 0, 0);
+        for (int q = 0; q < QW; ++q) {
+            __nv_bfloat16* dst = Ws + (stage * BN + ((tid + q * THREADS) >> 2)) * PITCH + ch8;
+            if (w_ok[q] && k_ok) cp_async16(smem_addr(dst), w_at[q] + k0);
+            else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
         }
     };
 
@@ -93,34 +105,33 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
     const int a_row = (lane & 7) + 8 * ((lane >> 3) & 1), a_col = 8 * (lane >> 4);
     const int b_row = (lane & 7) + 8 * (lane >> 4), b_col = 8 * ((lane >> 3) & 1);
     const int n_steps = (p.K + BK - 1) / BK;
-    load(0, 0);
-    cp_async_commit();
+#pragma unroll
+    for (int s = 0; s < STAGES - 1; ++s) {
+        if (s < n_steps) load(s, s * BK);
+        cp_async_commit();
+    }
     for (int s = 0; s < n_steps; ++s) {
-        if (s + 1 < n_steps) {
-            load((s + 1) & 1, (s + 1) * BK);
-            cp_async_commit();
-            cp_async_wait<1>();
-        } else {
-            cp_async_wait<0>();
-        }
-        __syncthreads();
-        const int buf = s & 1;
+        cp_async_wait<STAGES - 2>();
+        __syncthreads();                           // step s is here; nobody reads the stage of step s - 1 any more
+        if (s + STAGES - 1 < n_steps) load((s + STAGES - 1) % STAGES, (s + STAGES - 1) * BK);
+        cp_async_commit();
+        const __nv_bfloat16* At = As + (s % STAGES) * BM * PITCH;
+        const __nv_bfloat16* Wt = Ws + (s % STAGES) * BN * PITCH;
 #pragma unroll
         for (int kk = 0; kk < BK; kk += 16) {
             uint32_t a[MT][4], b[NT][2];
 #pragma unroll
             for (int i = 0; i < MT; ++i)
-                ldmatrix_x4(smem_addr(&As[buf][m_base + i * 16 + a_row][kk + a_col]), a[i][0], a[i][1], a[i][2], a[i][3]);
+                ldmatrix_x4(smem_addr(At + (m_base + i * 16 + a_row) * PITCH + kk + a_col), a[i][0], a[i][1], a[i][2], a[i][3]);
 #pragma unroll
             for (int j = 0; j < NT / 2; ++j)
-                ldmatrix_x4(smem_addr(&Ws[buf][n_base + j * 16 + b_row][kk + b_col]), b[2 * j][0], b[2 * j][1], b[2 * j + 1][0],
+                ldmatrix_x4(smem_addr(Wt + (n_base + j * 16 + b_row) * PITCH + kk + b_col), b[2 * j][0], b[2 * j][1], b[2 * j + 1][0],
                             b[2 * j + 1][1]);
 #pragma unroll
             for (int i = 0; i < MT; ++i)
 #pragma unroll
                 for (int j = 0; j < NT; ++j) mma16816(acc[i][j], a[i], b[j][0], b[j][1]);
         }
-        __syncthreads();
     }
 #pragma unroll
     for (int i = 0; i < MT; ++i)
@@ -168,6 +179,26 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
             }
         }
 }
+
+template <int BM, int BN, int WM, int WN, bool GATE>
+int launch_grouped(const GroupedMmaParams& p, dim3 grid, cudaStream_t s) {
+    constexpr size_t smem = (size_t)STAGES * (BM + BN) * PITCH * sizeof(__nv_bfloat16);
+    auto kern = grouped_gemm_mma_kernel<BM, BN, WM, WN, GATE>;
+    if (smem > 48 * 1024) {                        // the opt-in is a property of (kernel, device): asked for once on each
+        static std::atomic<bool> allowed[64];
+        int dev = 0;
+        cudaError_t e = cudaGetDevice(&dev);
+        if (e != cudaSuccess) return (int)e;
+        if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
+        if (!allowed[dev].load(std::memory_order_acquire)) {
+            e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (e != cudaSuccess) return (int)e;
+            allowed[dev].store(true, std::memory_order_release);
+        }
+    }
+    kern<<<grid, WM * WN * 32, smem, s>>>(p);
+    return rs_launch_result();
+}
 }  // namespace
 
 // Rows of one expert per CTA: the tile for few rows per expert (large == 0) and the one for prompt portions.
@@ -183,9 +214,9 @@ RS_EXPORT int rs_grouped_gemm_mma(const void* a, long a_stride, int a_div, const
         return (int)cudaErrorInvalidValue;
     GroupedMmaParams p{a, RS_BF16, a_stride, a_div, 0, (const __nv_bfloat16*)w, w_expert_stride, w_rows, nullptr, 0, out, out_dt,
                        out_stride, 0, order, tiles, n_tiles, 0, 1, K, gated, OutputGate{nullptr, 0, 0, 1.0f}};
-    if (large) grouped_gemm_mma_kernel<128, 128, 2, 4, false><<<dim3((w_rows + 127) / 128, max_tiles), 256, 0, (cudaStream_t)stream>>>(p);
-    else grouped_gemm_mma_kernel<64, 64, 2, 2, false><<<dim3((w_rows + 63) / 64, max_tiles), 128, 0, (cudaStream_t)stream>>>(p);
-    return rs_launch_result();
+    const cudaStream_t s = (cudaStream_t)stream;
+    if (large) return launch_grouped<128, 128, 2, 4, false>(p, dim3((w_rows + 127) / 128, max_tiles), s);
+    return launch_grouped<64, 64, 2, 2, false>(p, dim3((w_rows + 63) / 64, max_tiles), s);
 }
 
 // The block-diagonal product of sequence_parts.cu (rs_block_linear) for more than a few rows, through the same kernel:
@@ -206,10 +237,7 @@ RS_EXPORT int rs_block_linear_mma(const void* x, int x_dt, long x_stride, long i
                        out_bs, nullptr, nullptr, nullptr, T, tiles_per, I, 0, OutputGate{gate, gate_stride, gate_per_block, out_scale}};
     const cudaStream_t s = (cudaStream_t)stream;
     const dim3 wide((O + 127) / 128, tiles_per * B), narrow((O + 63) / 64, tiles_per * B);
-    if (gate != nullptr || out_scale != 1.0f) {
-        if (bm == 128) grouped_gemm_mma_kernel<128, 128, 2, 4, true><<<wide, 256, 0, s>>>(p);
-        else grouped_gemm_mma_kernel<64, 64, 2, 2, true><<<narrow, 128, 0, s>>>(p);
-    } else if (bm == 128) grouped_gemm_mma_kernel<128, 128, 2, 4, false><<<wide, 256, 0, s>>>(p);
-    else grouped_gemm_mma_kernel<64, 64, 2, 2, false><<<narrow, 128, 0, s>>>(p);
-    return rs_launch_result();
+    if (gate != nullptr || out_scale != 1.0f)
+        return bm == 128 ? launch_grouped<128, 128, 2, 4, true>(p, wide, s) : launch_grouped<64, 64, 2, 2, true>(p, narrow, s);
+    return bm == 128 ? launch_grouped<128, 128, 2, 4, false>(p, wide, s) : launch_grouped<64, 64, 2, 2, false>(p, narrow, s);
 }
