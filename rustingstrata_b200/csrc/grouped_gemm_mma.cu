@@ -1,10 +1,10 @@
 // One launch for the products of all experts of a mixture, on the warp-level tensor cores (mma.sync m16n8k16,
 // bfloat16 operands, float32 accumulation): the bfloat16 engine's form of the grouped product in moe_simt.cu, with
-// the same work list (moe_route: the step's (token, k) pairs sorted by expert and cut into row tiles of 64 or 128).
+// the same work list (moe_route: the step's (token, k) pairs sorted by expert and cut into row tiles of 16, 64 or 128).
 //
-// A CTA takes one row tile of one expert and a tile of rows of the expert's matrix (64 x 64 with 4 warps, or 128 x 128
-// with 8); it gathers its input rows through the sorted list (pair p reads row p / a_div of A), streams A and W in steps
-// of 32 of k through four shared-memory stages with cp.async, and writes every pair's result to the pair's own row of the
+// A CTA takes one row tile of one expert and a tile of rows of the expert's matrix (16 x 64, 64 x 64 or 128 x 128); it
+// gathers its input rows through the sorted list (pair p reads row p / a_div of A), streams A and W in steps of k through
+// several shared-memory stages with cp.async, and writes every pair's result to the pair's own row of the
 // output.  Epilogues: plain store (float32 or bfloat16), or SiLU(gate) * up for a matrix whose rows
 // alternate gate, up: the two lie in neighbouring accumulator columns of one thread, and the output has half the columns.
 // Every output element accumulates k in ascending order, whatever else is in the batch.
@@ -12,7 +12,10 @@
 #include <atomic>
 
 namespace {
-constexpr int BK = 32, PITCH = BK + 8, STAGES = 4;
+// A form's tile and pipeline: BM rows x BN matrix rows a CTA, steps of BK of k, STAGES of them in shared memory, WM x WN warps.
+struct Tile128 { static constexpr int BM = 128, BN = 128, BK = 32, STAGES = 4, WM = 2, WN = 4; };    // prompt portions
+struct Tile64 { static constexpr int BM = 64, BN = 64, BK = 32, STAGES = 4, WM = 2, WN = 2; };       // some rows per expert
+struct Tile16 { static constexpr int BM = 16, BN = 64, BK = 64, STAGES = 6, WM = 1, WN = 4; };       // single tokens
 
 struct GroupedMmaParams {
     const void* a; int a_dt; long a_stride; int a_div;             // bfloat16, or float32 rounded to bfloat16 on the way in
@@ -26,13 +29,14 @@ struct GroupedMmaParams {
     OutputGate gate;                                               // GATE: the result times gate.factor(row, expert, column)
 };
 
-// BM x BN: the CTA's tile; WM x WN warps, each owning (BM / WM) x (BN / WN) of it.  64 x 64 with 2 x 2 warps where an
-// expert has few rows (a decode step reads every expert's matrix for a handful of rows: the weights are the cost), 128 x
-// 128 with 2 x 4 warps for prompt portions, where the traffic from L2 per multiply-add halves with the tile's edge.
+// 16 x 64 where an expert has a handful of rows (a decode step reads every chosen expert's matrix for them: the weights are the
+// cost, fetched 128 bytes a row and step, six steps ahead), 64 x 64 for some rows, 128 x 128 for prompt portions, where the
+// traffic from L2 per multiply-add halves with the tile's edge.
 // GATE (plain products): the epilogue of a product behind a gate, compiled apart because it costs registers.
-template <int BM, int BN, int WM, int WN, bool GATE>
-__global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const GroupedMmaParams p) {
-    constexpr int THREADS = WM * WN * 32, MT = BM / WM / 16, NT = BN / WN / 8;
+template <class F, bool GATE>
+__global__ void __launch_bounds__(F::WM * F::WN * 32) grouped_gemm_mma_kernel(const GroupedMmaParams p) {
+    constexpr int BM = F::BM, BN = F::BN, BK = F::BK, STAGES = F::STAGES, WM = F::WM, WN = F::WN, PITCH = BK + 8;
+    constexpr int THREADS = WM * WN * 32, MT = BM / WM / 16, NT = BN / WN / 8, CH = BK / 8;      // CH: 16-byte columns of a step
     int e, row0, rows;
     if (p.tiles != nullptr) {
         if ((int)blockIdx.y >= p.n_tiles[0]) return;
@@ -52,20 +56,21 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
     __syncthreads();
 
     // a thread fetches the same 16-byte column of the same rows at every step: their addresses are found once
-    constexpr int QA = BM * 4 / THREADS, QW = BN * 4 / THREADS;
-    const int ch8 = (tid & 3) * 8;
+    constexpr int QA = BM * CH / THREADS, QW = BN * CH / THREADS;
+    static_assert(THREADS % CH == 0 && QA * THREADS == BM * CH && QW * THREADS == BN * CH, "the tile's pieces divide by the threads");
+    const int ch8 = (tid % CH) * 8;
     size_t a_at[QA];
     const __nv_bfloat16* w_at[QW];
     bool a_ok[QA], w_ok[QW];
 #pragma unroll
     for (int q = 0; q < QA; ++q) {
-        const int pr = pair_of_row[(tid + q * THREADS) >> 2];
+        const int pr = pair_of_row[(tid + q * THREADS) / CH];
         a_ok[q] = pr >= 0;
         a_at[q] = a_ok[q] ? (size_t)(pr / p.a_div) * p.a_stride + (size_t)e * p.a_expert_cols + ch8 : 0;
     }
 #pragma unroll
     for (int q = 0; q < QW; ++q) {
-        const int gn = n0 + ((tid + q * THREADS) >> 2);
+        const int gn = n0 + (tid + q * THREADS) / CH;
         w_ok[q] = gn < p.w_rows;
         w_at[q] = p.w + (size_t)e * p.w_expert_stride + (w_ok[q] ? (size_t)gn * p.K + ch8 : 0);
     }
@@ -73,7 +78,7 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
         const bool k_ok = k0 + ch8 < p.K;
 #pragma unroll
         for (int q = 0; q < QA; ++q) {
-            __nv_bfloat16* dst = As + (stage * BM + ((tid + q * THREADS) >> 2)) * PITCH + ch8;
+            __nv_bfloat16* dst = As + (stage * BM + (tid + q * THREADS) / CH) * PITCH + ch8;
             if (a_ok[q] && k_ok) {
                 if (p.a_dt == RS_BF16) {
                     cp_async16(smem_addr(dst), reinterpret_cast<const __nv_bfloat16*>(p.a) + a_at[q] + k0);
@@ -90,7 +95,7 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
         }
 #pragma unroll
         for (int q = 0; q < QW; ++q) {
-            __nv_bfloat16* dst = Ws + (stage * BN + ((tid + q * THREADS) >> 2)) * PITCH + ch8;
+            __nv_bfloat16* dst = Ws + (stage * BN + (tid + q * THREADS) / CH) * PITCH + ch8;
             if (w_ok[q] && k_ok) cp_async16(smem_addr(dst), w_at[q] + k0);
             else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
         }
@@ -180,10 +185,11 @@ __global__ void __launch_bounds__(WM * WN * 32) grouped_gemm_mma_kernel(const Gr
         }
 }
 
-template <int BM, int BN, int WM, int WN, bool GATE>
-int launch_grouped(const GroupedMmaParams& p, dim3 grid, cudaStream_t s) {
-    constexpr size_t smem = (size_t)STAGES * (BM + BN) * PITCH * sizeof(__nv_bfloat16);
-    auto kern = grouped_gemm_mma_kernel<BM, BN, WM, WN, GATE>;
+// Launches a form for ``row_tiles`` tiles of rows (times blocks).
+template <class F, bool GATE>
+int launch_grouped(const GroupedMmaParams& p, int row_tiles, cudaStream_t s) {
+    constexpr size_t smem = (size_t)F::STAGES * (F::BM + F::BN) * (F::BK + 8) * sizeof(__nv_bfloat16);
+    auto kern = grouped_gemm_mma_kernel<F, GATE>;
     if (smem > 48 * 1024) {                        // the opt-in is a property of (kernel, device): asked for once on each
         static std::atomic<bool> allowed[64];
         int dev = 0;
@@ -196,27 +202,27 @@ int launch_grouped(const GroupedMmaParams& p, dim3 grid, cudaStream_t s) {
             allowed[dev].store(true, std::memory_order_release);
         }
     }
-    kern<<<grid, WM * WN * 32, smem, s>>>(p);
+    kern<<<dim3((p.w_rows + F::BN - 1) / F::BN, row_tiles), F::WM * F::WN * 32, smem, s>>>(p);
     return rs_launch_result();
 }
 }  // namespace
 
-// Rows of one expert per CTA: the tile for few rows per expert (large == 0) and the one for prompt portions.
-RS_EXPORT int rs_grouped_gemm_mma_rows_per_tile(int large) { return large ? 128 : 64; }
+// Rows of one expert per CTA of form 0 (single tokens), 1 (some rows per expert) and 2 (prompt portions).
+RS_EXPORT int rs_grouped_gemm_mma_rows_per_tile(int form) { return form == 2 ? Tile128::BM : form == 1 ? Tile64::BM : Tile16::BM; }
 
 // a: bfloat16 [*, K] rows 16-byte aligned; w: bfloat16 [E][w_rows][K]; out: [pairs, w_rows] (or w_rows / 2 when gated,
 // the rows of w alternating gate, up).  K a multiple of 8.
 RS_EXPORT int rs_grouped_gemm_mma(const void* a, long a_stride, int a_div, const void* w, long w_expert_stride, int w_rows,
                                   void* out, int out_dt, long out_stride, const int* order, const int* tiles,
-                                  const int* n_tiles, int max_tiles, int K, int gated, int large, void* stream) {
+                                  const int* n_tiles, int max_tiles, int K, int gated, int form, void* stream) {
     if (max_tiles <= 0 || w_rows <= 0) return 0;
-    if (K <= 0 || K % 8 || a_stride % 8 || w_expert_stride % 8 || ((size_t)a & 15) || ((size_t)w & 15) || (gated == 1 && w_rows % 2) || gated < 0 || gated > 2)
+    if (K <= 0 || K % 8 || a_stride % 8 || w_expert_stride % 8 || ((size_t)a & 15) || ((size_t)w & 15) || (gated == 1 && w_rows % 2) || gated < 0 || gated > 2 || form < 0 || form > 2)
         return (int)cudaErrorInvalidValue;
     GroupedMmaParams p{a, RS_BF16, a_stride, a_div, 0, (const __nv_bfloat16*)w, w_expert_stride, w_rows, nullptr, 0, out, out_dt,
                        out_stride, 0, order, tiles, n_tiles, 0, 1, K, gated, OutputGate{nullptr, 0, 0, 1.0f}};
     const cudaStream_t s = (cudaStream_t)stream;
-    if (large) return launch_grouped<128, 128, 2, 4, false>(p, dim3((w_rows + 127) / 128, max_tiles), s);
-    return launch_grouped<64, 64, 2, 2, false>(p, dim3((w_rows + 63) / 64, max_tiles), s);
+    if (form == 2) return launch_grouped<Tile128, false>(p, max_tiles, s);
+    return form == 1 ? launch_grouped<Tile64, false>(p, max_tiles, s) : launch_grouped<Tile16, false>(p, max_tiles, s);
 }
 
 // The block-diagonal product of sequence_parts.cu (rs_block_linear) for more than a few rows, through the same kernel:
@@ -236,8 +242,7 @@ RS_EXPORT int rs_block_linear_mma(const void* x, int x_dt, long x_stride, long i
     GroupedMmaParams p{x, x_dt, x_stride, 1, in_bs, (const __nv_bfloat16*)w, (long)O * I, O, bias, bias_dt, out, out_dt, out_stride,
                        out_bs, nullptr, nullptr, nullptr, T, tiles_per, I, 0, OutputGate{gate, gate_stride, gate_per_block, out_scale}};
     const cudaStream_t s = (cudaStream_t)stream;
-    const dim3 wide((O + 127) / 128, tiles_per * B), narrow((O + 63) / 64, tiles_per * B);
     if (gate != nullptr || out_scale != 1.0f)
-        return bm == 128 ? launch_grouped<128, 128, 2, 4, true>(p, wide, s) : launch_grouped<64, 64, 2, 2, true>(p, narrow, s);
-    return bm == 128 ? launch_grouped<128, 128, 2, 4, false>(p, wide, s) : launch_grouped<64, 64, 2, 2, false>(p, narrow, s);
+        return bm == 128 ? launch_grouped<Tile128, true>(p, tiles_per * B, s) : launch_grouped<Tile64, true>(p, tiles_per * B, s);
+    return bm == 128 ? launch_grouped<Tile128, false>(p, tiles_per * B, s) : launch_grouped<Tile64, false>(p, tiles_per * B, s);
 }

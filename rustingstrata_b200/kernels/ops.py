@@ -1383,7 +1383,7 @@ def moe_route(ids: Optional[torch.Tensor], table: torch.Tensor, n_experts: int, 
             raise KernelError(f"moe_route: {name} must be contiguous int32")
     if order.numel() < n_tokens * top or (ids.numel() if ids is not None else V) < n_tokens:
         raise KernelError("moe_route: order must hold tokens * top entries")
-    if rows_per_tile not in (grouped_rows_per_tile(True), grouped_rows_per_tile(False), GROUPED_ROWS_LARGE):
+    if rows_per_tile not in (grouped_rows_per_tile(True), grouped_rows_per_tile(False)) + GROUPED_MMA_ROWS:
         raise KernelError("moe_route: rows_per_tile must be a tile size of the grouped product")
     _check(core().rs_moe_route(_ptr(ids), _ptr(table), V, top, n_experts, int(identity), n_tokens, rows_per_tile, _ptr(order), _ptr(tiles),
                                _ptr(n_tiles), tiles.numel() // 3, _ptr(status), _stream()), "moe_route")
@@ -1421,15 +1421,20 @@ def grouped_gemm_mma_ok(a: torch.Tensor, weight: torch.Tensor) -> bool:
             and weight.data_ptr() % 16 == 0)
 
 
-GROUPED_ROWS_LARGE = 128      # row tile of the tensor-core grouped product's form for prompt portions
+GROUPED_MMA_ROWS = (16, 64, 128)     # row tiles of the tensor-core grouped product's forms: single tokens, some rows, prompt portions
+GROUPED_MMA_FORMS = (0, 8, 96)       # pairs per expert on average from which a form is taken
+
+
+def grouped_mma_form(pairs: int, n_experts: int) -> int:
+    """The form of :func:`grouped_gemm_mma` for so many (token, k) pairs among so many experts."""
+    return max(i for i, least in enumerate(GROUPED_MMA_FORMS) if pairs >= least * n_experts)
 
 
 def grouped_gemm_mma(a: torch.Tensor, a_div: int, weight: torch.Tensor, out: torch.Tensor, order: torch.Tensor,
-                     tiles: torch.Tensor, n_tiles: torch.Tensor, max_tiles: int, gated: bool, large: bool = False,
+                     tiles: torch.Tensor, n_tiles: torch.Tensor, max_tiles: int, gated: bool, form: int = 1,
                      relu2: bool = False) -> None:
     """The grouped product of :func:`grouped_linear` on the tensor cores (csrc/grouped_gemm_mma.cu), for the row tiles
-    that ``moe_route`` lists: of ``GROUPED_ROWS_TILED`` rows (64 x 64 tiles, for few rows per expert), or with ``large`` of
-    ``GROUPED_ROWS_LARGE`` (128 x 128 tiles, for prompt portions).  ``gated``: the rows of every expert's matrix alternate
+    that ``moe_route`` lists, of ``GROUPED_MMA_ROWS[form]`` rows (:func:`grouped_mma_form`).  ``gated``: the rows of every expert's matrix alternate
     gate, up and out = SiLU(gate) * up has half as many columns as the matrix has rows.  ``relu2`` (plain products only):
     out = max(a W.T, 0)^2."""
     _cuda(a, weight, out, order, tiles, n_tiles)
@@ -1442,12 +1447,11 @@ def grouped_gemm_mma(a: torch.Tensor, a_div: int, weight: torch.Tensor, out: tor
     if a.shape[1] != K or out.shape[1] != (rows // 2 if gated else rows) or (gated and rows % 2) or max_tiles * 3 > tiles.numel():
         raise KernelError(f"grouped_gemm_mma: a {tuple(a.shape)} x weight {tuple(weight.shape)} -> out {tuple(out.shape)} "
                           f"does not fit")
-    if (int(bf16lib().rs_grouped_gemm_mma_rows_per_tile(0)), int(bf16lib().rs_grouped_gemm_mma_rows_per_tile(1))) != \
-            (GROUPED_ROWS_TILED, GROUPED_ROWS_LARGE):
+    if int(bf16lib().rs_grouped_gemm_mma_rows_per_tile(form)) != GROUPED_MMA_ROWS[form]:
         raise KernelError("grouped_gemm_mma: the compiled kernel's row tiles differ from the launcher's")
     _check(bf16lib().rs_grouped_gemm_mma(_ptr(a), a.stride(0), a_div, _ptr(weight), weight.stride(0), rows, _ptr(out),
                                          dtype_code(out), out.stride(0), _ptr(order), _ptr(tiles), _ptr(n_tiles), max_tiles,
-                                         K, 1 if gated else (2 if relu2 else 0), 1 if large else 0, _stream()), "grouped_gemm_mma")
+                                         K, 1 if gated else (2 if relu2 else 0), form, _stream()), "grouped_gemm_mma")
 
 
 def moe_combine(pair_out: torch.Tensor, top: int, weight: float, out: torch.Tensor, n_tokens: int,

@@ -54,7 +54,6 @@ class TableMoE(FeedForward):
     tensors: table [vocab, top]; expert_gate / expert_up / expert_down: name patterns with ``{e}`` for the expert's
     number; shared_gate, shared_up, shared_down, shared_scale [1, hidden] when there is a shared expert."""
     SMALL_PAIRS_PER_EXPERT = 4      # up to this many (token, k) pairs per expert on average the row-streaming form runs
-    LARGE_PAIRS_PER_EXPERT = 96     # from this many on average the tensor-core product takes its 128 x 128 tiles
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -130,8 +129,8 @@ class TableMoE(FeedForward):
         # bfloat16 engine: one tensor-core launch per projection for all experts, whatever the step's size
         tensor_cores = self.interleaved
         small = not tensor_cores and pairs <= self.SMALL_PAIRS_PER_EXPERT * self.n_experts
-        large = tensor_cores and pairs >= self.LARGE_PAIRS_PER_EXPERT * self.n_experts
-        rows = ops.GROUPED_ROWS_LARGE if large else _ROWS_PER_TILE[small]
+        form = ops.grouped_mma_form(pairs, self.n_experts)
+        rows = ops.GROUPED_MMA_ROWS[form] if tensor_cores else _ROWS_PER_TILE[small]
         max_tiles = self._max_tiles(pairs, rows)
         order = rt.get_scratch("moe_order", torch.int32).view(-1)
         tiles = rt.get_scratch("moe_tiles", torch.int32).view(-1)
@@ -140,8 +139,8 @@ class TableMoE(FeedForward):
         pair_out = rt.get_scratch("moe_pair_out", torch.float32)[:, : self.hidden]
         ops.moe_route(ctx.token_ids, self.table, self.n_experts, T, rows, order, tiles, n_tiles, ctx.status)
         if tensor_cores:
-            ops.grouped_gemm_mma(h, top, self.w_gate_up, act, order, tiles, n_tiles, max_tiles, gated=True, large=large)
-            ops.grouped_gemm_mma(act, 1, self.w_down, pair_out, order, tiles, n_tiles, max_tiles, gated=False, large=large)
+            ops.grouped_gemm_mma(h, top, self.w_gate_up, act, order, tiles, n_tiles, max_tiles, gated=True, form=form)
+            ops.grouped_gemm_mma(act, 1, self.w_down, pair_out, order, tiles, n_tiles, max_tiles, gated=False, form=form)
         else:
             ops.grouped_linear(h, top, self.w_gate_up, act, order, tiles, n_tiles, max_tiles, gated=True, small=small)
             ops.grouped_linear(act, 1, self.w_down, pair_out, order, tiles, n_tiles, max_tiles, gated=False, small=small)
@@ -183,7 +182,6 @@ class RoutedMoE(FeedForward):
     whose product with h is one more row of the router's.  The step's (token, k) pairs are sorted
     by expert on the device and one grouped product per projection serves all experts, as in :class:`TableMoE`."""
     SMALL_PAIRS_PER_EXPERT = TableMoE.SMALL_PAIRS_PER_EXPERT
-    LARGE_PAIRS_PER_EXPERT = TableMoE.LARGE_PAIRS_PER_EXPERT
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -298,8 +296,8 @@ class RoutedMoE(FeedForward):
         pairs = T * top
         tensor_cores = self.tensor_cores
         small = not tensor_cores and pairs <= self.SMALL_PAIRS_PER_EXPERT * self.n_experts
-        large = tensor_cores and pairs >= self.LARGE_PAIRS_PER_EXPERT * self.n_experts
-        rows = ops.GROUPED_ROWS_LARGE if large else _ROWS_PER_TILE[small]
+        form = ops.grouped_mma_form(pairs, self.n_experts)
+        rows = ops.GROUPED_MMA_ROWS[form] if tensor_cores else _ROWS_PER_TILE[small]
         max_tiles = self._max_tiles(pairs, rows)
         order = rt.get_scratch("moe_order", torch.int32).view(-1)
         tiles = rt.get_scratch("moe_tiles", torch.int32).view(-1)
@@ -315,9 +313,9 @@ class RoutedMoE(FeedForward):
                         renormalize=self.renormalize, group_worth=self.group_worth)
         ops.moe_route(None, choice.view(T, top), self.n_experts, T, rows, order, tiles, n_tiles, ctx.status, identity=self.identity)
         if tensor_cores:
-            ops.grouped_gemm_mma(h, top, self.w_up, act, order, tiles, n_tiles, max_tiles, gated=self.gated, large=large,
+            ops.grouped_gemm_mma(h, top, self.w_up, act, order, tiles, n_tiles, max_tiles, gated=self.gated, form=form,
                                  relu2=not self.gated)
-            ops.grouped_gemm_mma(act, 1, self.w_down, pair_out, order, tiles, n_tiles, max_tiles, gated=False, large=large)
+            ops.grouped_gemm_mma(act, 1, self.w_down, pair_out, order, tiles, n_tiles, max_tiles, gated=False, form=form)
         else:
             ops.grouped_linear(h, top, self.w_up, act, order, tiles, n_tiles, max_tiles, gated=self.gated, small=small,
                                relu2=not self.gated)
