@@ -509,7 +509,7 @@ class OpTimer:
              "stream_update", "router_topk", "conv_norm_kv_write", "sigmoid_gate", "talking_attention_prep", "talking_attention", "talking_attention_mma", "grouped_attention_mma",
              "state_recurrence", "state_recurrence_chunked", "hgrn2_prep", "delta_prep", "head_norm_gate", "activation", "scale_rows", "retention_prep",
              "mamba2_prep", "low_rank_decay", "pad_heads", "gated_group_norm", "add_embed", "embed_rmsnorm",
-             "gelu_table_gate", "cast_rows", "softcap_rows")
+             "gelu_table_gate", "cast_rows", "softcap_rows", "router_route", "latent_queries")
 
     def __init__(self):
         self.events, self.real = [], {}

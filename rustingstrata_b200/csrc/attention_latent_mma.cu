@@ -74,6 +74,8 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_kernel(const LatP
     float* stat_l = stat_m + ROWS;
     float* stat_c = stat_l + ROWS;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    pdl_launch_dependents();
+    pdl_wait();
 
     int seq, q_off, n_q_tok;
     if (p.decode) { seq = p.work[blockIdx.x]; q_off = 0; n_q_tok = 1; }
@@ -103,7 +105,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_kernel(const LatP
         const int tl = r / p.hc, h = head0 + r % p.hc;
         uint4 v = make_uint4(0, 0, 0, 0);
         if (tl < n_q_tok && h < p.n_heads)
-            v = *reinterpret_cast<const uint4*>(p.q + (size_t)(row0 + q_off + tl) * p.q_stride + (size_t)h * lat + ch * 8);
+            v = ld_dep(reinterpret_cast<const uint4*>(p.q + (size_t)(row0 + q_off + tl) * p.q_stride + (size_t)h * lat + ch * 8));
         *reinterpret_cast<uint4*>(Qs + r * pitch + ch * 8) = v;
     }
     if (tid < ROWS) { stat_m[tid] = -INFINITY; stat_l[tid] = 0.f; stat_c[tid] = 1.f; }
@@ -273,7 +275,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_kernel(const LatP
             for (int n = 0; n < NT_MAX; ++n) {
                 if (n < my_nt) {
                     const int d = dim_lo + n * 8 + (lane & 3) * 2;
-                    dst[d] = acc[n][2 * half]; dst[d + 1] = acc[n][2 * half + 1];
+                    *reinterpret_cast<float2*>(dst + d) = make_float2(acc[n][2 * half], acc[n][2 * half + 1]);
                 }
             }
             if (warp == 0 && (lane & 3) == 0) { dst[lat] = stat_m[r]; dst[lat + 1] = stat_l[r]; }
@@ -333,7 +335,7 @@ __global__ void __launch_bounds__(WTHREADS, 1) latent_portion_kernel(const LatPa
         const int tl = r / p.hc, h = head0 + r - tl * p.hc;
         uint4 v = make_uint4(0, 0, 0, 0);
         if (r < n_rows && h < p.n_heads)
-            v = *reinterpret_cast<const uint4*>(p.q + (size_t)(row0 + q_off + tl) * p.q_stride + (size_t)h * lat + ch * 8);
+            v = ld_dep(reinterpret_cast<const uint4*>(p.q + (size_t)(row0 + q_off + tl) * p.q_stride + (size_t)h * lat + ch * 8));
         *reinterpret_cast<uint4*>(Qs + r * pitch + ch * 8) = v;
     }
     if (tid < WR) { stat_m[tid] = -INFINITY; stat_l[tid] = 0.f; stat_c[tid] = 1.f; }
@@ -497,53 +499,59 @@ size_t wide_smem_bytes(int lat) {
     return (size_t)(WR + 2 * WK) * pitch * 2 + (size_t)WR * WS_PITCH * 4 + 2 * (size_t)WR * WP_PITCH * 2 + 3 * WR * 4;
 }
 
-// out[token of seq, head, :] = sum_s acc_s e^(m_s - M) / sum_s l_s e^(m_s - M), splits in ascending order
-__global__ void latent_merge_kernel(const LatParams p) {
-    const int w = blockIdx.x, h = blockIdx.y;
+// out[token of seq, head, :] = sum_s acc_s e^(m_s - M) / (sum_s l_s e^(m_s - M) + e^(sink - M)), splits in ascending order.
+// A lane takes a split's maximum and denominator (further ones in turn), the weights of up to MERGE_CACHED splits stay in shared
+// memory (a sequence with more recomputes the rest), and a thread adds up two columns over the splits, eight loads at a time.
+__global__ void __launch_bounds__(256) latent_merge_kernel(const LatParams p) {
+    __shared__ float ws[MERGE_CACHED];
+    __shared__ float stats[2];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int w = blockIdx.x, h = blockIdx.y, lat = p.lat;
     const int seq = p.work[w];
     const int kv_len = p.kv_len[seq];
     const int key_lo = p.window > 0 ? max(0, kv_len - p.window) : 0;
     const int n_splits = (kv_len + p.split_keys - 1) / p.split_keys - key_lo / p.split_keys;
-    const int lat = p.lat;
     if ((size_t)p.split_start[w] + n_splits > (size_t)p.partial_slots) {
         if (threadIdx.x == 0) atomicOr(p.status, RS_STATUS_BAD_PLAN);
         return;
     }
     const float* base = p.partial + ((size_t)p.split_start[w] * p.n_heads + h) * (lat + 2);
     const size_t split_stride = (size_t)p.n_heads * (lat + 2);
-    // every thread takes the splits' maxima in (the loads are independent of each other), then the weights of up to
-    // MERGE_CACHED splits and the denominator are kept in shared memory; a sequence with more splits recomputes them
-    __shared__ float ws[MERGE_CACHED];
-    __shared__ float stats[2];
-    float M = -INFINITY;
-#pragma unroll 4
-    for (int s = 0; s < n_splits; ++s) M = fmaxf(M, base[s * split_stride + lat]);
-    if (p.sink != nullptr) M = fmaxf(M, p.sink[h]);
     if (threadIdx.x < 32) {
-        float den = p.sink != nullptr && threadIdx.x == 0 ? __expf(p.sink[h] - M) : 0.f;
-        // lanes take splits in turn, added lane by lane: a fixed order
-        for (int s = threadIdx.x; s < n_splits; s += 32) {
-            const float* ps = base + s * split_stride;
-            const float e = __expf(ps[lat] - M);
+        const int lane = threadIdx.x;
+        float M = -INFINITY;
+        for (int s = lane; s < n_splits; s += 32) M = fmaxf(M, ld_dep(base + s * split_stride + lat));
+        M = warp_max(M);
+        if (p.sink != nullptr) M = fmaxf(M, p.sink[h]);
+        float den = p.sink != nullptr && lane == 0 ? __expf(p.sink[h] - M) : 0.f;
+        for (int s = lane; s < n_splits; s += 32) {           // lane by lane, then over the lanes: a fixed order
+            const float2 ml = ld_dep(reinterpret_cast<const float2*>(base + s * split_stride + lat));
+            const float e = __expf(ml.x - M);
             if (s < MERGE_CACHED) ws[s] = e;
-            den = fmaf(ps[lat + 1], e, den);
+            den = fmaf(ml.y, e, den);
         }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
-        if (threadIdx.x == 0) stats[0] = den;
+        den = warp_sum(den);
+        if (lane == 0) { stats[0] = den; stats[1] = M; }
     }
     __syncthreads();
-    const float inv = 1.0f / stats[0];
+    const float inv = 1.0f / stats[0], M = stats[1];
     __nv_bfloat16* dst = p.out + (size_t)p.q_start[seq] * p.out_stride + (size_t)h * lat;
-    for (int d = threadIdx.x; d < p.v_cols; d += blockDim.x) {
-        float num = 0.f;
-#pragma unroll 4
-        for (int s = 0; s < n_splits; ++s) {
-            const float* ps = base + s * split_stride;
-            const float e = s < MERGE_CACHED ? ws[s] : __expf(ps[lat] - M);
-            num = fmaf(ps[d], e, num);
+    for (int d = 2 * threadIdx.x; d < p.v_cols; d += 2 * blockDim.x) {
+        float2 num = make_float2(0.f, 0.f);
+        for (int s0 = 0; s0 < n_splits; s0 += 8) {
+            float2 v[8];
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+                v[u] = s0 + u < n_splits ? ld_dep(reinterpret_cast<const float2*>(base + (s0 + u) * split_stride + d)) : make_float2(0.f, 0.f);
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                if (s0 + u >= n_splits) break;
+                const float e = s0 + u < MERGE_CACHED ? ws[s0 + u] : __expf(ld_dep(base + (s0 + u) * split_stride + lat) - M);
+                num.x = fmaf(v[u].x, e, num.x); num.y = fmaf(v[u].y, e, num.y);
+            }
         }
-        dst[d] = __float2bfloat16_rn(num * inv);
+        *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16(num.x * inv, num.y * inv);
     }
 }
 
@@ -588,7 +596,7 @@ RS_EXPORT int rs_attention_latent_bf16(const void* q, long q_stride, void* out, 
         return (int)cudaErrorInvalidValue;
     if (v_cols <= 0 || v_cols % 8 || v_cols > lat || (wide && decode)) return (int)cudaErrorInvalidValue;
     if (decode && (split_keys % KT || split_keys <= 0 || max_splits <= 0 || partial == nullptr || partial_slots <= 0 ||
-                   split_start == nullptr))
+                   split_start == nullptr || ((size_t)partial & 7)))
         return (int)cudaErrorInvalidValue;
     LatParams p;
     p.q = (const __nv_bfloat16*)q; p.q_stride = q_stride; p.out = (__nv_bfloat16*)out; p.out_stride = out_stride;
@@ -626,10 +634,7 @@ RS_EXPORT int rs_attention_latent_bf16(const void* q, long q_stride, void* out, 
     // Wider rows read the query fragments from shared memory: kept in registers (20 or 36 steps) they cost a CTA 175 to
     // 231 registers a thread, one CTA fits an SM instead of two, and the kernel got slower (593 against 431 us for 2,048
     // tokens, 8 heads, rows of 320).
-    if (lat <= 128) latent_attention_kernel<8><<<grid, THREADS, smem, s>>>(p);
-    else latent_attention_kernel<0><<<grid, THREADS, smem, s>>>(p);
-    e = cudaGetLastError();
-    if (e != cudaSuccess || !decode) return (int)e;
-    latent_merge_kernel<<<dim3(n_work, n_heads), 128, 0, s>>>(p);
-    return rs_launch_result();
+    const int rc = rs_launch_pdl(lat <= 128 ? latent_attention_kernel<8> : latent_attention_kernel<0>, grid, dim3(THREADS), smem, s, p);
+    if (rc != 0 || !decode) return rc;
+    return rs_launch_pdl(latent_merge_kernel, dim3(n_work, n_heads), dim3(v_cols > 256 ? 256 : 128), 0, s, p);
 }

@@ -74,7 +74,7 @@ struct OutputGate {
     const float* g; long stride; int per_block; float scale;
     __device__ __forceinline__ float factor(long row, int block, int col) const {
         if (g == nullptr) return scale;
-        return scale / (1.0f + expf(-g[row * stride + (per_block ? block : col)]));
+        return scale / (1.0f + expf(-__ldcg(g + row * stride + (per_block ? block : col))));
     }
 };
 
@@ -139,6 +139,12 @@ static inline int rs_launch_result() { return (int)cudaGetLastError(); }
 template <typename T> __device__ __forceinline__ T ld_dep(const T* p) { return __ldcg(p); }
 __device__ __forceinline__ float ld_dep_f32(const __nv_bfloat16* p) {
     return __bfloat162float(__ushort_as_bfloat16(__ldcg(reinterpret_cast<const unsigned short*>(p))));
+}
+
+// an element of either type, or of a type known at run time, read from L2
+__device__ __forceinline__ float ld_dep_f32(const float* p) { return __ldcg(p); }
+__device__ __forceinline__ float ld_dep_any(const void* p, int dt, size_t i) {
+    return dt == RS_F32 ? ld_dep_f32(reinterpret_cast<const float*>(p) + i) : ld_dep_f32(reinterpret_cast<const __nv_bfloat16*>(p) + i);
 }
 
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }

@@ -38,9 +38,12 @@ __global__ void __launch_bounds__(F::WM * F::WN * 32) grouped_gemm_mma_kernel(co
     constexpr int BM = F::BM, BN = F::BN, BK = F::BK, STAGES = F::STAGES, WM = F::WM, WN = F::WN, PITCH = BK + 8;
     constexpr int THREADS = WM * WN * 32, MT = BM / WM / 16, NT = BN / WN / 8, CH = BK / 8;      // CH: 16-byte columns of a step
     int e, row0, rows;
+    pdl_launch_dependents();
+    pdl_wait();
     if (p.tiles != nullptr) {
-        if ((int)blockIdx.y >= p.n_tiles[0]) return;
-        e = p.tiles[3 * blockIdx.y]; row0 = p.tiles[3 * blockIdx.y + 1]; rows = p.tiles[3 * blockIdx.y + 2];
+        if ((int)blockIdx.y >= ld_dep(p.n_tiles)) return;
+        const int* tile = p.tiles + 3 * blockIdx.y;
+        e = ld_dep(tile); row0 = ld_dep(tile + 1); rows = ld_dep(tile + 2);
     } else {
         e = blockIdx.y / p.tiles_per_expert;
         row0 = (blockIdx.y % p.tiles_per_expert) * BM;
@@ -52,7 +55,7 @@ __global__ void __launch_bounds__(F::WM * F::WN * 32) grouped_gemm_mma_kernel(co
     __shared__ int pair_of_row[BM];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int n0 = blockIdx.x * BN;
-    if (tid < BM) pair_of_row[tid] = tid < rows ? (p.order != nullptr ? p.order[row0 + tid] : row0 + tid) : -1;
+    if (tid < BM) pair_of_row[tid] = tid < rows ? (p.order != nullptr ? ld_dep(p.order + row0 + tid) : row0 + tid) : -1;
     __syncthreads();
 
     // a thread fetches the same 16-byte column of the same rows at every step: their addresses are found once
@@ -84,7 +87,7 @@ __global__ void __launch_bounds__(F::WM * F::WN * 32) grouped_gemm_mma_kernel(co
                     cp_async16(smem_addr(dst), reinterpret_cast<const __nv_bfloat16*>(p.a) + a_at[q] + k0);
                 } else {
                     const float* src = reinterpret_cast<const float*>(p.a) + a_at[q] + k0;
-                    const float4 lo = *reinterpret_cast<const float4*>(src), hi = *reinterpret_cast<const float4*>(src + 4);
+                    const float4 lo = ld_dep(reinterpret_cast<const float4*>(src)), hi = ld_dep(reinterpret_cast<const float4*>(src + 4));
                     uint4 u;
                     u.x = pack_bf16(lo.x, lo.y); u.y = pack_bf16(lo.z, lo.w); u.z = pack_bf16(hi.x, hi.y); u.w = pack_bf16(hi.z, hi.w);
                     *reinterpret_cast<uint4*>(dst) = u;
@@ -202,8 +205,7 @@ int launch_grouped(const GroupedMmaParams& p, int row_tiles, cudaStream_t s) {
             allowed[dev].store(true, std::memory_order_release);
         }
     }
-    kern<<<dim3((p.w_rows + F::BN - 1) / F::BN, row_tiles), F::WM * F::WN * 32, smem, s>>>(p);
-    return rs_launch_result();
+    return rs_launch_pdl(kern, dim3((p.w_rows + F::BN - 1) / F::BN, row_tiles), dim3(F::WM * F::WN * 32), smem, s, p);
 }
 }  // namespace
 

@@ -58,10 +58,80 @@ __global__ void rmsnorm_add_kernel(float* __restrict__ x, long x_stride, const f
         store_any(out, out_dt, (size_t)r * out_stride + i, xr[i] * s2 * load_any(w2, w2_dt, w2_n == 1 ? 0 : i));
 }
 
+// The same with the rows in registers (n a multiple of 4 up to 1024 V, 16-byte aligned rows): 256 threads, V pieces of four
+// columns each; the gains are fetched before the kernel before is waited for.
+namespace {
+template <int V>
+__global__ void __launch_bounds__(256) rmsnorm_add_vec_kernel(float* x, long x_stride, const float* delta, long d_stride,
+                                                              const void* __restrict__ g, int g_dt, int g_n, float eps,
+                                                              const void* __restrict__ w2, int w2_dt, int w2_n, float eps2, void* out,
+                                                              int out_dt, long out_stride, int n) {
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    const int n4 = n >> 2;
+    auto gains = [&](const void* w, int dt, int count, int i) {
+        if (count == 1) { const float one = load_any(w, dt, 0); return make_float4(one, one, one, one); }
+        return load_weights4(w, dt, i);
+    };
+    float4 gv[V], wv[V];
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int i = threadIdx.x + u * 256;
+        gv[u] = i < n4 ? gains(g, g_dt, g_n, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        wv[u] = i < n4 && out != nullptr ? gains(w2, w2_dt, w2_n, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    pdl_wait();
+    const int r = blockIdx.x;
+    float4* xr = reinterpret_cast<float4*>(x + (size_t)r * x_stride);
+    const float4* dr = reinterpret_cast<const float4*>(delta + (size_t)r * d_stride);
+    float4 d[V], v[V];
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int i = threadIdx.x + u * 256;
+        d[u] = i < n4 ? ld_dep(dr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[u] = i < n4 ? ld_dep(xr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss = fmaf(d[u].x, d[u].x, ss); ss = fmaf(d[u].y, d[u].y, ss); ss = fmaf(d[u].z, d[u].z, ss); ss = fmaf(d[u].w, d[u].w, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float s = 1.0f / sqrtf(ss / (float)n + eps);
+    float ss2 = 0.f;
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int i = threadIdx.x + u * 256;
+        v[u].x += d[u].x * s * gv[u].x; v[u].y += d[u].y * s * gv[u].y; v[u].z += d[u].z * s * gv[u].z; v[u].w += d[u].w * s * gv[u].w;
+        if (i < n4) xr[i] = v[u];
+        ss2 = fmaf(v[u].x, v[u].x, ss2); ss2 = fmaf(v[u].y, v[u].y, ss2); ss2 = fmaf(v[u].z, v[u].z, ss2); ss2 = fmaf(v[u].w, v[u].w, ss2);
+    }
+    if (out == nullptr) return;
+    ss2 = block_sum(ss2, scratch);
+    const float s2 = 1.0f / sqrtf(ss2 / (float)n + eps2);
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int i = threadIdx.x + u * 256;
+        if (i >= n4) continue;
+        const float4 y = make_float4(v[u].x * s2 * wv[u].x, v[u].y * s2 * wv[u].y, v[u].z * s2 * wv[u].z, v[u].w * s2 * wv[u].w);
+        if (out_dt == RS_F32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + (size_t)r * out_stride + 4 * i) = y;
+        else *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out) + (size_t)r * out_stride + 4 * i) = pack_bf16x4(y.x, y.y, y.z, y.w);
+    }
+}
+}  // namespace
+
 RS_EXPORT int rs_rmsnorm_add(float* x, long x_stride, const float* delta, long d_stride, const void* g, int g_dt, int g_n,
                              float eps, const void* w2, int w2_dt, int w2_n, float eps2, void* out, int out_dt,
                              long out_stride, int n_rows, int n, void* stream) {
     if (n_rows <= 0) return 0;
+    auto ok = [](const void* q, int dt, long stride) { return q == nullptr || ((size_t)q % (dt == RS_F32 ? 16 : 8) == 0 && stride % 4 == 0); };
+    if (n % 4 == 0 && n <= 8192 && ok(x, RS_F32, x_stride) && ok(delta, RS_F32, d_stride) && ok(out, out_dt, out_stride) &&
+        ok(g_n == 1 ? nullptr : g, g_dt, 0) && ok(w2_n == 1 ? nullptr : w2, w2_dt, 0)) {
+        cudaStream_t s = (cudaStream_t)stream;
+#define RS_NORM_ADD(V) rs_launch_pdl(rmsnorm_add_vec_kernel<V>, dim3(n_rows), dim3(256), 0, s, x, x_stride, delta, d_stride, g, g_dt, g_n, eps, w2, w2_dt, w2_n, eps2, out, out_dt, out_stride, n)
+        if (n <= 1024) return RS_NORM_ADD(1);
+        if (n <= 2048) return RS_NORM_ADD(2);
+        if (n <= 4096) return RS_NORM_ADD(4);
+        return RS_NORM_ADD(8);
+#undef RS_NORM_ADD
+    }
     const int threads = n >= 2048 ? 512 : (n >= 512 ? 256 : 128);
     rmsnorm_add_kernel<<<n_rows, threads, 0, (cudaStream_t)stream>>>(x, x_stride, delta, d_stride, g, g_dt, g_n, eps, w2,
                                                                      w2_dt, w2_n, eps2, out, out_dt, out_stride, n);
@@ -266,8 +336,17 @@ RS_EXPORT int rs_short_conv(const void* in, int in_dt, long in_stride, const voi
 // out[t, b * out_bs + o] = (bias[b * O + o] + sum_i W[b, o, i] * in[t, b * in_bs + i]) * f,  o < O, i < I, b < B,
 // f = out_scale * sigmoid(gate) in float32, gate one float32 number per token and block (gate_per_block) or per token and
 // output, or f = out_scale without a gate.  W: [B, O, I] contiguous.  Tiles of 64 x 64 outputs, k ascending per output element.
+// A rotated tail (the form for few rows only): out[t, b * out_bs + O + j] = rotate(in[t, b * in_bs + at + j]) for j < rot, zeros
+// for rot <= j < pad; the rotation as in latent_kv_write below.
 namespace {
 constexpr int BL_BM = 64, BL_BN = 64, BL_BK = 16;
+
+struct RotatedTail {
+    const float* cos_sin; int n_rot, table_rows;
+    const int* positions; int pos_stride;
+    int at, rot, pad;
+    int* status;
+};
 
 struct BlockLinearParams {
     const void* in; int in_dt; long in_stride; long in_bs;
@@ -276,7 +355,14 @@ struct BlockLinearParams {
     void* out; int out_dt; long out_stride; long out_bs;
     int T, O, I;
     OutputGate gate;
+    RotatedTail tail;
 };
+
+__device__ __forceinline__ float turned(float own, float partner, const float* cs, int n_rot, int j) {
+    // coordinate j of a rotated part whose pairs are (2i, 2i + 1); own = v[j], partner = v[j ^ 1], j < n_rot
+    const float c = cs[j >> 1], s = cs[(n_rot >> 1) + (j >> 1)];
+    return (j & 1) ? fmaf(own, c, partner * s) : fmaf(own, c, -partner * s);
+}
 
 __global__ void __launch_bounds__(256) block_linear_kernel(const BlockLinearParams p) {
     __shared__ float As[BL_BK][BL_BM + 1];
@@ -392,15 +478,148 @@ __global__ void __launch_bounds__(256) block_linear_rows_kernel(const BlockLinea
         }
     }
 }
+
+// The same for bfloat16 weights in 16-byte pieces and up to 768 inputs per block: a warp owns two output columns, its weights
+// are on their way before the rows of the kernel before are waited for, and the eight rows' sums of a column are added up over
+// the lanes together (each exchange halves how many of them a lane still carries).
+constexpr int BV_COLS = 16, BV_NI = 3;
+
+template <typename TX>
+__global__ void __launch_bounds__(256) block_linear_rows_vec_kernel(const BlockLinearParams p) {
+    __shared__ __align__(16) TX xs[BR_ROWS][BV_NI * 256];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, b = blockIdx.y;
+    const int o0 = blockIdx.x * BV_COLS + warp * 2;
+    pdl_launch_dependents();
+    uint4 w[2][BV_NI];
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int i = 0; i < BV_NI; ++i) {
+            const int k = (lane + 32 * i) * 8;
+            w[c][i] = k < p.I && o0 + c < p.O
+                ? *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.w) + ((size_t)b * p.O + o0 + c) * p.I + k)
+                : make_uint4(0, 0, 0, 0);
+        }
+    pdl_wait();
+    constexpr int VX = 16 / sizeof(TX);
+    const int per_row = p.I / VX;
+    for (int i = tid; i < p.T * per_row; i += 256) {
+        const int r = i / per_row, k = (i - r * per_row) * VX;
+        *reinterpret_cast<uint4*>(&xs[r][k]) =
+            __ldcg(reinterpret_cast<const uint4*>(reinterpret_cast<const TX*>(p.in) + (size_t)r * p.in_stride + (size_t)b * p.in_bs + k));
+    }
+    __syncthreads();
+    float acc[2][BR_ROWS];
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int r = 0; r < BR_ROWS; ++r) acc[c][r] = 0.f;
+#pragma unroll
+    for (int i = 0; i < BV_NI; ++i) {
+        const int k = (lane + 32 * i) * 8;
+        if (k >= p.I) continue;
+        float wf[2][8];
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+            const __nv_bfloat162* w2 = reinterpret_cast<const __nv_bfloat162*>(&w[c][i]);
+#pragma unroll
+            for (int q = 0; q < 4; ++q) { wf[c][2 * q] = __low2float(w2[q]); wf[c][2 * q + 1] = __high2float(w2[q]); }
+        }
+#pragma unroll
+        for (int r = 0; r < BR_ROWS; ++r) {
+            if (r >= p.T) continue;                               // the same for every lane
+            float x[8];
+#pragma unroll
+            for (int v = 0; v < 8 / VX; ++v) {
+                const uint4 raw = *reinterpret_cast<const uint4*>(&xs[r][k + v * VX]);
+                const TX* e = reinterpret_cast<const TX*>(&raw);
+#pragma unroll
+                for (int q = 0; q < VX; ++q) x[v * VX + q] = to_f32<TX>(e[q]);
+            }
+#pragma unroll
+            for (int q = 0; q < 8; ++q) { acc[0][r] = fmaf(x[q], wf[0][q], acc[0][r]); acc[1][r] = fmaf(x[q], wf[1][q], acc[1][r]); }
+        }
+    }
+    // lane l ends with the sum of row (bit 4, bit 3, bit 2 of l)
+    const int row = ((lane >> 4) & 1) * 4 + ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        float v[BR_ROWS];
+#pragma unroll
+        for (int r = 0; r < BR_ROWS; ++r) v[r] = acc[c][r];
+#pragma unroll
+        for (int n = 4, bit = 16; n > 0; n >>= 1, bit >>= 1) {
+            const bool up = lane & bit;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                if (j < n) {
+                    const float send = up ? v[j] : v[j + n], keep = up ? v[j + n] : v[j];
+                    v[j] = keep + __shfl_xor_sync(0xffffffffu, send, bit);
+                }
+            }
+        }
+        float t = v[0];
+        t += __shfl_xor_sync(0xffffffffu, t, 2);
+        t += __shfl_xor_sync(0xffffffffu, t, 1);
+        const int o = o0 + c;
+        if ((lane & 3) == 0 && row < p.T && o < p.O) {
+            if (p.bias != nullptr) t += load_any(p.bias, p.bias_dt, (size_t)b * p.O + o);
+            t *= p.gate.factor(row, b, b * p.O + o);
+            store_any(p.out, p.out_dt, (size_t)row * p.out_stride + (size_t)b * p.out_bs + o, t);
+        }
+    }
+    if (p.tail.pad > 0 && blockIdx.x == 0) {
+        const TX* in = reinterpret_cast<const TX*>(p.in);
+        for (int i = tid; i < p.T * p.tail.pad; i += 256) {
+            const int r = i / p.tail.pad, j = i - r * p.tail.pad;
+            float v = 0.f;
+            if (j < p.tail.rot) {
+                const TX* part = in + (size_t)r * p.in_stride + (size_t)b * p.in_bs + p.tail.at;
+                v = ld_dep_f32(part + j);
+                if (p.tail.cos_sin != nullptr && j < p.tail.n_rot) {
+                    const int pos = __ldcg(p.tail.positions + (size_t)r * p.tail.pos_stride);
+                    if (pos < 0 || pos >= p.tail.table_rows) {
+                        atomicOr(p.tail.status, RS_STATUS_BAD_PLAN);
+                        continue;
+                    }
+                    v = turned(v, ld_dep_f32(part + (j ^ 1)), p.tail.cos_sin + (size_t)pos * p.tail.n_rot, p.tail.n_rot, j);
+                }
+            }
+            store_any(p.out, p.out_dt, (size_t)r * p.out_stride + (size_t)b * p.out_bs + p.O + j, v);
+        }
+    }
+}
+
+bool rows_vec_ok(const BlockLinearParams& p) {
+    const int vx = p.in_dt == RS_F32 ? 4 : 8;
+    return p.w_dt == RS_BF16 && p.I % 8 == 0 && p.I <= BV_NI * 256 && ((size_t)p.w & 15) == 0 && ((size_t)p.in & 15) == 0 &&
+           p.in_stride % vx == 0 && p.in_bs % vx == 0;
+}
 }  // namespace
+
+// Whether the form for few rows that can rotate a tail takes these operands.
+RS_EXPORT int rs_block_linear_takes_tail(const void* in, int in_dt, long in_stride, long in_bs, const void* w, int w_dt, int T, int I) {
+    BlockLinearParams p{};
+    p.in = in; p.in_dt = in_dt; p.in_stride = in_stride; p.in_bs = in_bs; p.w = w; p.w_dt = w_dt; p.I = I;
+    return T > 0 && T <= BR_ROWS && rows_vec_ok(p);
+}
 
 RS_EXPORT int rs_block_linear(const void* in, int in_dt, long in_stride, long in_bs, const void* w, int w_dt,
                               const void* bias, int bias_dt, void* out, int out_dt, long out_stride, long out_bs, int T,
                               int B, int O, int I, const float* gate, long gate_stride, int gate_per_block, float out_scale,
-                              void* stream) {
+                              const float* tail_cos_sin, int tail_n_rot, int tail_table_rows, const int* tail_positions,
+                              int tail_pos_stride, int tail_at, int tail_rot, int tail_pad, int* status, void* stream) {
     if (T <= 0 || B <= 0 || O <= 0) return 0;
     BlockLinearParams p{in, in_dt, in_stride, in_bs, w, w_dt, bias, bias_dt, out, out_dt, out_stride, out_bs, T, O, I,
-                        OutputGate{gate, gate_stride, gate_per_block, out_scale}};
+                        OutputGate{gate, gate_stride, gate_per_block, out_scale},
+                        RotatedTail{tail_cos_sin, tail_n_rot, tail_table_rows, tail_positions, tail_pos_stride, tail_at, tail_rot,
+                                    tail_pad, status}};
+    if (tail_pad > 0 && (T > BR_ROWS || !rows_vec_ok(p) || tail_n_rot % 2 || tail_n_rot > tail_rot || tail_rot > tail_pad))
+        return (int)cudaErrorInvalidValue;
+    if (T <= BR_ROWS && rows_vec_ok(p)) {
+        const dim3 grid((O + BV_COLS - 1) / BV_COLS, B);
+        RS_DISPATCH_DTYPE(in_dt, TX, return rs_launch_pdl(block_linear_rows_vec_kernel<TX>, grid, dim3(256), 0, (cudaStream_t)stream, p));
+    }
     if (T <= BR_ROWS) {
         block_linear_rows_kernel<<<dim3((O + BR_COLS - 1) / BR_COLS, B), 256, 0, (cudaStream_t)stream>>>(p);
         return rs_launch_result();
@@ -565,6 +784,7 @@ RS_EXPORT int rs_gated_linear_recurrence(const float* gates, long gates_stride, 
 // cos_sin[position][i] and cos_sin[position][n_rot / 2 + i]; coordinates from n_rot on pass unchanged.
 // A query that comes through a latent of its own: c_q[t] = cq[t] * rsqrt(mean(cq^2) + eps) * cq_w besides; the rotation of the
 // queries, which are made from c_q, is then a launch of its own (cache == null).
+namespace {
 struct LatentParams {
     const float* dkv; long dkv_stride;
     const void* norm_w; int norm_dt; float eps;
@@ -579,18 +799,45 @@ struct LatentParams {
     int* status;
 };
 
+// rotated part of a row v (own = v[j], partner = v[j ^ 1]); cs: the position's row of the table, or null
 __device__ __forceinline__ float rotated(const LatentParams& p, const float* cs, float own, float partner, int j) {
-    // j: index within the rotated part; own = v[j], partner = v[j ^ 1]
-    if (cs == nullptr || j >= p.n_rot) return own;
-    const int i = j >> 1, half = p.n_rot >> 1;
-    const float c = cs[i], s = cs[half + i];
-    return (j & 1) ? fmaf(own, c, partner * s) : fmaf(own, c, -partner * s);
+    return cs == nullptr || j >= p.n_rot ? own : turned(own, partner, cs, p.n_rot, j);
 }
 
-__global__ void latent_kv_write_kernel(const LatentParams p) {
+constexpr int LAT_THREADS = 128, LAT_KEPT = 8;
+
+// put(i, x[i] * rsqrt(mean(x^2) + eps)) for i < n: the row stays in registers as far as it fits
+template <typename Put>
+__device__ __forceinline__ void normed_row(const float* x, int n, float eps, float* scratch, Put put) {
+    float v[LAT_KEPT], ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < LAT_KEPT; ++u) {
+        const int i = threadIdx.x + u * LAT_THREADS;
+        v[u] = i < n ? ld_dep(x + i) : 0.f;
+        ss = fmaf(v[u], v[u], ss);
+    }
+    for (int i = threadIdx.x + LAT_KEPT * LAT_THREADS; i < n; i += LAT_THREADS) { const float e = ld_dep(x + i); ss = fmaf(e, e, ss); }
+    ss = block_sum(ss, scratch);
+    const float s = 1.0f / sqrtf(ss / (float)n + eps);
+#pragma unroll
+    for (int u = 0; u < LAT_KEPT; ++u) { const int i = threadIdx.x + u * LAT_THREADS; if (i < n) put(i, v[u] * s); }
+    for (int i = threadIdx.x + LAT_KEPT * LAT_THREADS; i < n; i += LAT_THREADS) put(i, ld_dep(x + i) * s);
+}
+
+// One block per token and job: the cache row, the query latent, or 128 values of the queries' rotated parts.
+__global__ void __launch_bounds__(LAT_THREADS) latent_kv_write_kernel(const LatentParams p) {
     __shared__ float scratch[33];
+    pdl_launch_dependents();
+    pdl_wait();
     const int t = blockIdx.x;
-    const int pos = p.positions[(size_t)t * p.pos_stride];
+    int job = blockIdx.y;
+    if (p.cq_out != nullptr && job-- == 0) {
+        normed_row(p.cq + (size_t)t * p.cq_stride, p.q_rank, p.eps, scratch, [&](int i, float v) {
+            store_any(p.cq_out, p.cq_dt, (size_t)t * p.cq_out_stride + i, v * load_any(p.cq_w, p.cq_w_dt, i));
+        });
+        return;
+    }
+    const int pos = ld_dep(p.positions + (size_t)t * p.pos_stride);
     const float* cs = nullptr;
     if (p.cos_sin != nullptr) {
         if (pos < 0 || pos >= p.table_rows) {
@@ -599,49 +846,37 @@ __global__ void latent_kv_write_kernel(const LatentParams p) {
         }
         cs = p.cos_sin + (size_t)pos * p.n_rot;
     }
-    // queries: the rotated part of every head
-    for (int i = threadIdx.x; i < p.heads * (p.lat - p.rank); i += blockDim.x) {
-        const int h = i / (p.lat - p.rank), j = i % (p.lat - p.rank);
-        float v = 0.f;
-        if (j < p.rot) {
-            const size_t base = (size_t)t * p.q_stride + (size_t)h * p.q_head + p.q_nope;
-            const float own = load_any(p.q, p.q_dt, base + j);
-            const float partner = (j < p.n_rot) ? load_any(p.q, p.q_dt, base + (j ^ 1)) : 0.f;
-            v = rotated(p, cs, own, partner, j);
+    if (p.cache != nullptr && job-- == 0) {
+        const int page = p.block_table[(size_t)ld_dep(p.seq_of_token + t) * p.table_stride + pos / p.page_size];
+        if (page < 0 || page >= p.num_pages) {
+            if (threadIdx.x == 0) atomicOr(p.status, RS_STATUS_BAD_PAGE);
+            return;
         }
-        store_any(p.q_lat, p.q_lat_dt, (size_t)t * p.q_lat_stride + (size_t)h * p.lat + p.rank + j, v);
-    }
-    if (p.cq_out != nullptr) {
-        const float* row = p.cq + (size_t)t * p.cq_stride;
-        float ss = 0.f;
-        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
-        ss = block_sum(ss, scratch);
-        const float s = 1.0f / sqrtf(ss / (float)p.q_rank + p.eps);
-        for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x)
-            store_any(p.cq_out, p.cq_dt, (size_t)t * p.cq_out_stride + i, row[i] * s * load_any(p.cq_w, p.cq_w_dt, i));
-    }
-    if (p.cache == nullptr) return;
-    const int page = p.block_table[(size_t)p.seq_of_token[t] * p.table_stride + pos / p.page_size];
-    if (page < 0 || page >= p.num_pages) {
-        if (threadIdx.x == 0) atomicOr(p.status, RS_STATUS_BAD_PAGE);
+        const float* row = p.dkv + (size_t)t * p.dkv_stride;
+        const size_t dst = (size_t)page * p.page_stride + (size_t)(pos % p.page_size) * p.lat;
+        for (int i = p.rank + threadIdx.x; i < p.lat; i += LAT_THREADS) {
+            const int j = i - p.rank;
+            float v = 0.f;
+            if (j < p.rot) v = rotated(p, cs, ld_dep(row + i), j < p.n_rot ? ld_dep(row + p.rank + (j ^ 1)) : 0.f, j);
+            store_any(p.cache, p.cache_dt, dst + i, v);
+        }
+        normed_row(row, p.rank, p.eps, scratch, [&](int i, float v) {
+            store_any(p.cache, p.cache_dt, dst + i, v * load_any(p.norm_w, p.norm_dt, i));
+        });
         return;
     }
-    const float* row = p.dkv + (size_t)t * p.dkv_stride;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < p.rank; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
-    ss = block_sum(ss, scratch);
-    const float s = 1.0f / sqrtf(ss / (float)p.rank + p.eps);
-    const size_t dst = (size_t)page * p.page_stride + (size_t)(pos % p.page_size) * p.lat;
-    for (int i = threadIdx.x; i < p.lat; i += blockDim.x) {
-        float v = 0.f;
-        if (i < p.rank) v = row[i] * s * load_any(p.norm_w, p.norm_dt, i);
-        else if (i < p.rank + p.rot) {
-            const int j = i - p.rank;
-            v = rotated(p, cs, row[i], (j < p.n_rot) ? row[p.rank + (j ^ 1)] : 0.f, j);
-        }
-        store_any(p.cache, p.cache_dt, dst + i, v);
+    const int tail = p.lat - p.rank, i = job * LAT_THREADS + threadIdx.x;
+    if (i >= p.heads * tail) return;
+    const int h = i / tail, j = i - h * tail;
+    float v = 0.f;
+    if (j < p.rot) {
+        const size_t base = (size_t)t * p.q_stride + (size_t)h * p.q_head + p.q_nope;
+        v = rotated(p, cs, ld_dep_any(p.q, p.q_dt, base + j), j < p.n_rot ? ld_dep_any(p.q, p.q_dt, base + (j ^ 1)) : 0.f, j);
     }
+    store_any(p.q_lat, p.q_lat_dt, (size_t)t * p.q_lat_stride + (size_t)h * p.lat + p.rank + j, v);
 }
+
+}  // namespace
 
 RS_EXPORT int rs_latent_kv_write(const float* dkv, long dkv_stride, const void* norm_w, int norm_dt, float eps, const void* q,
                                  int q_dt, long q_stride, int q_head, int q_nope, void* q_lat, int q_lat_dt,
@@ -657,8 +892,9 @@ RS_EXPORT int rs_latent_kv_write(const float* dkv, long dkv_stride, const void* 
                    cos_sin, n_rot, table_rows, positions, pos_stride, seq_of_token, block_table, table_stride, page_size,
                    cache, cache_dt, page_stride, num_pages, rank, rot, lat, heads, n_tokens, cq, cq_stride, cq_w, cq_w_dt, cq_out,
                    cq_dt, cq_out_stride, q_rank, status};
-    latent_kv_write_kernel<<<n_tokens, 128, 0, (cudaStream_t)stream>>>(p);
-    return rs_launch_result();
+    const int jobs = (cache != nullptr) + (cq_out != nullptr) + (heads * (lat - rank) + LAT_THREADS - 1) / LAT_THREADS;
+    if (jobs == 0) return 0;
+    return rs_launch_pdl(latent_kv_write_kernel, dim3(n_tokens, jobs), dim3(LAT_THREADS), 0, (cudaStream_t)stream, p);
 }
 
 // --------------------------------------------------------------------------- activations

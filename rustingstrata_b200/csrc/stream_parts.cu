@@ -165,90 +165,6 @@ __global__ void stream_update_kernel(const StreamUpdateParams p) {
                   (size_t)r * p.next.out_stride, scratch);
 }
 
-// one warp per token: scores = softmax(logits), or sigmoid(logits) each for itself (``sigmoid``); the `top` largest of
-// scores + correction are chosen (the lower index on a tie); with ``n_groups`` > 0 the experts form that many equal
-// groups of neighbours, a group is worth the sum of its two largest scores + correction (``worth_one``: its largest), and only experts of the
-// ``keep`` groups worth most can be chosen (the lower index on a tie); weights = the chosen experts' scores times
-// ``scale``, divided by (their sum + 1e-20) first when ``renorm`` is set
-__global__ void router_topk_kernel(const float* __restrict__ logits, long l_stride, const void* __restrict__ corr,
-                                   int corr_dt, int E, int top, int n_tokens, int sigmoid, int n_groups, int keep, int worth_one, float scale,
-                                   int renorm, int* __restrict__ choice, float* __restrict__ weight, int* status) {
-    extern __shared__ float sm[];
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, wpb = blockDim.x >> 5;
-    const int t = blockIdx.x * wpb + warp;
-    if (t >= n_tokens) return;
-    float* score = sm + (size_t)warp * (2 * E + 2 * n_groups);
-    float* pick = score + E;
-    float* worth = pick + E;                 // [n_groups]
-    float* kept = worth + n_groups;          // [n_groups] 1: the group's experts can be chosen
-    const float* z = logits + (size_t)t * l_stride;
-    if (sigmoid) {
-        bool bad = false;
-        for (int e = lane; e < E; e += 32) {
-            const float v = z[e];
-            bad |= !isfinite(v);
-            score[e] = 1.0f / (1.0f + expf(-v));
-        }
-        if (__any_sync(0xffffffffu, bad) && lane == 0) atomicOr(status, RS_STATUS_NON_FINITE);
-    } else {
-        float m = -INFINITY;
-        for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
-        m = warp_max(m);
-        float sum = 0.f;
-        for (int e = lane; e < E; e += 32) { const float v = expf(z[e] - m); score[e] = v; sum += v; }
-        sum = warp_sum(sum);
-        if (!(sum > 0.f) || !isfinite(sum)) { if (lane == 0) atomicOr(status, RS_STATUS_NON_FINITE); }
-        for (int e = lane; e < E; e += 32) score[e] = score[e] / sum;
-    }
-    for (int e = lane; e < E; e += 32) pick[e] = corr != nullptr ? score[e] + load_any(corr, corr_dt, e) : score[e];
-    __syncwarp();
-    if (n_groups > 0) {
-        const int per = E / n_groups;
-        for (int g = lane; g < n_groups; g += 32) {
-            float a = -INFINITY, b = -INFINITY;              // the group's largest and second largest
-            for (int e = g * per; e < (g + 1) * per; ++e) {
-                const float v = pick[e];
-                if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
-            }
-            worth[g] = per > 1 && !worth_one ? a + b : a;
-            kept[g] = 0.f;
-        }
-        __syncwarp();
-        for (int k = 0; k < keep; ++k) {
-            float best = -INFINITY; int bi = 0x7FFFFFFF;
-            for (int g = lane; g < n_groups; g += 32) { const float v = worth[g]; if (kept[g] == 0.f && (v > best || bi == 0x7FFFFFFF)) { best = v; bi = g; } }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-                if (oi != 0x7FFFFFFF && (bi == 0x7FFFFFFF || ov > best || (ov == best && oi < bi))) { best = ov; bi = oi; }
-            }
-            if (bi >= 0 && bi < n_groups && lane == 0) kept[bi] = 1.f;
-            __syncwarp();
-        }
-        for (int e = lane; e < E; e += 32) if (kept[e / per] == 0.f) pick[e] = -INFINITY;
-        __syncwarp();
-    }
-    float total = 0.f;
-    for (int k = 0; k < top; ++k) {
-        float best = -INFINITY; int bi = 0x7FFFFFFF;
-        for (int e = lane; e < E; e += 32) { const float v = pick[e]; if (v > best) { best = v; bi = e; } }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
-        }
-        if (bi < 0 || bi >= E) bi = 0;                           // nothing finite left: every lane agrees
-        const float s = score[bi];
-        total += s;
-        if (lane == 0) { choice[(size_t)t * top + k] = bi; weight[(size_t)t * top + k] = s; pick[bi] = -INFINITY; }
-        __syncwarp();
-    }
-    const float f = renorm ? scale / (total + 1e-20f) : scale;
-    __syncwarp();
-    for (int k = lane; k < top; k += 32) weight[(size_t)t * top + k] *= f;
-}
 }  // namespace
 
 RS_EXPORT int rs_embed_sum(const void* tok, int tok_dt, int V, const void* bigram, int bigram_dt, int buckets, long mul_prev,
@@ -300,19 +216,5 @@ RS_EXPORT int rs_stream_update(float* x, long x_stride, const float* y, long y_s
     else if (S <= 4) stream_update_kernel<4><<<n_rows, threads, smem, st>>>(p);
     else if (S <= 8) stream_update_kernel<8><<<n_rows, threads, smem, st>>>(p);
     else stream_update_kernel<16><<<n_rows, threads, smem, st>>>(p);
-    return rs_launch_result();
-}
-
-RS_EXPORT int rs_router_topk(const float* logits, long l_stride, const void* corr, int corr_dt, int E, int top, int n_tokens,
-                             int sigmoid, int n_groups, int keep, int worth_one, float scale, int renorm, int* choice, float* weight, int* status,
-                             void* stream) {
-    if (n_tokens <= 0) return 0;
-    if (E <= 0 || top <= 0 || top > E || E > 1024) return (int)cudaErrorInvalidValue;
-    if (n_groups < 0 || (n_groups > 0 && (E % n_groups || keep < 1 || keep > n_groups || top > keep * (E / n_groups))))
-        return (int)cudaErrorInvalidValue;
-    const int wpb = 4;
-    router_topk_kernel<<<(n_tokens + wpb - 1) / wpb, wpb * 32, (size_t)wpb * (2 * E + 2 * n_groups) * sizeof(float),
-                         (cudaStream_t)stream>>>(
-        logits, l_stride, corr, corr_dt, E, top, n_tokens, sigmoid, n_groups, keep, worth_one, scale, renorm, choice, weight, status);
     return rs_launch_result();
 }

@@ -116,7 +116,9 @@ def core():
                                       c_int, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                       c_int, c_int, c_void_p]
         lib.rs_block_linear.argtypes = [c_void_p, c_int, c_long, c_long, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int,
-                                        c_long, c_long, c_int, c_int, c_int, c_int, c_void_p, c_long, c_int, c_float, c_void_p]
+                                        c_long, c_long, c_int, c_int, c_int, c_int, c_void_p, c_long, c_int, c_float, c_void_p, c_int, c_int, c_void_p,
+                                        c_int, c_int, c_int, c_int, c_void_p, c_void_p]
+        lib.rs_block_linear_takes_tail.argtypes = [c_void_p, c_int, c_long, c_long, c_void_p, c_int, c_int, c_int]
         lib.rs_gated_linear_recurrence.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_void_p, c_int,
                                                    c_void_p, c_int, c_void_p, c_int, c_long, c_void_p, c_long, c_void_p,
                                                    c_void_p, c_int, c_int, c_float, c_int, c_void_p]
@@ -136,6 +138,12 @@ def core():
         lib.rs_moe_combine.argtypes = [c_void_p, c_long, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int, c_long, c_void_p,
                                        c_int, c_long, c_void_p, c_int, c_void_p, c_long, c_void_p, c_long, c_float, c_int,
                                        c_void_p, c_int, c_long, c_int, c_int, c_void_p]
+        lib.rs_router_topk.argtypes = [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
+                                       c_void_p, c_void_p, c_void_p, c_void_p]
+        lib.rs_router_route_supported.argtypes = [c_int, c_int, c_int, c_int]
+        lib.rs_router_route.argtypes = [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                        c_float, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                        c_void_p]
         lib.rs_embed_rmsnorm.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_long, c_int, c_int, c_int,
                                          c_void_p, c_void_p]
         lib.rs_gelu_table_gate.argtypes = [c_void_p, c_long, c_void_p, c_int, c_long, c_int, c_int, c_void_p, c_void_p, c_int,
@@ -1214,12 +1222,15 @@ BLOCK_LINEAR_ROWS_FORM = 8     # up to this many rows the CUDA-core kernel's row
 
 def block_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_rows: int, in_block_stride: int,
                  out_block_stride: int, bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                 out_scale: float = 1.0) -> None:
+                 out_scale: float = 1.0, tail=None) -> None:
     """out[t, b * out_block_stride + o] = bias[b, o] + sum_i weight[b, o, i] * x[t, b * in_block_stride + i]: one small
     matrix per block of channels (a block-diagonal product), float32 accumulation.  weight [B, O, I] contiguous.
 
     ``gate`` float32 [T, B] or [T, B * O] (rows may be strided) and ``out_scale``: the result is multiplied, still in
-    float32, by out_scale * sigmoid(gate) of its block or of its own column."""
+    float32, by out_scale * sigmoid(gate) of its block or of its own column.
+
+    ``tail`` (cos_sin or None, n_rot, positions, at, rot, pad, status), for shapes ``rs_block_linear_takes_tail`` takes: behind a
+    block's outputs follow pad more values, rotate(x[t, b * in_block_stride + at : ... + rot]) and zeros."""
     _cuda(x, weight, out, bias, gate)
     _rows_contiguous(x, "block_linear x")
     _rows_contiguous(out, "block_linear out")
@@ -1236,6 +1247,16 @@ def block_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_row
                              or gate.stride(1) != 1):
         raise KernelError("block_linear: the gate holds float32 rows of one value per block or per output")
     gate_args = (_ptr(gate), 0 if gate is None else gate.stride(0), 1 if gate is not None and gate.shape[1] == B else 0, float(out_scale))
+    tail_args = (None, 0, 0, None, 0, 0, 0, 0, None)
+    if tail is not None:
+        cos_sin, n_rot, positions, at, rot, pad, status = tail
+        _cuda(cos_sin, positions, status)
+        if positions.dtype != torch.int32 or at + rot > in_block_stride or (B - 1) * in_block_stride + at + rot > x.shape[1] \
+                or (B - 1) * out_block_stride + O + pad > out.shape[1] or rot > pad or positions.shape[0] < n_rows \
+                or (cos_sin is not None and (cos_sin.dtype != torch.float32 or cos_sin.shape[1] != n_rot or not cos_sin.is_contiguous())):
+            raise KernelError("block_linear: the tail's part does not lie within the blocks, or its table or positions do not fit")
+        tail_args = (_ptr(cos_sin), n_rot if cos_sin is not None else 0, 0 if cos_sin is None else cos_sin.shape[0], _ptr(positions),
+                     1 if positions.dim() == 1 else positions.shape[1], at, rot, pad, _ptr(status))
     per16 = 4 if x.dtype == torch.float32 else 8
     if (n_rows > BLOCK_LINEAR_ROWS_FORM and weight.dtype == torch.bfloat16 and x.dtype in (torch.bfloat16, torch.float32)
             and out.dtype in (torch.bfloat16, torch.float32) and I % 8 == 0 and in_block_stride % per16 == 0
@@ -1248,7 +1269,23 @@ def block_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, n_row
         return
     _check(core().rs_block_linear(_ptr(x), dtype_code(x), x.stride(0), in_block_stride, _ptr(weight), dtype_code(weight),
                                   _ptr(bias), _any_code(bias), _ptr(out), dtype_code(out), out.stride(0), out_block_stride,
-                                  n_rows, B, O, I, *gate_args, _stream()), "block_linear")
+                                  n_rows, B, O, I, *gate_args, *tail_args, _stream()), "block_linear")
+
+
+def latent_queries(q: torch.Tensor, weight: torch.Tensor, q_lat: torch.Tensor, n_rows: int, q_head: int, lat: int, cos_sin, n_rot: int,
+                   rot: int, positions: torch.Tensor, seq_of_token: torch.Tensor, block_table: torch.Tensor, page_size: int,
+                   status: torch.Tensor) -> None:
+    """Queries against a latent: q_lat[t, h * lat : ...] = [weight[h] @ q[t, h, : dim] | rotate(q[t, h, dim : dim + rot]) | 0...],
+    weight [heads, rank, dim].  One launch for few rows, a product and a launch for the rotated parts otherwise."""
+    H, rank, dim = weight.shape
+    if lat > rank and core().rs_block_linear_takes_tail(_ptr(q), dtype_code(q), q.stride(0), q_head, _ptr(weight), dtype_code(weight),
+                                                        n_rows, dim):
+        block_linear(q, weight, q_lat, n_rows, q_head, lat, tail=(cos_sin, n_rot, positions, dim, rot, lat - rank, status))
+        return
+    block_linear(q, weight, q_lat, n_rows, q_head, lat)
+    if lat > rank:
+        latent_kv_write(None, None, 0.0, q, q_head, dim, q_lat, cos_sin, n_rot, positions, seq_of_token, block_table, page_size, None,
+                        rank, rot, lat, H, n_rows, status)
 
 
 def gated_linear_recurrence(gates: torch.Tensor, u: torch.Tensor, y: torch.Tensor, y_bias: Optional[torch.Tensor],
@@ -1370,6 +1407,16 @@ def grouped_rows_per_tile(small: bool) -> int:
     return GROUPED_ROWS_SMALL if small else GROUPED_ROWS_TILED
 
 
+def _check_route(who: str, pairs: int, rows_per_tile: int, order, tiles, n_tiles) -> None:
+    for name, t in (("order", order), ("tiles", tiles), ("n_tiles", n_tiles)):
+        if t.dtype != torch.int32 or not t.is_contiguous():
+            raise KernelError(f"{who}: {name} must be contiguous int32")
+    if order.numel() < pairs:
+        raise KernelError(f"{who}: order must hold tokens * top entries")
+    if rows_per_tile not in (grouped_rows_per_tile(True), grouped_rows_per_tile(False)) + GROUPED_MMA_ROWS:
+        raise KernelError(f"{who}: rows_per_tile must be a tile size of the grouped product")
+
+
 def moe_route(ids: Optional[torch.Tensor], table: torch.Tensor, n_experts: int, n_tokens: int, rows_per_tile: int,
               order: torch.Tensor, tiles: torch.Tensor, n_tiles: torch.Tensor, status: torch.Tensor, identity: int = 0) -> None:
     """Sorts the step's (token, k) pairs by the expert that ``table[ids[t], k]`` names: ``order`` [T * top] pair ids
@@ -1378,15 +1425,64 @@ def moe_route(ids: Optional[torch.Tensor], table: torch.Tensor, n_experts: int, 
     choice is one of the ``identity`` numbers behind the last expert (experts without matrices) are left out of the lists."""
     _cuda(ids, table, order, tiles, n_tiles, status)
     V, top = table.shape
-    for name, t in (("ids", ids), ("table", table), ("order", order), ("tiles", tiles), ("n_tiles", n_tiles)):
+    for name, t in (("ids", ids), ("table", table)):
         if t is not None and (t.dtype != torch.int32 or not t.is_contiguous()):
             raise KernelError(f"moe_route: {name} must be contiguous int32")
-    if order.numel() < n_tokens * top or (ids.numel() if ids is not None else V) < n_tokens:
-        raise KernelError("moe_route: order must hold tokens * top entries")
-    if rows_per_tile not in (grouped_rows_per_tile(True), grouped_rows_per_tile(False)) + GROUPED_MMA_ROWS:
-        raise KernelError("moe_route: rows_per_tile must be a tile size of the grouped product")
+    if (ids.numel() if ids is not None else V) < n_tokens:
+        raise KernelError("moe_route: one id, or one row of the table, per token")
+    _check_route("moe_route", n_tokens * top, rows_per_tile, order, tiles, n_tiles)
     _check(core().rs_moe_route(_ptr(ids), _ptr(table), V, top, n_experts, int(identity), n_tokens, rows_per_tile, _ptr(order), _ptr(tiles),
                                _ptr(n_tiles), tiles.numel() // 3, _ptr(status), _stream()), "moe_route")
+
+
+def _check_router(who: str, logits, correction, top, n_tokens, choice, weights, groups, keep, group_worth) -> None:
+    E = logits.shape[1]
+    _rows_contiguous(logits, f"{who} logits")
+    if logits.dtype != torch.float32 or choice.dtype != torch.int32 or weights.dtype != torch.float32 \
+            or not choice.is_contiguous() or not weights.is_contiguous() or min(choice.numel(), weights.numel()) < n_tokens * top:
+        raise KernelError(f"{who}: logits float32 [T, E], choice int32 and weights float32 [T * top] contiguous")
+    if not 1 <= top <= E <= 1024 or (correction is not None and correction.numel() != E):
+        raise KernelError(f"{who}: top {top} of {E} experts (up to 1024), one correction per expert")
+    if group_worth not in ("top2", "max"):
+        raise KernelError(f"{who}: unknown group worth '{group_worth}'")
+    if groups and (E % groups or not 1 <= keep <= groups or top > keep * (E // groups)):
+        raise KernelError(f"{who}: {groups} groups of {E} experts, {keep} kept, top {top}")
+
+
+def router_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, n_tokens: int, choice: torch.Tensor,
+                weights: torch.Tensor, status: torch.Tensor, sigmoid: bool = False, groups: int = 0, keep: int = 0,
+                scale: float = 1.0, renormalize: bool = True, group_worth: str = "top2") -> None:
+    """scores = softmax(logits[t]) (float32 [T, E]; ``sigmoid``: the sigmoid of every logit); choice[t] = the ``top``
+    experts with the largest score + correction (int32 [T, top], the lower index on a tie); with ``groups`` > 0 only
+    experts of the ``keep`` best of that many equal groups of neighbours (a group is worth its two largest scores +
+    correction added, or with ``group_worth`` "max" its largest); weights[t] = their scores times ``scale``, over (the sum of their scores + 1e-20) first if
+    ``renormalize``."""
+    _cuda(logits, correction, choice, weights, status)
+    _check_router("router_topk", logits, correction, top, n_tokens, choice, weights, groups, keep, group_worth)
+    _check(core().rs_router_topk(_ptr(logits), logits.stride(0), _ptr(correction), _any_code(correction), logits.shape[1], top,
+                                 n_tokens, 1 if sigmoid else 0, int(groups), int(keep), 1 if group_worth == "max" else 0, float(scale),
+                                 1 if renormalize else 0, _ptr(choice), _ptr(weights), _ptr(status), _stream()), "router_topk")
+
+
+def router_route(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, n_tokens: int, choice: torch.Tensor,
+                 weights: torch.Tensor, n_experts: int, rows_per_tile: int, order: torch.Tensor, tiles: torch.Tensor,
+                 n_tiles: torch.Tensor, status: torch.Tensor, identity: int = 0, sigmoid: bool = False, groups: int = 0, keep: int = 0,
+                 scale: float = 1.0, renormalize: bool = True, group_worth: str = "top2") -> None:
+    """:func:`router_topk` and :func:`moe_route` on what it chose; one launch where the step is small, else the two."""
+    if logits.shape[1] != n_experts + identity:
+        raise KernelError(f"router_route: {logits.shape[1]} logits for {n_experts} experts and {identity} identity experts")
+    if not core().rs_router_route_supported(n_tokens, n_experts + identity, int(groups), n_experts):
+        router_topk(logits, correction, top, n_tokens, choice, weights, status, sigmoid, groups, keep, scale, renormalize, group_worth)
+        moe_route(None, choice[: n_tokens * top].view(n_tokens, top), n_experts, n_tokens, rows_per_tile, order, tiles, n_tiles, status,
+                  identity)
+        return
+    _cuda(logits, correction, choice, weights, order, tiles, n_tiles, status)
+    _check_router("router_route", logits, correction, top, n_tokens, choice, weights, groups, keep, group_worth)
+    _check_route("router_route", n_tokens * top, rows_per_tile, order, tiles, n_tiles)
+    _check(core().rs_router_route(_ptr(logits), logits.stride(0), _ptr(correction), _any_code(correction), n_experts, int(identity), top,
+                                  n_tokens, 1 if sigmoid else 0, int(groups), int(keep), 1 if group_worth == "max" else 0, float(scale),
+                                  1 if renormalize else 0, _ptr(choice), _ptr(weights), rows_per_tile, _ptr(order), _ptr(tiles),
+                                  _ptr(n_tiles), tiles.numel() // 3, _ptr(status), _stream()), "router_route")
 
 
 def grouped_linear(a: torch.Tensor, a_div: int, weight: torch.Tensor, out: torch.Tensor, order: torch.Tensor,
@@ -1519,8 +1615,6 @@ def streamlib():
         lib.rs_stream_update.argtypes = [c_void_p, c_long, c_void_p, c_long, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int,
                                          c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_long, c_int, c_int, c_int,
                                          c_void_p]
-        lib.rs_router_topk.argtypes = [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
-                                       c_void_p, c_void_p, c_void_p, c_void_p]
         lib.rs_conv_norm_kv_write.argtypes = [c_void_p, c_int, c_long, c_void_p, c_int, c_void_p, c_long, c_int, c_int, c_int,
                                               c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_long, c_void_p, c_long,
                                               c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
@@ -1620,32 +1714,6 @@ def stream_update(x: torch.Tensor, n_streams: int, y: torch.Tensor, mix: torch.T
         _ptr(next_coef), _any_code(next_coef), _ptr(next_weight), _any_code(next_weight), _ptr(next_bias),
         _any_code(next_bias), float(next_eps), _ptr(next_out), _any_code(next_out),
         0 if next_out is None else next_out.stride(0), n_streams, D, n_rows, _stream()), "stream_update")
-
-
-def router_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, n_tokens: int, choice: torch.Tensor,
-                weights: torch.Tensor, status: torch.Tensor, sigmoid: bool = False, groups: int = 0, keep: int = 0,
-                scale: float = 1.0, renormalize: bool = True, group_worth: str = "top2") -> None:
-    """scores = softmax(logits[t]) (float32 [T, E]; ``sigmoid``: the sigmoid of every logit); choice[t] = the ``top``
-    experts with the largest score + correction (int32 [T, top], the lower index on a tie); with ``groups`` > 0 only
-    experts of the ``keep`` best of that many equal groups of neighbours (a group is worth its two largest scores +
-    correction added, or with ``group_worth`` "max" its largest); weights[t] = their scores times ``scale``, over (the sum of their scores + 1e-20) first if
-    ``renormalize``."""
-    _cuda(logits, correction, choice, weights, status)
-    _rows_contiguous(logits, "router_topk logits")
-    E = logits.shape[1]
-    if logits.dtype != torch.float32 or choice.dtype != torch.int32 or weights.dtype != torch.float32 \
-            or not choice.is_contiguous() or not weights.is_contiguous() or min(choice.numel(), weights.numel()) < n_tokens * top:
-        raise KernelError("router_topk: logits float32 [T, E], choice int32 and weights float32 [T * top] contiguous")
-    if not 1 <= top <= E <= 1024 or (correction is not None and correction.numel() != E):
-        raise KernelError(f"router_topk: top {top} of {E} experts (up to 1024), one correction per expert")
-    if group_worth not in ("top2", "max"):
-        raise KernelError(f"router_topk: unknown group worth '{group_worth}'")
-    if groups and (E % groups or not 1 <= keep <= groups or top > keep * (E // groups)):
-        raise KernelError(f"router_topk: {groups} groups of {E} experts, {keep} kept, top {top}")
-    _check(streamlib().rs_router_topk(_ptr(logits), logits.stride(0), _ptr(correction), _any_code(correction), E, top,
-                                      n_tokens, 1 if sigmoid else 0, int(groups), int(keep), 1 if group_worth == "max" else 0, float(scale),
-                                      1 if renormalize else 0, _ptr(choice), _ptr(weights), _ptr(status), _stream()),
-           "router_topk")
 
 
 def conv_norm_kv_write(proj: torch.Tensor, conv_weight: Optional[torch.Tensor], tails: Optional[torch.Tensor], n_q: int,

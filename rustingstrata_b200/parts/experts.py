@@ -308,10 +308,9 @@ class RoutedMoE(FeedForward):
         choice = rt.get_scratch("router_choice", torch.int32).view(-1)[:pairs]
         weights = rt.get_scratch("router_weights", torch.float32).view(-1)[:pairs]
         ops.linear(h, self.w_router, logits, T, status=ctx.status)
-        ops.router_topk(logits[:, : self.n_choices], self.correction, top, T, choice, weights, ctx.status,
-                        sigmoid=self.score == "sigmoid", groups=self.groups, keep=self.keep, scale=self.route_scale,
-                        renormalize=self.renormalize, group_worth=self.group_worth)
-        ops.moe_route(None, choice.view(T, top), self.n_experts, T, rows, order, tiles, n_tiles, ctx.status, identity=self.identity)
+        ops.router_route(logits[:, : self.n_choices], self.correction, top, T, choice, weights, self.n_experts, rows, order, tiles,
+                         n_tiles, ctx.status, identity=self.identity, sigmoid=self.score == "sigmoid", groups=self.groups,
+                         keep=self.keep, scale=self.route_scale, renormalize=self.renormalize, group_worth=self.group_worth)
         if tensor_cores:
             ops.grouped_gemm_mma(h, top, self.w_up, act, order, tiles, n_tiles, max_tiles, gated=self.gated, form=form,
                                  relu2=not self.gated)

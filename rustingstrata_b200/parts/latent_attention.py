@@ -210,9 +210,8 @@ class LatentAttention(PagedAttention):
             ops.latent_kv_write(*row, None, 0, 0, None, *where, call.cache, *sizes, cq=dkv[:, self.cq_at: self.gate_at],
                                 cq_weight=self.q_latent_norm, cq_out=cq)
             ops.linear(cq, self.w_q, q, T, status=ctx.status)
-            ops.block_linear(q, self.w_uk_t, q_lat, T, self.q_head, self.lat)
-            if self.lat > self.rank:
-                ops.latent_kv_write(None, None, 0.0, *query, *where, None, *sizes)
+            rot, n_rot, *place = where
+            ops.latent_queries(q, self.w_uk_t, q_lat, T, self.q_head, self.lat, rot, n_rot, self.rot_dim, *place, ctx.status)
         out = self._attend(q_lat, ctx, call)
         ops.block_linear(out, self.w_uv, o, T, self.lat, self.vdim, gate=dkv[:, self.gate_at:] if self.gate else None,
                          out_scale=self.out_scale)

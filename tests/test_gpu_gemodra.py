@@ -350,6 +350,33 @@ def test_router_choice_with_groups_worth_their_best_score():
         assert torch.allclose(weights.view(T, top).cpu().double(), s.gather(1, got) * scale, rtol=1e-5, atol=1e-6)
 
 
+@pytest.mark.parametrize("T", [1, 5, 32])
+def test_choice_and_lists_in_one_launch(T):
+    """The joint launch for small steps gives the two launches' choices, weights and tiles, and deals every pair once."""
+    from rustingstrata_b200.kernels import ops
+    g = torch.Generator().manual_seed(T)
+    for E, identity, top, groups, keep in [(12, 4, 3, 4, 2), (40, 0, 5, 0, 0), (3, 9, 2, 2, 1)]:
+        n = E + identity
+        logits, corr = torch.randn(T, n + 1, generator=g).cuda()[:, :n], torch.randn(n, generator=g).cuda()
+        outs = []
+        for joint in (True, False):
+            i32 = lambda k: torch.full((k,), -1, dtype=torch.int32, device="cuda")                  # noqa: E731
+            choice, weights, order, tiles, n_tiles, status = i32(T * top), torch.zeros(T * top, device="cuda"), i32(T * top), i32(3 * (T * top + E)), i32(1), _status()
+            kw = dict(groups=groups, keep=keep, scale=1.5, renormalize=False, group_worth="max")
+            if joint:
+                assert ops.core().rs_router_route_supported(T, n, groups, E)
+                ops.router_route(logits, corr, top, T, choice, weights, E, 16, order, tiles, n_tiles, status, identity=identity, **kw)
+            else:
+                ops.router_topk(logits, corr, top, T, choice, weights, status, **kw)
+                ops.moe_route(None, choice.view(T, top), E, T, 16, order, tiles, n_tiles, status, identity=identity)
+            assert int(status.item()) == 0
+            nt = int(n_tiles.item())
+            outs.append((choice.tolist(), weights.tolist(), tiles[: 3 * nt].tolist()))
+            rows = sum(outs[-1][2][2::3])
+            assert sorted(order[:rows].tolist()) == [i for i, c in enumerate(outs[-1][0]) if c < E]
+        assert outs[0] == outs[1]
+
+
 def test_identity_choices_get_no_rows_in_the_lists():
     from rustingstrata_b200.kernels import ops
     T, top, E, identity, rows = 300, 3, 5, 4, 64
@@ -482,6 +509,51 @@ def test_attention_over_latents_with_a_sink(dtype, H, lat, v, window):
         for h in range(H):
             assert rel_err(got[:, h, :v], want[:, h, :v]) <= (2e-5 if dtype == torch.float32 else 1.2e-2), (form, h, float(sink[h]))
         assert dtype == torch.float32 or not got[:, :, v:].any()
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("rows", [1, 6, 8, 30])
+def test_queries_against_a_latent(rows, dtype):
+    """The key map folded into the queries with the rotated parts behind it: one launch for few rows, two for many."""
+    from rustingstrata_b200.kernels import ops
+    g = torch.Generator().manual_seed(rows)
+    for H, dim, rot, rank in [(3, 16, 8, 24), (5, 40, 32, 64), (2, 24, 0, 21), (4, 12, 6, 20), (2, 576, 16, 32), (2, 800, 16, 32)]:
+        lat = (rank + rot + 15) // 16 * 16
+        q = torch.randn(rows, H * (dim + rot), generator=g).to(dtype)
+        w = (torch.randn(H, rank, dim, generator=g) / dim ** 0.5).to(torch.bfloat16 if dtype == torch.bfloat16 else dtype)
+        pos = torch.randint(0, 50, (rows,), generator=g).to(torch.int32)
+        ang = pos.double()[:, None] * 100.0 ** (-2.0 * torch.arange(max(rot, 2) // 2, dtype=torch.float64) / max(rot, 2))
+        table = torch.arange(50, dtype=torch.float64)[:, None] * 100.0 ** (-2.0 * torch.arange(max(rot, 2) // 2, dtype=torch.float64) / max(rot, 2))
+        cos_sin = torch.cat([table.cos(), table.sin()], 1).float().cuda() if rot else None
+        out, status = torch.full((rows, H * lat), 7.0, dtype=dtype, device="cuda"), _status()
+        zero = torch.zeros(rows, dtype=torch.int32, device="cuda")
+        ops.latent_queries(q.cuda(), w.cuda(), out, rows, dim + rot, lat, cos_sin, rot, rot, pos.cuda()[:, None], zero, zero[:1, None], 16, status)
+        assert int(status.item()) == 0
+        x = q.double().view(rows, H, dim + rot)
+        want = torch.zeros(rows, H, lat, dtype=torch.float64)
+        want[..., :rank] = torch.einsum("thd,hrd->thr", x[..., :dim], w.double())
+        if rot:
+            c, s = ang.cos()[:, None], ang.sin()[:, None]
+            u, v = x[..., dim::2], x[..., dim + 1::2]
+            want[..., rank: rank + rot: 2], want[..., rank + 1: rank + rot: 2] = u * c - v * s, v * c + u * s
+        assert rel_err(out.float().cpu(), want.view(rows, -1)) <= (1e-5 if dtype == torch.float32 else 6e-3), (H, dim, rot, rank)
+
+
+@pytest.mark.parametrize("n", [256, 1028, 4096, 8192, 75])
+def test_norm_of_a_sublayer_into_the_stream(n):
+    """x += norm(delta) and the next reader's norm, in the form that keeps rows in registers and the one for other widths."""
+    from rustingstrata_b200.kernels import ops
+    g = torch.Generator().manual_seed(n)
+    x, d = torch.randn(5, n, generator=g), torch.randn(5, n, generator=g)
+    gain, w2 = torch.randn(n, generator=g), torch.randn(n, generator=g).to(torch.bfloat16)
+    want = x.double() + P.rms_norm(d.double(), gain.double(), 1e-5)
+    for dtype, tol in ((torch.float32, 2e-6), (torch.bfloat16, 5e-3)):
+        xs, out = x.cuda(), torch.zeros(5, n, dtype=dtype, device="cuda")
+        ops.rmsnorm_add(xs, d.cuda(), gain.cuda(), 1e-5, 5, w2.cuda(), 1e-3, out)
+        assert rel_err(xs.cpu(), want) <= 2e-6 and rel_err(out.float().cpu(), P.rms_norm(want, w2.double(), 1e-3)) <= tol
+    xs = x.cuda()
+    ops.rmsnorm_add(xs, d.cuda(), gain[:1].cuda(), 1e-5, 5)
+    assert rel_err(xs.cpu(), x.double() + P.rms_norm(d.double(), gain[:1].double(), 1e-5)) <= 2e-6
 
 
 def test_small_row_kernels():
