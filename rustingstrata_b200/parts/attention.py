@@ -173,6 +173,8 @@ class PagedAttention(Mixer):
 
     def build_plan(self, batch: HostBatch):
         """Work lists: sequences with one query take the split (decode) form, the rest are cut into query tiles."""
+        if self.q_per_cta is None:
+            self.plan_key()                       # asks the kernels for their tile sizes
         single = batch.q_lens == 1
         qpc = self._tile_tokens(batch.q_lens[~single])
         dec = np.nonzero(single)[0].astype(np.int32)
