@@ -1,6 +1,6 @@
 // Memory-bound kernels of the step: token embedding, RMSNorm (optionally gathering
 // rows), per-head QK-norm + rotary encoding + write of K and V into cache pages,
-// SiLU(gate)*up.  Each is templated on the activation element type so the 32-bit and
+// SiLU(gate)*up, a projection gated by a token's table row, capped logits.  Each is templated on the activation element type so the 32-bit and
 // the bfloat16 engine run the same code; reductions and the rotation are float32.
 //
 // Reference counterparts (RustingStrata, src/cuda/kernels.cu): rms_norm :1504-1552,

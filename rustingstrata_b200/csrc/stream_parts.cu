@@ -3,10 +3,7 @@
 //     to every residual stream; the previous token of a request's next portion lives in its state slot;
 //   * stream_layernorm: layer norm (weight and bias) of a weighted sum of the residual streams of a token;
 //   * stream_update: all streams at once from the old ones, x_t <- sum_s mix[s, t] x_s + out[t] y, and in the same
-//     pass the layer norm of the next reader's weighted sum;
-//   * router_topk: softmax or sigmoid over expert logits, choice by score + correction (within the best groups of
-//     experts, if they form groups), weights from the uncorrected scores
-//     of the chosen experts divided by their sum.
+//     pass the layer norm of the next reader's weighted sum.
 // Everything here is float32 whatever the activation type is; a token's row is computed in an order that only the
 // row's own width fixes, never the batch.
 #include "common.cuh"

@@ -33,7 +33,7 @@ NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "-Xcompil
 LIBRARIES: Dict[str, Dict[str, List[str]]] = {
     "core": {"sources": ["elementwise.cu", "linear_simt.cu", "attention_simt.cu", "sampling.cu", "sequence_parts.cu",
                          "moe_simt.cu"], "link": []},
-    # several residual streams, summed embedding tables, routers, convolved and gated attention (both engines)
+    # several residual streams, summed embedding tables, convolved and gated attention (both engines)
     "stream": {"sources": ["stream_parts.cu", "conv_attention_parts.cu"], "link": []},
     # mixers that keep a state matrix per head (gated write, delta rule, decay per head), attention with scores mixed across heads,
     # a sink and head gates, and the activations that go with them (both engines)

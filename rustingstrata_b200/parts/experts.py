@@ -1,5 +1,6 @@
-"""Feed-forwards beyond the gated one: a plain two-matrix layer with a squared ReLU, and a mixture of experts whose
-choice is a table from token id to expert ids (no router to evaluate), with an optional shared expert.
+"""Feed-forwards beyond the gated one: a plain two-matrix layer with a squared ReLU, a mixture of experts whose choice is
+a table from token id to expert ids (no router to evaluate), and a mixture whose experts a router chooses per token, both
+with an optional shared expert.
 
 ``table_moe``: every token uses the ``top`` experts its id names, each with weight 1 / top; an expert is
 down(SiLU(gate h) * (up h)) without biases.  A shared expert of the same form runs for every token and is added,
